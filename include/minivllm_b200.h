@@ -20,8 +20,8 @@
 extern "C" {
 #endif
 
-/* Element types of q/k/v and of a non-quantised cache. */
-enum mv_dtype { MV_F16 = 0, MV_BF16 = 1 };
+/* Element types of activations, weights and of a non-quantised cache (each entry point says which it takes). */
+enum mv_dtype { MV_F16 = 0, MV_BF16 = 1, MV_F32 = 2 };
 
 enum mv_status {
   MV_OK = 0,
@@ -412,6 +412,96 @@ int mv_add_rmsnorm(void* out, const void* x, const void* residual_in,
  */
 int mv_silu_mul(void* out, const void* gate_up, int64_t gate_up_stride,
                 int64_t rows, int inter, int dtype, void* stream);
+
+/*
+ * Steps between the sublayers of a decoder with an fp32 residual stream x (rows, width), updated in place, and RMS
+ * norms over `groups` equal runs of channels.  dtype (MV_BF16 or MV_F32) is that of every void* operand; *_stride
+ * are row strides in elements.  No counterpart in the reference.
+ *   mv_embed_norm           x = embed[ids];  out = norm(x) * w_next
+ *   mv_gated_residual_norm  y' = y * sigmoid(gate + gate_bias) (gate may be null);
+ *                           x += mult * norm(y') * w_post;  out = norm(x) * w_next
+ *   mv_moe_residual_norm    the same with y = sum_k top_weights[t, k] * expert_rows[pos[t, k]]
+ *                           + sigmoid(shared_gate[t]) * shared[t]   (shared may be null)
+ *   mv_gated_group_norm     out = norm(y * silu(z)) * w
+ *   mv_gate_mul             out = y * act(gate), act 0 = sigmoid, 1 = silu; a row of y is `heads` pieces
+ *                           y_head_stride elements apart
+ */
+int mv_embed_norm(void* out, float* x, const int64_t* ids, const void* embed, int64_t vocab, const
+    void* w_next, int64_t rows, int width, int groups, float eps, int dtype, void* stream);
+int mv_gated_residual_norm(void* out, float* x, const void* y, int64_t y_stride, const void* gate,
+    int64_t gate_stride, const void* gate_bias, const void* w_post, const void* w_next, float mult,
+    int64_t rows, int width, int groups, float eps, int dtype, void* stream);
+int mv_moe_residual_norm(void* out, float* x, const void* expert_rows, const int32_t* pos, const
+    float* top_weights, int top, const void* shared, int64_t shared_stride, const void* shared_gate,
+    int64_t shared_gate_stride, const void* gate, int64_t gate_stride, const void* gate_bias, const
+    void* w_post, const void* w_next, float mult, int64_t rows, int width, int groups, float eps,
+    int dtype, void* stream);
+int mv_gated_group_norm(void* out, const void* y, int64_t y_stride, const void* z, int64_t z_stride,
+    const void* w, int64_t rows, int width, int groups, float eps, int dtype, void* stream);
+int mv_gate_mul(void* out, const void* y, int64_t y_stride, int64_t y_head_stride, int heads,
+    const void* gate, int64_t gate_stride, int act, int64_t rows, int cols, int dtype, void* stream);
+
+/*
+ * Latent attention over a paged cache (num_blocks, block_size, rank + rot_dim) of rows [c | rotated key part].
+ *   mv_latent_prep  down (tokens, rank + rot_dim, row stride): c = rms_norm(down[:rank]) * c_weight, rotary on the
+ *                   shared key part and, in place, on the last rot_dim entries of every head of q (tokens,
+ *                   heads * (dim + rot_dim)); rows go to latent_out (contiguous, may be null) and to cache[slot]
+ *                   (slot < 0 skips).  cos/sin tables (max_position, rope_dims / 2) fp32.
+ *   mv_latent_attention_rows  out[t, h] = sum_j softmax_j((q_lat . c_j + q_rot . k_j) * scale) c_j over keys
+ *                   j <= positions[t] (token and head strides of out, q_lat and q_rot in elements), with exp(sink[h]) added to the denominator (sink may be null).  Token t belongs
+ *                   to the sequence of cu_q (null: token t is row t of block_tables).  Any sizes up to rank 1,024.
+ * dtype MV_BF16 or MV_F32.  No counterpart in the reference.
+ */
+int mv_latent_prep(void* q, int64_t q_stride, const void* down, int64_t down_stride, const void*
+    c_weight, const int64_t* positions, const float* cos_table, const float* sin_table, int64_t
+    max_position, void* latent_out, void* cache, const int64_t* slot_mapping, int64_t num_slots,
+    int64_t tokens, int heads, int dim, int rot_dim, int rope_dims, int rank, float eps, int dtype,
+    void* stream);
+int mv_latent_attention_rows(void* out, int64_t out_stride, int64_t out_head_stride, const void* q_lat,
+    int64_t q_lat_stride, int64_t q_lat_head_stride, const void* q_rot,
+    int64_t q_rot_stride, int64_t q_rot_head_stride, const void* cache, const int32_t* block_tables,
+    int64_t bt_stride, int max_blocks, int block_size, int64_t num_blocks, const int32_t* cu_q, int
+    num_seqs, const int64_t* positions, const void* sink, int64_t tokens, int heads, int rank, int
+    rot_dim, float scale, int dtype, void* stream);
+
+/*
+ * State-space mixer over a packed batch.  Sequence s has tokens cu[s] .. cu[s + 1] (cu null: one token each), slot
+ * slots[s] and start[s] earlier tokens; start 0 reads the slot as zeros, start < 0 marks a padding row.
+ *   mv_conv_silu          out (tokens, channels) = silu(causal depthwise convolution of u with w (channels, taps))
+ *   mv_conv_state_update  state (num_slots, taps - 1, channels): the last inputs, oldest first
+ *   mv_ssm_scan           xbc = [x: heads * vdim | B: groups * state_dim | C: the same] per token, dt before
+ *                         bias and softplus; state (num_slots, heads, state_dim, vdim) fp32, updated
+ * dtype MV_BF16 or MV_F32.  No counterpart in the reference.
+ */
+int mv_conv_silu(void* out, const void* u, int64_t u_stride, const void* w, const void* bias, int
+    taps, int channels, const int32_t* cu, int num_seqs, int64_t tokens, const int32_t* slots, const
+    int32_t* start, const void* state, int num_slots, int dtype, void* stream);
+int mv_conv_state_update(void* state, const void* u, int64_t u_stride, int taps, int channels, const
+    int32_t* cu, int num_seqs, const int32_t* slots, const int32_t* start, int num_slots, int dtype,
+    void* stream);
+int mv_ssm_scan(void* y, const void* xbc, const void* dt, int64_t dt_stride, const void* dt_bias,
+    const void* A_log, const void* D, const int32_t* cu, int num_seqs, const int32_t* slots, const
+    int32_t* start, float* state, int num_slots, int heads, int vdim, int state_dim, int groups, int
+    dtype, void* stream);
+
+/*
+ * Mixture of experts; the routing never leaves the device.
+ *   mv_moe_route    idx, weight (tokens, top): largest logits + bias, softmax over them
+ *   mv_moe_sort     stable sort of the tokens * top entries by expert: pos[entry] = row, row_token[row] = token,
+ *                   offsets (experts + 1) = row ranges
+ *   mv_gather_rows  out[r] = x[row_token[r]]
+ *   mv_grouped_rows rows of expert e times w[e]^T (out_dim, in_dim); gated: w[e] = [gate; up], silu(gate) * up
+ * No counterpart in the reference.
+ */
+int mv_moe_route(int32_t* idx, float* weight, const float* logits, int64_t logits_stride, const
+    float* bias, int64_t tokens, int experts, int top, void* stream);
+int64_t mv_moe_sort_workspace_bytes(int64_t tokens, int experts, int top);
+int mv_moe_sort(int32_t* pos, int32_t* row_token, int32_t* offsets, const int32_t* idx, int64_t
+    tokens, int experts, int top, void* workspace, int64_t workspace_bytes, void* stream);
+int mv_gather_rows(void* out, const void* x, int64_t x_stride, const int32_t* row_token, int64_t
+    rows, int width, int dtype, void* stream);
+int mv_grouped_rows(void* out, const void* x, const void* w, const int32_t* offsets, int experts,
+    int64_t rows, int in_dim, int out_dim, int gated, int dtype, void* stream);
 
 #ifdef __cplusplus
 }

@@ -13,7 +13,7 @@ import torch
 _HERE = os.path.dirname(os.path.abspath(__file__))
 LIB_PATH = os.path.join(_HERE, "csrc", "libminivllm_b200.so")
 
-MV_F16, MV_BF16 = 0, 1
+MV_F16, MV_BF16, MV_F32 = 0, 1, 2
 
 _c_i64 = ctypes.c_int64
 _c_int = ctypes.c_int
@@ -67,21 +67,58 @@ SIGNATURES = {
     "mv_add_rmsnorm": (_c_int, [_c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_i64, _c_i64, _c_ptr, _c_f32, _c_i64, _c_int,
                                 _c_int, _c_ptr]),
     "mv_silu_mul": (_c_int, [_c_ptr, _c_ptr, _c_i64, _c_i64, _c_int, _c_int, _c_ptr]),
+    "mv_embed_norm": (_c_int, [_c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_i64, _c_ptr, _c_i64, _c_int, _c_int, _c_f32,
+        _c_int, _c_ptr]),
+    "mv_gated_residual_norm": (_c_int, [_c_ptr, _c_ptr, _c_ptr, _c_i64, _c_ptr, _c_i64, _c_ptr, _c_ptr, _c_ptr,
+        _c_f32, _c_i64, _c_int, _c_int, _c_f32, _c_int, _c_ptr]),
+    "mv_moe_residual_norm": (_c_int, [_c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_int, _c_ptr, _c_i64, _c_ptr,
+        _c_i64, _c_ptr, _c_i64, _c_ptr, _c_ptr, _c_ptr, _c_f32, _c_i64, _c_int, _c_int, _c_f32, _c_int, _c_ptr]),
+    "mv_gated_group_norm": (_c_int, [_c_ptr, _c_ptr, _c_i64, _c_ptr, _c_i64, _c_ptr, _c_i64, _c_int, _c_int, _c_f32,
+        _c_int, _c_ptr]),
+    "mv_gate_mul": (_c_int, [_c_ptr, _c_ptr, _c_i64, _c_i64, _c_int, _c_ptr, _c_i64, _c_int, _c_i64, _c_int, _c_int,
+        _c_ptr]),
+    "mv_latent_prep": (_c_int, [_c_ptr, _c_i64, _c_ptr, _c_i64, _c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_i64, _c_ptr,
+        _c_ptr, _c_ptr, _c_i64, _c_i64, _c_int, _c_int, _c_int, _c_int, _c_int, _c_f32, _c_int, _c_ptr]),
+    "mv_latent_attention_rows": (_c_int, [_c_ptr, _c_i64, _c_i64, _c_ptr, _c_i64, _c_i64, _c_ptr, _c_i64, _c_i64, _c_ptr, _c_ptr, _c_i64,
+        _c_int, _c_int, _c_i64, _c_ptr, _c_int, _c_ptr, _c_ptr, _c_i64, _c_int, _c_int, _c_int, _c_f32, _c_int,
+        _c_ptr]),
+    "mv_conv_silu": (_c_int, [_c_ptr, _c_ptr, _c_i64, _c_ptr, _c_ptr, _c_int, _c_int, _c_ptr, _c_int, _c_i64,
+        _c_ptr, _c_ptr, _c_ptr, _c_int, _c_int, _c_ptr]),
+    "mv_conv_state_update": (_c_int, [_c_ptr, _c_ptr, _c_i64, _c_int, _c_int, _c_ptr, _c_int, _c_ptr, _c_ptr,
+        _c_int, _c_int, _c_ptr]),
+    "mv_ssm_scan": (_c_int, [_c_ptr, _c_ptr, _c_ptr, _c_i64, _c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_int, _c_ptr, _c_ptr,
+        _c_ptr, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_ptr]),
+    "mv_moe_route": (_c_int, [_c_ptr, _c_ptr, _c_ptr, _c_i64, _c_ptr, _c_i64, _c_int, _c_int, _c_ptr]),
+    "mv_moe_sort_workspace_bytes": (_c_i64, [_c_i64, _c_int, _c_int]),
+    "mv_moe_sort": (_c_int, [_c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_i64, _c_int, _c_int, _c_ptr, _c_i64, _c_ptr]),
+    "mv_gather_rows": (_c_int, [_c_ptr, _c_ptr, _c_i64, _c_ptr, _c_i64, _c_int, _c_int, _c_ptr]),
+    "mv_grouped_rows": (_c_int, [_c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_int, _c_i64, _c_int, _c_int, _c_int, _c_int,
+        _c_ptr]),
 }
 
 _lib = None
+_lib_path = LIB_PATH
+
+
+def use_library(path):
+    """Selects the library to load: one that holds the kernels of a single model family (csrc/build.py)."""
+    global _lib, _lib_path
+    if path != _lib_path:
+        _lib, _lib_path = None, path
 
 
 def lib():
     """Loads the shared library once; raises if it is missing."""
     global _lib
     if _lib is None:
-        if not os.path.exists(LIB_PATH):
+        if not os.path.exists(_lib_path):
             raise RuntimeError(
-                f"{LIB_PATH} is missing: build it with `python -m minivllm_b200.csrc.build` "
+                f"{_lib_path} is missing: build it with `python -m minivllm_b200.csrc.build` "
                 "(this package has no fallback path)")
-        handle = ctypes.CDLL(LIB_PATH)
+        handle = ctypes.CDLL(_lib_path)
         for name, (restype, argtypes) in SIGNATURES.items():
+            if _lib_path != LIB_PATH and not hasattr(handle, name):
+                continue             # another family's kernel
             fn = getattr(handle, name)
             fn.restype = restype
             fn.argtypes = argtypes
@@ -105,6 +142,19 @@ def dtype_code(dt):
     if dt == torch.bfloat16:
         return MV_BF16
     raise ValueError(f"minivllm_b200 kernels take float16 or bfloat16 tensors, got {dt}")
+
+
+def layer_dtype_code(dt):
+    """Element type of the operators that run in bf16 or in 32-bit."""
+    if dt == torch.bfloat16:
+        return MV_BF16
+    if dt == torch.float32:
+        return MV_F32
+    raise ValueError(f"this operator takes bfloat16 or float32 tensors, got {dt}")
+
+
+def logits_dtype_code(dt):
+    return MV_F32 if dt == torch.float32 else dtype_code(dt)
 
 
 def stream_ptr():

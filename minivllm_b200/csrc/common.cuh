@@ -49,6 +49,12 @@ template <> struct Elem<__nv_bfloat16> {
   }
 };
 
+template <> struct Elem<float> {
+  using T2 = float2;
+  static __device__ __forceinline__ float to_f(float x) { return x; }
+  static __device__ __forceinline__ float from_f(float x) { return x; }
+};
+
 // 16-byte streaming load that does not allocate in L1 (data is used once).
 __device__ __forceinline__ uint4 ld_stream16(const void* p) {
   uint4 v;

@@ -1,0 +1,364 @@
+// What stands between two sublayers of a decoder whose residual stream is fp32 and whose RMS norms work on
+// groups of channels: one launch takes a sublayer's result (or the embedding row, or the pieces of a mixture of
+// experts), gates it element by element, normalises it, adds it to the residual stream, normalises the sum and
+// writes the next sublayer's input.  Plus the gated group norm that ends a state-space mixer, and a sigmoid gate.
+//
+// HBM-bound.  A CTA owns a row and keeps it in shared memory as fp32; every group of channels belongs to a fixed
+// set of warps, so sums are formed in a fixed order whatever the batch.
+#include <algorithm>
+#include "vec.cuh"
+
+namespace mv {
+
+constexpr int kNormThreads = 256;
+constexpr int kNormWarps = kNormThreads / 32;
+
+enum { SRC_EMBED = 0, SRC_ROWS = 1, SRC_EXPERTS = 2 };
+
+template <typename T> struct ResidualParams {
+  T* out;                  // (rows, width): normalised residual
+  float* x;                // (rows, width): residual stream, updated (SRC_EMBED: written)
+  const T* y; int64_t y_stride;                 // SRC_ROWS: sublayer result;  SRC_EXPERTS: expert rows (sorted)
+  const T* gate; int64_t gate_stride; const T* gate_bias;   // logits of the element gate (null: no gate)
+  const T* w_post;         // norm of the sublayer's result
+  const T* w_next;         // norm of the new residual
+  const int64_t* ids; const T* embed; int64_t vocab;        // SRC_EMBED
+  const int32_t* pos; const float* topw; int top;           // SRC_EXPERTS: row of (token, k) and its weight
+  const T* shared; int64_t shared_stride; const T* sg; int64_t sg_stride;   // shared expert and its scalar gate
+  float mult;
+  int width, groups;
+  float eps;
+};
+
+// Which warps sum which group: `wpg` warps each, `cg` groups at a time.
+struct GroupPlan {
+  int wpg, cg, g0, sub, chunks, gs;
+  __device__ __forceinline__ GroupPlan(int width, int groups, int V, int warp) {
+    wpg = groups >= kNormWarps ? 1 : kNormWarps / groups;
+    cg = kNormWarps / wpg;
+    g0 = warp / wpg;
+    sub = warp - g0 * wpg;
+    gs = width / groups;
+    chunks = gs / V;
+    if (g0 >= cg) g0 = groups;   // left-over warps
+  }
+};
+__device__ __forceinline__ float group_rs(const float* part, int g, int wpg, int gs, float eps) {
+  float s = 0.f;
+  for (int k = 0; k < wpg; ++k) s += part[g * wpg + k];
+  return 1.f / sqrtf(s / static_cast<float>(gs) + eps);
+}
+
+template <typename T, int V, int SRC>
+__global__ void __launch_bounds__(kNormThreads) residual_norm_kernel(const ResidualParams<T> p) {
+  extern __shared__ __align__(16) float s_row[];
+  float* part = s_row + ((p.width + 3) & ~3);
+  float* part2 = part + (p.groups < kNormWarps ? kNormWarps : p.groups);
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+  const int64_t row = blockIdx.x;
+  const GroupPlan gp(p.width, p.groups, V, warp);
+  float* x = p.x + row * p.width;
+  float sgate = 0.f;
+  int64_t token = 0;
+  if (SRC == SRC_EMBED) {
+    token = p.ids[row];
+    if (token < 0 || token >= p.vocab) token = 0;   // placeholder rows of a padded batch
+  }
+  if (SRC == SRC_EXPERTS && p.shared) sgate = p.sg ? sigmoid_f(Elem<T>::to_f(p.sg[row * p.sg_stride])) : 1.f;
+
+  for (int g = gp.g0; g < p.groups; g += gp.cg) {
+    float acc = 0.f;
+    for (int i = gp.sub * 32 + lane; i < gp.chunks; i += gp.wpg * 32) {
+      const int c = g * gp.gs + i * V;
+      float v[V];
+      if (SRC == SRC_EMBED) {
+        Vec<T, V>::load(p.embed + token * p.width + c, v);
+        Vec<float, V>::store(x + c, v);
+      } else {
+        if (SRC == SRC_ROWS) {
+          Vec<T, V>::load(p.y + row * p.y_stride + c, v);
+        } else {
+#pragma unroll
+          for (int e = 0; e < V; ++e) v[e] = 0.f;
+          for (int k = 0; k < p.top; ++k) {
+            const float w = p.topw[row * p.top + k];
+            float t[V];
+            Vec<T, V>::load(p.y + static_cast<int64_t>(p.pos[row * p.top + k]) * p.y_stride + c, t);
+#pragma unroll
+            for (int e = 0; e < V; ++e) v[e] = fmaf(w, t[e], v[e]);
+          }
+          if (p.shared) {
+            float t[V];
+            Vec<T, V>::load(p.shared + row * p.shared_stride + c, t);
+#pragma unroll
+            for (int e = 0; e < V; ++e) v[e] = fmaf(sgate, t[e], v[e]);
+          }
+        }
+        if (p.gate) {
+          float t[V], b[V];
+          Vec<T, V>::load(p.gate + row * p.gate_stride + c, t);
+          Vec<T, V>::load(p.gate_bias + c, b);
+#pragma unroll
+          for (int e = 0; e < V; ++e) v[e] *= sigmoid_f(t[e] + b[e]);
+        }
+      }
+#pragma unroll
+      for (int e = 0; e < V; ++e) acc = fmaf(v[e], v[e], acc);
+      Vec<float, V>::store(s_row + c, v);
+    }
+    acc = warp_sum(acc);
+    if (lane == 0) part[g * gp.wpg + gp.sub] = acc;
+  }
+  __syncthreads();
+  const float* fin = part;
+  if (SRC != SRC_EMBED) {
+    for (int g = gp.g0; g < p.groups; g += gp.cg) {
+      const float rs = group_rs(part, g, gp.wpg, gp.gs, p.eps);
+      float acc = 0.f;
+      for (int i = gp.sub * 32 + lane; i < gp.chunks; i += gp.wpg * 32) {
+        const int c = g * gp.gs + i * V;
+        float v[V], w[V], r[V];
+        Vec<float, V>::load(s_row + c, v);
+        Vec<T, V>::load(p.w_post + c, w);
+        Vec<float, V>::load(x + c, r);
+#pragma unroll
+        for (int e = 0; e < V; ++e) {
+          r[e] = fmaf(p.mult, v[e] * rs * w[e], r[e]);
+          acc = fmaf(r[e], r[e], acc);
+        }
+        Vec<float, V>::store(x + c, r);
+        Vec<float, V>::store(s_row + c, r);
+      }
+      acc = warp_sum(acc);
+      if (lane == 0) part2[g * gp.wpg + gp.sub] = acc;
+    }
+    __syncthreads();
+    fin = part2;
+  }
+  for (int g = gp.g0; g < p.groups; g += gp.cg) {
+    const float rs = group_rs(fin, g, gp.wpg, gp.gs, p.eps);
+    for (int i = gp.sub * 32 + lane; i < gp.chunks; i += gp.wpg * 32) {
+      const int c = g * gp.gs + i * V;
+      float v[V], w[V];
+      Vec<float, V>::load(s_row + c, v);
+      Vec<T, V>::load(p.w_next + c, w);
+#pragma unroll
+      for (int e = 0; e < V; ++e) v[e] = v[e] * rs * w[e];
+      Vec<T, V>::store(p.out + row * p.width + c, v);
+    }
+  }
+}
+
+// out = group_rms_norm(y * silu(z)) * w
+template <typename T, int V>
+__global__ void __launch_bounds__(kNormThreads)
+gated_group_norm_kernel(T* __restrict__ out, const T* __restrict__ y, int64_t y_stride, const T* __restrict__ z,
+                        int64_t z_stride, const T* __restrict__ w, int width, int groups, float eps) {
+  extern __shared__ __align__(16) float s_row[];
+  float* part = s_row + ((width + 3) & ~3);
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+  const int64_t row = blockIdx.x;
+  const GroupPlan gp(width, groups, V, warp);
+  for (int g = gp.g0; g < groups; g += gp.cg) {
+    float acc = 0.f;
+    for (int i = gp.sub * 32 + lane; i < gp.chunks; i += gp.wpg * 32) {
+      const int c = g * gp.gs + i * V;
+      float v[V], t[V];
+      Vec<T, V>::load(y + row * y_stride + c, v);
+      Vec<T, V>::load(z + row * z_stride + c, t);
+#pragma unroll
+      for (int e = 0; e < V; ++e) {
+        v[e] *= silu_f(t[e]);
+        acc = fmaf(v[e], v[e], acc);
+      }
+      Vec<float, V>::store(s_row + c, v);
+    }
+    acc = warp_sum(acc);
+    if (lane == 0) part[g * gp.wpg + gp.sub] = acc;
+  }
+  __syncthreads();
+  for (int g = gp.g0; g < groups; g += gp.cg) {
+    const float rs = group_rs(part, g, gp.wpg, gp.gs, eps);
+    for (int i = gp.sub * 32 + lane; i < gp.chunks; i += gp.wpg * 32) {
+      const int c = g * gp.gs + i * V;
+      float v[V], t[V];
+      Vec<float, V>::load(s_row + c, v);
+      Vec<T, V>::load(w + c, t);
+#pragma unroll
+      for (int e = 0; e < V; ++e) v[e] = v[e] * rs * t[e];
+      Vec<T, V>::store(out + row * width + c, v);
+    }
+  }
+}
+
+// out = y * act(gate); row r of y is `heads` pieces of cols / heads elements, y_head_stride apart
+template <typename T, int V>
+__global__ void __launch_bounds__(kNormThreads)
+gate_mul_kernel(T* __restrict__ out, const T* __restrict__ y, int64_t y_stride, int64_t y_head_stride, int head_cols,
+                const T* __restrict__ gate, int64_t gate_stride, int act, int64_t rows, int cols) {
+  const int per = cols / V;
+  const int64_t total = rows * per;
+  for (int64_t i = static_cast<int64_t>(blockIdx.x) * kNormThreads + threadIdx.x; i < total;
+       i += static_cast<int64_t>(gridDim.x) * kNormThreads) {
+    const int64_t row = i / per;
+    const int c = static_cast<int>(i - row * per) * V, h = c / head_cols;
+    float v[V], g[V];
+    Vec<T, V>::load(y + row * y_stride + h * y_head_stride + (c - h * head_cols), v);
+    Vec<T, V>::load(gate + row * gate_stride + c, g);
+#pragma unroll
+    for (int e = 0; e < V; ++e) v[e] *= act ? silu_f(g[e]) : sigmoid_f(g[e]);
+    Vec<T, V>::store(out + row * cols + c, v);
+  }
+}
+
+static size_t norm_smem(int width, int groups) {
+  return sizeof(float) * (((width + 3) & ~3) + 2 * (groups < kNormWarps ? kNormWarps : groups));
+}
+template <typename K> static int allow_smem(K kernel, size_t bytes, const char* what) {
+  if (bytes > 227 * 1024) return fail(MV_ERR_LIMIT, "%s: a row does not fit in shared memory", what);
+  if (bytes > 48 * 1024) {
+    const cudaError_t e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(bytes));
+    if (e != cudaSuccess) return fail(MV_ERR_CUDA, "%s: %s", what, cudaGetErrorString(e));
+  }
+  return MV_OK;
+}
+
+template <typename T, int V, int SRC>
+static int launch_residual(const ResidualParams<T>& p, int64_t rows, cudaStream_t st) {
+  const size_t smem = norm_smem(p.width, p.groups);
+  const int rc = allow_smem(residual_norm_kernel<T, V, SRC>, smem, "residual_norm");
+  if (rc) return rc;
+  residual_norm_kernel<T, V, SRC><<<static_cast<unsigned>(rows), kNormThreads, smem, st>>>(p);
+  return check_launch("residual_norm");
+}
+template <typename T, int SRC>
+static int launch_residual_v(const ResidualParams<T>& p, int64_t rows, cudaStream_t st) {
+  const int eb = sizeof(T);
+  bool v8 = (p.width / p.groups) % 8 == 0 && aligned16(p.out) && aligned16(p.x) && aligned16(p.w_next) &&
+            vec8_ok(p.y, p.y_stride, eb) && vec8_ok(p.gate, p.gate_stride, eb) && vec8_ok(p.gate_bias, 0, eb) &&
+            vec8_ok(p.w_post, 0, eb) && vec8_ok(p.embed, p.width, eb) && vec8_ok(p.shared, p.shared_stride, eb);
+  return v8 ? launch_residual<T, 8, SRC>(p, rows, st) : launch_residual<T, 1, SRC>(p, rows, st);
+}
+static int check_norm(const char* what, int width, int groups, int dtype) {
+  if (dtype != MV_BF16 && dtype != MV_F32) return fail(MV_ERR_DTYPE, "%s: dtype %d", what, dtype);
+  if (width <= 0 || groups <= 0 || width % groups) return fail(MV_ERR_SHAPE, "%s: width %d in %d groups", what, width, groups);
+  return MV_OK;
+}
+
+}  // namespace mv
+
+extern "C" int mv_embed_norm(void* out, float* x, const int64_t* ids, const void* embed, int64_t vocab,
+                             const void* w_next, int64_t rows, int width, int groups, float eps, int dtype,
+                             void* stream) {
+  using namespace mv;
+  int rc = check_norm("embed_norm", width, groups, dtype);
+  if (rc || rows == 0) return rc;
+  if (!out || !x || !ids || !embed || !w_next) return fail(MV_ERR_NULL, "embed_norm: null pointer");
+  auto run = [&](auto tag) {
+    using T = decltype(tag);
+    ResidualParams<T> p{};
+    p.out = static_cast<T*>(out); p.x = x; p.ids = ids; p.embed = static_cast<const T*>(embed); p.vocab = vocab;
+    p.w_next = static_cast<const T*>(w_next); p.width = width; p.groups = groups; p.eps = eps;
+    return launch_residual_v<T, SRC_EMBED>(p, rows, static_cast<cudaStream_t>(stream));
+  };
+  return dtype == MV_F32 ? run(float{}) : run(__nv_bfloat16{});
+}
+
+extern "C" int mv_gated_residual_norm(void* out, float* x, const void* y, int64_t y_stride, const void* gate,
+                                      int64_t gate_stride, const void* gate_bias, const void* w_post,
+                                      const void* w_next, float mult, int64_t rows, int width, int groups, float eps,
+                                      int dtype, void* stream) {
+  using namespace mv;
+  int rc = check_norm("gated_residual_norm", width, groups, dtype);
+  if (rc || rows == 0) return rc;
+  if (!out || !x || !y || !w_post || !w_next || (gate && !gate_bias))
+    return fail(MV_ERR_NULL, "gated_residual_norm: null pointer");
+  auto run = [&](auto tag) {
+    using T = decltype(tag);
+    ResidualParams<T> p{};
+    p.out = static_cast<T*>(out); p.x = x; p.y = static_cast<const T*>(y); p.y_stride = y_stride;
+    p.gate = static_cast<const T*>(gate); p.gate_stride = gate_stride; p.gate_bias = static_cast<const T*>(gate_bias);
+    p.w_post = static_cast<const T*>(w_post); p.w_next = static_cast<const T*>(w_next);
+    p.mult = mult; p.width = width; p.groups = groups; p.eps = eps;
+    return launch_residual_v<T, SRC_ROWS>(p, rows, static_cast<cudaStream_t>(stream));
+  };
+  return dtype == MV_F32 ? run(float{}) : run(__nv_bfloat16{});
+}
+
+extern "C" int mv_moe_residual_norm(void* out, float* x, const void* expert_rows, const int32_t* pos,
+                                    const float* top_weights, int top, const void* shared, int64_t shared_stride,
+                                    const void* shared_gate, int64_t shared_gate_stride, const void* gate,
+                                    int64_t gate_stride, const void* gate_bias, const void* w_post, const void* w_next,
+                                    float mult, int64_t rows, int width, int groups, float eps, int dtype,
+                                    void* stream) {
+  using namespace mv;
+  int rc = check_norm("moe_residual_norm", width, groups, dtype);
+  if (rc || rows == 0) return rc;
+  if (!out || !x || !expert_rows || !pos || !top_weights || !w_post || !w_next || (gate && !gate_bias))
+    return fail(MV_ERR_NULL, "moe_residual_norm: null pointer");
+  if (top <= 0) return fail(MV_ERR_SHAPE, "moe_residual_norm: top %d", top);
+  auto run = [&](auto tag) {
+    using T = decltype(tag);
+    ResidualParams<T> p{};
+    p.out = static_cast<T*>(out); p.x = x; p.y = static_cast<const T*>(expert_rows); p.y_stride = width;
+    p.pos = pos; p.topw = top_weights; p.top = top;
+    p.shared = static_cast<const T*>(shared); p.shared_stride = shared_stride;
+    p.sg = static_cast<const T*>(shared_gate); p.sg_stride = shared_gate_stride;
+    p.gate = static_cast<const T*>(gate); p.gate_stride = gate_stride; p.gate_bias = static_cast<const T*>(gate_bias);
+    p.w_post = static_cast<const T*>(w_post); p.w_next = static_cast<const T*>(w_next);
+    p.mult = mult; p.width = width; p.groups = groups; p.eps = eps;
+    return launch_residual_v<T, SRC_EXPERTS>(p, rows, static_cast<cudaStream_t>(stream));
+  };
+  return dtype == MV_F32 ? run(float{}) : run(__nv_bfloat16{});
+}
+
+extern "C" int mv_gated_group_norm(void* out, const void* y, int64_t y_stride, const void* z, int64_t z_stride,
+                                   const void* w, int64_t rows, int width, int groups, float eps, int dtype,
+                                   void* stream) {
+  using namespace mv;
+  int rc = check_norm("gated_group_norm", width, groups, dtype);
+  if (rc || rows == 0) return rc;
+  if (!out || !y || !z || !w) return fail(MV_ERR_NULL, "gated_group_norm: null pointer");
+  const size_t smem = norm_smem(width, groups);
+  auto run = [&](auto tag) {
+    using T = decltype(tag);
+    const int eb = sizeof(T);
+    auto go = [&](auto kernel) {
+      const int r = allow_smem(kernel, smem, "gated_group_norm");
+      if (r) return r;
+      kernel<<<static_cast<unsigned>(rows), kNormThreads, smem, static_cast<cudaStream_t>(stream)>>>(
+          static_cast<T*>(out), static_cast<const T*>(y), y_stride, static_cast<const T*>(z), z_stride,
+          static_cast<const T*>(w), width, groups, eps);
+      return check_launch("gated_group_norm");
+    };
+    if ((width / groups) % 8 == 0 && vec8_ok(out, width, eb) && vec8_ok(y, y_stride, eb) && vec8_ok(z, z_stride, eb) &&
+        aligned16(w))
+      return go(gated_group_norm_kernel<T, 8>);
+    return go(gated_group_norm_kernel<T, 1>);
+  };
+  return dtype == MV_F32 ? run(float{}) : run(__nv_bfloat16{});
+}
+
+extern "C" int mv_gate_mul(void* out, const void* y, int64_t y_stride, int64_t y_head_stride, int heads,
+                           const void* gate, int64_t gate_stride, int act, int64_t rows, int cols, int dtype,
+                           void* stream) {
+  using namespace mv;
+  int rc = check_norm("gate_mul", cols, heads, dtype);
+  if (rc || rows == 0) return rc;
+  if (!out || !y || !gate) return fail(MV_ERR_NULL, "gate_mul: null pointer");
+  auto run = [&](auto tag) {
+    using T = decltype(tag);
+    const int eb = sizeof(T), hc = cols / heads;
+    const bool v8 = hc % 8 == 0 && aligned16(out) && vec8_ok(y, y_stride, eb) && vec8_ok(y, y_head_stride, eb) &&
+                    vec8_ok(gate, gate_stride, eb);
+    const int64_t work = rows * (v8 ? cols / 8 : cols);
+    const unsigned grid = static_cast<unsigned>(std::min<int64_t>((work + kNormThreads - 1) / kNormThreads, kNumSMs * 16));
+    auto* o = static_cast<T*>(out);
+    auto *a = static_cast<const T*>(y), *b = static_cast<const T*>(gate);
+    auto st = static_cast<cudaStream_t>(stream);
+    if (v8) gate_mul_kernel<T, 8><<<grid, kNormThreads, 0, st>>>(o, a, y_stride, y_head_stride, hc, b, gate_stride, act, rows, cols);
+    else gate_mul_kernel<T, 1><<<grid, kNormThreads, 0, st>>>(o, a, y_stride, y_head_stride, hc, b, gate_stride, act, rows, cols);
+    return check_launch("gate_mul");
+  };
+  return dtype == MV_F32 ? run(float{}) : run(__nv_bfloat16{});
+}

@@ -56,7 +56,7 @@ argmax_rows_kernel(const T* __restrict__ logits, int64_t row_stride, int64_t col
       have = true;
     }
   };
-  const int64_t chunks = aligned ? cols / 8 : 0;  // 16-byte chunks when every row starts on a 16-byte boundary
+  const int64_t chunks = sizeof(T) == 2 && aligned ? cols / 8 : 0;  // 16-byte chunks when every row starts on a 16-byte boundary
   // Per chunk of eight logits only its maximum is computed (packed 16-bit maxima, exact, NaN-propagating) and
   // compared with the running one; the chunk that raised it is kept and searched for the position at the end.
   // Chunks are visited in increasing order and only a strictly larger maximum replaces the kept chunk, so the
@@ -66,6 +66,7 @@ argmax_rows_kernel(const T* __restrict__ logits, int64_t row_stride, int64_t col
   int64_t best_chunk = -1;
   float cbest = -INFINITY;
   bool cbest_nan = false;
+  if constexpr (sizeof(T) == 2) {
   for (int64_t c0 = threadIdx.x; c0 < chunks; c0 += static_cast<int64_t>(kArgmaxThreads) * kUnroll) {
     uint4 raw[kUnroll];
 #pragma unroll
@@ -98,6 +99,7 @@ argmax_rows_kernel(const T* __restrict__ logits, int64_t row_stride, int64_t col
       offer(f.x, static_cast<uint32_t>(best_chunk * 8 + 2 * j));
       offer(f.y, static_cast<uint32_t>(best_chunk * 8 + 2 * j + 1));
     }
+  }
   }
   for (int64_t i = chunks * 8 + threadIdx.x; i < cols; i += kArgmaxThreads)   // ragged tail
     offer(Elem<T>::to_f(row[i]), static_cast<uint32_t>(i));
@@ -188,8 +190,9 @@ sample_rows_kernel(const T* __restrict__ logits, int64_t row_stride, int64_t col
     return race_noise(lane == 0 ? r.x : lane == 1 ? r.y : lane == 2 ? r.z : r.w);
   };
   // 16-byte chunks of eight logits = two Philox groups, when rows and the shard start on such boundaries
-  const bool fast = aligned && (index_offset & 7u) == 0;
+  const bool fast = sizeof(T) == 2 && aligned && (index_offset & 7u) == 0;
   const int64_t chunks = fast ? cols / 8 : 0;
+  if constexpr (sizeof(T) == 2) {
   for (int64_t c = threadIdx.x; c < chunks; c += kArgmaxThreads) {
     const uint4 raw = ld_stream16(row + c * 8);
     const T2* p2 = reinterpret_cast<const T2*>(&raw);
@@ -210,6 +213,7 @@ sample_rows_kernel(const T* __restrict__ logits, int64_t row_stride, int64_t col
     }
 #pragma unroll
     for (int j = 0; j < 8; ++j) offer(v[j], static_cast<uint32_t>(c * 8 + j));
+  }
   }
   for (int64_t i = chunks * 8 + threadIdx.x; i < cols; i += kArgmaxThreads) {
     float v = Elem<T>::to_f(row[i]);
@@ -251,7 +255,7 @@ __global__ void argmax_decode_kernel(const long long* __restrict__ keys, int sha
 extern "C" int mv_argmax_rows(const void* logits, int64_t row_stride, int64_t rows, int64_t cols,
                               int64_t index_offset, int64_t* keys, int64_t* tokens, int dtype, void* stream) {
   using namespace mv;
-  if (dtype != MV_F16 && dtype != MV_BF16) return fail(MV_ERR_DTYPE, "argmax_rows: dtype %d", dtype);
+  if (dtype < MV_F16 || dtype > MV_F32) return fail(MV_ERR_DTYPE, "argmax_rows: dtype %d", dtype);
   if (rows < 0 || cols <= 0 || index_offset < 0) return fail(MV_ERR_SHAPE, "argmax_rows: negative or zero size");
   if (rows == 0) return MV_OK;
   if (!logits || (!keys && !tokens)) return fail(MV_ERR_NULL, "argmax_rows: null pointer");
@@ -264,6 +268,10 @@ extern "C" int mv_argmax_rows(const void* logits, int64_t row_stride, int64_t ro
   if (dtype == MV_F16)
     argmax_rows_kernel<__half><<<grid, kArgmaxThreads, 0, st>>>(
         static_cast<const __half*>(logits), row_stride, cols, static_cast<uint32_t>(index_offset), aligned,
+        reinterpret_cast<long long*>(keys), reinterpret_cast<long long*>(tokens));
+  else if (dtype == MV_F32)
+    argmax_rows_kernel<float><<<grid, kArgmaxThreads, 0, st>>>(
+        static_cast<const float*>(logits), row_stride, cols, static_cast<uint32_t>(index_offset), aligned,
         reinterpret_cast<long long*>(keys), reinterpret_cast<long long*>(tokens));
   else
     argmax_rows_kernel<__nv_bfloat16><<<grid, kArgmaxThreads, 0, st>>>(
@@ -289,7 +297,7 @@ extern "C" int mv_sample_rows(const void* logits, int64_t row_stride, int64_t ro
                               const float* temperatures, uint64_t seed, const int64_t* step, int64_t* keys,
                               int64_t* tokens, int dtype, void* stream) {
   using namespace mv;
-  if (dtype != MV_F16 && dtype != MV_BF16) return fail(MV_ERR_DTYPE, "sample_rows: dtype %d", dtype);
+  if (dtype < MV_F16 || dtype > MV_F32) return fail(MV_ERR_DTYPE, "sample_rows: dtype %d", dtype);
   if (rows < 0 || cols <= 0 || index_offset < 0) return fail(MV_ERR_SHAPE, "sample_rows: negative or zero size");
   if (rows == 0) return MV_OK;
   if (!logits || !temperatures || !step || (!keys && !tokens)) return fail(MV_ERR_NULL, "sample_rows: null pointer");
@@ -302,6 +310,11 @@ extern "C" int mv_sample_rows(const void* logits, int64_t row_stride, int64_t ro
   if (dtype == MV_F16)
     sample_rows_kernel<__half><<<grid, kArgmaxThreads, 0, st>>>(
         static_cast<const __half*>(logits), row_stride, cols, static_cast<uint32_t>(index_offset), aligned, temperatures,
+        seed, reinterpret_cast<const long long*>(step), reinterpret_cast<long long*>(keys),
+        reinterpret_cast<long long*>(tokens));
+  else if (dtype == MV_F32)
+    sample_rows_kernel<float><<<grid, kArgmaxThreads, 0, st>>>(
+        static_cast<const float*>(logits), row_stride, cols, static_cast<uint32_t>(index_offset), aligned, temperatures,
         seed, reinterpret_cast<const long long*>(step), reinterpret_cast<long long*>(keys),
         reinterpret_cast<long long*>(tokens));
   else

@@ -109,6 +109,14 @@ class BlockManager:
             self.free_slots.append(seq.slot)
         seq.slot = -1
         seq.synced_blocks = 0
+        seq.on_device = False
+
+    def reserve(self, seq):
+        """Blocks for every token the sequence holds now (tokens were added to a sequence that has a table)."""
+        while len(seq.block_table) < seq.num_blocks:
+            if not self.free_blocks:
+                raise RuntimeError("no free cache block")
+            seq.block_table.append(self._fresh())
 
     def can_append(self, seq):
         """The decode step writes the KV of the last token (position len-1): it needs a new block

@@ -25,7 +25,9 @@ class LLMEngine:
             max_num_batched_tokens=_cfg(config, "max_num_batched_tokens", default=1024),
             num_blocks=num_blocks, block_size=self.block_size, eos=config.get("eos", -1),
             num_slots=self.model_runner.max_num_seqs,
-            prefix_caching=config.get("enable_prefix_caching", False))
+            prefix_caching=config.get("enable_prefix_caching", False),
+            chunked_prefill=self.model_runner.chunked_prefill)
+        self._scored = {}            # request id -> Sequence of score_step
         self.stats = dict(prefill_tokens=0, decode_tokens=0, prefill_s=0.0, decode_s=0.0, steps=0)
 
     def add_prompt(self, token_ids, sampling_params: SamplingParams = None):
@@ -39,7 +41,10 @@ class LLMEngine:
         return seq
 
     def _account(self, seqs, is_prefill, dt):
-        n = sum(len(s) - 1 - s.num_cached_tokens for s in seqs) if is_prefill else len(seqs)
+        if self.scheduler.chunked_prefill:
+            n = sum(s.num_scheduled_tokens for s in seqs)
+        else:
+            n = sum(len(s) - 1 - s.num_cached_tokens for s in seqs) if is_prefill else len(seqs)
         key = "prefill" if is_prefill else "decode"
         self.stats[key + "_tokens"] += n
         self.stats[key + "_s"] += dt
@@ -100,6 +105,39 @@ class LLMEngine:
             t_last = now
         resolve()
         return {"token_ids": [s.completion_token_ids for s in seqs]}
+
+    def score_step(self, entries, end=()):
+        """One step on given tokens instead of sampled ones: entries = [(request id, token ids, wanted places)].
+        The entries run as one batch, from the cache and state that earlier steps left; a request is admitted at its
+        first entry and gives back what it holds when its id is in `end`.  Returns the logits at the wanted places,
+        in the order of the entries, as an fp32 CPU tensor (wanted, vocab)."""
+        bm, batch = self.scheduler.block_manager, []
+        for rid, tokens, want in entries:
+            if not tokens:
+                raise ValueError(f"request '{rid}': an entry without tokens")
+            if any(not 0 <= w < len(tokens) for w in want):
+                raise ValueError(f"request '{rid}': a wanted place outside its tokens")
+            seq = self._scored.get(rid)
+            if seq is None:
+                seq = Sequence(tokens, block_size=self.block_size)
+                if not bm.can_allocate(seq):
+                    raise RuntimeError(f"request '{rid}': no free cache blocks or state slot")
+                bm.allocate(seq)
+                self._scored[rid] = seq
+            else:
+                for t in tokens:
+                    seq.append_token(t)
+                bm.reserve(seq)
+            if len(seq) > self.model_runner.max_model_len:
+                raise ValueError(f"request '{rid}' is longer than max_model_length")
+            batch.append((seq, len(tokens), list(want)))
+        logits = self.model_runner.step_logits(batch)
+        for seq, n, _ in batch:
+            seq.num_cached_tokens += n
+            seq.on_device = True
+        for rid in end:
+            bm.deallocate(self._scored.pop(rid))
+        return logits
 
     def exit(self):
         self.model_runner.exit()

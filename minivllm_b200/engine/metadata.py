@@ -67,6 +67,7 @@ class SequenceStateTable:
             out["cu_seqlens_q"].data_ptr(), out["cu_seqlens_k"].data_ptr(), out["positions"].data_ptr(),
             out["slot_mapping"].data_ptr(), out["last_token_index"].data_ptr(), _cabi.stream_ptr())
         _cabi.check(rc)
+        out["slots"], out["seq_lens"], out["starts"] = dev[0], dev[1], dev[2]
         out["max_seqlen_q"] = max(int(l) - int(c) for l, c in zip(seq_lens, cached))
         out["max_seqlen_k"] = max(int(l) for l in seq_lens)
         return out

@@ -25,7 +25,8 @@ from ..layers.attention import _error_word
 from ..utils.context import get_context, reset_context, set_context
 from .metadata import SequenceStateTable
 from ..layers.sampler import greedy_tokens, sampled_tokens
-from .qwen3 import Qwen3Config, Qwen3ForCausalLM
+from . import cache
+from .registry import build_model, family_of
 
 
 def _cfg(config, *names, default=None):
@@ -53,12 +54,28 @@ class ModelRunner:
         if self.kv_int8 and config.get("enable_prefix_caching", False):
             raise ValueError("kv_cache_dtype='int8' cannot be combined with prefix caching: the prefix-aware prefill "
                              "kernel reads fp16/bf16 caches only")
-        mcfg = Qwen3Config.from_dict(config)
+        # mixed steps (portions of prompts beside decoded tokens); models whose prefill always runs from the cache
+        # take the same path for whole prompts
+        self.chunked_prefill = bool(config.get("chunked_prefill", False))
+        if self.chunked_prefill and self.kv_int8:
+            raise ValueError("kv_cache_dtype='int8' cannot be combined with chunked prefill: portions of prompts read "
+                             "the cache through the fp16/bf16 paged prefill kernel")
+        family = family_of(config)
+        mcfg = family.config.from_dict(config)
         mcfg.max_position = max(mcfg.max_position, self.max_model_len)
         self.model_cfg = mcfg
-        self.model = model if model is not None else Qwen3ForCausalLM(
-            mcfg, tp_rank=rank, tp_size=self.world_size, dtype=self.dtype, device=self.device,
-            seed=config.get("seed", 0))
+        if not getattr(family.model, "tensor_parallel", True) and self.world_size > 1:
+            raise ValueError(f"{family.name} runs on one GPU")
+        self.model = model if model is not None else build_model(config, mcfg, rank, self.world_size, self.dtype,
+                                                                 self.device)
+        self.mixed_steps = self.chunked_prefill or getattr(self.model, "mixed_steps", False)
+        self.kv_layers = sum(hasattr(m, "k_cache") and hasattr(m, "v_cache") for m in self.model.modules())
+        self.has_state = bool(cache.state_modules(self.model))
+        if self.has_state and config.get("enable_prefix_caching", False):
+            raise ValueError("prefix caching needs every layer's past in the paged cache; this model keeps "
+                             "per-sequence state")
+        if self.dtype == torch.float32:
+            torch.backends.cuda.matmul.allow_tf32 = False    # a 32-bit model is 32-bit in its matrix products too
         self.comm, self.comm_note = None, "single rank"
         if self.world_size > 1:
             self._attach_communicator()
@@ -70,7 +87,7 @@ class ModelRunner:
         # one step counter in stream order.
         self.prefill_lanes, self._prefill_at = [], 0
         want = int(config.get("prefill_streams", 2 if self.comm is not None else 1))
-        if want >= 2 and self.greedy and self.device.type == "cuda":
+        if want >= 2 and self.greedy and not self.mixed_steps and self.device.type == "cuda":
             lanes = []
             for _ in range(2):
                 comm = self._new_communicator(staged=True) if self.comm is not None else None
@@ -97,6 +114,8 @@ class ModelRunner:
         self.decode_workspace = None
         self._stage, self._stage_at, self._stage_dev = None, 0, None
         self._readback, self._readback_at = None, 0
+        self.keep_logits = config.get("keep_logits", False)    # step_logits: decode graphs keep their logits
+        self.logits = None
         self.allocate_kv_cache()
         if not self.enforce_eager:
             self.capture_cudagraph()
@@ -104,6 +123,9 @@ class ModelRunner:
     # ------------------------------------------------------------------ memory ---
     def kv_block_bytes(self):
         c = self.model_cfg
+        latent = cache.latent_block_bytes(self.model, self.block_size, self.dtype)
+        if not self.kv_layers:
+            return latent
         rows = self.block_size * 2 * c.num_layers * (c.num_kv_heads // self.world_size)
         if self.kv_int8:
             return rows * (c.head_dim + 2)             # int8 codes + one fp16 scale per row
@@ -120,13 +142,21 @@ class ModelRunner:
             free, _ = torch.cuda.mem_get_info(self.device)
             util = self.config.get("gpu_memory_utilization", 0.9)
             reserve = self.config.get("activation_reserve_bytes", self._activation_reserve())
-            num_blocks = int((free * util - reserve) // self.kv_block_bytes())
+            reserve += self.num_slots * cache.slot_bytes(self.model, self.dtype)
+            if self.kv_block_bytes():
+                num_blocks = int((free * util - reserve) // self.kv_block_bytes())
+            else:            # no paged layer: blocks only count positions
+                num_blocks = self.max_num_seqs * self.max_blocks_per_seq
             if self.world_size > 1:  # every rank must agree on the pool size: the scheduler state is replicated
                 t = torch.tensor([num_blocks], device=self.device, dtype=torch.int64)
                 dist.all_reduce(t, op=dist.ReduceOp.MIN)
                 num_blocks = int(t.item())
         assert num_blocks >= 1, f"not enough memory for one KV block on rank {self.rank}"
         self.num_kv_blocks = num_blocks
+        self.pools = cache.bind(self.model, num_blocks, self.block_size, self.num_slots, self.dtype, self.device)
+        self.kv_cache = self.kv_scale = None
+        if not self.kv_layers:
+            return
         kvh = c.num_kv_heads // self.world_size
         self.kv_cache = torch.zeros(2, c.num_layers, num_blocks, self.block_size, kvh, c.head_dim,
                                     dtype=torch.int8 if self.kv_int8 else self.dtype, device=self.device)
@@ -146,6 +176,8 @@ class ModelRunner:
         """Peak activation bytes of the largest prefill wave (logits of the last tokens included), estimated
         from shapes instead of the reference's warm-up run."""
         c, t = self.model_cfg, self.max_num_batched_tokens
+        if hasattr(c, "widest_activation"):
+            return t * c.widest_activation() * 4 + self.max_num_seqs * c.vocab_size * 8 + (2 << 30)
         per_tok = (c.hidden_size * 6 + (c.num_heads + 2 * c.num_kv_heads) * c.head_dim * 3 // self.world_size +
                    3 * c.intermediate_size * 2 // self.world_size) * 4
         return t * per_tok + self.max_num_seqs * c.vocab_size * 8 + (2 << 30)
@@ -180,6 +212,39 @@ class ModelRunner:
                     meta["slot_mapping"], None, tables, positions=meta["positions"],
                     last_token_index=meta["last_token_index"])
         return input_ids
+
+    def prepare_mixed(self, seqs, counts, want=None):
+        """A step of counts[i] tokens of sequence i behind its num_cached_tokens.  One-token sequences are put first
+        (they take the decode kernels).  Returns the input ids and the order of the sequences in the batch.  A token
+        that the host does not know yet (-1) is the device's last sampled one.  `want`: per sequence, the places among
+        its tokens whose rows go to the LM head (default: the last)."""
+        order = sorted(range(len(seqs)), key=lambda i: counts[i] != 1)
+        seqs, counts = [seqs[i] for i in order], [counts[i] for i in order]
+        nd = sum(n == 1 for n in counts)
+        self._sync_tables(seqs)
+        ids = [t for s, n in zip(seqs, counts) for t in s.token_ids[s.num_cached_tokens:s.num_cached_tokens + n]]
+        input_ids = torch.tensor(ids, dtype=torch.int64).pin_memory().to(self.device, non_blocking=True)
+        meta = self.state.build_prefill([s.slot for s in seqs], [s.num_cached_tokens + n for s, n in zip(seqs, counts)],
+                                        [s.num_cached_tokens for s in seqs])
+        if any(t < 0 for t in ids):
+            assert all(t >= 0 for t in ids[nd:]), "a portion of a prompt holds a token that is not known yet"
+            known = input_ids[:nd]
+            last = self.state.last_token.index_select(0, meta["slots"][:nd].long())
+            input_ids[:nd] = torch.where(known < 0, last, known)
+        rows = meta["last_token_index"]
+        if want is not None:
+            at, flat = [0] * len(seqs), 0
+            for k, n in enumerate(counts):
+                at[order[k]], flat = flat, flat + n
+            rows = torch.tensor([at[i] + w for i in range(len(seqs)) for w in want[i]], dtype=torch.int64)
+            rows = rows.pin_memory().to(self.device, non_blocking=True) if rows.numel() else rows.to(self.device)
+        cu_q, cu_k = meta["cu_seqlens_q"], meta["cu_seqlens_k"]
+        set_context(True, cu_q, cu_k, meta["max_seqlen_q"], meta["max_seqlen_k"], meta["slot_mapping"],
+                    meta["seq_lens"], self.state.tables.index_select(0, meta["slots"].long()),
+                    positions=meta["positions"], last_token_index=rows, num_decode=nd,
+                    portion_cu_q=cu_q[nd:] - cu_q[nd], portion_cu_k=cu_k[nd:] - cu_k[nd],
+                    state_slots=meta["slots"], state_starts=meta["starts"])
+        return input_ids, order
 
     def _attach_communicator(self):
         """The fused all-reduce + residual + RMSNorm over NVLink peer memory (layers/allreduce.py) replaces the
@@ -244,12 +309,14 @@ class ModelRunner:
             n_active_buf = torch.empty(1, dtype=torch.int32, device=self.device)
         self._upload_slots(seqs, slots_buf, n_active_buf)
         self.state.build_decode(slots_buf, n_active_buf, bufs)
-        self._set_decode_context(bufs)
+        self._set_decode_context(bufs, slots_buf)
         return bufs["input_ids"], slots_buf
 
-    def _set_decode_context(self, bufs):
+    def _set_decode_context(self, bufs, slots_buf):
+        starts = (bufs["context_lens"] - 1).to(torch.int32) if self.has_state else None     # -1: padding row
         set_context(False, None, None, 0, 0, bufs["slot_mapping"], bufs["context_lens"], bufs["block_tables"],
-                    positions=bufs["positions"], decode_workspace=self.decode_workspace)
+                    positions=bufs["positions"], decode_workspace=self.decode_workspace,
+                    num_decode=slots_buf.shape[0], state_slots=slots_buf, state_starts=starts)
 
     # ---------------------------------------------------------------- sampling ---
     def next_tokens(self, hidden, temperatures=None):
@@ -267,6 +334,8 @@ class ModelRunner:
         else:
             logits = self.model.compute_logits(hidden)
             offset, world = 0, 1
+        if self.keep_logits:
+            self.logits = logits
         if self.greedy or temperatures is None:
             return greedy_tokens(logits, offset, None, world)
         tokens = sampled_tokens(logits, temperatures, self.sample_seed, self.sample_step, offset, None, world)
@@ -320,7 +389,54 @@ class ModelRunner:
         done.record()
         return host, done, n
 
+    def _mixed_body(self, seqs, temps):
+        counts = [s.num_scheduled_tokens if self.chunked_prefill else len(s) - s.num_cached_tokens for s in seqs]
+        input_ids, order = self.prepare_mixed(seqs, counts)
+        slots = get_context().state_slots.long()
+        moved = order != list(range(len(seqs)))
+        if moved:
+            perm = torch.tensor(order, dtype=torch.int64).pin_memory().to(self.device, non_blocking=True)
+            temps = temps[perm] if temps is not None else None
+        tokens = self.next_tokens(self.run_model(input_ids, True), temps)
+        self.state.last_token.index_copy_(0, slots, tokens)
+        if moved:
+            tokens = torch.empty_like(tokens).index_copy_(0, perm, tokens)
+        return torch.cat([tokens, self.error_word.to(torch.int64)])
+
+    @torch.inference_mode()
+    def step_logits(self, batch):
+        """One step on given tokens: batch = [(sequence, tokens of this step, wanted places among them)].  Tokens that
+        continue sequences one by one take the decode step (the captured graph, when there is one), everything else
+        the mixed step.  Returns the logits at the wanted places, fp32 on the CPU."""
+        seqs, counts, want = [b[0] for b in batch], [b[1] for b in batch], [b[2] for b in batch]
+        if all(n == 1 for n in counts) and all(s.on_device for s in seqs):
+            slots = torch.tensor([s.slot for s in seqs], dtype=torch.int64).to(self.device)
+            self.state.last_token.index_copy_(0, slots, torch.tensor([s.last_token for s in seqs]).to(self.device))
+            temps = None if self.greedy else torch.zeros(len(seqs), device=self.device)
+            if self.enforce_eager or not self.graphs:
+                input_ids, _ = self.prepare_decode(seqs)
+                logits = self.model.compute_logits(self.run_model(input_ids, False))
+            else:
+                self._replay(seqs, temps)
+                logits = self.graph_vars["logits"][next(b for b in sorted(self.graphs) if b >= len(seqs))]
+            logits = logits[[i for i, w in enumerate(want) for _ in w]]
+        elif self.mixed_steps:
+            input_ids, _ = self.prepare_mixed(seqs, counts, want)
+            hidden = self.run_model(input_ids, True)
+            logits = self.model.compute_logits(hidden) if any(want) else None
+        else:
+            raise ValueError("this model takes given tokens in mixed steps only: set chunked_prefill")
+        reset_context()
+        out = logits.float().cpu() if logits is not None else torch.empty(0, self.model_cfg.vocab_size)
+        code = int(self.error_word.item())
+        if code:
+            self.error_word.zero_()
+            raise RuntimeError(f"a bounded wait inside a kernel ran out of time (error word {code:#x})")
+        return out
+
     def _prefill_body(self, seqs, temps):
+        if self.mixed_steps:
+            return self._mixed_body(seqs, temps)
         input_ids = self.prepare_prefill(seqs)
         tokens = self.next_tokens(self.run_model(input_ids, True), temps)
         slots = torch.tensor([s.slot for s in seqs], dtype=torch.int64).pin_memory().to(self.device,
@@ -374,7 +490,7 @@ class ModelRunner:
         """The whole decode step on static buffers; captured once per padded batch size."""
         bufs = {k: t[:bp] for k, t in v["bufs"].items()}
         self.state.build_decode(v["slots"][:bp], v["n_active"], bufs)
-        self._set_decode_context(bufs)
+        self._set_decode_context(bufs, v["slots"][:bp])
         tokens = self.next_tokens(self.model(bufs["input_ids"]), None if self.greedy else v["temps"][:bp])
         v["tokens"][:bp].copy_(tokens)
         v["tokens"][self.max_num_seqs:].copy_(self.error_word)
@@ -390,9 +506,11 @@ class ModelRunner:
                  tokens=torch.zeros(max_bs + 1, dtype=torch.int64, device=self.device))
         c = self.model_cfg
         from .. import _cabi
-        need = _cabi.lib().mv_paged_decode_workspace_bytes(max_bs, c.num_heads // self.world_size,
-                                                           c.num_kv_heads // self.world_size, c.head_dim,
-                                                           self.max_blocks_per_seq, self.block_size)
+        need = 0
+        if self.kv_layers:
+            need = _cabi.lib().mv_paged_decode_workspace_bytes(max_bs, c.num_heads // self.world_size,
+                                                               c.num_kv_heads // self.world_size, c.head_dim,
+                                                               self.max_blocks_per_seq, self.block_size)
         self.decode_workspace = torch.zeros(max(need, 1), dtype=torch.uint8, device=self.device)
         sizes = [b for b in [1, 2, 4, 8] if b <= max_bs] + list(range(16, max_bs + 1, 16))
         if max_bs not in sizes:
@@ -407,6 +525,8 @@ class ModelRunner:
                 self._decode_body(v, bp)
             pool = pool or g.pool()
             self.graphs[bp] = g
+            if self.keep_logits:
+                v.setdefault("logits", {})[bp] = self.logits
         torch.cuda.synchronize()
         reset_context()
 

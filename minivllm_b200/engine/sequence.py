@@ -33,6 +33,8 @@ class Sequence:
         self.block_size = block_size
         self.block_table = []
         self.num_cached_tokens = 0
+        self.num_scheduled_tokens = 0  # tokens of the step being run (mixed steps)
+        self.on_device = False       # the next input token is the device's own last sampled one
         self.slot = -1               # row of the device-resident state while running
         self.synced_blocks = 0       # how many block-table entries the device row already holds
         self.temperature, self.max_tokens, self.ignore_eos = sp.temperature, sp.max_tokens, sp.ignore_eos

@@ -331,7 +331,18 @@ class Attention(nn.Module):
         if ctx.is_prefill:
             if ctx.cu_seqlens_q is None:
                 raise ValueError("cu_seqlens_q must be provided for varlen attention")
-            if ctx.block_tables is not None and ctx.cu_seqlens_k is not None and has_cache:
+            nd = ctx.num_decode
+            if nd:
+                # mixed step: the first nd rows are decoded tokens, the rest portions of prompts
+                o = torch.empty_like(q, memory_format=torch.contiguous_format)
+                o[:nd] = paged_attention_decode(q[:nd], k_cache, v_cache, ctx.block_tables[:nd], ctx.context_lens[:nd],
+                                                scale, self.num_heads, self.num_kv_heads, self.head_dim,
+                                                k_cache.shape[1])
+                if q.shape[0] > nd:
+                    o[nd:] = flash_attention_prefill_paged(q[nd:], k_cache, v_cache, ctx.portion_cu_q, ctx.portion_cu_k,
+                                                           ctx.block_tables[nd:], scale, self.num_heads,
+                                                           self.num_kv_heads, self.head_dim)
+            elif ctx.block_tables is not None and ctx.cu_seqlens_k is not None and has_cache:
                 # some sequence has a cached prefix: attend through the paged cache (this step's K/V are in it)
                 o = flash_attention_prefill_paged(q, k_cache, v_cache, ctx.cu_seqlens_q, ctx.cu_seqlens_k,
                                                   ctx.block_tables, scale, self.num_heads, self.num_kv_heads,

@@ -19,7 +19,7 @@ from .. import _cabi
 
 
 def argmax_rows(logits, index_offset=0, want_keys=True, want_tokens=False):
-    """logits (rows, cols) fp16/bf16, last dim contiguous.  Returns (keys, tokens): int64 (rows,) each or None.
+    """logits (rows, cols) fp16/bf16/fp32, last dim contiguous.  Returns (keys, tokens): int64 (rows,) each or None.
 
     A key orders first by logit (NaN highest, as torch.argmax), then by lower index `index_offset + column`.
     `tokens` are the indices of this shard's maxima."""
@@ -33,7 +33,7 @@ def argmax_rows(logits, index_offset=0, want_keys=True, want_tokens=False):
         _cabi.check(_cabi.lib().mv_argmax_rows(
             logits.data_ptr(), logits.stride(0), rows, cols, int(index_offset),
             keys.data_ptr() if want_keys else None, tokens.data_ptr() if want_tokens else None,
-            _cabi.dtype_code(logits.dtype), _cabi.stream_ptr()))
+            _cabi.logits_dtype_code(logits.dtype), _cabi.stream_ptr()))
     return keys, tokens
 
 
@@ -62,7 +62,7 @@ def greedy_tokens(shard_logits, index_offset=0, group=None, world_size=1):
 def sample_rows(logits, temperatures, seed, step, index_offset=0, want_keys=True, want_tokens=False):
     """Exponential-race scores of this vocabulary shard reduced to one key per row.
 
-    logits (rows, cols) fp16/bf16; temperatures (rows,) fp32 on the device (0 = greedy row); seed: Python int
+    logits (rows, cols) fp16/bf16/fp32; temperatures (rows,) fp32 on the device (0 = greedy row); seed: Python int
     (64 bits); step: int64 device tensor with one element, read by the kernel (advance it between calls, e.g.
     `step.add_(1)` inside a captured graph).  Returns (keys, tokens) like `argmax_rows`."""
     _cabi.require_cuda(logits, temperatures, step)
@@ -79,7 +79,7 @@ def sample_rows(logits, temperatures, seed, step, index_offset=0, want_keys=True
         _cabi.check(_cabi.lib().mv_sample_rows(
             logits.data_ptr(), logits.stride(0), rows, cols, int(index_offset), temperatures.data_ptr(),
             int(seed) & 0xffffffffffffffff, step.data_ptr(), keys.data_ptr() if want_keys else None,
-            tokens.data_ptr() if want_tokens else None, _cabi.dtype_code(logits.dtype), _cabi.stream_ptr()))
+            tokens.data_ptr() if want_tokens else None, _cabi.logits_dtype_code(logits.dtype), _cabi.stream_ptr()))
     return keys, tokens
 
 

@@ -32,6 +32,12 @@ class Context:
     positions: Optional[torch.Tensor] = None        # (num_tokens,) int64 RoPE positions
     last_token_index: Optional[torch.Tensor] = None  # (num_seqs,) int64 rows fed to the LM head
     decode_workspace: Optional[torch.Tensor] = None  # split-K scratch shared by all layers
+    # --- mixed steps (portions of prompts beside decoded tokens) and layers with per-sequence state ---
+    num_decode: int = 0                              # the first num_decode sequences have one token each
+    portion_cu_q: Optional[torch.Tensor] = None      # cu_seqlens_q / _k of the sequences behind them, from 0
+    portion_cu_k: Optional[torch.Tensor] = None
+    state_slots: Optional[torch.Tensor] = None       # (num_seqs,) int32 slot of each sequence
+    state_starts: Optional[torch.Tensor] = None      # (num_seqs,) int32 tokens behind this step (-1: padding row)
 
 
 class _Holder:
