@@ -190,7 +190,7 @@ def random_weights(config, seed=0, scale=1.0):
         if layer.get("mlp"):
             p, e = l + "mlp.", layer["mlp"]
             n = e["router"]["experts"]
-            w[p + "router"], w[p + "router.b"] = mat(n, W, 2.0), around(n, 0.0, 0.5)
+            w[p + "router"], w[p + "router.b"] = mat(n, W), around(n, 0.0, 1.5)
             names = [(f"e{j}.", e["expert"]["ff"]) for j in range(n)]
             if e.get("shared"):
                 names.append(("shared.", e["shared"]["ff"]))
