@@ -503,6 +503,61 @@ int mv_gather_rows(void* out, const void* x, int64_t x_stride, const int32_t* ro
 int mv_grouped_rows(void* out, const void* x, const void* w, const int32_t* offsets, int experts,
     int64_t rows, int in_dim, int out_dim, int gated, int dtype, void* stream);
 
+/*
+ * mv_grouped_rows on the tensor cores (tcgen05), bf16, in_dim a multiple of 8.  A bounded wait that runs out is
+ * reported in *error_word, as by mv_prefill_varlen.
+ */
+int mv_grouped_gemm(void* out, const void* x, const void* w, const int32_t* offsets, int experts,
+    int64_t rows, int in_dim, int out_dim, int gated, int* error_word, void* stream);
+
+/*
+ * mv_latent_attention_rows for one query row per sequence on tensor cores, bf16: rank a multiple of 64 up to 512,
+ * rot_dim a multiple of 32, at most 1,024 rows (workspace_bytes returns -1 otherwise).  Sequence b has
+ * positions[b] + 1 keys; rows with active[b] < 0 (active may be null) have none and give zeros.
+ */
+int64_t mv_latent_decode_workspace_bytes(int batch, int heads, int rank, int rot_dim);
+int mv_latent_decode(void* out, int64_t out_stride, int64_t out_head_stride, const void* q_lat,
+    int64_t q_lat_stride, int64_t q_lat_head_stride, const void* q_rot, int64_t q_rot_stride,
+    int64_t q_rot_head_stride, const void* cache, const int32_t* block_tables, int64_t bt_stride,
+    int max_blocks, int block_size, int64_t num_blocks, const int64_t* positions, const int32_t*
+    active, const void* sink, int batch, int heads, int rank, int rot_dim, float scale, void*
+    workspace, int64_t workspace_bytes, void* stream);
+
+/*
+ * Prefill of latent attention with keys and values expanded per head, bf16, tcgen05.
+ *   mv_latent_gather   out[cu_k[s] + j] = cache row of position j of sequence s (bf16 or fp32, rows of whole 16 bytes)
+ *   mv_latent_prefill  q (tokens, heads * (dim + rot_dim)), k (keys, heads * dim), k_rot (keys, rot_dim) shared by the
+ *                      heads, v (keys, heads * vdim); row strides in elements; sequence s has queries cu_q[s] .. at the
+ *                      end of its keys cu_k[s] ..; sizes multiples of 8, 64-column boxes: at most three for dim and
+ *                      rot_dim together, two for vdim; sink may be null.  Bounded waits report in *error_word.
+ */
+int mv_latent_gather(void* out, const void* cache, const int32_t* cu_k, int num_seqs, int64_t keys,
+    const int32_t* block_tables, int64_t bt_stride, int max_blocks, int block_size, int64_t
+    num_blocks, int row, int dtype, void* stream);
+int mv_latent_prefill(void* out, int64_t out_stride, const void* q, int64_t q_stride, const void* k,
+    int64_t k_stride, const void* k_rot, int64_t k_rot_stride, const void* v, int64_t v_stride,
+    const int32_t* cu_q, const int32_t* cu_k, int num_seqs, int64_t tokens, int64_t keys, int heads,
+    int dim, int rot_dim, int vdim, float scale, const void* sink, int* error_word, void* stream);
+
+/*
+ * mv_ssm_scan in chunks of 64 tokens on tensor cores, bf16; every sequence of cu must be a portion.  `takes` tells
+ * whether the sizes are supported (state 32, 64 or 128, vdim a multiple of 8).
+ */
+int mv_ssm_chunk_takes(int vdim, int state_dim);
+int mv_ssm_chunk_scan(void* y, int64_t y_stride, const void* xbc, int64_t xbc_stride, const void*
+    dt, int64_t dt_stride, const void* dt_bias, const void* A_log, const void* D, const int32_t* cu,
+    int num_seqs, const int32_t* slots, const int32_t* start, float* state, int num_slots, int
+    heads, int vdim, int state_dim, int groups, void* stream);
+
+/*
+ * One token per sequence, convolution included: u holds the rows before it, conv_state is read only (advance it with
+ * mv_conv_state_update afterwards); state as in mv_ssm_scan.  vdim and state_dim multiples of 4.
+ */
+int mv_ssm_step(void* y, const void* u, int64_t u_stride, const void* w, const void* bias, int taps,
+    const void* conv_state, const void* dt, int64_t dt_stride, const void* dt_bias, const void*
+    A_log, const void* D, int num_seqs, const int32_t* slots, const int32_t* start, float* state,
+    int num_slots, int heads, int vdim, int state_dim, int groups, int dtype, void* stream);
+
 #ifdef __cplusplus
 }
 #endif

@@ -94,6 +94,21 @@ SIGNATURES = {
     "mv_gather_rows": (_c_int, [_c_ptr, _c_ptr, _c_i64, _c_ptr, _c_i64, _c_int, _c_int, _c_ptr]),
     "mv_grouped_rows": (_c_int, [_c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_int, _c_i64, _c_int, _c_int, _c_int, _c_int,
         _c_ptr]),
+    "mv_grouped_gemm": (_c_int, [_c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_int, _c_i64, _c_int, _c_int, _c_int, _c_ptr,
+        _c_ptr]),
+    "mv_latent_decode_workspace_bytes": (_c_i64, [_c_int, _c_int, _c_int, _c_int]),
+    "mv_latent_decode": (_c_int, [_c_ptr, _c_i64, _c_i64, _c_ptr, _c_i64, _c_i64, _c_ptr, _c_i64, _c_i64, _c_ptr,
+        _c_ptr, _c_i64, _c_int, _c_int, _c_i64, _c_ptr, _c_ptr, _c_ptr, _c_int, _c_int, _c_int, _c_int, _c_f32,
+        _c_ptr, _c_i64, _c_ptr]),
+    "mv_latent_gather": (_c_int, [_c_ptr, _c_ptr, _c_ptr, _c_int, _c_i64, _c_ptr, _c_i64, _c_int, _c_int, _c_i64,
+        _c_int, _c_int, _c_ptr]),
+    "mv_latent_prefill": (_c_int, [_c_ptr, _c_i64, _c_ptr, _c_i64, _c_ptr, _c_i64, _c_ptr, _c_i64, _c_ptr, _c_i64,
+        _c_ptr, _c_ptr, _c_int, _c_i64, _c_i64, _c_int, _c_int, _c_int, _c_int, _c_f32, _c_ptr, _c_ptr, _c_ptr]),
+    "mv_ssm_chunk_takes": (_c_int, [_c_int, _c_int]),
+    "mv_ssm_chunk_scan": (_c_int, [_c_ptr, _c_i64, _c_ptr, _c_i64, _c_ptr, _c_i64, _c_ptr, _c_ptr, _c_ptr, _c_ptr,
+        _c_int, _c_ptr, _c_ptr, _c_ptr, _c_int, _c_int, _c_int, _c_int, _c_int, _c_ptr]),
+    "mv_ssm_step": (_c_int, [_c_ptr, _c_ptr, _c_i64, _c_ptr, _c_ptr, _c_int, _c_ptr, _c_ptr, _c_i64, _c_ptr, _c_ptr,
+        _c_ptr, _c_int, _c_ptr, _c_ptr, _c_ptr, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_ptr]),
 }
 
 _lib = None

@@ -17,7 +17,8 @@ COMMON = ["api.cu", "metadata.cu", "sampling.cu"]
 GROUPS = {
     "qwen3": ["store_kvcache.cu", "paged_decode.cu", "paged_decode_int8.cu", "prefill_varlen.cu",
               "paged_decode_static.cu", "pre_attention.cu", "comm.cu"],
-    "sipazen": ["norms.cu", "latent_attention.cu", "mamba2.cu", "moe.cu"],
+    "sipazen": ["norms.cu", "latent_attention.cu", "latent_decode.cu", "latent_prefill.cu", "mamba2.cu",
+                "mamba2_chunk.cu", "moe.cu", "grouped_gemm.cu"],
 }
 SOURCES = COMMON + [s for g in GROUPS.values() for s in g]
 NVCC_FLAGS = [

@@ -1,0 +1,403 @@
+// Prefill attention of a latent-attention layer on the Blackwell tensor cores, with keys and values expanded per head
+// (k = [W_uk c | shared rotated part], v = W_uv c): causal, packed batch, an optional sink per head.
+//
+// Every head has keys of its own, so the two 128-row problems of a CTA are two consecutive query tiles of ONE head:
+// they share each K/V tile.  The K operand is assembled by TMA from two tensors, 64-column boxes of the expanded
+// unrotated part and one box of the rotated part that all heads share; a box that is wider than its tensor reads
+// zeros, so any sizes that are multiples of eight up to 192 query/key and 128 value dimensions run here.
+//   warps 0-3 / 4-7  softmax of the lower / upper query tile (thread = row = TMEM lane)
+//   warp 8           TMA producer, warp 9 MMA issuer (S = Q K^T from shared memory, O += P V with P in TMEM)
+// Sequence s has queries cu_q[s] .. and keys cu_k[s] .. of the packed tensors; its first query sits at position
+// (keys - queries).  Same roles, tensor-memory layout and lazy rescaling as prefill_varlen.cu.
+//
+// Tensor-bound: FLOPs = 2 * heads * (dim + rot_dim + vdim) * (number of visible (query, key) pairs).
+#include <algorithm>
+#include "mma.cuh"
+#include "tcgen05.cuh"
+#include "tmap.cuh"
+#include "vec.cuh"
+
+namespace mv {
+
+constexpr int kLfThreads = 384, kLfTile = 128;
+constexpr int kLfBox = kLfTile * 128;                 // one 64-column box of a 128-row tile
+constexpr float kLfRescale = 8.f;                     // log2 units
+
+template <int NQ, int NV> struct LfShape {
+  static constexpr int kVStages = NQ == 3 ? (NV == 2 ? 1 : 2) : 2;
+  static constexpr int kQBytes = NQ * kLfBox, kVBytes = NV * kLfBox;
+  static constexpr int kSmem = 4 * kQBytes + kVStages * kVBytes + 1024;
+};
+
+struct LfParams {
+  __nv_bfloat16* out; int64_t out_stride; int vdim;
+  const int32_t* cu_q; const int32_t* cu_k;
+  int num_seqs, nd, dim, rot_dim;                     // nd: boxes of the unrotated part
+  float scale_log2;
+  const __nv_bfloat16* sink;
+  int* error_word;
+};
+
+enum { LB_Q = 0, LB_KFULL = 1, LB_KEMPTY = 3, LB_VFULL = 5, LB_VEMPTY = 7, LB_SFULL = 9, LB_PREADY = 11, LB_ODONE = 13,
+       LB_DRAIN = 15, LB_COUNT = 16 };
+
+template <int NQ, int NV>
+__global__ void __launch_bounds__(kLfThreads, 1)
+latent_prefill_kernel(const __grid_constant__ CUtensorMap tm_qn, const __grid_constant__ CUtensorMap tm_qr,
+                      const __grid_constant__ CUtensorMap tm_kn, const __grid_constant__ CUtensorMap tm_kr,
+                      const __grid_constant__ CUtensorMap tm_v, const LfParams p) {
+  using Sh = LfShape<NQ, NV>;
+  constexpr int VS = Sh::kVStages;
+  extern __shared__ unsigned char smem_raw[];
+  __shared__ __align__(8) uint64_t bars[LB_COUNT];
+  __shared__ uint32_t s_tmem;
+  __shared__ int s_tile[2], s_scan[kLfThreads / 32], s_abort, s_sticky;
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const uint32_t q_smem = (smem_u32(smem_raw) + 1023u) & ~1023u;      // [tile 2][box][128][128B]
+  const uint32_t k_smem = q_smem + 2 * Sh::kQBytes;                   // [stage 2][box]
+  const uint32_t v_smem = k_smem + 2 * Sh::kQBytes;                   // [stage VS][box]
+  const uint32_t bar0 = smem_u32(bars);
+  auto bar = [&](int i) { return bar0 + 8u * i; };
+  volatile int* abort_flag = &s_abort;
+
+  // which (sequence, 256-row tile) is blockIdx.x: tiles of a sequence in descending order
+  if (tid == 0) {
+    s_tile[0] = -1;
+    s_tile[1] = 0;
+    s_abort = 0;
+    s_sticky = *reinterpret_cast<volatile int*>(p.error_word);
+  }
+  __syncthreads();
+  int carry = 0;
+  for (int base = 0; base < p.num_seqs; base += kLfThreads) {
+    const int s = base + tid;
+    int n = 0;
+    if (s < p.num_seqs) n = (max(p.cu_q[s + 1] - p.cu_q[s], 0) + 2 * kLfTile - 1) / (2 * kLfTile);
+    int incl = n;
+#pragma unroll
+    for (int o = 1; o < 32; o <<= 1) {
+      const int v = __shfl_up_sync(0xffffffffu, incl, o);
+      if (lane >= o) incl += v;
+    }
+    if (lane == 31) s_scan[warp] = incl;
+    __syncthreads();
+    int before = 0, tot = 0;
+    for (int w = 0; w < kLfThreads / 32; ++w) {
+      if (w < warp) before += s_scan[w];
+      tot += s_scan[w];
+    }
+    const int start = carry + before + incl - n, x = static_cast<int>(blockIdx.x);
+    if (n > 0 && x >= start && x < start + n) { s_tile[0] = s; s_tile[1] = n - 1 - (x - start); }
+    carry += tot;
+    __syncthreads();
+  }
+  const int seq = s_tile[0];
+  if (seq < 0 || s_sticky != 0) return;      // uniform: the grid is an upper bound; an earlier wait ran out
+  const int head = blockIdx.y;
+  const int q_start = p.cu_q[seq], q_len = p.cu_q[seq + 1] - q_start;
+  const int k_start = p.cu_k[seq], k_len = p.cu_k[seq + 1] - k_start;
+  const int q0 = s_tile[1] * 2 * kLfTile;
+  const int first_pos = k_len - q_len + q0;
+  // KV tiles up to the position of each query tile's last row
+  const int n_a = (k_len - q_len + min(q0 + kLfTile, q_len) + kLfTile - 1) / kLfTile;
+  const int n_b = q0 + kLfTile < q_len ? (k_len - q_len + min(q0 + 2 * kLfTile, q_len) + kLfTile - 1) / kLfTile : 0;
+  const int n_kv = max(n_a, n_b);
+
+  if (tid == 0) {
+    tc::mbar_init(bar(LB_Q), 1);
+    for (int s = 0; s < 2; ++s) {
+      tc::mbar_init(bar(LB_KFULL + s), 1);
+      tc::mbar_init(bar(LB_KEMPTY + s), 1);
+      tc::mbar_init(bar(LB_VFULL + s), 1);
+      tc::mbar_init(bar(LB_VEMPTY + s), 1);
+      tc::mbar_init(bar(LB_SFULL + s), 1);
+      tc::mbar_init(bar(LB_PREADY + s), 128);
+      tc::mbar_init(bar(LB_ODONE + s), 1);
+    }
+    tc::mbar_init(bar(LB_DRAIN), 1);
+    tc::mbar_fence_init();
+  }
+  if (warp == 8) {
+    tc::tmem_alloc(smem_u32(&s_tmem), 512);
+    tc::tmem_relinquish();
+  }
+  tc::fence_before_sync();
+  __syncthreads();
+  tc::fence_after_sync();
+  const uint32_t tmem = s_tmem;
+
+  if (warp >= 8) {
+    tc::setmaxnreg_dec_40();
+    if (warp == 8) {
+      if (lane == 0) {
+        const int tiles = n_b > 0 ? 2 : 1;
+        tc::mbar_expect_tx(bar(LB_Q), tiles * Sh::kQBytes);
+        for (int t = 0; t < tiles; ++t)
+          for (int b = 0; b < NQ; ++b) {
+            const uint32_t dst = q_smem + t * Sh::kQBytes + b * kLfBox;
+            const int row = q_start + q0 + t * kLfTile;
+            if (b < p.nd) tc::tma_load_3d(dst, &tm_qn, 64 * b, head, row, bar(LB_Q));
+            else tc::tma_load_3d(dst, &tm_qr, 64 * (b - p.nd), head, row, bar(LB_Q));
+          }
+        for (int j = 0; j < n_kv; ++j) {
+          const int s = j & 1, row = k_start + j * kLfTile;
+          tc::mbar_wait(bar(LB_KEMPTY + s), ((j / 2) & 1) ^ 1, abort_flag, p.error_word, 1);
+          tc::mbar_expect_tx(bar(LB_KFULL + s), Sh::kQBytes);
+          for (int b = 0; b < NQ; ++b) {
+            const uint32_t dst = k_smem + s * Sh::kQBytes + b * kLfBox;
+            if (b < p.nd) tc::tma_load_3d(dst, &tm_kn, 64 * b, head, row, bar(LB_KFULL + s));
+            else tc::tma_load_3d(dst, &tm_kr, 64 * (b - p.nd), 0, row, bar(LB_KFULL + s));
+          }
+          const int vs = j % VS;
+          tc::mbar_wait(bar(LB_VEMPTY + vs), ((j / VS) & 1) ^ 1, abort_flag, p.error_word, 2);
+          tc::mbar_expect_tx(bar(LB_VFULL + vs), Sh::kVBytes);
+          for (int b = 0; b < NV; ++b)
+            tc::tma_load_3d(v_smem + vs * Sh::kVBytes + b * kLfBox, &tm_v, 64 * b, head, row, bar(LB_VFULL + vs));
+        }
+        if (*abort_flag) {       // copies in flight must land before the shared memory goes away
+          tc::mbar_wait_timed(bar(LB_Q), 0);
+          for (int j = max(n_kv - 2, 0); j < n_kv; ++j) {
+            tc::mbar_wait_timed(bar(LB_KFULL + (j & 1)), (j / 2) & 1);
+            if (j >= n_kv - VS) tc::mbar_wait_timed(bar(LB_VFULL + j % VS), (j / VS) & 1);
+          }
+        }
+      }
+    } else if (warp == 9) {
+      const uint32_t idesc_qk = tc::instr_desc_f16(1, 1, false, 128, 128);
+      const uint32_t idesc_pv = tc::instr_desc_f16(1, 1, true, 128, 64 * NV);
+      const uint32_t q_lo = tc::desc_lo(q_smem, 16), k_lo = tc::desc_lo(k_smem, 16), v_lo = tc::desc_lo(v_smem, kLfBox);
+      auto issue_qk = [&](int t, int s) {
+#pragma unroll
+        for (int b = 0; b < NQ; ++b)
+          tc::mma_ss_k64(tmem + t * 128, tc::desc64(q_lo + ((t * Sh::kQBytes + b * kLfBox) >> 4), tc::kDescHiSw128Sbo1024),
+                         tc::desc64(k_lo + ((s * Sh::kQBytes + b * kLfBox) >> 4), tc::kDescHiSw128Sbo1024), idesc_qk, b > 0);
+        tc::commit_elected(bar(LB_SFULL + t), 0, false);
+      };
+      tc::mbar_wait(bar(LB_Q), 0, abort_flag, p.error_word, 3);
+      tc::mbar_wait(bar(LB_KFULL + 0), 0, abort_flag, p.error_word, 4);
+      tc::fence_after_sync();
+      __syncwarp();
+      issue_qk(0, 0);
+      if (n_b > 0) issue_qk(1, 0);
+      tc::commit_elected(bar(LB_KEMPTY + 0), 0, false);
+      for (int j = 0; j < n_kv; ++j) {
+        const int vs = j % VS, s1 = (j + 1) & 1;
+        const bool more = j + 1 < n_kv;
+        tc::mbar_wait(bar(LB_VFULL + vs), (j / VS) & 1, abort_flag, p.error_word, 5);
+        if (more) tc::mbar_wait(bar(LB_KFULL + s1), ((j + 1) / 2) & 1, abort_flag, p.error_word, 6);
+        for (int t = 0; t < 2; ++t) {
+          const int n_t = t == 0 ? n_a : n_b;
+          if (j >= n_t) continue;
+          tc::mbar_wait(bar(LB_PREADY + t), j & 1, abort_flag, p.error_word, 7);
+          tc::fence_after_sync();
+          __syncwarp();
+          tc::mma_ts_k128_commit(tmem + 256 + t * 128, tmem + t * 128,
+                                 tc::desc64(v_lo + ((vs * Sh::kVBytes) >> 4), tc::kDescHiSw128Sbo1024), idesc_pv, j > 0,
+                                 bar(LB_ODONE + t));
+          if (j + 1 < n_t) issue_qk(t, s1);
+        }
+        tc::commit_elected(bar(LB_VEMPTY + vs), bar(LB_KEMPTY + s1), more);
+      }
+      if (*abort_flag) {
+        __syncwarp();
+        tc::commit_elected(bar(LB_DRAIN), 0, false);
+        tc::mbar_wait_timed(bar(LB_DRAIN), 0);
+      }
+    }
+  } else {
+    tc::setmaxnreg_inc_232();
+    const int t = warp >> 2, n_t = t == 0 ? n_a : n_b;
+    if (n_t > 0) {
+      const int row = (warp & 3) * 32 + lane;
+      const uint32_t lane_addr = static_cast<uint32_t>((warp & 3) * 32) << 16;
+      const uint32_t s_addr = tmem + lane_addr + t * 128, o_addr = tmem + lane_addr + 256 + t * 128;
+      float m_used = -INFINITY, l = 0.f;
+      for (int j = 0; j < n_t; ++j) {
+        tc::mbar_wait(bar(LB_SFULL + t), j & 1, abort_flag, p.error_word, 8);
+        tc::fence_after_sync();
+        // key 128j + col is visible to this row when col <= vis
+        const int vis = first_pos + t * kLfTile + row - j * kLfTile;
+        uint32_t sv[4][32];
+#pragma unroll
+        for (int c = 0; c < 4; ++c) tc::tmem_ld32(s_addr + c * 32, sv[c]);
+        tc::wait_ld();
+        if (first_pos + t * kLfTile - j * kLfTile < kLfTile - 1) {     // the tile reaches past the first row's position
+#pragma unroll
+          for (int c = 0; c < 4; ++c)
+#pragma unroll
+            for (int i = 0; i < 32; ++i)
+              if (c * 32 + i > vis) sv[c][i] = 0xff800000u;
+        }
+        float mxs[8];
+#pragma unroll
+        for (int i = 0; i < 8; ++i) mxs[i] = -INFINITY;
+#pragma unroll
+        for (int c = 0; c < 4; ++c)
+#pragma unroll
+          for (int i = 0; i < 16; ++i)
+            mxs[i & 7] = tc::max3(mxs[i & 7], __uint_as_float(sv[c][2 * i]), __uint_as_float(sv[c][2 * i + 1]));
+        float mx = fmaxf(tc::max3(mxs[0], mxs[1], mxs[2]), tc::max3(mxs[3], mxs[4], mxs[5]));
+        mx = tc::max3(mx, mxs[6], mxs[7]) * p.scale_log2;
+        const bool grow = mx > m_used + kLfRescale;
+        if (j > 0 && __any_sync(0xffffffffu, grow)) {    // rare: move the reference maximum, rescale O
+          const float alpha = grow ? fast_exp2(m_used - mx) : 1.f;
+          tc::mbar_wait(bar(LB_ODONE + t), (j - 1) & 1, abort_flag, p.error_word, 9);
+          tc::fence_after_sync();
+#pragma unroll 1
+          for (int c = 0; c < 2 * NV; ++c) {
+            uint32_t ov[32];
+            tc::tmem_ld32(o_addr + c * 32, ov);
+            tc::wait_ld();
+#pragma unroll
+            for (int i = 0; i < 32; ++i) ov[i] = __float_as_uint(__uint_as_float(ov[i]) * alpha);
+            tc::tmem_st32(o_addr + c * 32, ov);
+          }
+          tc::wait_st();
+          l *= alpha;
+        }
+        if (grow) m_used = mx;
+        const float2 sc2 = make_float2(p.scale_log2, p.scale_log2), nm2 = make_float2(-m_used, -m_used);
+        float2 sums[4] = {make_float2(0.f, 0.f), make_float2(0.f, 0.f), make_float2(0.f, 0.f), make_float2(0.f, 0.f)};
+#pragma unroll
+        for (int c2 = 0; c2 < 2; ++c2) {
+          uint32_t pk[32];
+#pragma unroll
+          for (int i = 0; i < 32; ++i) {
+            const int c = 2 * c2 + (i >> 4), k = (i & 15) * 2;
+            const float2 x = tc::fma2(make_float2(__uint_as_float(sv[c][k]), __uint_as_float(sv[c][k + 1])), sc2, nm2);
+            float2 e;
+            if ((i & 3) == 3) {
+              e = tc::ex2_poly2(x);
+            } else {
+              e.x = tc::ex2_mufu(x.x);
+              e.y = tc::ex2_mufu(x.y);
+            }
+            sums[i & 3] = tc::add2(sums[i & 3], e);
+            pk[i] = pack2<__nv_bfloat16>(e.x, e.y);
+          }
+          tc::tmem_st32(s_addr + c2 * 32, pk);
+        }
+        const float2 s01 = tc::add2(sums[0], sums[1]), s23 = tc::add2(sums[2], sums[3]);
+        l += (s01.x + s01.y) + (s23.x + s23.y);
+        tc::wait_st();
+        tc::fence_before_sync();
+        tc::mbar_arrive(bar(LB_PREADY + t));
+      }
+      tc::mbar_wait(bar(LB_ODONE + t), (n_t - 1) & 1, abort_flag, p.error_word, 10);
+      tc::fence_after_sync();
+      float f = 1.f;
+      if (p.sink) {
+        const float sk = __bfloat162float(p.sink[head]) * 1.4426950408889634f, mm = fmaxf(m_used, sk);
+        f = exp2f(m_used - mm);
+        l = l * f + exp2f(sk - mm);
+      }
+      const float inv = l > 0.f ? f / l : 0.f;
+      const int qrow = q0 + t * kLfTile + row;
+      __nv_bfloat16* orow = p.out + static_cast<int64_t>(q_start + qrow) * p.out_stride + static_cast<int64_t>(head) * p.vdim;
+#pragma unroll
+      for (int c = 0; c < 2 * NV; ++c) {
+        uint32_t ov[32];
+        tc::tmem_ld32(o_addr + c * 32, ov);
+        tc::wait_ld();
+        if (qrow < q_len) {
+#pragma unroll
+          for (int i = 0; i < 4; ++i) {
+            if (c * 32 + i * 8 >= p.vdim) continue;
+            uint4 w;
+            w.x = pack2<__nv_bfloat16>(__uint_as_float(ov[8 * i + 0]) * inv, __uint_as_float(ov[8 * i + 1]) * inv);
+            w.y = pack2<__nv_bfloat16>(__uint_as_float(ov[8 * i + 2]) * inv, __uint_as_float(ov[8 * i + 3]) * inv);
+            w.z = pack2<__nv_bfloat16>(__uint_as_float(ov[8 * i + 4]) * inv, __uint_as_float(ov[8 * i + 5]) * inv);
+            w.w = pack2<__nv_bfloat16>(__uint_as_float(ov[8 * i + 6]) * inv, __uint_as_float(ov[8 * i + 7]) * inv);
+            st_global16(orow + c * 32 + i * 8, w);
+          }
+        }
+      }
+    }
+  }
+  __syncwarp();
+  tc::fence_before_sync();
+  __syncthreads();
+  if (warp == 8) {
+    tc::fence_after_sync();
+    tc::tmem_dealloc(tmem, 512);
+  }
+}
+
+// Rows of the paged latent cache of every sequence, packed: out[cu_k[s] + j] = cache row of position j of sequence s.
+// Rows without a block read as zero.
+__global__ void __launch_bounds__(256)
+latent_gather_kernel(uint4* __restrict__ out, const uint4* __restrict__ cache, const int32_t* __restrict__ cu_k,
+                     int num_seqs, int64_t keys, const int32_t* __restrict__ tables, int64_t bt_stride, int max_blocks,
+                     int block_size, int64_t num_blocks, int chunks) {
+  const int lane = threadIdx.x & 31;
+  for (int64_t r = static_cast<int64_t>(blockIdx.x) * 8 + (threadIdx.x >> 5); r < keys; r += static_cast<int64_t>(gridDim.x) * 8) {
+    const int s = seq_of_token(cu_k, num_seqs, static_cast<int>(r));
+    const int pos = static_cast<int>(r) - cu_k[s], blk = pos / block_size;
+    const int32_t phys = blk < max_blocks ? tables[static_cast<int64_t>(s) * bt_stride + blk] : -1;
+    const bool ok = phys >= 0 && phys < num_blocks;
+    const int64_t src = ok ? (static_cast<int64_t>(phys) * block_size + (pos - blk * block_size)) * chunks : 0;
+    for (int c = lane; c < chunks; c += 32) out[r * chunks + c] = ok ? cache[src + c] : make_uint4(0, 0, 0, 0);
+  }
+}
+
+template <int NQ, int NV>
+static int launch_latent_prefill(const CUtensorMap (&tm)[5], const LfParams& p, int64_t tokens, int heads, cudaStream_t st) {
+  const cudaError_t e = cudaFuncSetAttribute(latent_prefill_kernel<NQ, NV>, cudaFuncAttributeMaxDynamicSharedMemorySize, LfShape<NQ, NV>::kSmem);
+  if (e != cudaSuccess) return fail(MV_ERR_CUDA, "latent_prefill: %s", cudaGetErrorString(e));
+  const dim3 grid(static_cast<unsigned>(tokens / (2 * kLfTile) + std::min<int64_t>(p.num_seqs, tokens)), heads);
+  latent_prefill_kernel<NQ, NV><<<grid, kLfThreads, LfShape<NQ, NV>::kSmem, st>>>(tm[0], tm[1], tm[2], tm[3], tm[4], p);
+  return check_launch("latent_prefill");
+}
+
+}  // namespace mv
+
+extern "C" int mv_latent_gather(void* out, const void* cache, const int32_t* cu_k, int num_seqs, int64_t keys,
+                                const int32_t* block_tables, int64_t bt_stride, int max_blocks, int block_size,
+                                int64_t num_blocks, int row, int dtype, void* stream) {
+  using namespace mv;
+  if (dtype != MV_BF16 && dtype != MV_F32) return fail(MV_ERR_DTYPE, "latent_gather: dtype %d", dtype);
+  const int bytes = row * (dtype == MV_F32 ? 4 : 2);
+  if (keys < 0 || num_seqs < 0 || block_size <= 0 || row <= 0 || bytes % 16) return fail(MV_ERR_SHAPE, "latent_gather: row %d", row);
+  if (keys == 0 || num_seqs == 0) return MV_OK;
+  if (!out || !cache || !cu_k || !block_tables) return fail(MV_ERR_NULL, "latent_gather: null pointer");
+  if (!aligned16(out) || !aligned16(cache)) return fail(MV_ERR_ALIGN, "latent_gather: alignment");
+  const unsigned grid = static_cast<unsigned>(std::min<int64_t>((keys + 7) / 8, kNumSMs * 16));
+  latent_gather_kernel<<<grid, 256, 0, static_cast<cudaStream_t>(stream)>>>(
+      static_cast<uint4*>(out), static_cast<const uint4*>(cache), cu_k, num_seqs, keys, block_tables, bt_stride, max_blocks, block_size,
+      num_blocks, bytes / 16);
+  return check_launch("latent_gather");
+}
+
+extern "C" int mv_latent_prefill(void* out, int64_t out_stride, const void* q, int64_t q_stride, const void* k,
+                                 int64_t k_stride, const void* k_rot, int64_t k_rot_stride, const void* v,
+                                 int64_t v_stride, const int32_t* cu_q, const int32_t* cu_k, int num_seqs,
+                                 int64_t tokens, int64_t keys, int heads, int dim, int rot_dim, int vdim, float scale,
+                                 const void* sink, int* error_word, void* stream) {
+  using namespace mv;
+  if (num_seqs < 0 || tokens < 0 || keys < tokens || heads <= 0 || dim <= 0 || rot_dim < 0 || vdim <= 0 || !(scale > 0.f))
+    return fail(MV_ERR_SHAPE, "latent_prefill: heads %d dim %d rot_dim %d vdim %d", heads, dim, rot_dim, vdim);
+  const int nd = (dim + 63) / 64, nq = nd + (rot_dim + 63) / 64, nv = (vdim + 63) / 64;
+  if (dim % 8 || rot_dim % 8 || vdim % 8 || nq > 3 || nv > 2)
+    return fail(MV_ERR_LIMIT, "latent_prefill: dim %d rot_dim %d vdim %d", dim, rot_dim, vdim);
+  if (tokens == 0 || num_seqs == 0) return MV_OK;
+  if (!out || !q || !k || (rot_dim && !k_rot) || !v || !cu_q || !cu_k || !error_word) return fail(MV_ERR_NULL, "latent_prefill: null pointer");
+  if (!vec8_ok(out, out_stride, 2) || !vec8_ok(q, q_stride, 2) || !vec8_ok(k, k_stride, 2) || !vec8_ok(k_rot, k_rot_stride, 2) ||
+      !vec8_ok(v, v_stride, 2))
+    return fail(MV_ERR_ALIGN, "latent_prefill: rows must start on 16-byte boundaries");
+  const char* w = "latent_prefill";
+  CUtensorMap tm[5];
+  const auto* qb = static_cast<const __nv_bfloat16*>(q);
+  int rc = make_tmap_bf16(&tm[0], q, dim, heads, tokens, dim + rot_dim, q_stride, 1, kLfTile, w);
+  if (!rc) rc = make_tmap_bf16(&tm[2], k, dim, heads, keys, dim, k_stride, 1, kLfTile, w);
+  if (!rc && rot_dim) rc = make_tmap_bf16(&tm[1], qb + dim, rot_dim, heads, tokens, dim + rot_dim, q_stride, 1, kLfTile, w);
+  if (!rc && rot_dim) rc = make_tmap_bf16(&tm[3], k_rot, rot_dim, 1, keys, rot_dim, k_rot_stride, 1, kLfTile, w);
+  if (!rc) rc = make_tmap_bf16(&tm[4], v, vdim, heads, keys, vdim, v_stride, 1, kLfTile, w);
+  if (rc) return rc;
+  if (!rot_dim) { tm[1] = tm[0]; tm[3] = tm[2]; }
+  LfParams p{static_cast<__nv_bfloat16*>(out), out_stride, vdim, cu_q, cu_k, num_seqs, nd, dim, rot_dim,
+             scale * 1.4426950408889634f, static_cast<const __nv_bfloat16*>(sink), error_word};
+  auto st = static_cast<cudaStream_t>(stream);
+  if (nq == 1) return nv == 1 ? launch_latent_prefill<1, 1>(tm, p, tokens, heads, st) : launch_latent_prefill<1, 2>(tm, p, tokens, heads, st);
+  if (nq == 2) return nv == 1 ? launch_latent_prefill<2, 1>(tm, p, tokens, heads, st) : launch_latent_prefill<2, 2>(tm, p, tokens, heads, st);
+  return nv == 1 ? launch_latent_prefill<3, 1>(tm, p, tokens, heads, st) : launch_latent_prefill<3, 2>(tm, p, tokens, heads, st);
+}

@@ -4,7 +4,10 @@
 // assigns.  Sequence s of the batch has tokens cu[s] .. cu[s+1] and `start[s]` tokens behind it; start 0 means that
 // the slot's contents belong to somebody else and count as zero.
 //
-// conv_silu_kernel      every token and channel of the step (reads the slot, does not change it)
+// conv_silu_kernel      every token and channel of the step (reads the slot, does not change it); conv_silu_vec_kernel
+//                       is the same with eight channels per thread and the taps in registers
+// ssm_step_kernel       one token per sequence: convolution of the head's channels and one step of S, which is read
+//                       and written once, in whole rows (HBM-bound: 8 * heads * N * P bytes per sequence)
 // ssm_scan_kernel       token by token, S in shared memory: any sizes, bf16 or fp32
 // conv_state_kernel     writes the slot's convolution inputs for the next step
 #include <algorithm>
@@ -52,6 +55,61 @@ conv_silu_kernel(T* __restrict__ out, const T* __restrict__ u, int64_t u_stride,
     for (int k = 0; k < taps; ++k)
       acc = fmaf(Elem<T>::to_f(wc[k]), conv_input(u, u_stride, first, j - hist + k, c, st, hist, channels), acc);
     out[t * channels + c] = Elem<T>::from_f(silu_f(acc));
+  }
+}
+
+// Eight channels per thread, up to kCvRun consecutive tokens, the last taps - 1 inputs kept in registers.
+template <typename T, int TAPS>
+__global__ void __launch_bounds__(kCvThreads)
+conv_silu_vec_kernel(T* __restrict__ out, const T* __restrict__ u, int64_t u_stride, const T* __restrict__ w,
+                     const T* __restrict__ bias, int channels, const int32_t* __restrict__ cu, int num_seqs,
+                     int64_t tokens, const int32_t* __restrict__ slots, const int32_t* __restrict__ start,
+                     const T* __restrict__ state, int num_slots, int run) {
+  constexpr int HIST = TAPS - 1;
+  const int c = (blockIdx.x * kCvThreads + threadIdx.x) * 8;
+  if (c >= channels) return;
+  float wt[TAPS][8], b[8], win[HIST][8];
+#pragma unroll
+  for (int e = 0; e < 8; ++e) {
+    b[e] = bias ? Elem<T>::to_f(bias[c + e]) : 0.f;
+#pragma unroll
+    for (int k = 0; k < TAPS; ++k) wt[k][e] = Elem<T>::to_f(w[static_cast<int64_t>(c + e) * TAPS + k]);
+  }
+  const int64_t t0 = static_cast<int64_t>(blockIdx.y) * run, t1 = min(t0 + run, tokens);
+  int64_t end = -1;
+  for (int64_t t = t0; t < t1; ++t) {
+    if (t >= end) {                      // first token of this thread, or of a sequence: fetch what lies before it
+      const int s = seq_of_token(cu, num_seqs, static_cast<int>(t));
+      const int64_t first = cu ? cu[s] : t;
+      end = cu ? cu[s + 1] : t + 1;
+      const int slot = slots[s];
+      const T* st = start[s] > 0 && slot >= 0 && slot < num_slots ? state + static_cast<int64_t>(slot) * HIST * channels : nullptr;
+#pragma unroll
+      for (int k = 0; k < HIST; ++k) {
+        const int64_t j = t - first - HIST + k;
+        if (j >= 0) {
+          Vec<T, 8>::load(u + (first + j) * u_stride + c, win[k]);
+        } else if (st && HIST + j >= 0) {
+          Vec<T, 8>::load(st + (HIST + j) * channels + c, win[k]);
+        } else {
+#pragma unroll
+          for (int e = 0; e < 8; ++e) win[k][e] = 0.f;
+        }
+      }
+    }
+    float v[8], r[8];
+    Vec<T, 8>::load(u + t * u_stride + c, v);
+#pragma unroll
+    for (int e = 0; e < 8; ++e) {
+      float a = b[e];
+#pragma unroll
+      for (int k = 0; k < HIST; ++k) a = fmaf(wt[k][e], win[k][e], a);
+      r[e] = silu_f(fmaf(wt[HIST][e], v[e], a));
+#pragma unroll
+      for (int k = 0; k + 1 < HIST; ++k) win[k][e] = win[k + 1][e];
+      if (HIST > 0) win[HIST - 1][e] = v[e];
+    }
+    Vec<T, 8>::store(out + t * channels + c, r);
   }
 }
 
@@ -142,6 +200,87 @@ ssm_scan_kernel(T* __restrict__ y, const T* __restrict__ xbc, const T* __restric
   }
 }
 
+constexpr int kStThreads = 256;
+constexpr int kStBatch = 8;      // rows of S a thread has in flight
+
+// One CTA per (sequence, head), one token: u is the row before the convolution.
+template <typename T>
+__global__ void __launch_bounds__(kStThreads)
+ssm_step_kernel(T* __restrict__ y, const T* __restrict__ u, int64_t u_stride, const T* __restrict__ w,
+                const T* __restrict__ bias, int taps, const T* __restrict__ conv_state, const T* __restrict__ dt,
+                int64_t dt_stride, const T* __restrict__ dt_bias, const T* __restrict__ A_log, const T* __restrict__ D,
+                const int32_t* __restrict__ slots, const int32_t* __restrict__ start, float* __restrict__ state,
+                int num_slots, int heads, int P, int N, int groups) {
+  extern __shared__ __align__(16) float sm[];
+  const int s = blockIdx.x, h = blockIdx.y, tid = threadIdx.x;
+  const int g = h / (heads / groups), inner = heads * P, channels = inner + 2 * groups * N, hist = taps - 1;
+  float *sx = sm, *sB = sx + P, *sC = sB + N, *red = sC + N;      // red: [rows][P]
+  const int slot = slots[s], st0 = start[s];
+  const bool live = slot >= 0 && slot < num_slots && st0 >= 0;
+  T* yr = y + static_cast<int64_t>(s) * inner + h * P;
+  if (!live) {
+    for (int i = tid; i < P; i += kStThreads) yr[i] = Elem<T>::from_f(0.f);
+    return;
+  }
+  const int PQ = P / 4, rows = kStThreads / PQ, q = tid % PQ, r = tid / PQ;
+  const bool on = r < rows;
+  float4* gS = reinterpret_cast<float4*>(state + (static_cast<int64_t>(slot) * heads + h) * N * P);
+  float4 v[kStBatch];
+  auto fetch = [&](int n0) {
+#pragma unroll
+    for (int i = 0; i < kStBatch; ++i) {
+      const int n = n0 + i * rows + r;
+      v[i] = on && n < N && st0 > 0 ? gS[static_cast<int64_t>(n) * PQ + q] : make_float4(0.f, 0.f, 0.f, 0.f);
+    }
+  };
+  fetch(0);                                     // in flight while the convolution is computed
+  const T* cs = conv_state + static_cast<int64_t>(slot) * hist * channels;
+  for (int i = tid; i < P + 2 * N; i += kStThreads) {
+    const int c = i < P ? h * P + i : i < P + N ? inner + g * N + i - P : inner + (groups + g) * N + i - P - N;
+    float a = bias ? Elem<T>::to_f(bias[c]) : 0.f;
+    const T* wc = w + static_cast<int64_t>(c) * taps;
+    if (st0 > 0)
+      for (int k = 0; k < hist; ++k) a = fmaf(Elem<T>::to_f(wc[k]), Elem<T>::to_f(cs[static_cast<int64_t>(k) * channels + c]), a);
+    a = fmaf(Elem<T>::to_f(wc[hist]), Elem<T>::to_f(u[s * u_stride + c]), a);
+    sm[i] = Elem<T>::to_f(Elem<T>::from_f(silu_f(a)));       // rounded as the prompt path stores it
+  }
+  const float d = softplus_f(Elem<T>::to_f(dt[s * dt_stride + h]) + Elem<T>::to_f(dt_bias[h]));
+  const float decay = expf(-expf(Elem<T>::to_f(A_log[h])) * d);
+  __syncthreads();
+  float4 acc = make_float4(0.f, 0.f, 0.f, 0.f);
+  const float4 x = on ? *reinterpret_cast<const float4*>(sx + q * 4) : make_float4(0.f, 0.f, 0.f, 0.f);
+  const float4 dx = make_float4(d * x.x, d * x.y, d * x.z, d * x.w);
+  for (int n0 = 0; n0 < N; n0 += kStBatch * rows) {
+    if (n0) fetch(n0);
+#pragma unroll
+    for (int i = 0; i < kStBatch; ++i) {
+      const int n = n0 + i * rows + r;
+      if (on && n < N) {
+        const float b = sB[n], c = sC[n];
+        v[i].x = fmaf(decay, v[i].x, b * dx.x);
+        v[i].y = fmaf(decay, v[i].y, b * dx.y);
+        v[i].z = fmaf(decay, v[i].z, b * dx.z);
+        v[i].w = fmaf(decay, v[i].w, b * dx.w);
+        gS[static_cast<int64_t>(n) * PQ + q] = v[i];
+        acc.x = fmaf(v[i].x, c, acc.x);
+        acc.y = fmaf(v[i].y, c, acc.y);
+        acc.z = fmaf(v[i].z, c, acc.z);
+        acc.w = fmaf(v[i].w, c, acc.w);
+      }
+    }
+  }
+  if (on) {
+    float* o = red + r * P + q * 4;
+    o[0] = acc.x; o[1] = acc.y; o[2] = acc.z; o[3] = acc.w;
+  }
+  __syncthreads();
+  for (int i = tid; i < P; i += kStThreads) {
+    float a = Elem<T>::to_f(D[h]) * sx[i];
+    for (int k = 0; k < rows; ++k) a += red[k * P + i];
+    yr[i] = Elem<T>::from_f(a);
+  }
+}
+
 }  // namespace mv
 
 static int check_ssm(const char* what, int dtype, int num_seqs, int channels, int taps) {
@@ -162,6 +301,18 @@ extern "C" int mv_conv_silu(void* out, const void* u, int64_t u_stride, const vo
   if (grid.y > 65535) return fail(MV_ERR_LIMIT, "conv_silu: %lld tokens", static_cast<long long>(tokens));
   auto run = [&](auto tag) {
     using T = decltype(tag);
+    const int eb = sizeof(T);
+    if (taps >= 2 && taps <= 4 && channels % 8 == 0 && vec8_ok(out, channels, eb) && vec8_ok(u, u_stride, eb) && vec8_ok(state, channels, eb)) {
+      const int len = tokens > 4096 ? 32 : tokens > 512 ? 8 : 2;      // longer runs re-read fewer inputs
+      const dim3 vg((channels / 8 + kCvThreads - 1) / kCvThreads, static_cast<unsigned>((tokens + len - 1) / len));
+      auto go = [&](auto kernel) {
+        kernel<<<vg, kCvThreads, 0, static_cast<cudaStream_t>(stream)>>>(
+            static_cast<T*>(out), static_cast<const T*>(u), u_stride, static_cast<const T*>(w), static_cast<const T*>(bias),
+            channels, cu, num_seqs, tokens, slots, start, static_cast<const T*>(state), num_slots, len);
+        return check_launch("conv_silu");
+      };
+      return taps == 2 ? go(conv_silu_vec_kernel<T, 2>) : taps == 3 ? go(conv_silu_vec_kernel<T, 3>) : go(conv_silu_vec_kernel<T, 4>);
+    }
     conv_silu_kernel<T><<<grid, kCvThreads, 0, static_cast<cudaStream_t>(stream)>>>(
         static_cast<T*>(out), static_cast<const T*>(u), u_stride, static_cast<const T*>(w), static_cast<const T*>(bias),
         taps, channels, cu, num_seqs, tokens, slots, start, static_cast<const T*>(state), num_slots);
@@ -213,6 +364,33 @@ extern "C" int mv_ssm_scan(void* y, const void* xbc, const void* dt, int64_t dt_
         static_cast<const T*>(dt_bias), static_cast<const T*>(A_log), static_cast<const T*>(D), cu, num_seqs, slots,
         start, state, num_slots, heads, vdim, state_dim, groups, pb);
     return check_launch("ssm_scan");
+  };
+  return dtype == MV_F32 ? run(float{}) : run(__nv_bfloat16{});
+}
+
+extern "C" int mv_ssm_step(void* y, const void* u, int64_t u_stride, const void* w, const void* bias, int taps,
+                           const void* conv_state, const void* dt, int64_t dt_stride, const void* dt_bias,
+                           const void* A_log, const void* D, int num_seqs, const int32_t* slots, const int32_t* start,
+                           float* state, int num_slots, int heads, int vdim, int state_dim, int groups, int dtype,
+                           void* stream) {
+  using namespace mv;
+  const int rc = check_ssm("ssm_step", dtype, num_seqs, heads, taps);
+  if (rc || num_seqs == 0) return rc;
+  if (vdim <= 0 || vdim % 4 || vdim > 4 * kStThreads || state_dim <= 0 || state_dim % 4 || groups <= 0 || heads % groups)
+    return fail(MV_ERR_SHAPE, "ssm_step: heads %d groups %d vdim %d state %d", heads, groups, vdim, state_dim);
+  if (!y || !u || !w || (taps > 1 && !conv_state) || !dt || !dt_bias || !A_log || !D || !slots || !start || !state)
+    return fail(MV_ERR_NULL, "ssm_step: null pointer");
+  if (!aligned16(state)) return fail(MV_ERR_ALIGN, "ssm_step: state");
+  const int rows = kStThreads / (vdim / 4);
+  const size_t smem = sizeof(float) * (static_cast<size_t>(vdim) + 2 * state_dim + rows * vdim);
+  if (smem > 48 * 1024) return fail(MV_ERR_LIMIT, "ssm_step: state %d", state_dim);
+  auto run = [&](auto tag) {
+    using T = decltype(tag);
+    ssm_step_kernel<T><<<dim3(num_seqs, heads), kStThreads, smem, static_cast<cudaStream_t>(stream)>>>(
+        static_cast<T*>(y), static_cast<const T*>(u), u_stride, static_cast<const T*>(w), static_cast<const T*>(bias), taps,
+        static_cast<const T*>(conv_state), static_cast<const T*>(dt), dt_stride, static_cast<const T*>(dt_bias),
+        static_cast<const T*>(A_log), static_cast<const T*>(D), slots, start, state, num_slots, heads, vdim, state_dim, groups);
+    return check_launch("ssm_step");
   };
   return dtype == MV_F32 ? run(float{}) : run(__nv_bfloat16{});
 }

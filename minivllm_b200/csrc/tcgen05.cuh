@@ -63,7 +63,7 @@ __device__ __forceinline__ bool mbar_wait(uint32_t bar, uint32_t parity, volatil
 // that warp shares an instruction cache with the (large) softmax loop, and with the spin loops unrolled its code
 // is pushed out of the cache at every unit boundary (measured: 0.61 ms against 0.51 ms on the 32-sequence
 // benchmark).  The part that runs when a wait is long is a call.
-__device__ __noinline__ bool mbar_wait_long(uint32_t bar, uint32_t parity, volatile int* abort_flag, int* error_word,
+static __device__ __noinline__ bool mbar_wait_long(uint32_t bar, uint32_t parity, volatile int* abort_flag, int* error_word,
                                             int where) {
   const unsigned long long t0 = global_ns();
   for (;;) {
@@ -210,6 +210,23 @@ __device__ __forceinline__ void mma_ss_k128_commit(uint32_t d_tmem, uint64_t a_d
       "@pe tcgen05.mma.cta_group::1.kind::f16 [%0], da, db, %3, pt;\n\t"
       "@pe tcgen05.commit.cta_group::1.mbarrier::arrive::one.shared::cluster.b64 [%4];\n\t}"
       ::"r"(d_tmem), "l"(a_desc), "l"(b_desc), "r"(idesc), "r"(commit_bar) : "memory");
+}
+// The four K = 16 steps of one 64-column slab (A and B K-major, 128B swizzle), without a commit.
+__device__ __forceinline__ void mma_ss_k64(uint32_t d_tmem, uint64_t a_desc, uint64_t b_desc, uint32_t idesc, bool accum) {
+  const uint32_t acc = accum ? 1u : 0u;
+  asm volatile(
+      "{\n\t.reg .pred pe, pt, pf;\n\t.reg .b64 da, db;\n\t"
+      "elect.sync _|pe, 0xffffffff;\n\t"
+      "setp.eq.u32 pt, %3, %3;\n\t"
+      "setp.ne.u32 pf, %4, 0;\n\t"
+      "@pe tcgen05.mma.cta_group::1.kind::f16 [%0], %1, %2, %3, pf;\n\t"
+      "add.s64 da, %1, 2;\n\tadd.s64 db, %2, 2;\n\t"
+      "@pe tcgen05.mma.cta_group::1.kind::f16 [%0], da, db, %3, pt;\n\t"
+      "add.s64 da, %1, 4;\n\tadd.s64 db, %2, 4;\n\t"
+      "@pe tcgen05.mma.cta_group::1.kind::f16 [%0], da, db, %3, pt;\n\t"
+      "add.s64 da, %1, 6;\n\tadd.s64 db, %2, 6;\n\t"
+      "@pe tcgen05.mma.cta_group::1.kind::f16 [%0], da, db, %3, pt;\n\t}"
+      ::"r"(d_tmem), "l"(a_desc), "l"(b_desc), "r"(idesc), "r"(acc) : "memory");
 }
 //   D[tmem] (+)= A[tmem] * B[smem]; A holds two 16-bit values per column (8 columns per MMA), B is an MN-major
 //   tile whose 16-row slices are 2048 bytes apart.

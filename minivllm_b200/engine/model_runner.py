@@ -242,6 +242,8 @@ class ModelRunner:
         set_context(True, cu_q, cu_k, meta["max_seqlen_q"], meta["max_seqlen_k"], meta["slot_mapping"],
                     meta["seq_lens"], self.state.tables.index_select(0, meta["slots"].long()),
                     positions=meta["positions"], last_token_index=rows, num_decode=nd,
+                    portion_keys=sum(s.num_cached_tokens + n for s, n in zip(seqs[nd:], counts[nd:])),
+                    portion_fresh=all(s.num_cached_tokens == 0 for s in seqs[nd:]),
                     portion_cu_q=cu_q[nd:] - cu_q[nd], portion_cu_k=cu_k[nd:] - cu_k[nd],
                     state_slots=meta["slots"], state_starts=meta["starts"])
         return input_ids, order

@@ -1,8 +1,11 @@
 """Latent attention: low-rank key/value rows in a paged cache, one rotated key part shared by all heads, a learned
 sink per head and a sigmoid gate on the heads (csrc/latent_attention.cu).
 
-The cache holds one row [c | rotated key part] per token.  Attention runs in the absorbed form: the key
-up-projection is applied to the queries, the value up-projection to the weighted sum of the c's.
+The cache holds one row [c | rotated key part] per token.  Decoded tokens run in the absorbed form: the key
+up-projection is applied to the queries, the value up-projection to the weighted sum of the c's.  Portions of
+prompts expand keys and values per head (one product over the packed latent rows, gathered from the cache when a
+sequence has tokens behind it) and run tcgen05 prefill attention.  Sizes those kernels do not take, and 32-bit
+models, use the absorbed form with a kernel for any sizes.
 """
 import torch
 import torch.nn as nn
@@ -10,6 +13,7 @@ import torch.nn.functional as F
 
 from .. import _cabi
 from ..utils.context import get_context
+from .attention import _error_word
 from .group_norm import gate_mul
 from .linear import StackedLinear
 
@@ -59,6 +63,52 @@ def latent_attention_rows(q_lat, q_rot, cache, block_tables, cu_q, positions, si
     return out
 
 
+def latent_decode(q_lat, q_rot, cache, block_tables, positions, sink, scale, workspace=None):
+    """latent_attention_rows for one row per sequence on tensor cores; None when the kernel does not take the sizes."""
+    _cabi.require_cuda(q_lat, q_rot, cache, block_tables, positions)
+    batch, heads, rank = q_lat.shape
+    rot = q_rot.shape[2]
+    L = _cabi.lib()
+    need = L.mv_latent_decode_workspace_bytes(batch, heads, rank, rot)
+    if need < 0 or q_lat.dtype != torch.bfloat16:
+        return None
+    if workspace is None:
+        workspace = torch.empty(need, dtype=torch.uint8, device=q_lat.device)
+    out = torch.empty((heads, batch, rank), dtype=q_lat.dtype, device=q_lat.device).transpose(0, 1)
+    _cabi.check(L.mv_latent_decode(
+        out.data_ptr(), out.stride(0), out.stride(1), q_lat.data_ptr(), q_lat.stride(0), q_lat.stride(1),
+        q_rot.data_ptr(), q_rot.stride(0), q_rot.stride(1), cache.data_ptr(), block_tables.data_ptr(),
+        block_tables.stride(0), block_tables.shape[1], cache.shape[1], cache.shape[0], positions.data_ptr(), None,
+        sink.data_ptr() if sink is not None else None, batch, heads, rank, rot, scale, workspace.data_ptr(),
+        workspace.numel(), _cabi.stream_ptr()))
+    return out
+
+
+def latent_gather(cache, cu_k, keys, block_tables):
+    """Packed latent rows (keys, row) of the sequences of cu_k, from position 0, out of the paged cache."""
+    row = cache.shape[2]
+    out = torch.empty((keys, row), dtype=cache.dtype, device=cache.device)
+    _cabi.check(_cabi.lib().mv_latent_gather(
+        out.data_ptr(), cache.data_ptr(), cu_k.data_ptr(), cu_k.numel() - 1, keys, block_tables.data_ptr(),
+        block_tables.stride(0), block_tables.shape[1], cache.shape[1], cache.shape[0], row,
+        _cabi.layer_dtype_code(cache.dtype), _cabi.stream_ptr()))
+    return out
+
+
+def latent_prefill(q, kv, k_rot, cu_q, cu_k, heads, dim, rot_dim, vdim, scale, sink):
+    """q (tokens, heads * (dim + rot_dim)), kv (keys, heads * (dim + vdim)): all keys, then all values; k_rot (keys,
+    rot_dim).  Returns (tokens, heads * vdim)."""
+    _cabi.require_cuda(q, kv, k_rot, cu_q, cu_k)
+    out = torch.empty((q.shape[0], heads * vdim), dtype=q.dtype, device=q.device)
+    v = kv[:, heads * dim:]
+    _cabi.check(_cabi.lib().mv_latent_prefill(
+        out.data_ptr(), out.stride(0), q.data_ptr(), q.stride(0), kv.data_ptr(), kv.stride(0), k_rot.data_ptr(),
+        k_rot.stride(0), v.data_ptr(), v.stride(0), cu_q.data_ptr(), cu_k.data_ptr(), cu_q.numel() - 1, q.shape[0],
+        kv.shape[0], heads, dim, rot_dim, vdim, scale, sink.data_ptr() if sink is not None else None,
+        _error_word(q.device).data_ptr(), _cabi.stream_ptr()))
+    return out
+
+
 class LatentAttention(nn.Module):
     def __init__(self, m, width, eps, load, extra=None, max_position=4096):
         super().__init__()
@@ -70,8 +120,7 @@ class LatentAttention(nn.Module):
                                       "g": load("g", (H * vd, width)), **(extra or {})})
         param = lambda t: nn.Parameter(t, requires_grad=False)
         self.c_norm, self.sink = param(load("dkv.norm", (rank,))), param(load("sink", (H,)))
-        self.uk_w = param(load("uk", (H * d, rank)))                    # (heads * dim, rank)
-        self.uv_w = param(load("uv", (H * vd, rank)))                   # (heads * vdim, rank)
+        self.ukv_w = param(torch.cat([load("uk", (H * d, rank)), load("uv", (H * vd, rank))]))
         self.o_w = param(load("o", (width, H * vd)))
         self.cos_t, self.sin_t = rope_table(m["rot"]["base"], self.rope_dims, max_position, self.o_w.device)
         self.latent_cache = None        # (blocks, block_size, rank + rot_dim), assigned by the model runner
@@ -80,21 +129,65 @@ class LatentAttention(nn.Module):
     def latent_row(self):
         return self.rank + self.rot_dim
 
+    @property
+    def uk_w(self):
+        return self.ukv_w[:self.heads * self.dim].view(self.heads, self.dim, self.rank)
+
+    @property
+    def uv_w(self):
+        return self.ukv_w[self.heads * self.dim:].view(self.heads, self.vdim, self.rank)
+
+    def _expands(self, dtype):
+        """Does the tensor-core prefill kernel take this layer's sizes?"""
+        d, r, vd = self.dim, self.rot_dim, self.vdim
+        return dtype == torch.bfloat16 and d % 8 == 0 and r % 8 == 0 and vd % 8 == 0 and self.rank % 8 == 0 and \
+            -(-d // 64) - (-r // 64) <= 3 and vd <= 128 and self.scale > 0
+
     def _absorbed(self, q, block_tables, cu_q, positions):
-        """q (tokens, heads, dim + rot_dim) -> (tokens, heads, vdim) view of a head-major tensor."""
-        H, d = self.heads, self.dim
-        q_lat = torch.bmm(q[:, :, :d].transpose(0, 1), self.uk_w.view(H, d, self.rank))      # (heads, tokens, rank)
-        o = latent_attention_rows(q_lat.transpose(0, 1), q[:, :, d:], self.latent_cache, block_tables, cu_q, positions,
-                                  self.sink, self.scale)
-        return torch.bmm(o.transpose(0, 1), self.uv_w.view(H, self.vdim, self.rank).transpose(1, 2)).transpose(0, 1)
+        """q (tokens, heads, dim + rot_dim) -> (tokens, heads, vdim) view of a head-major tensor.  cu_q None: one
+        token per row of block_tables."""
+        d = self.dim
+        q_lat = torch.bmm(q[:, :, :d].transpose(0, 1), self.uk_w).transpose(0, 1)            # (tokens, heads, rank)
+        o = None
+        if cu_q is None:
+            o = latent_decode(q_lat, q[:, :, d:], self.latent_cache, block_tables, positions, self.sink, self.scale)
+        if o is None:
+            o = latent_attention_rows(q_lat, q[:, :, d:], self.latent_cache, block_tables, cu_q, positions, self.sink,
+                                      self.scale)
+        return torch.bmm(o.transpose(0, 1), self.uv_w.transpose(1, 2)).transpose(0, 1)
+
+    def _portions(self, ctx, q2, lat, nd):
+        """The rows behind the decoded ones -> (tokens, heads * vdim) or (tokens, heads, vdim)."""
+        H, d, r, rank = self.heads, self.dim, self.rot_dim, self.rank
+        tokens, tables, positions = q2.shape[0], ctx.block_tables[nd:], ctx.positions[nd:]
+        q = q2.unflatten(1, (H, d + r))
+        if not self._expands(q2.dtype):
+            return self._absorbed(q, tables, ctx.portion_cu_q, positions)
+        if tokens <= 16 and ctx.portion_keys >= 2048:
+            # a few tokens far into a sequence: expanding every key would cost more than decoding them
+            at = torch.arange(tokens, device=q.device, dtype=torch.int32)
+            seq = torch.bucketize(at, ctx.portion_cu_q[1:], right=True)
+            return self._absorbed(q, tables.index_select(0, seq), None, positions)
+        if ctx.portion_fresh:
+            cu_k = ctx.portion_cu_q
+        else:
+            cu_k = ctx.portion_cu_k
+            lat = latent_gather(self.latent_cache, cu_k, ctx.portion_keys, tables)
+        kv = F.linear(lat[:, :rank], self.ukv_w)
+        return latent_prefill(q2, kv, lat[:, rank:], ctx.portion_cu_q, cu_k, H, d, r, self.vdim, self.scale, self.sink)
 
     def forward(self, h):
         """h (tokens, width) -> (mixer output (tokens, width), {extra parts of the stacked projection})."""
         ctx = get_context()
         p = self.stacked(h)
         H, d, r = self.heads, self.dim, self.rot_dim
-        latent_prep(p["q"], p["dkv"], self.c_norm, ctx.positions, self.cos_t, self.sin_t, H, d, r, self.rope_dims,
-                    self.rank, self.eps, self.latent_cache, ctx.slot_mapping)
-        q = p["q"].unflatten(1, (H, d + r))
-        o = self._absorbed(q, ctx.block_tables, ctx.cu_seqlens_q, ctx.positions)
-        return F.linear(gate_mul(o, p["g"]), self.o_w), p
+        q, g, nd = p["q"], p["g"], ctx.num_decode
+        lat = latent_prep(q, p["dkv"], self.c_norm, ctx.positions, self.cos_t, self.sin_t, H, d, r, self.rope_dims,
+                          self.rank, self.eps, self.latent_cache, ctx.slot_mapping)
+        o = torch.empty((h.shape[0], H * self.vdim), dtype=h.dtype, device=h.device)
+        if nd:
+            y = self._absorbed(q[:nd].unflatten(1, (H, d + r)), ctx.block_tables[:nd], None, ctx.positions[:nd])
+            gate_mul(y, g[:nd], out=o[:nd])
+        if h.shape[0] > nd:
+            gate_mul(self._portions(ctx, q[nd:], lat[nd:], nd), g[nd:], out=o[nd:])
+        return F.linear(o, self.o_w), p

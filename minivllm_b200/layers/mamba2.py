@@ -33,16 +33,40 @@ def conv_state_update(state, u, taps, cu, slots, starts):
         _cabi.stream_ptr()))
 
 
-def ssm_scan(xbc, dt, dt_bias, A_log, D, cu, slots, starts, state, heads, vdim, state_dim, groups):
+def ssm_scan(xbc, dt, dt_bias, A_log, D, cu, slots, starts, state, heads, vdim, state_dim, groups, out=None,
+             chunked=None):
     """xbc (tokens, heads*vdim + 2*groups*state_dim) contiguous, dt (tokens, heads); returns y (tokens, heads*vdim)
-    and advances `state` (slots, heads, state_dim, vdim) fp32."""
+    and advances `state` (slots, heads, state_dim, vdim) fp32.  bf16 takes the chunked tensor-core kernel when it has
+    the sizes."""
     _cabi.require_cuda(xbc, dt, state)
-    y = torch.empty((xbc.shape[0], heads * vdim), dtype=xbc.dtype, device=xbc.device)
-    _cabi.check(_cabi.lib().mv_ssm_scan(
+    L = _cabi.lib()
+    y = torch.empty((xbc.shape[0], heads * vdim), dtype=xbc.dtype, device=xbc.device) if out is None else out
+    if chunked is None:
+        chunked = xbc.dtype == torch.bfloat16 and cu is not None and bool(L.mv_ssm_chunk_takes(vdim, state_dim))
+    if chunked:
+        _cabi.check(L.mv_ssm_chunk_scan(
+            y.data_ptr(), y.stride(0), xbc.data_ptr(), xbc.stride(0), dt.data_ptr(), dt.stride(0), dt_bias.data_ptr(),
+            A_log.data_ptr(), D.data_ptr(), cu.data_ptr(), slots.numel(), slots.data_ptr(), starts.data_ptr(),
+            state.data_ptr(), state.shape[0], heads, vdim, state_dim, groups, _cabi.stream_ptr()))
+        return y
+    _cabi.check(L.mv_ssm_scan(
         y.data_ptr(), xbc.data_ptr(), dt.data_ptr(), dt.stride(0), dt_bias.data_ptr(), A_log.data_ptr(), D.data_ptr(),
         cu.data_ptr() if cu is not None else None, slots.numel(), slots.data_ptr(), starts.data_ptr(),
         state.data_ptr(), state.shape[0], heads, vdim, state_dim, groups, _cabi.layer_dtype_code(xbc.dtype),
         _cabi.stream_ptr()))
+    return y
+
+
+def ssm_step(u, conv_w, conv_b, conv_state, dt, dt_bias, A_log, D, slots, starts, state, heads, vdim, state_dim,
+             groups, out=None):
+    """One token per sequence: convolution (conv_state is only read) and one step of the recurrence."""
+    _cabi.require_cuda(u, dt, state)
+    y = torch.empty((u.shape[0], heads * vdim), dtype=u.dtype, device=u.device) if out is None else out
+    _cabi.check(_cabi.lib().mv_ssm_step(
+        y.data_ptr(), u.data_ptr(), u.stride(0), conv_w.data_ptr(), conv_b.data_ptr(), conv_w.shape[1],
+        conv_state.data_ptr(), dt.data_ptr(), dt.stride(0), dt_bias.data_ptr(), A_log.data_ptr(), D.data_ptr(),
+        slots.numel(), slots.data_ptr(), starts.data_ptr(), state.data_ptr(), state.shape[0], heads, vdim, state_dim,
+        groups, _cabi.layer_dtype_code(u.dtype), _cabi.stream_ptr()))
     return y
 
 
@@ -73,11 +97,24 @@ class Mamba2(nn.Module):
         """h (tokens, width) -> (mixer output (tokens, width), {extra parts of the stacked projection})."""
         ctx = get_context()
         p = self.stacked(h)
-        cu, slots, starts = ctx.cu_seqlens_q, ctx.state_slots, ctx.state_starts
+        slots, starts, nd = ctx.state_slots, ctx.state_starts, ctx.num_decode
         conv, ssm = self.slot_state["conv"], self.slot_state["ssm"]
-        xbc = conv_silu(p["xbc"], self.conv_w, self.conv_b, cu, slots, starts, conv)
-        y = ssm_scan(xbc, p["dt"], self.dt_bias, self.A_log, self.D, cu, slots, starts, ssm, self.heads, self.vdim,
-                     self.state, self.groups)
-        conv_state_update(conv, p["xbc"], self.taps, cu, slots, starts)
+        u, dt = p["xbc"], p["dt"]
+        y = torch.empty((h.shape[0], self.inner), dtype=h.dtype, device=h.device)
+        if nd:                           # sequences with one token come first
+            w = (self.conv_w, self.conv_b)
+            par = (self.dt_bias, self.A_log, self.D)
+            dims = (self.heads, self.vdim, self.state, self.groups)
+            if self.vdim % 4 == 0 and self.state % 4 == 0:
+                ssm_step(u[:nd], *w, conv, dt[:nd], *par, slots[:nd], starts[:nd], ssm, *dims, out=y[:nd])
+            else:
+                xbc = conv_silu(u[:nd], *w, None, slots[:nd], starts[:nd], conv)
+                ssm_scan(xbc, dt[:nd], *par, None, slots[:nd], starts[:nd], ssm, *dims, out=y[:nd])
+        if h.shape[0] > nd:
+            cu = ctx.portion_cu_q
+            xbc = conv_silu(u[nd:], self.conv_w, self.conv_b, cu, slots[nd:], starts[nd:], conv)
+            ssm_scan(xbc, dt[nd:], self.dt_bias, self.A_log, self.D, cu, slots[nd:], starts[nd:], ssm, self.heads,
+                     self.vdim, self.state, self.groups, out=y[nd:])
+        conv_state_update(conv, u, self.taps, ctx.cu_seqlens_q, slots, starts)
         y = gated_group_norm(y, p["z"], self.norm_w, self.norm_groups, self.eps)
         return F.linear(y, self.o_w), p

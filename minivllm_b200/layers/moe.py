@@ -10,6 +10,7 @@ import torch.nn as nn
 import torch.nn.functional as F
 
 from .. import _cabi
+from .attention import _error_word
 from .group_norm import gate_mul, moe_residual_norm
 from .linear import StackedLinear, router_logits
 
@@ -49,15 +50,23 @@ def gather_rows(x, row_token):
     return out
 
 
-def grouped_linear(x, weight, offsets, gated=False):
+def grouped_linear(x, weight, offsets, gated=False, tensor_cores=None):
     """x (rows, in) sorted by expert, weight (experts, out, in) -> (rows, out).  With `gated`, weight is
-    (experts, 2 * out, in), gate rows first, and the result silu(gate) * up."""
+    (experts, 2 * out, in), gate rows first, and the result silu(gate) * up.  bf16 runs on the tensor cores when the rows
+    are whole 16-byte pieces."""
     _cabi.require_cuda(x, weight, offsets)
     experts, out_dim, in_dim = weight.shape
     if gated:
         out_dim //= 2
     rows = x.shape[0]
     out = torch.empty((rows, out_dim), dtype=x.dtype, device=x.device)
+    if tensor_cores is None:
+        tensor_cores = x.dtype == torch.bfloat16 and in_dim % 8 == 0
+    if tensor_cores:
+        _cabi.check(_cabi.lib().mv_grouped_gemm(out.data_ptr(), x.data_ptr(), weight.data_ptr(), offsets.data_ptr(),
+                                                experts, rows, in_dim, out_dim, 1 if gated else 0,
+                                                _error_word(x.device).data_ptr(), _cabi.stream_ptr()))
+        return out
     _cabi.check(_cabi.lib().mv_grouped_rows(out.data_ptr(), x.data_ptr(), weight.data_ptr(), offsets.data_ptr(),
                                             experts, rows, in_dim, out_dim, 1 if gated else 0,
                                             _cabi.layer_dtype_code(x.dtype), _cabi.stream_ptr()))

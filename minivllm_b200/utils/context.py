@@ -36,6 +36,8 @@ class Context:
     num_decode: int = 0                              # the first num_decode sequences have one token each
     portion_cu_q: Optional[torch.Tensor] = None      # cu_seqlens_q / _k of the sequences behind them, from 0
     portion_cu_k: Optional[torch.Tensor] = None
+    portion_keys: int = 0                            # cu_seqlens_k's total over those sequences
+    portion_fresh: bool = False                      # none of them has tokens behind it
     state_slots: Optional[torch.Tensor] = None       # (num_seqs,) int32 slot of each sequence
     state_starts: Optional[torch.Tensor] = None      # (num_seqs,) int32 tokens behind this step (-1: padding row)
 
