@@ -793,8 +793,9 @@ def main():
     ap.add_argument("--steps", type=int, default=None)
     ap.add_argument("--warmup", type=int, default=None)
     ap.add_argument("--impl", default="ours", choices=["ours", "reference"])
-    ap.add_argument("--workload", default="engine", choices=["engine", "decode", "allreduce", "ops"])
-    ap.add_argument("--case", default="store_kvcache_bf16", help="operator case of --workload ops: " + ", ".join(OP_CASES))
+    ap.add_argument("--workload", default="engine", choices=["engine", "decode", "allreduce", "ops", "sipazen"])
+    ap.add_argument("--case", default=None, help="operator case of --workload ops: " + ", ".join(OP_CASES) +
+                    "; of --workload sipazen: one of its kernels")
     ap.add_argument("--cpu-seconds", type=float, default=10.0)
     ap.add_argument("--no-extras", action="store_true", help="skip the secondary operator numbers and the CPU leg")
     ap.add_argument("--small", action="store_true",
@@ -809,7 +810,10 @@ def main():
         if not ours:
             args.steps = min(args.steps, 2)      # each CPU step is ~20-40 s of host work
             args.warmup = min(args.warmup, 1)    # (a short pass that touches every weight once)
+    elif args.workload == "sipazen":
+        args.steps, args.warmup = 20 if args.steps is None else args.steps, 3
     elif args.workload == "ops":
+        args.case = args.case or "store_kvcache_bf16"
         args.steps = 3 if args.steps is None else args.steps
         args.warmup = 3
     else:
@@ -841,6 +845,9 @@ def main():
         line = run_engine(args, rank, world, local, device, dist_on, pk)
     elif args.workload == "allreduce":
         line = run_allreduce(args, rank, world, local, device, dist_on, pk)
+    elif args.workload == "sipazen":
+        import bench_sipazen
+        line = bench_sipazen.run(device, pk, args.steps, args.case)
     elif args.workload == "ops":
         line = run_ops(args, device, pk)
     else:
