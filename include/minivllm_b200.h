@@ -511,8 +511,9 @@ int mv_grouped_gemm(void* out, const void* x, const void* w, const int32_t* offs
     int64_t rows, int in_dim, int out_dim, int gated, int* error_word, void* stream);
 
 /*
- * mv_latent_attention_rows for one query row per sequence on tensor cores, bf16: rank a multiple of 64 up to 512,
- * rot_dim a multiple of 32, at most 1,024 rows (workspace_bytes returns -1 otherwise).  Sequence b has
+ * mv_latent_attention_rows for one query row per sequence on tensor cores, bf16: rank a multiple of 16 up to 512,
+ * rank + rot_dim a multiple of 32 up to 576, at most 1,024 rows (workspace_bytes returns -1 otherwise).  Bounded waits
+ * report in *error_word.  Sequence b has
  * positions[b] + 1 keys; rows with active[b] < 0 (active may be null) have none and give zeros.
  */
 int64_t mv_latent_decode_workspace_bytes(int batch, int heads, int rank, int rot_dim);
@@ -521,7 +522,7 @@ int mv_latent_decode(void* out, int64_t out_stride, int64_t out_head_stride, con
     int64_t q_rot_head_stride, const void* cache, const int32_t* block_tables, int64_t bt_stride,
     int max_blocks, int block_size, int64_t num_blocks, const int64_t* positions, const int32_t*
     active, const void* sink, int batch, int heads, int rank, int rot_dim, float scale, void*
-    workspace, int64_t workspace_bytes, void* stream);
+    workspace, int64_t workspace_bytes, int* error_word, void* stream);
 
 /*
  * Prefill of latent attention with keys and values expanded per head, bf16, tcgen05.

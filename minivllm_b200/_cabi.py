@@ -99,7 +99,7 @@ SIGNATURES = {
     "mv_latent_decode_workspace_bytes": (_c_i64, [_c_int, _c_int, _c_int, _c_int]),
     "mv_latent_decode": (_c_int, [_c_ptr, _c_i64, _c_i64, _c_ptr, _c_i64, _c_i64, _c_ptr, _c_i64, _c_i64, _c_ptr,
         _c_ptr, _c_i64, _c_int, _c_int, _c_i64, _c_ptr, _c_ptr, _c_ptr, _c_int, _c_int, _c_int, _c_int, _c_f32,
-        _c_ptr, _c_i64, _c_ptr]),
+        _c_ptr, _c_i64, _c_ptr, _c_ptr]),
     "mv_latent_gather": (_c_int, [_c_ptr, _c_ptr, _c_ptr, _c_int, _c_i64, _c_ptr, _c_i64, _c_int, _c_int, _c_i64,
         _c_int, _c_int, _c_ptr]),
     "mv_latent_prefill": (_c_int, [_c_ptr, _c_i64, _c_ptr, _c_i64, _c_ptr, _c_i64, _c_ptr, _c_i64, _c_ptr, _c_i64,

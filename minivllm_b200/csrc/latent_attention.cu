@@ -63,6 +63,84 @@ latent_prep_kernel(T* __restrict__ q, int64_t q_stride, const T* __restrict__ do
   }
 }
 
+// The same in 16-byte pieces: rank, dim and half of the rotated dimensions are multiples of 8 and rot_dim is rotated whole.
+constexpr int kLvThreads = 128;
+template <typename T>
+__global__ void __launch_bounds__(kLvThreads)
+latent_prep_vec_kernel(T* __restrict__ q, int64_t q_stride, const T* __restrict__ down, int64_t down_stride,
+                       const T* __restrict__ c_weight, const int64_t* __restrict__ positions,
+                       const float* __restrict__ cos_t, const float* __restrict__ sin_t, int64_t max_position,
+                       T* __restrict__ latent_out, T* __restrict__ cache, const int64_t* __restrict__ slot_mapping,
+                       int64_t num_slots, int heads, int dim, int rot_dim, int rank, float eps) {
+  const int64_t t = blockIdx.x;
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+  const int half = rot_dim / 2, row = rank + rot_dim, hv = half / 8;
+  const T* d = down + t * down_stride;
+  const int64_t slot = slot_mapping ? slot_mapping[t] : -1;
+  T* lo = latent_out ? latent_out + t * row : nullptr;
+  T* co = cache && slot >= 0 && slot < num_slots ? cache + slot * row : nullptr;
+  if (warp == 0) {
+    constexpr int kHold = 2;            // pieces of the row a lane keeps in registers (rank 512); longer rows re-read
+    float hold[kHold][8];
+    float acc = 0.f;
+    for (int i = lane, k = 0; i < rank / 8; i += 32, ++k) {
+      float v[8];
+      Vec<T, 8>::load(d + i * 8, v);
+#pragma unroll
+      for (int e = 0; e < 8; ++e) acc = fmaf(v[e], v[e], acc);
+#pragma unroll
+      for (int h = 0; h < kHold; ++h)
+        if (k == h)
+#pragma unroll
+          for (int e = 0; e < 8; ++e) hold[h][e] = v[e];
+    }
+    const float rs = 1.f / sqrtf(warp_sum(acc) / static_cast<float>(rank) + eps);
+    for (int i = lane, k = 0; i < rank / 8; i += 32, ++k) {
+      float v[8], w[8];
+      Vec<T, 8>::load(c_weight + i * 8, w);
+      if (k >= kHold) Vec<T, 8>::load(d + i * 8, v);
+#pragma unroll
+      for (int h = 0; h < kHold; ++h)
+        if (k == h)
+#pragma unroll
+          for (int e = 0; e < 8; ++e) v[e] = hold[h][e];
+#pragma unroll
+      for (int e = 0; e < 8; ++e) v[e] = v[e] * rs * w[e];
+      if (lo) Vec<T, 8>::store(lo + i * 8, v);
+      if (co) Vec<T, 8>::store(co + i * 8, v);
+    }
+    return;
+  }
+  const int64_t pos = min(positions[t], max_position - 1);
+  const float* ct = cos_t + pos * half;
+  const float* st = sin_t + pos * half;
+  // items: heads * hv pieces of the queries, then hv of the shared key part
+  for (int i = threadIdx.x - 32; i < (heads + 1) * hv; i += kLvThreads - 32) {
+    const int h = i / hv, j = (i - h * hv) * 8;
+    const bool key = h == heads;
+    const T* src = key ? d + rank : q + t * q_stride + static_cast<int64_t>(h) * (dim + rot_dim) + dim;
+    float u[8], v[8], c[8], s[8];
+    Vec<T, 8>::load(src + j, u);
+    Vec<T, 8>::load(src + j + half, v);
+    Vec<float, 8>::load(ct + j, c);
+    Vec<float, 8>::load(st + j, s);
+#pragma unroll
+    for (int e = 0; e < 8; ++e) {
+      const float a = u[e] * c[e] - v[e] * s[e];
+      v[e] = v[e] * c[e] + u[e] * s[e];
+      u[e] = a;
+    }
+    if (!key) {
+      T* dst = q + t * q_stride + static_cast<int64_t>(h) * (dim + rot_dim) + dim;
+      Vec<T, 8>::store(dst + j, u);
+      Vec<T, 8>::store(dst + j + half, v);
+    } else {
+      if (lo) { Vec<T, 8>::store(lo + rank + j, u); Vec<T, 8>::store(lo + rank + j + half, v); }
+      if (co) { Vec<T, 8>::store(co + rank + j, u); Vec<T, 8>::store(co + rank + j + half, v); }
+    }
+  }
+}
+
 constexpr int kLaThreads = 256;
 constexpr int kLaHeads = 4;    // heads per CTA
 constexpr int kLaKeys = 32;    // keys per tile
@@ -191,6 +269,16 @@ extern "C" int mv_latent_prep(void* q, int64_t q_stride, const void* down, int64
     return fail(MV_ERR_NULL, "latent_prep: null pointer");
   auto run = [&](auto tag) {
     using T = decltype(tag);
+    const int eb = sizeof(T);
+    if (rank % 8 == 0 && dim % 8 == 0 && rot_dim % 16 == 0 && rope_dims == rot_dim && vec8_ok(q, q_stride, eb) &&
+        vec8_ok(down, down_stride, eb) && aligned16(c_weight) && aligned16(cos_table) && aligned16(sin_table) &&
+        aligned16(latent_out) && aligned16(cache)) {
+      latent_prep_vec_kernel<T><<<static_cast<unsigned>(tokens), kLvThreads, 0, static_cast<cudaStream_t>(stream)>>>(
+          static_cast<T*>(q), q_stride, static_cast<const T*>(down), down_stride, static_cast<const T*>(c_weight),
+          positions, cos_table, sin_table, max_position, static_cast<T*>(latent_out), static_cast<T*>(cache),
+          slot_mapping, num_slots, heads, dim, rot_dim, rank, eps);
+      return check_launch("latent_prep");
+    }
     latent_prep_kernel<T><<<static_cast<unsigned>(tokens), kLpThreads, 0, static_cast<cudaStream_t>(stream)>>>(
         static_cast<T*>(q), q_stride, static_cast<const T*>(down), down_stride, static_cast<const T*>(c_weight),
         positions, cos_table, sin_table, max_position, static_cast<T*>(latent_out), static_cast<T*>(cache),

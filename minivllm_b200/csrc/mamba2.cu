@@ -54,7 +54,7 @@ conv_silu_kernel(T* __restrict__ out, const T* __restrict__ u, int64_t u_stride,
     float acc = b;
     for (int k = 0; k < taps; ++k)
       acc = fmaf(Elem<T>::to_f(wc[k]), conv_input(u, u_stride, first, j - hist + k, c, st, hist, channels), acc);
-    out[t * channels + c] = Elem<T>::from_f(silu_f(acc));
+    out[t * channels + c] = Elem<T>::from_f(silu_t<T>(acc));
   }
 }
 
@@ -76,7 +76,8 @@ conv_silu_vec_kernel(T* __restrict__ out, const T* __restrict__ u, int64_t u_str
     for (int k = 0; k < TAPS; ++k) wt[k][e] = Elem<T>::to_f(w[static_cast<int64_t>(c + e) * TAPS + k]);
   }
   const int64_t t0 = static_cast<int64_t>(blockIdx.y) * run, t1 = min(t0 + run, tokens);
-  int64_t end = -1;
+  int64_t end = -1, ahead = -1;
+  Raw8<T> raw[4];
   for (int64_t t = t0; t < t1; ++t) {
     if (t >= end) {                      // first token of this thread, or of a sequence: fetch what lies before it
       const int s = seq_of_token(cu, num_seqs, static_cast<int>(t));
@@ -97,6 +98,43 @@ conv_silu_vec_kernel(T* __restrict__ out, const T* __restrict__ u, int64_t u_str
         }
       }
     }
+    // four tokens at a time: their loads go out together, and the window needs no register moves
+    if (t + 4 <= min(end, t1)) {
+      float v[HIST + 4][8];
+      if (ahead != t) {
+#pragma unroll
+        for (int k = 0; k < 4; ++k) raw[k].load(u + (t + k) * u_stride + c);
+      }
+#pragma unroll
+      for (int k = 0; k < 4; ++k) raw[k].get(v[HIST + k]);
+      if (t + 8 <= min(end, t1)) {       // the next four are on their way while these are worked on
+        ahead = t + 4;
+#pragma unroll
+        for (int k = 0; k < 4; ++k) raw[k].load(u + (t + 4 + k) * u_stride + c);
+      }
+#pragma unroll
+      for (int k = 0; k < HIST; ++k)
+#pragma unroll
+        for (int e = 0; e < 8; ++e) v[k][e] = win[k][e];
+#pragma unroll
+      for (int n = 0; n < 4; ++n) {
+        float r[8];
+#pragma unroll
+        for (int e = 0; e < 8; ++e) {
+          float a = b[e];
+#pragma unroll
+          for (int k = 0; k < TAPS; ++k) a = fmaf(wt[k][e], v[n + k][e], a);
+          r[e] = silu_t<T>(a);
+        }
+        Vec<T, 8>::store(out + (t + n) * channels + c, r);
+      }
+#pragma unroll
+      for (int k = 0; k < HIST; ++k)
+#pragma unroll
+        for (int e = 0; e < 8; ++e) win[k][e] = v[4 + k][e];
+      t += 3;
+      continue;
+    }
     float v[8], r[8];
     Vec<T, 8>::load(u + t * u_stride + c, v);
 #pragma unroll
@@ -104,10 +142,10 @@ conv_silu_vec_kernel(T* __restrict__ out, const T* __restrict__ u, int64_t u_str
       float a = b[e];
 #pragma unroll
       for (int k = 0; k < HIST; ++k) a = fmaf(wt[k][e], win[k][e], a);
-      r[e] = silu_f(fmaf(wt[HIST][e], v[e], a));
+      r[e] = silu_t<T>(fmaf(wt[HIST][e], v[e], a));
 #pragma unroll
       for (int k = 0; k + 1 < HIST; ++k) win[k][e] = win[k + 1][e];
-      if (HIST > 0) win[HIST - 1][e] = v[e];
+      win[HIST - 1][e] = v[e];
     }
     Vec<T, 8>::store(out + t * channels + c, r);
   }
@@ -242,7 +280,7 @@ ssm_step_kernel(T* __restrict__ y, const T* __restrict__ u, int64_t u_stride, co
     if (st0 > 0)
       for (int k = 0; k < hist; ++k) a = fmaf(Elem<T>::to_f(wc[k]), Elem<T>::to_f(cs[static_cast<int64_t>(k) * channels + c]), a);
     a = fmaf(Elem<T>::to_f(wc[hist]), Elem<T>::to_f(u[s * u_stride + c]), a);
-    sm[i] = Elem<T>::to_f(Elem<T>::from_f(silu_f(a)));       // rounded as the prompt path stores it
+    sm[i] = Elem<T>::to_f(Elem<T>::from_f(silu_t<T>(a)));       // rounded as the prompt path stores it
   }
   const float d = softplus_f(Elem<T>::to_f(dt[s * dt_stride + h]) + Elem<T>::to_f(dt_bias[h]));
   const float decay = expf(-expf(Elem<T>::to_f(A_log[h])) * d);

@@ -3,9 +3,9 @@
 // One CTA walks the tokens of a (sequence, head, block of value columns) in chunks of 64, with the state S (N x P) as
 // fp32 accumulators in registers.  With c_t the running sum of the log decays inside the chunk:
 //   Y = exp(c_t) (C S_prev) + (M X) + D X,   M[t, j] = exp(c_t - c_j) dt_j (C_t . B_j) for j <= t
-//   S = exp(c_last) S_prev + (W B)^T X,       W_t = exp(c_last - c_t) dt_t
+//   S = exp(c_last) S_prev + B^T (W X),       W_t = exp(c_last - c_t) dt_t
 // C, B and X are the bf16 outputs of the convolution and enter the products as they are.  What the recurrence forms
-// itself (M, W B, S) is fp32 and enters a product as two bf16 terms, the value and its rounding residue, so that the
+// itself (M, W X, S) is fp32 and enters a product as two bf16 terms, the value and its rounding residue, so that the
 // products carry 16 bits of it and nothing of the state is rounded to bf16.
 // Two CTAs per SM: one computes while the other waits for its loads.
 //
@@ -21,7 +21,8 @@ constexpr int kCsThreads = 256, kCsQ = 64;
 template <int N, int PB> struct CsShape {
   static constexpr int kXs = PB + 8, kBs = (N > PB ? N : PB) + 8, kMs = kCsQ + 8;  // row strides, elements (Y passes through C)
   static constexpr int kX = kCsQ * kXs, kB = kCsQ * kBs, kS = N * kXs;
-  static constexpr int kM2 = 2 * kCsQ * kMs > kB ? 2 * kCsQ * kMs : kB;           // M (two terms), later the residue of W B
+  static constexpr int kM2 = 2 * kCsQ * kMs;                                      // M (two terms), later the residue of W X
+  static_assert(kM2 >= kX, "the residue of W X lies over M");
   static constexpr int kElems = kX + 2 * kB + kM2 + 2 * kS;
   static constexpr int kBytes = kElems * 2;
 };
@@ -114,6 +115,15 @@ __global__ void __launch_bounds__(kCsThreads, 2) ssm_chunk_kernel(const CsParams
       cp_async16(c_s + (t * Sh::kBs + c) * 2, src + p.groups * N, ok ? 16 : 0);
     }
     cp_async_commit();
+    {  // the next chunk's lines on their way to L2
+      const int t = tid >> 2, part = tid & 3;
+      if (t0 + kCsQ + t < n_tok) {
+        const __nv_bfloat16* row = p.xbc + (static_cast<int64_t>(first) + t0 + kCsQ + t) * p.xbc_stride;
+        const __nv_bfloat16* at = part == 0 ? row + h * p.P + p0 : row + inner + (part == 1 ? g : part == 2 ? p.groups + g : g) * N + (part == 3 ? N / 2 : 0);
+        asm volatile("prefetch.global.L2 [%0];" ::"l"(at));
+        if (part == 2 && N > 64) asm volatile("prefetch.global.L2 [%0];" ::"l"(at + N / 2));
+      }
+    }
     if (warp == 0) {       // dt and the running log2 decay; two tokens per lane
       float d[2], c[2];
 #pragma unroll
@@ -163,8 +173,8 @@ __global__ void __launch_bounds__(kCsThreads, 2) ssm_chunk_kernel(const CsParams
           for (int half = 0; half < 2; ++half) {
             const int row = ym * 16 + r8 + half * 8;
             const float ct = half ? ct1 : ct0;
-            const float m0 = col <= row ? G[j][half * 2] * exp2f(ct - cj0) * d0 : 0.f;
-            const float m1 = col + 1 <= row ? G[j][half * 2 + 1] * exp2f(ct - cj1) * d1 : 0.f;
+            const float m0 = col <= row ? G[j][half * 2] * fast_exp2(ct - cj0) * d0 : 0.f;
+            const float m1 = col + 1 <= row ? G[j][half * 2 + 1] * fast_exp2(ct - cj1) * d1 : 0.f;
             uint32_t hi, lo;
             split2(m0, m1, hi, lo);
             *reinterpret_cast<uint32_t*>(sM + row * Sh::kMs + col) = hi;
@@ -193,7 +203,7 @@ __global__ void __launch_bounds__(kCsThreads, 2) ssm_chunk_kernel(const CsParams
             Mma::run(acc[i + 1], a, b[2], b[3]);
           }
       }
-      const float e0 = exp2f(ct0), e1 = exp2f(ct1);
+      const float e0 = fast_exp2(ct0), e1 = fast_exp2(ct1);
 #pragma unroll
       for (int i = 0; i < YN; ++i) {
         acc[i][0] *= e0; acc[i][1] *= e0; acc[i][2] *= e1; acc[i][3] *= e1;
@@ -229,18 +239,18 @@ __global__ void __launch_bounds__(kCsThreads, 2) ssm_chunk_kernel(const CsParams
     }
     __syncthreads();                       // M has been read, Y is complete
     const float cl = s_c[kCsQ - 1];
-    for (int i = tid; i < kCsQ * (N / 8); i += kCsThreads) {    // W B in two terms: the value in place, the residue over M
-      const int t = i / (N / 8), c = (i % (N / 8)) * 8;
-      const float w = exp2f(cl - s_c[t]) * s_dt[t];
+    for (int i = tid; i < kCsQ * (PB / 8); i += kCsThreads) {    // W X in two terms: the value in place, the residue over M
+      const int t = i / (PB / 8), c = (i % (PB / 8)) * 8;
+      const float w = fast_exp2(cl - s_c[t]) * s_dt[t];
       float v[8], lo[8];
-      Vec<__nv_bfloat16, 8>::load(sB + t * Sh::kBs + c, v);
+      Vec<__nv_bfloat16, 8>::load(sX + t * Sh::kXs + c, v);
 #pragma unroll
       for (int e = 0; e < 8; ++e) {
         v[e] *= w;
         lo[e] = v[e] - __bfloat162float(__float2bfloat16_rn(v[e]));
       }
-      Vec<__nv_bfloat16, 8>::store(sB + t * Sh::kBs + c, v);
-      Vec<__nv_bfloat16, 8>::store(sM + t * Sh::kBs + c, lo);
+      Vec<__nv_bfloat16, 8>::store(sX + t * Sh::kXs + c, v);
+      Vec<__nv_bfloat16, 8>::store(sM + t * Sh::kXs + c, lo);
     }
     for (int i = tid; i < nt * (PB / 8); i += kCsThreads) {
       const int t = i / (PB / 8), c = (i % (PB / 8)) * 8;
@@ -250,31 +260,31 @@ __global__ void __launch_bounds__(kCsThreads, 2) ssm_chunk_kernel(const CsParams
     }
     __syncthreads();
     {  // S = exp(c_last) S + (W B)^T X
-      const float e = exp2f(cl);
+      const float e = fast_exp2(cl);
 #pragma unroll
       for (int a = 0; a < MPW; ++a)
 #pragma unroll
         for (int b = 0; b < SN; ++b)
 #pragma unroll
           for (int q = 0; q < 4; ++q) S[a][b][q] *= e;
-      const uint32_t xa = x_s + ((l7 + l8 * 8) * Sh::kXs + sn0 * 8 + l16 * 8) * 2;
+      const uint32_t xo = ((l7 + l8 * 8) * Sh::kXs + sn0 * 8 + l16 * 8) * 2;
 #pragma unroll
       for (int k = 0; k < kCsQ; k += 16) {
+        uint32_t bt[MPW][4];
 #pragma unroll
-        for (int a = 0; a < MPW; ++a) {
-          const uint32_t at = ((k + l7 + l16 * 8) * Sh::kBs + (sm0 + a) * 16 + l8 * 8) * 2;
-          uint32_t hi[4], lo[4], b[4];
-          ldmatrix_x4_trans(hi, b_s + at);
-          ldmatrix_x4_trans(lo, m_s + at);
+        for (int a = 0; a < MPW; ++a)
+          ldmatrix_x4_trans(bt[a], b_s + ((k + l7 + l16 * 8) * Sh::kBs + (sm0 + a) * 16 + l8 * 8) * 2);
 #pragma unroll
-          for (int i = 0; i < SN; i += 2) {
-            ldmatrix_x4_trans(b, xa + (k * Sh::kXs + i * 8) * 2);
-            Mma::run(S[a][i], hi, b[0], b[1]);
-            Mma::run(S[a][i], lo, b[0], b[1]);
-            if (i + 1 < SN) {
-              Mma::run(S[a][i + 1 < SN ? i + 1 : i], hi, b[2], b[3]);
-              Mma::run(S[a][i + 1 < SN ? i + 1 : i], lo, b[2], b[3]);
-            }
+        for (int i = 0; i < SN; i += 2) {
+          uint32_t hi[4], lo[4];
+          ldmatrix_x4_trans(hi, x_s + xo + (k * Sh::kXs + i * 8) * 2);
+          ldmatrix_x4_trans(lo, m_s + xo + (k * Sh::kXs + i * 8) * 2);
+#pragma unroll
+          for (int a = 0; a < MPW; ++a) {
+            Mma::run(S[a][i], bt[a], hi[0], hi[1]);
+            if (i + 1 < SN) Mma::run(S[a][i + 1 < SN ? i + 1 : i], bt[a], hi[2], hi[3]);
+            Mma::run(S[a][i], bt[a], lo[0], lo[1]);
+            if (i + 1 < SN) Mma::run(S[a][i + 1 < SN ? i + 1 : i], bt[a], lo[2], lo[3]);
           }
         }
       }

@@ -13,15 +13,17 @@ constexpr int kRtThreads = 256;
 constexpr int kRtMaxPer = 32;      // experts per lane: up to 1024 experts
 
 // One warp per token: the `top` largest logits (ties: lower index) and the softmax over them.
+// kPer: experts per lane.
+template <int kPer>
 __global__ void __launch_bounds__(kRtThreads)
 moe_route_kernel(int32_t* __restrict__ idx, float* __restrict__ weight, const float* __restrict__ logits,
                  int64_t stride, const float* __restrict__ bias, int64_t tokens, int experts, int top) {
   const int lane = threadIdx.x & 31;
   const int64_t t = static_cast<int64_t>(blockIdx.x) * (kRtThreads / 32) + (threadIdx.x >> 5);
   if (t >= tokens) return;
-  float z[kRtMaxPer];
+  float z[kPer];
 #pragma unroll
-  for (int i = 0; i < kRtMaxPer; ++i) {
+  for (int i = 0; i < kPer; ++i) {
     const int e = i * 32 + lane;
     z[i] = e < experts ? logits[t * stride + e] + (bias ? bias[e] : 0.f) : -INFINITY;
   }
@@ -31,7 +33,7 @@ moe_route_kernel(int32_t* __restrict__ idx, float* __restrict__ weight, const fl
     float best = -INFINITY;
     int at = 0x7fffffff;
 #pragma unroll
-    for (int i = 0; i < kRtMaxPer; ++i) {
+    for (int i = 0; i < kPer; ++i) {
       const int e = i * 32 + lane;
       if (e < experts && !((taken >> i) & 1u) && (z[i] > best || at == 0x7fffffff)) { best = z[i]; at = e; }
     }
@@ -68,29 +70,44 @@ moe_count_kernel(int32_t* __restrict__ hist, const int32_t* __restrict__ idx, in
 }
 
 // One CTA: hist[b][e] becomes the first row of block b's entries of expert e; offsets[e] the expert's first row.
+// The 1,024 threads are `ep` experts (a power of two) times 1,024 / ep runs of blocks.
 __global__ void __launch_bounds__(1024)
-moe_scan_kernel(int32_t* __restrict__ hist, int32_t* __restrict__ offsets, int blocks, int experts) {
-  __shared__ int s_tot[1024];
-  const int tid = threadIdx.x;
-  int total = 0;
-  if (tid < experts) {
-#pragma unroll 4
-    for (int b = 0; b < blocks; ++b) total += hist[static_cast<int64_t>(b) * experts + tid];
+moe_scan_kernel(int32_t* __restrict__ hist, int32_t* __restrict__ offsets, int blocks, int experts, int ep) {
+  __shared__ int s_run[1024], s_tot[1024];
+  const int tid = threadIdx.x, e = tid & (ep - 1), seg = tid / ep, segs = 1024 / ep;
+  const int per = (blocks + segs - 1) / segs, b0 = min(seg * per, blocks), b1 = min(b0 + per, blocks);
+  int sum = 0;
+  if (e < experts) {
+#pragma unroll 8
+    for (int b = b0; b < b1; ++b) sum += hist[static_cast<int64_t>(b) * experts + e];
   }
-  s_tot[tid] = total;
+  s_run[tid] = sum;
+  s_tot[tid] = 0;
   __syncthreads();
-  for (int o = 1; o < 1024; o <<= 1) {
+  if (seg == 0) {
+    int total = 0;
+    for (int k = 0; k < segs; ++k) {
+      const int v = s_run[k * ep + e];
+      s_run[k * ep + e] = total;       // entries of the runs before
+      total += v;
+    }
+    s_tot[e] = total;
+  }
+  __syncthreads();
+  const int mine = s_tot[tid];
+  for (int o = 1; o < ep; o <<= 1) {
     const int v = tid >= o ? s_tot[tid - o] : 0;
     __syncthreads();
     s_tot[tid] += v;
     __syncthreads();
   }
-  if (tid >= experts) return;
-  int run = s_tot[tid] - total;
-  offsets[tid] = run;
+  if (tid < experts) offsets[tid] = s_tot[tid] - mine;
   if (tid == experts - 1) offsets[experts] = s_tot[tid];
-  for (int b = 0; b < blocks; ++b) {
-    const int64_t a = static_cast<int64_t>(b) * experts + tid;
+  if (e >= experts) return;
+  int run = (e ? s_tot[e - 1] : 0) + s_run[tid];
+#pragma unroll 4
+  for (int b = b0; b < b1; ++b) {
+    const int64_t a = static_cast<int64_t>(b) * experts + e;
     const int n = hist[a];
     hist[a] = run;
     run += n;
@@ -250,7 +267,12 @@ extern "C" int mv_moe_route(int32_t* idx, float* weight, const float* logits, in
   if (tokens == 0) return MV_OK;
   if (!idx || !weight || !logits) return fail(MV_ERR_NULL, "moe_route: null pointer");
   const unsigned grid = static_cast<unsigned>((tokens + kRtThreads / 32 - 1) / (kRtThreads / 32));
-  moe_route_kernel<<<grid, kRtThreads, 0, static_cast<cudaStream_t>(stream)>>>(idx, weight, logits, logits_stride, bias, tokens, experts, top);
+  auto go = [&](auto kernel) {
+    kernel<<<grid, kRtThreads, 0, static_cast<cudaStream_t>(stream)>>>(idx, weight, logits, logits_stride, bias, tokens, experts, top);
+  };
+  if (experts <= 64) go(moe_route_kernel<2>);
+  else if (experts <= 256) go(moe_route_kernel<8>);
+  else go(moe_route_kernel<kRtMaxPer>);
   return check_launch("moe_route");
 }
 
@@ -277,7 +299,9 @@ extern "C" int mv_moe_sort(int32_t* pos, int32_t* row_token, int32_t* offsets, c
   if (!workspace || workspace_bytes < static_cast<int64_t>(blocks) * experts * 4) return fail(MV_ERR_WORKSPACE, "moe_sort: workspace");
   auto* hist = static_cast<int32_t*>(workspace);
   moe_count_kernel<<<blocks, kSortThreads, experts * sizeof(int), st>>>(hist, idx, entries, experts);
-  moe_scan_kernel<<<1, 1024, 0, st>>>(hist, offsets, blocks, experts);
+  int ep = 1;
+  while (ep < experts) ep *= 2;
+  moe_scan_kernel<<<1, 1024, 0, st>>>(hist, offsets, blocks, experts, ep);
   moe_place_kernel<<<blocks, kSortThreads, 0, st>>>(pos, row_token, hist, idx, entries, experts, top);
   return check_launch("moe_sort");
 }

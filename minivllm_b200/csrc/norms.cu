@@ -12,6 +12,7 @@ namespace mv {
 
 constexpr int kNormThreads = 256;
 constexpr int kNormWarps = kNormThreads / 32;
+constexpr int kMaxTop = 256;     // choices per token
 
 enum { SRC_EMBED = 0, SRC_ROWS = 1, SRC_EXPERTS = 2 };
 
@@ -64,6 +65,15 @@ __global__ void __launch_bounds__(kNormThreads) residual_norm_kernel(const Resid
     token = p.ids[row];
     if (token < 0 || token >= p.vocab) token = 0;   // placeholder rows of a padded batch
   }
+  __shared__ int s_pos[SRC == SRC_EXPERTS ? kMaxTop : 1];
+  __shared__ float s_w[SRC == SRC_EXPERTS ? kMaxTop : 1];
+  if (SRC == SRC_EXPERTS) {
+    for (int k = threadIdx.x; k < p.top; k += kNormThreads) {
+      s_pos[k] = p.pos[row * p.top + k];
+      s_w[k] = p.topw[row * p.top + k];
+    }
+    __syncthreads();
+  }
   if (SRC == SRC_EXPERTS && p.shared) sgate = p.sg ? sigmoid_f(Elem<T>::to_f(p.sg[row * p.sg_stride])) : 1.f;
 
   for (int g = gp.g0; g < p.groups; g += gp.cg) {
@@ -80,12 +90,18 @@ __global__ void __launch_bounds__(kNormThreads) residual_norm_kernel(const Resid
         } else {
 #pragma unroll
           for (int e = 0; e < V; ++e) v[e] = 0.f;
-          for (int k = 0; k < p.top; ++k) {
-            const float w = p.topw[row * p.top + k];
-            float t[V];
-            Vec<T, V>::load(p.y + static_cast<int64_t>(p.pos[row * p.top + k]) * p.y_stride + c, t);
+          constexpr int kAtOnce = 4;
+          for (int k0 = 0; k0 < p.top; k0 += kAtOnce) {
+            float t[kAtOnce][V];
 #pragma unroll
-            for (int e = 0; e < V; ++e) v[e] = fmaf(w, t[e], v[e]);
+            for (int k = 0; k < kAtOnce; ++k)
+              if (k0 + k < p.top) Vec<T, V>::load(p.y + static_cast<int64_t>(s_pos[k0 + k]) * p.y_stride + c, t[k]);
+#pragma unroll
+            for (int k = 0; k < kAtOnce; ++k)
+              if (k0 + k < p.top) {
+#pragma unroll
+                for (int e = 0; e < V; ++e) v[e] = fmaf(s_w[k0 + k], t[k][e], v[e]);
+              }
           }
           if (p.shared) {
             float t[V];
@@ -99,7 +115,7 @@ __global__ void __launch_bounds__(kNormThreads) residual_norm_kernel(const Resid
           Vec<T, V>::load(p.gate + row * p.gate_stride + c, t);
           Vec<T, V>::load(p.gate_bias + c, b);
 #pragma unroll
-          for (int e = 0; e < V; ++e) v[e] *= sigmoid_f(t[e] + b[e]);
+          for (int e = 0; e < V; ++e) v[e] *= sigmoid_t<T>(t[e] + b[e]);
         }
       }
 #pragma unroll
@@ -149,6 +165,145 @@ __global__ void __launch_bounds__(kNormThreads) residual_norm_kernel(const Resid
   }
 }
 
+// The same with the row in registers: at most eight groups, kCh pieces of eight channels per thread.  Everything a row
+// needs is requested at once; two block-wide sums follow.
+template <typename T, int SRC, int kCh>
+__global__ void __launch_bounds__(kNormThreads, SRC == SRC_EXPERTS ? (kCh == 1 ? 3 : 2) : 3) residual_norm_reg_kernel(const ResidualParams<T> p) {
+  __shared__ float part[kNormWarps], part2[kNormWarps];
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+  const int64_t row = blockIdx.x;
+  const GroupPlan gp(p.width, p.groups, 8, warp);
+  const bool on = gp.g0 < p.groups;
+  float* x = p.x + row * p.width;
+  int col[kCh];
+  bool has[kCh];
+#pragma unroll
+  for (int k = 0; k < kCh; ++k) {
+    const int i = gp.sub * 32 + lane + k * gp.wpg * 32;
+    has[k] = on && i < gp.chunks;
+    col[k] = gp.g0 * gp.gs + i * 8;
+  }
+  float v[kCh][8], r[kCh][8];
+  Raw8<T> gate[kCh], gb[kCh], wp[kCh], wn[kCh];
+  int64_t token = 0;
+  float sgate = 0.f;
+  if (SRC == SRC_EMBED) {
+    token = p.ids[row];
+    if (token < 0 || token >= p.vocab) token = 0;
+  }
+  if (SRC == SRC_EXPERTS && p.shared) sgate = p.sg ? sigmoid_f(Elem<T>::to_f(p.sg[row * p.sg_stride])) : 1.f;
+#pragma unroll
+  for (int k = 0; k < kCh; ++k)
+    if (has[k]) {
+      wn[k].load(p.w_next + col[k]);
+      if (SRC != SRC_EMBED) {
+        Vec<float, 8>::load(x + col[k], r[k]);
+        wp[k].load(p.w_post + col[k]);
+        if (p.gate) {
+          gate[k].load(p.gate + row * p.gate_stride + col[k]);
+          gb[k].load(p.gate_bias + col[k]);
+        }
+      }
+    }
+  if (SRC == SRC_EXPERTS) {
+    Raw8<T> sh[kCh];
+#pragma unroll
+    for (int k = 0; k < kCh; ++k) {
+      if (has[k] && p.shared) sh[k].load(p.shared + row * p.shared_stride + col[k]);
+#pragma unroll
+      for (int e = 0; e < 8; ++e) v[k][e] = 0.f;
+    }
+    constexpr int kAtOnce = kCh == 1 ? 6 : 4;
+    for (int k0 = 0; k0 < p.top; k0 += kAtOnce) {
+      int64_t at[kAtOnce];
+      float w[kAtOnce];
+#pragma unroll
+      for (int j = 0; j < kAtOnce; ++j) {
+        const bool ok = k0 + j < p.top;
+        at[j] = ok ? static_cast<int64_t>(p.pos[row * p.top + k0 + j]) * p.y_stride : 0;
+        w[j] = ok ? p.topw[row * p.top + k0 + j] : 0.f;
+      }
+#pragma unroll
+      for (int k = 0; k < kCh; ++k)
+        if (has[k]) {
+          Raw8<T> t[kAtOnce];
+#pragma unroll
+          for (int j = 0; j < kAtOnce; ++j)
+            if (k0 + j < p.top) t[j].load(p.y + at[j] + col[k]);
+#pragma unroll
+          for (int j = 0; j < kAtOnce; ++j)
+            if (k0 + j < p.top) {
+              float f[8];
+              t[j].get(f);
+#pragma unroll
+              for (int e = 0; e < 8; ++e) v[k][e] = fmaf(w[j], f[e], v[k][e]);
+            }
+        }
+    }
+#pragma unroll
+    for (int k = 0; k < kCh; ++k)
+      if (has[k] && p.shared) {
+        float f[8];
+        sh[k].get(f);
+#pragma unroll
+        for (int e = 0; e < 8; ++e) v[k][e] = fmaf(sgate, f[e], v[k][e]);
+      }
+  } else {
+#pragma unroll
+    for (int k = 0; k < kCh; ++k)
+      if (has[k]) Vec<T, 8>::load(SRC == SRC_EMBED ? p.embed + token * p.width + col[k] : p.y + row * p.y_stride + col[k], v[k]);
+  }
+  float acc = 0.f;
+#pragma unroll
+  for (int k = 0; k < kCh; ++k)
+    if (has[k]) {
+      if (SRC == SRC_EMBED) Vec<float, 8>::store(x + col[k], v[k]);
+      if (SRC != SRC_EMBED && p.gate) {
+        float t[8], b[8];
+        gate[k].get(t);
+        gb[k].get(b);
+#pragma unroll
+        for (int e = 0; e < 8; ++e) v[k][e] *= sigmoid_t<T>(t[e] + b[e]);
+      }
+#pragma unroll
+      for (int e = 0; e < 8; ++e) acc = fmaf(v[k][e], v[k][e], acc);
+    }
+  acc = warp_sum(acc);
+  if (lane == 0) part[warp] = acc;
+  __syncthreads();
+  const float* fin = part;
+  if (SRC != SRC_EMBED) {
+    const float rs = on ? group_rs(part, gp.g0, gp.wpg, gp.gs, p.eps) : 0.f;
+    acc = 0.f;
+#pragma unroll
+    for (int k = 0; k < kCh; ++k)
+      if (has[k]) {
+        float w[8];
+        wp[k].get(w);
+#pragma unroll
+        for (int e = 0; e < 8; ++e) {
+          v[k][e] = fmaf(p.mult, v[k][e] * rs * w[e], r[k][e]);
+          acc = fmaf(v[k][e], v[k][e], acc);
+        }
+        Vec<float, 8>::store(x + col[k], v[k]);
+      }
+    acc = warp_sum(acc);
+    if (lane == 0) part2[warp] = acc;
+    __syncthreads();
+    fin = part2;
+  }
+  const float rs = on ? group_rs(fin, gp.g0, gp.wpg, gp.gs, p.eps) : 0.f;
+#pragma unroll
+  for (int k = 0; k < kCh; ++k)
+    if (has[k]) {
+      float w[8];
+      wn[k].get(w);
+#pragma unroll
+      for (int e = 0; e < 8; ++e) v[k][e] = v[k][e] * rs * w[e];
+      Vec<T, 8>::store(p.out + row * p.width + col[k], v[k]);
+    }
+}
+
 // out = group_rms_norm(y * silu(z)) * w
 template <typename T, int V>
 __global__ void __launch_bounds__(kNormThreads)
@@ -168,7 +323,7 @@ gated_group_norm_kernel(T* __restrict__ out, const T* __restrict__ y, int64_t y_
       Vec<T, V>::load(z + row * z_stride + c, t);
 #pragma unroll
       for (int e = 0; e < V; ++e) {
-        v[e] *= silu_f(t[e]);
+        v[e] *= silu_t<T>(t[e]);
         acc = fmaf(v[e], v[e], acc);
       }
       Vec<float, V>::store(s_row + c, v);
@@ -206,7 +361,7 @@ gate_mul_kernel(T* __restrict__ out, const T* __restrict__ y, int64_t y_stride, 
     Vec<T, V>::load(y + row * y_stride + h * y_head_stride + (c - h * head_cols), v);
     Vec<T, V>::load(gate + row * gate_stride + c, g);
 #pragma unroll
-    for (int e = 0; e < V; ++e) v[e] *= act ? silu_f(g[e]) : sigmoid_f(g[e]);
+    for (int e = 0; e < V; ++e) v[e] *= act ? silu_t<T>(g[e]) : sigmoid_t<T>(g[e]);
     Vec<T, V>::store(out + row * cols + c, v);
   }
 }
@@ -237,6 +392,14 @@ static int launch_residual_v(const ResidualParams<T>& p, int64_t rows, cudaStrea
   bool v8 = (p.width / p.groups) % 8 == 0 && aligned16(p.out) && aligned16(p.x) && aligned16(p.w_next) &&
             vec8_ok(p.y, p.y_stride, eb) && vec8_ok(p.gate, p.gate_stride, eb) && vec8_ok(p.gate_bias, 0, eb) &&
             vec8_ok(p.w_post, 0, eb) && vec8_ok(p.embed, p.width, eb) && vec8_ok(p.shared, p.shared_stride, eb);
+  if (v8 && p.groups <= kNormWarps) {
+    const int lanes = kNormWarps / p.groups * 32, per = (p.width / p.groups / 8 + lanes - 1) / lanes;
+    if (per <= 2) {
+      if (per == 1) residual_norm_reg_kernel<T, SRC, 1><<<static_cast<unsigned>(rows), kNormThreads, 0, st>>>(p);
+      else residual_norm_reg_kernel<T, SRC, 2><<<static_cast<unsigned>(rows), kNormThreads, 0, st>>>(p);
+      return check_launch("residual_norm");
+    }
+  }
   return v8 ? launch_residual<T, 8, SRC>(p, rows, st) : launch_residual<T, 1, SRC>(p, rows, st);
 }
 static int check_norm(const char* what, int width, int groups, int dtype) {
@@ -296,7 +459,7 @@ extern "C" int mv_moe_residual_norm(void* out, float* x, const void* expert_rows
   if (rc || rows == 0) return rc;
   if (!out || !x || !expert_rows || !pos || !top_weights || !w_post || !w_next || (gate && !gate_bias))
     return fail(MV_ERR_NULL, "moe_residual_norm: null pointer");
-  if (top <= 0) return fail(MV_ERR_SHAPE, "moe_residual_norm: top %d", top);
+  if (top <= 0 || top > kMaxTop) return fail(MV_ERR_SHAPE, "moe_residual_norm: top %d", top);
   auto run = [&](auto tag) {
     using T = decltype(tag);
     ResidualParams<T> p{};

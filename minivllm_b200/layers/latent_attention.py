@@ -80,7 +80,7 @@ def latent_decode(q_lat, q_rot, cache, block_tables, positions, sink, scale, wor
         q_rot.data_ptr(), q_rot.stride(0), q_rot.stride(1), cache.data_ptr(), block_tables.data_ptr(),
         block_tables.stride(0), block_tables.shape[1], cache.shape[1], cache.shape[0], positions.data_ptr(), None,
         sink.data_ptr() if sink is not None else None, batch, heads, rank, rot, scale, workspace.data_ptr(),
-        workspace.numel(), _cabi.stream_ptr()))
+        workspace.numel(), _error_word(q_lat.device).data_ptr(), _cabi.stream_ptr()))
     return out
 
 
