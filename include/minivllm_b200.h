@@ -512,8 +512,8 @@ int mv_grouped_gemm(void* out, const void* x, const void* w, const int32_t* offs
 
 /*
  * mv_latent_attention_rows for one query row per sequence on tensor cores, bf16: rank a multiple of 16 up to 512,
- * rank + rot_dim a multiple of 32 up to 576, at most 1,024 rows (workspace_bytes returns -1 otherwise).  Bounded waits
- * report in *error_word.  Sequence b has
+ * rank + rot_dim a multiple of 32 up to 576, at most 1,024 rows (workspace_bytes returns -1 otherwise), blocks of 8, 16,
+ * 32 or a multiple of 64 tokens.  Cache rows must hold finite values.  Bounded waits report in *error_word.  Sequence b has
  * positions[b] + 1 keys; rows with active[b] < 0 (active may be null) have none and give zeros.
  */
 int64_t mv_latent_decode_workspace_bytes(int batch, int heads, int rank, int rot_dim);

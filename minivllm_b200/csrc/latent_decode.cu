@@ -5,8 +5,8 @@
 // The batch's 64-key tiles form one stream that is cut into equal ranges, one per persistent CTA (the grid depends on
 // shapes only; the cut on the device-side lengths).  A CTA's range may end or begin inside a sequence: those pieces go
 // to the workspace as (m, l, unnormalised sum) and latent_combine_kernel joins them; whole sequences are written
-// directly.  Rows arrive by bulk copies (one per row, issued by one warp, two tiles in flight across sequence borders)
-// in shared-memory rows padded by 16 bytes, so that ldmatrix meets no bank conflicts.  16 heads per CTA are the 16 rows
+// directly.  Tiles arrive by TMA as 64-column boxes with the 128-byte swizzle (no bank conflicts under ldmatrix), two in
+// flight across sequence borders; block table entries are read one tile ahead of their use.  16 heads per CTA are the 16 rows
 // of m16n8k16 MMAs (the kernel is HBM-bound, and mma.sync needs no wider tile).  16 warps: for the scores, eight key
 // groups times two halves of the row, the query fragments of its half in registers; one softmax row per warp, fp32;
 // for the sum, 16-column units of c.  The weights enter the product as two bf16 terms (value and rounding residue).
@@ -16,6 +16,7 @@
 #include <algorithm>
 #include "mma.cuh"
 #include "tcgen05.cuh"
+#include "tmap.cuh"
 #include "vec.cuh"
 
 namespace mv {
@@ -24,6 +25,8 @@ constexpr int kLdThreads = 512, kLdWarps = 16;
 constexpr int kLdKeys = 64, kLdHeads = 16;
 constexpr int kLdMaxSeqs = 1024, kLdMaxRank = 512, kLdMaxRow = 576;
 constexpr int kLdUnits = kLdMaxRank / 16 / kLdWarps;   // 16-column units of the sum per warp
+constexpr int kLdBox = kLdKeys * 128;       // bytes of a 64-key, 64-column box
+constexpr int kLdAhead = 128;                // tiles whose cache rows are known ahead
 constexpr int kLdSStride = kLdKeys + 4;    // floats per score row
 constexpr int kLdPStride = kLdKeys + 8;    // bf16 per weight row
 
@@ -31,7 +34,7 @@ struct LdParams {
   __nv_bfloat16* out; int64_t out_stride, out_head_stride;
   const __nv_bfloat16* q_lat; int64_t q_lat_stride, q_lat_head_stride;
   const __nv_bfloat16* q_rot; int64_t q_rot_stride, q_rot_head_stride;
-  const __nv_bfloat16* cache;
+  int box_rows;                  // rows of one TMA box: 64, or the block size when that is smaller
   const int32_t* tables; int64_t bt_stride; int max_blocks, block_size; int64_t num_blocks;
   const int64_t* positions;      // keys of sequence b: positions[b] + 1
   const int32_t* active;         // null, or per sequence < 0: a padding row without keys
@@ -74,18 +77,19 @@ __device__ __forceinline__ int ld_cut(int total, int c, int ctas) { return stati
 
 // kHalf: 32-column steps of a score half row that the query fragments have registers for.
 template <int kHalf>
-__global__ void __launch_bounds__(kLdThreads, 1) latent_decode_kernel(const LdParams p) {
-  extern __shared__ __align__(128) unsigned char raw[];
+__global__ void __launch_bounds__(kLdThreads, 1) latent_decode_kernel(const __grid_constant__ CUtensorMap tmap, const LdParams p) {
+  extern __shared__ unsigned char raw[];
   __shared__ int s_start[kLdMaxSeqs + 1], s_keys[kLdMaxSeqs];
   __shared__ float s_m[kLdHeads], s_l[kLdHeads], s_c[kLdHeads];
   __shared__ __align__(8) uint64_t s_bar[2];
-  __shared__ int s_abort;
+  __shared__ int s_abort, s_row[kLdAhead][8];
   const int R = p.rank + p.rot_dim, row_bytes = R * 2 + 16;
-  unsigned char* kv = raw;                                   // [2][64][row_bytes]
-  unsigned char* sq = kv + 2 * kLdKeys * row_bytes;          // [16][row_bytes]
+  const int boxes = (R + 63) / 64;
+  const uint32_t kv_s = (smem_u32(raw) + 1023u) & ~1023u;    // [2][box][64][128B], swizzled
+  unsigned char* sq = raw + (kv_s - smem_u32(raw)) + 2 * boxes * kLdBox;   // [16][row_bytes]
   float* ss = reinterpret_cast<float*>(sq + kLdHeads * row_bytes);                       // [2 halves][16][kLdSStride]
   __nv_bfloat16* sp = reinterpret_cast<__nv_bfloat16*>(ss + 2 * kLdHeads * kLdSStride);  // [2 terms][16][kLdPStride]
-  const uint32_t kv_s = smem_u32(kv), q_s = smem_u32(sq), p_s = smem_u32(sp), bar0 = smem_u32(s_bar);
+  const uint32_t q_s = smem_u32(sq), p_s = smem_u32(sp), bar0 = smem_u32(s_bar);
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const int h0 = blockIdx.y * kLdHeads, nh = min(kLdHeads, p.heads - h0);
   if (tid == 0) {
@@ -98,70 +102,49 @@ __global__ void __launch_bounds__(kLdThreads, 1) latent_decode_kernel(const LdPa
   const int total = s_abort ? 0 : s_start[p.batch], ctas = gridDim.x, c = blockIdx.x;
   const int g0 = ld_cut(total, c, ctas), g1 = ld_cut(total, c + 1, ctas);
   if (g0 >= g1) return;
-  const int start_b = [&] {     // the sequence of tile g0: the last b with s_start[b] <= g0
+  // Cache rows of the tiles ahead, looked up by all threads for 64 tiles at a time (a lookup in the block table takes
+  // as long as a tile's scores).  A missing block is a row outside the tensor and reads as zeros.
+  const int groups = kLdKeys / p.box_rows;        // boxes of rows per tile
+  auto find = [&](int g) {      // the sequence of tile g: the last b with s_start[b] <= g
     int lo = 0, hi = p.batch - 1;
     while (lo < hi) {
       const int mid = (lo + hi + 1) >> 1;
-      if (s_start[mid] <= g0) lo = mid; else hi = mid - 1;
+      if (s_start[mid] <= g) lo = mid; else hi = mid - 1;
     }
     return lo;
-  }();
-  int load_b = start_b;
-  int32_t phys[2] = {-1, -1};      // blocks of this lane's rows of the tile that is copied next: read one tile ahead
-  int off[2] = {0, 0};
-  auto look = [&](int g) {
-    if (g >= g1) return;
-    while (g >= s_start[load_b + 1]) ++load_b;
-    const int n = s_keys[load_b];
-    const int32_t* table = p.tables + static_cast<int64_t>(load_b) * p.bt_stride;
-#pragma unroll
-    for (int i = 0; i < 2; ++i) {
-      const int pos = (g - s_start[load_b]) * kLdKeys + i * 32 + lane, blk = pos / p.block_size;
-      off[i] = pos - blk * p.block_size;
-      phys[i] = pos < n ? table[blk] : -1;
+  };
+  auto look = [&](int first, int tiles) {
+    for (int i = tid; i < tiles * groups; i += kLdThreads) {
+      const int g = first + i / groups, r = i % groups;
+      if (g >= g1) break;
+      const int sb = find(g), pos = (g - s_start[sb]) * kLdKeys + r * p.box_rows, blk = pos / p.block_size;
+      const int32_t phys = pos < s_keys[sb] ? p.tables[static_cast<int64_t>(sb) * p.bt_stride + blk] : -1;
+      s_row[(g - g0) % kLdAhead][r] = phys >= 0 && phys < p.num_blocks ? phys * p.block_size + (pos - blk * p.block_size)
+                                                                      : static_cast<int>(p.num_blocks) * p.block_size;
     }
   };
-  // Warp 0: two rows per lane.  A row without a key is not copied; its score is masked, and its weight of zero must
-  // meet finite numbers, so it is cleared.
+  // Warp x copies box x of a tile: nine copies issued by one thread would take longer than the tile's products.
   auto load = [&](int g, int buf) {
-    if (g >= g1) return;
-    const __nv_bfloat16* src[2];
-    int rows = 0;
-#pragma unroll
-    for (int i = 0; i < 2; ++i) {
-      src[i] = phys[i] >= 0 && phys[i] < p.num_blocks ? p.cache + (static_cast<int64_t>(phys[i]) * p.block_size + off[i]) * R : nullptr;
-      rows += src[i] != nullptr;
-    }
-    look(g + 1);
-#pragma unroll
-    for (int o = 16; o; o >>= 1) rows += __shfl_xor_sync(0xffffffffu, rows, o);
-#pragma unroll
-    for (int i = 0; i < 2; ++i)
-      if (!src[i]) {
-        uint4* z = reinterpret_cast<uint4*>(kv + (buf * kLdKeys + i * 32 + lane) * row_bytes);
-        for (int k = 0; k < R / 8; ++k) z[k] = make_uint4(0, 0, 0, 0);
-      }
-    if (rows < kLdKeys) asm volatile("fence.proxy.async.shared::cta;" ::: "memory");   // cleared rows, before later copies
-    if (lane == 0) tc::mbar_expect_tx(bar0 + 8 * buf, rows * R * 2);
-    __syncwarp();
-#pragma unroll
-    for (int i = 0; i < 2; ++i)
-      if (src[i])
-        asm volatile("cp.async.bulk.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1], %2, [%3];"
-                     ::"r"(kv_s + (buf * kLdKeys + i * 32 + lane) * row_bytes), "l"(src[i]), "r"(R * 2), "r"(bar0 + 8 * buf) : "memory");
+    if (g >= g1 || warp >= boxes) return;
+    if (tid == 0) tc::mbar_expect_tx(bar0 + 8 * buf, boxes * kLdBox);
+    if (lane < groups)
+      tc::tma_load_3d(kv_s + (buf * boxes + warp) * kLdBox + lane * p.box_rows * 128, &tmap, warp * 64,
+                      s_row[(g - g0) % kLdAhead][lane], 0, bar0 + 8 * buf);
   };
-  if (warp == 0) {
-    look(g0);
-    load(g0, 0);
-    load(g0 + 1, 1);
-  }
+  look(g0, kLdAhead);
+  __syncthreads();
+  load(g0, 0);
+  load(g0 + 1, 1);
 
   const int steps = R / 32, half = warp >> 3, kt = warp & 7;      // score role: key group kt, half of the row
   const int k_first = half ? (steps + 1) / 2 : 0, k_num = half ? steps / 2 : (steps + 1) / 2;
   const int units = p.rank / 16;
+  // The products below run without branches, so that loads and MMAs of several steps overlap: a step or unit that the
+  // sizes do not have works on zeros (queries) or on keys that are there, and its result is not stored.
   uint32_t qf[kHalf][8];
   float acc[kLdUnits][8];
-  int b = start_b, first_g = g0;
+  int b = find(g0), first_g = g0;
+  float m_row = -INFINITY, l_lane = 0.f;     // softmax row of this warp: running maximum, this lane's part of the sum
   bool fresh = true;
   int nkeys = 0;
   for (int g = g0; g < g1; ++g) {
@@ -179,7 +162,8 @@ __global__ void __launch_bounds__(kLdThreads, 1) latent_decode_kernel(const LdPa
                                                            : p.q_rot + b * p.q_rot_stride + (h0 + h) * p.q_rot_head_stride + col - p.rank);
         *reinterpret_cast<uint4*>(sq + h * row_bytes + col * 2) = v;
       }
-      if (tid < kLdHeads) { s_m[tid] = -INFINITY; s_l[tid] = 0.f; }
+      m_row = -INFINITY;
+      l_lane = 0.f;
 #pragma unroll
       for (int i = 0; i < kLdUnits; ++i)
 #pragma unroll
@@ -187,36 +171,31 @@ __global__ void __launch_bounds__(kLdThreads, 1) latent_decode_kernel(const LdPa
       __syncthreads();
       const uint32_t qa = q_s + ((lane & 7) + ((lane >> 3) & 1) * 8) * row_bytes + (lane >> 4) * 16 + k_first * 64;
 #pragma unroll
-      for (int k = 0; k < kHalf; ++k)
+      for (int k = 0; k < kHalf; ++k) {
+        uint32_t a[4] = {0, 0, 0, 0}, e[4] = {0, 0, 0, 0};
         if (k < k_num) {
-          uint32_t a[4];
           ldmatrix_x4(a, qa + k * 64);
-          qf[k][0] = a[0]; qf[k][1] = a[1]; qf[k][2] = a[2]; qf[k][3] = a[3];
-          ldmatrix_x4(a, qa + k * 64 + 32);
-          qf[k][4] = a[0]; qf[k][5] = a[1]; qf[k][6] = a[2]; qf[k][7] = a[3];
+          ldmatrix_x4(e, qa + k * 64 + 32);
         }
+#pragma unroll
+        for (int j = 0; j < 4; ++j) { qf[k][j] = a[j]; qf[k][4 + j] = e[j]; }
+      }
       fresh = false;
     }
-    const bool ok = tc::mbar_wait(bar0 + 8 * buf, ((g - g0) >> 1) & 1, &s_abort, p.error_word, 0x50);
-    if (!__syncthreads_and(ok)) {      // every thread leaves here; the copies in flight must have landed
-      if (tid == 0)
-        for (int d = 0; d < 2 && g + d < g1; ++d) tc::mbar_wait_timed(bar0 + 8 * ((g + d - g0) & 1), ((g + d - g0) >> 1) & 1);
-      __syncthreads();
-      return;
-    }
-    const uint32_t kb = kv_s + buf * kLdKeys * row_bytes;
+    tc::mbar_wait(bar0 + 8 * buf, ((g - g0) >> 1) & 1, &s_abort, p.error_word, 0x50);   // out of time: run on, the host learns of it
+    const uint32_t kb = kv_s + buf * boxes * kLdBox;
     {  // scores of 8 keys over half a row
       float d[2][4] = {};
-      const uint32_t ka = kb + (kt * 8 + (lane & 7)) * row_bytes + (lane >> 3) * 16 + k_first * 64;
+      const uint32_t ka = kb + (kt * 8 + (lane & 7)) * 128, sw0 = ((lane >> 3) ^ (lane & 7)) * 16, sw1 = sw0 ^ 64;
 #pragma unroll
-      for (int k = 0; k < kHalf; ++k)
-        if (k < k_num) {
-          uint32_t kf[4];
-          ldmatrix_x4(kf, ka + k * 64);
-          const uint32_t a0[4] = {qf[k][0], qf[k][1], qf[k][2], qf[k][3]}, a1[4] = {qf[k][4], qf[k][5], qf[k][6], qf[k][7]};
-          Mma16816<__nv_bfloat16>::run(d[0], a0, kf[0], kf[1]);
-          Mma16816<__nv_bfloat16>::run(d[1], a1, kf[2], kf[3]);
-        }
+      for (int k = 0; k < kHalf; ++k) {
+        uint32_t kf[4];
+        const int st = min(k_first + k, steps - 1);
+        ldmatrix_x4(kf, ka + (st >> 1) * kLdBox + (st & 1 ? sw1 : sw0));
+        const uint32_t a0[4] = {qf[k][0], qf[k][1], qf[k][2], qf[k][3]}, a1[4] = {qf[k][4], qf[k][5], qf[k][6], qf[k][7]};
+        Mma16816<__nv_bfloat16>::run(d[0], a0, kf[0], kf[1]);
+        Mma16816<__nv_bfloat16>::run(d[1], a1, kf[2], kf[3]);
+      }
       const int r = lane >> 2, col = kt * 8 + (lane & 3) * 2;
       float* o = ss + (half * kLdHeads + r) * kLdSStride + col;
       *reinterpret_cast<float2*>(o) = make_float2(d[0][0] + d[1][0], d[0][1] + d[1][1]);
@@ -231,22 +210,17 @@ __global__ void __launch_bounds__(kLdThreads, 1) latent_decode_kernel(const LdPa
       const float a = lane < left ? (r0[lane] + r1[lane]) * p.scale_log2 : -INFINITY;
       const float e = lane + 32 < left ? (r0[lane + 32] + r1[lane + 32]) * p.scale_log2 : -INFINITY;
       float mx = fmaxf(a, e);
-#pragma unroll
-      for (int o = 16; o; o >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, o));
-      const float m_old = s_m[h], m_new = fmaxf(m_old, mx);
+      asm("redux.sync.max.f32 %0, %1, 0xffffffff;" : "=f"(mx) : "f"(mx));
+      const float m_new = fmaxf(m_row, mx), corr = fast_exp2(m_row - m_new);
       const float pa = fast_exp2(a - m_new), pe = fast_exp2(e - m_new);    // key 0 of a tile is always visible
-      const float sum = warp_sum(pa + pe);
+      l_lane = fmaf(l_lane, corr, pa + pe);
+      m_row = m_new;
       const __nv_bfloat16 ha = __float2bfloat16_rn(pa), he = __float2bfloat16_rn(pe);
       sp[h * kLdPStride + lane] = ha;
       sp[h * kLdPStride + lane + 32] = he;
       sp[(kLdHeads + h) * kLdPStride + lane] = __float2bfloat16_rn(pa - __bfloat162float(ha));
       sp[(kLdHeads + h) * kLdPStride + lane + 32] = __float2bfloat16_rn(pe - __bfloat162float(he));
-      if (lane == 0) {
-        const float corr = fast_exp2(m_old - m_new);
-        s_c[h] = corr;
-        s_l[h] = s_l[h] * corr + sum;
-        s_m[h] = m_new;
-      }
+      if (lane == 0) s_c[h] = corr;
     }
     __syncthreads();
     {  // weighted sum: this warp's 16-column units, all 64 keys
@@ -256,33 +230,38 @@ __global__ void __launch_bounds__(kLdThreads, 1) latent_decode_kernel(const LdPa
 #pragma unroll
         for (int j = 0; j < 8; ++j) acc[i][j] *= (j & 2) ? c1 : c0;
       const uint32_t pa = p_s + (((lane & 7) + ((lane >> 3) & 1) * 8) * kLdPStride + (lane >> 4) * 8) * 2;
-      const uint32_t va = kb + ((lane & 7) + ((lane >> 3) & 1) * 8) * row_bytes + (warp * 16 + (lane >> 4) * 8) * 2;
-      if (warp < units) {
+      uint32_t va[kLdUnits];
 #pragma unroll
-        for (int k = 0; k < kLdKeys; k += 16) {
-          uint32_t hi[4], lo[4];
-          ldmatrix_x4(hi, pa + k * 2);
-          ldmatrix_x4(lo, pa + kLdHeads * kLdPStride * 2 + k * 2);
+      for (int i = 0; i < kLdUnits; ++i)
+        va[i] = kb + min((warp >> 2) + i * (kLdWarps / 4), boxes - 1) * kLdBox + ((lane & 7) + ((lane >> 3) & 1) * 8) * 128 +
+                ((((warp & 3) * 2 + (lane >> 4)) ^ (lane & 7)) * 16);
 #pragma unroll
-          for (int i = 0; i < kLdUnits; ++i)
-            if (warp + i * kLdWarps < units) {
-              uint32_t v[4];
-              ldmatrix_x4_trans(v, va + k * row_bytes + i * kLdWarps * 32);
-              float (&d0)[4] = *reinterpret_cast<float (*)[4]>(&acc[i][0]);
-              float (&d1)[4] = *reinterpret_cast<float (*)[4]>(&acc[i][4]);
-              Mma16816<__nv_bfloat16>::run(d0, hi, v[0], v[1]);
-              Mma16816<__nv_bfloat16>::run(d1, hi, v[2], v[3]);
-              Mma16816<__nv_bfloat16>::run(d0, lo, v[0], v[1]);
-              Mma16816<__nv_bfloat16>::run(d1, lo, v[2], v[3]);
-            }
+      for (int k = 0; k < kLdKeys; k += 16) {
+        uint32_t hi[4], lo[4];
+        ldmatrix_x4(hi, pa + k * 2);
+        ldmatrix_x4(lo, pa + kLdHeads * kLdPStride * 2 + k * 2);
+#pragma unroll
+        for (int i = 0; i < kLdUnits; ++i) {
+          uint32_t v[4];
+          ldmatrix_x4_trans(v, va[i] + k * 128);
+          float (&d0)[4] = *reinterpret_cast<float (*)[4]>(&acc[i][0]);
+          float (&d1)[4] = *reinterpret_cast<float (*)[4]>(&acc[i][4]);
+          Mma16816<__nv_bfloat16>::run(d0, hi, v[0], v[1]);
+          Mma16816<__nv_bfloat16>::run(d1, hi, v[2], v[3]);
+          Mma16816<__nv_bfloat16>::run(d0, lo, v[0], v[1]);
+          Mma16816<__nv_bfloat16>::run(d1, lo, v[2], v[3]);
         }
       }
     }
     __syncthreads();           // the buffer, the weights and the row statistics are free again
-    if (warp == 0) load(g + 2, buf);
+    load(g + 2, buf);
+    if ((g - g0) % (kLdAhead / 2) == kLdAhead / 2 - 1) look(g + 1 + kLdAhead / 2, kLdAhead / 2);   // over rows already used
     const bool last = g + 1 == s_start[b + 1];
     if (last || g + 1 == g1) {
       const bool whole = last && first_g == s_start[b];
+      const float l_row = warp_sum(l_lane);
+      if (lane == 0) { s_m[warp] = m_row; s_l[warp] = l_row; }
+      __syncthreads();
       const int r = lane >> 2, col = (lane & 3) * 2;
       float* piece = p.ws + ((static_cast<int64_t>(blockIdx.y) * ctas + c) * 2 + (first_g == g0 ? 0 : 1)) * ld_piece_floats(p.rank);
       if (!whole && tid < kLdHeads) { piece[tid] = s_m[tid]; piece[kLdHeads + tid] = s_l[tid]; }
@@ -317,6 +296,9 @@ __global__ void __launch_bounds__(kLdThreads, 1) latent_decode_kernel(const LdPa
       fresh = true;
     }
   }
+  if (*reinterpret_cast<volatile int*>(&s_abort) && tid == 0)      // copies in flight must land before the shared memory goes away
+    for (int g = max(g0, g1 - 2); g < g1; ++g) tc::mbar_wait_timed(bar0 + 8 * ((g - g0) & 1), ((g - g0) >> 1) & 1);
+  __syncthreads();
 }
 
 // One CTA per (sequence, head): joins the pieces of a sequence that several CTAs worked on.  Sequences without keys
@@ -412,17 +394,24 @@ extern "C" int mv_latent_decode(void* out, int64_t out_stride, int64_t out_head_
     return fail(MV_ERR_ALIGN, "latent_decode: rows must start on 16-byte boundaries");
   LdParams p{static_cast<__nv_bfloat16*>(out), out_stride, out_head_stride, static_cast<const __nv_bfloat16*>(q_lat),
              q_lat_stride, q_lat_head_stride, static_cast<const __nv_bfloat16*>(q_rot), q_rot_stride, q_rot_head_stride,
-             static_cast<const __nv_bfloat16*>(cache), block_tables, bt_stride, max_blocks, block_size, num_blocks,
+             block_size % kLdKeys == 0 ? kLdKeys : block_size, block_tables, bt_stride, max_blocks, block_size, num_blocks,
              positions, active, static_cast<const __nv_bfloat16*>(sink), batch, heads, rank, rot_dim,
              scale * 1.4426950408889634f, error_word, static_cast<float*>(workspace)};
+  if (block_size % kLdKeys && (kLdKeys % block_size || block_size < 8))
+    return fail(MV_ERR_SHAPE, "latent_decode: block_size %d", block_size);
+  if (num_blocks * block_size > 0x7fffff00LL) return fail(MV_ERR_LIMIT, "latent_decode: cache of %lld rows", static_cast<long long>(num_blocks * block_size));
+  CUtensorMap tm;
+  const int64_t cache_rows = num_blocks * block_size, R = rank + rot_dim;
+  const int rct = make_tmap_bf16(&tm, cache, R, cache_rows, 1, R, cache_rows * R, p.box_rows, 1, "latent_decode");
+  if (rct) return rct;
   const int row_bytes = (rank + rot_dim) * 2 + 16;
-  const size_t smem = static_cast<size_t>(2 * kLdKeys + kLdHeads) * row_bytes + 2 * kLdHeads * kLdSStride * 4 + 2 * kLdHeads * kLdPStride * 2;
+  const size_t smem = 1024 + static_cast<size_t>(2) * ((rank + rot_dim + 63) / 64) * kLdBox + kLdHeads * row_bytes + 2 * kLdHeads * kLdSStride * 4 + 2 * kLdHeads * kLdPStride * 2;
   const int ctas = ld_ctas(heads);
   auto st = static_cast<cudaStream_t>(stream);
   auto go = [&](auto kernel) {
     const cudaError_t e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem));
     if (e != cudaSuccess) return fail(MV_ERR_CUDA, "latent_decode: %s", cudaGetErrorString(e));
-    kernel<<<dim3(ctas, (heads + kLdHeads - 1) / kLdHeads), kLdThreads, smem, st>>>(p);
+    kernel<<<dim3(ctas, (heads + kLdHeads - 1) / kLdHeads), kLdThreads, smem, st>>>(tm, p);
     return check_launch("latent_decode");
   };
   const int rc = rank + rot_dim <= 320 ? go(latent_decode_kernel<5>) : go(latent_decode_kernel<9>);

@@ -70,7 +70,8 @@ def latent_decode(q_lat, q_rot, cache, block_tables, positions, sink, scale, wor
     rot = q_rot.shape[2]
     L = _cabi.lib()
     need = L.mv_latent_decode_workspace_bytes(batch, heads, rank, rot)
-    if need < 0 or q_lat.dtype != torch.bfloat16:
+    bs = cache.shape[1]
+    if need < 0 or q_lat.dtype != torch.bfloat16 or (bs % 64 and bs not in (8, 16, 32)):
         return None
     if workspace is None:
         workspace = torch.empty(need, dtype=torch.uint8, device=q_lat.device)
