@@ -140,10 +140,11 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmap, const LdParams p)
   auto load = [&](int g, int buf) {
     if (g >= g1) return;
     if (tid == 0) tc::mbar_expect_tx(bar0 + 8 * buf, boxes * kLdBox);
-    if (lane < groups)
-      for (int x = warp; x < boxes; x += kLdWarps)
-        tc::tma_load_3d(kv_s + (buf * boxes + x) * kLdBox + lane * p.box_rows * 128, &tmap, x * 64,
-                        s_row[(g - g0) % kLdAhead][lane], 0, bar0 + 8 * buf);
+    __syncwarp();
+    for (int x = warp; x < boxes; x += kLdWarps)
+      for (int r = 0; r < groups; ++r)
+        tc::tma_load_3d_elected(kv_s + (buf * boxes + x) * kLdBox + r * p.box_rows * 128, &tmap, x * 64,
+                                s_row[(g - g0) % kLdAhead][r], 0, bar0 + 8 * buf);
   };
   look(g0, kLdAhead);
   sync();
