@@ -48,7 +48,7 @@ __global__ void __launch_bounds__(kCsThreads, 2) ssm_chunk_kernel(const CsParams
   static_assert(SN >= 1, "more warps than column tiles");
   extern __shared__ __align__(128) __nv_bfloat16 sm[];
   __nv_bfloat16 *sX = sm, *sB = sX + Sh::kX, *sC = sB + Sh::kB, *sM = sC + Sh::kB, *sS = sM + Sh::kM2;
-  __shared__ float s_dt[kCsQ], s_c[kCsQ];
+  __shared__ __align__(8) float s_dts[2][kCsQ], s_cs[2][kCsQ];     // step sizes and running log2 decays of this chunk and the next
   const int s = blockIdx.x, h = blockIdx.y, p0 = blockIdx.z * PB, pw = min(PB, p.P - p0);
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const int g = h / (p.heads / p.groups), inner = p.heads * p.P;
@@ -88,49 +88,75 @@ __global__ void __launch_bounds__(kCsThreads, 2) ssm_chunk_kernel(const CsParams
   const int l7 = lane & 7, l8 = (lane >> 3) & 1, l16 = lane >> 4;
   const int ym = warp >> 1, yn = warp & 1;            // this warp's 16 rows and half of the columns of G and Y
 
+  // this thread's pieces of a chunk, as pointers that move from chunk to chunk
+  constexpr int XC = PB / 8, XR = kCsQ * XC / kCsThreads, BC = N / 8, BR = kCsQ * BC / kCsThreads;
+  static_assert(XR >= 1 && BR >= 1, "a chunk is at least one piece per thread");
+  const int xt = tid / XC, xc = (tid % XC) * 8, bt0 = tid / BC, bc = (tid % BC) * 8, c_off = p.groups * N;
+  const __nv_bfloat16* x_src = p.xbc + static_cast<int64_t>(first + xt) * p.xbc_stride + h * p.P + p0 + xc;
+  const __nv_bfloat16* b_src = p.xbc + static_cast<int64_t>(first + bt0) * p.xbc_stride + inner + g * N + bc;
+  __nv_bfloat16* y_dst = p.y + static_cast<int64_t>(first + xt) * p.y_stride + h * p.P + p0 + xc;
+  const __nv_bfloat16* ahead = p.xbc + static_cast<int64_t>(first + kCsQ + (tid >> 2)) * p.xbc_stride +
+      ((tid & 3) == 0 ? h * p.P + p0 : inner + ((tid & 3) == 2 ? p.groups + g : g) * N + ((tid & 3) == 3 ? N / 2 : 0));
+  // dt: warp 0 reads a chunk's values while the chunk before it is worked on, two tokens per lane
+  __nv_bfloat16 raw[2] = {__float2bfloat16_rn(0.f), __float2bfloat16_rn(0.f)};     // converted when used: nobody waits for the load
+  auto fetch_dt = [&](int t0) {
+#pragma unroll
+    for (int i = 0; i < 2; ++i)
+      if (t0 + lane * 2 + i < n_tok) raw[i] = p.dt[(static_cast<int64_t>(first) + t0 + lane * 2 + i) * p.dt_stride + h];
+  };
+  auto make_dt = [&](int t0) {
+    float d[2], c[2];
+#pragma unroll
+    for (int i = 0; i < 2; ++i) {
+      d[i] = t0 + lane * 2 + i < n_tok ? softplus_f(__bfloat162float(raw[i]) + db) : 0.f;
+      c[i] = a2 * d[i];
+    }
+    float run = c[0] + c[1];
+#pragma unroll
+    for (int o = 1; o < 32; o <<= 1) {
+      const float v = __shfl_up_sync(0xffffffffu, run, o);
+      if (lane >= o) run += v;
+    }
+    const int at = (t0 / kCsQ) & 1;
+    s_dts[at][lane * 2] = d[0];
+    s_dts[at][lane * 2 + 1] = d[1];
+    s_cs[at][lane * 2] = run - c[1];
+    s_cs[at][lane * 2 + 1] = run;
+  };
+  if (warp == 0) {
+    fetch_dt(0);
+    make_dt(0);
+  }
   for (int t0 = 0; t0 < n_tok; t0 += kCsQ) {
     const int nt = min(kCsQ, n_tok - t0);
-    for (int i = tid; i < kCsQ * (PB / 8); i += kCsThreads) {
-      const int t = i / (PB / 8), c = (i % (PB / 8)) * 8;
-      const bool ok = t < nt && c < pw;
-      cp_async16(x_s + (t * Sh::kXs + c) * 2, p.xbc + (static_cast<int64_t>(first + t0) + (ok ? t : 0)) * p.xbc_stride + h * p.P + p0 + (ok ? c : 0), ok ? 16 : 0);
+#pragma unroll
+    for (int i = 0; i < XR; ++i) {
+      const int t = xt + i * (kCsThreads / XC);
+      const bool ok = t < nt && xc < pw;
+      cp_async16(x_s + (t * Sh::kXs + xc) * 2, ok ? x_src + i * (kCsThreads / XC) * p.xbc_stride : p.xbc, ok ? 16 : 0);
     }
-    for (int i = tid; i < kCsQ * (N / 8); i += kCsThreads) {
-      const int t = i / (N / 8), c = (i % (N / 8)) * 8;
+#pragma unroll
+    for (int i = 0; i < BR; ++i) {
+      const int t = bt0 + i * (kCsThreads / BC);
       const bool ok = t < nt;
-      const __nv_bfloat16* src = p.xbc + (static_cast<int64_t>(first + t0) + (ok ? t : 0)) * p.xbc_stride + inner + g * N + c;
-      cp_async16(b_s + (t * Sh::kBs + c) * 2, src, ok ? 16 : 0);
-      cp_async16(c_s + (t * Sh::kBs + c) * 2, src + p.groups * N, ok ? 16 : 0);
+      const __nv_bfloat16* src = ok ? b_src + i * (kCsThreads / BC) * p.xbc_stride : p.xbc;
+      cp_async16(b_s + (t * Sh::kBs + bc) * 2, src, ok ? 16 : 0);
+      cp_async16(c_s + (t * Sh::kBs + bc) * 2, ok ? src + c_off : src, ok ? 16 : 0);
     }
     cp_async_commit();
+    x_src += kCsQ * p.xbc_stride;
+    b_src += kCsQ * p.xbc_stride;
     {  // the next chunk's lines on their way to L2
       const int t = tid >> 2, part = tid & 3;
       if (t0 + kCsQ + t < n_tok) {
-        const __nv_bfloat16* row = p.xbc + (static_cast<int64_t>(first) + t0 + kCsQ + t) * p.xbc_stride;
-        const __nv_bfloat16* at = part == 0 ? row + h * p.P + p0 : row + inner + (part == 1 ? g : part == 2 ? p.groups + g : g) * N + (part == 3 ? N / 2 : 0);
-        asm volatile("prefetch.global.L2 [%0];" ::"l"(at));
-        if (part == 2 && N > 64) asm volatile("prefetch.global.L2 [%0];" ::"l"(at + N / 2));
+        asm volatile("prefetch.global.L2 [%0];" ::"l"(ahead));
+        if (part == 2 && N > 64) asm volatile("prefetch.global.L2 [%0];" ::"l"(ahead + N / 2));
       }
+      ahead += kCsQ * p.xbc_stride;
     }
-    if (warp == 0) {       // dt and the running log2 decay; two tokens per lane
-      float d[2], c[2];
-#pragma unroll
-      for (int i = 0; i < 2; ++i) {
-        const int t = lane * 2 + i;
-        d[i] = t < nt ? softplus_f(__bfloat162float(p.dt[(static_cast<int64_t>(first) + t0 + t) * p.dt_stride + h]) + db) : 0.f;
-        c[i] = a2 * d[i];
-      }
-      float run = c[0] + c[1];
-#pragma unroll
-      for (int o = 1; o < 32; o <<= 1) {
-        const float v = __shfl_up_sync(0xffffffffu, run, o);
-        if (lane >= o) run += v;
-      }
-      s_dt[lane * 2] = d[0];
-      s_dt[lane * 2 + 1] = d[1];
-      s_c[lane * 2] = run - c[1];
-      s_c[lane * 2 + 1] = run;
-    }
+    const int cur = (t0 / kCsQ) & 1;
+    const float *s_dt = s_dts[cur], *s_c = s_cs[cur];
+    if (warp == 0) fetch_dt(t0 + kCsQ);
     cp_async_wait<0>();
     __syncthreads();
 
@@ -156,13 +182,13 @@ __global__ void __launch_bounds__(kCsThreads, 2) ssm_chunk_kernel(const CsParams
 #pragma unroll
         for (int j = 0; j < 4; ++j) {
           const int col = yn * 32 + j * 8 + c2;
-          const float cj0 = s_c[col], cj1 = s_c[col + 1], d0 = s_dt[col], d1 = s_dt[col + 1];
+          const float2 cj = *reinterpret_cast<const float2*>(s_c + col), dj = *reinterpret_cast<const float2*>(s_dt + col);
 #pragma unroll
           for (int half = 0; half < 2; ++half) {
             const int row = ym * 16 + r8 + half * 8;
             const float ct = half ? ct1 : ct0;
-            const float m0 = col <= row ? G[j][half * 2] * fast_exp2(ct - cj0) * d0 : 0.f;
-            const float m1 = col + 1 <= row ? G[j][half * 2 + 1] * fast_exp2(ct - cj1) * d1 : 0.f;
+            const float m0 = col <= row ? G[j][half * 2] * fast_exp2(ct - cj.x) * dj.x : 0.f;
+            const float m1 = col + 1 <= row ? G[j][half * 2 + 1] * fast_exp2(ct - cj.y) * dj.y : 0.f;
             *reinterpret_cast<uint32_t*>(sM + row * Sh::kMs + col) = pack2<__nv_bfloat16>(m0, m1);
           }
         }
@@ -217,6 +243,7 @@ __global__ void __launch_bounds__(kCsThreads, 2) ssm_chunk_kernel(const CsParams
           *reinterpret_cast<__nv_bfloat162*>(sC + row * Sh::kBs + col) = v;
         }
     }
+    if (warp == 0) make_dt(t0 + kCsQ);     // its rows have the fewest products
     __syncthreads();                       // M has been read, Y is complete
     const float cl = s_c[kCsQ - 1];
     for (int i = tid; i < kCsQ * (PB / 8); i += kCsThreads) {    // W X in two terms: the value in place, the residue over M
@@ -232,12 +259,13 @@ __global__ void __launch_bounds__(kCsThreads, 2) ssm_chunk_kernel(const CsParams
       Vec<__nv_bfloat16, 8>::store(sX + t * Sh::kXs + c, v);
       Vec<__nv_bfloat16, 8>::store(sM + t * Sh::kXs + c, lo);
     }
-    for (int i = tid; i < nt * (PB / 8); i += kCsThreads) {
-      const int t = i / (PB / 8), c = (i % (PB / 8)) * 8;
-      if (c < pw)
-        *reinterpret_cast<uint4*>(p.y + (static_cast<int64_t>(first) + t0 + t) * p.y_stride + h * p.P + p0 + c) =
-            *reinterpret_cast<const uint4*>(sC + t * Sh::kBs + c);
+#pragma unroll
+    for (int i = 0; i < XR; ++i) {
+      const int t = xt + i * (kCsThreads / XC);
+      if (t < nt && xc < pw)
+        *reinterpret_cast<uint4*>(y_dst + i * (kCsThreads / XC) * p.y_stride) = *reinterpret_cast<const uint4*>(sC + t * Sh::kBs + xc);
     }
+    y_dst += kCsQ * p.y_stride;
     __syncthreads();
     {  // S = exp(c_last) S + (W B)^T X
       const float e = fast_exp2(cl);
