@@ -416,7 +416,8 @@ extern "C" int mv_latent_decode(void* out, int64_t out_stride, int64_t out_head_
   if (!out || !q_lat || (rot_dim && !q_rot) || !cache || !block_tables || !positions || !workspace || !error_word)
     return fail(MV_ERR_NULL, "latent_decode: null pointer");
   if (workspace_bytes < mv_latent_decode_workspace_bytes(batch, heads, rank, rot_dim)) return fail(MV_ERR_WORKSPACE, "latent_decode: workspace");
-  if (!vec8_ok(q_lat, q_lat_stride, 2) || q_lat_head_stride % 8 || !vec8_ok(q_rot, q_rot_stride, 2) || q_rot_head_stride % 8 ||
+  if (!vec8_ok(q_lat, q_lat_stride, 2) || q_lat_head_stride % 8 ||
+      (rot_dim && (!vec8_ok(q_rot, q_rot_stride, 2) || q_rot_head_stride % 8)) ||
       !aligned16(cache) || !vec8_ok(out, out_stride, 2) || out_head_stride % 8 || !aligned16(workspace))
     return fail(MV_ERR_ALIGN, "latent_decode: rows must start on 16-byte boundaries");
   LdParams p{static_cast<__nv_bfloat16*>(out), out_stride, out_head_stride, static_cast<const __nv_bfloat16*>(q_lat),

@@ -71,6 +71,9 @@ def latent_decode(q_lat, q_rot, cache, block_tables, positions, sink, scale, wor
     L = _cabi.lib()
     need = L.mv_latent_decode_workspace_bytes(batch, heads, rank, rot)
     bs = cache.shape[1]
+    pieces = [t.data_ptr() // 2 | t.stride(0) | t.stride(1) for t in (q_lat, q_rot) if t.numel()]
+    if any(x % 8 for x in pieces):          # rows that are not whole 16-byte pieces
+        return None
     if need < 0 or q_lat.dtype != torch.bfloat16 or (bs % 64 and bs not in (8, 16, 32)):
         return None
     if workspace is None:

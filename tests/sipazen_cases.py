@@ -46,6 +46,16 @@ def even():
         ("latent_attention", _attention(16, 48, 64, 80, 256), _moe(8, 2, 64, 128))])
 
 
+def between():
+    """Sizes that some of the tensor-core kernels take and others do not."""
+    return _config(257, 136, 2, 0.9, [
+        ("latent_attention", _attention(3, 36, 28, 40, 68), _moe(9, 2, 44, 24)),
+        ("mamba2", _mamba(3, 20, 32, 1, 4, 3), _moe(3, 2, 40, 136)),
+        ("latent_attention", _attention(2, 36, 32, 24, 64, base=300.0), _moe(5, 2, 16, 20)),
+        ("mamba2", _mamba(2, 56, 32, 2, 5, 7), _moe(3, 1, 48, None)),
+        ("mamba2", _mamba(6, 24, 48, 3, 2, 1), _moe(6, 5, 8, 8))])
+
+
 def attention_only():
     return _config(200, 64, 1, 1.0, [("latent_attention", _attention(2, 16, 16, 16, 32), _moe(4, 2, 32, 32))] * 2)
 
@@ -54,13 +64,21 @@ def mamba_only():
     return _config(200, 64, 2, 0.6, [("mamba2", _mamba(2, 32, 16, 1, 4, 1), _moe(4, 2, 32, 32))] * 2)
 
 
-CONFIGS = {"odd": odd, "even": even, "attention_only": attention_only, "mamba_only": mamba_only}
+CONFIGS = {"odd": odd, "even": even, "between": between, "attention_only": attention_only, "mamba_only": mamba_only}
 
 
 @functools.lru_cache(maxsize=None)
 def model(name):
     cfg = CONFIGS[name]()
-    return cfg, oracle.random_weights(cfg, seed=len(name))
+    w = oracle.random_weights(cfg, seed=len(name))
+    if name == "between":
+        # few experts and many layers: spread the router's logits, so that rounding does not swap the last expert chosen
+        # with the first one that is not
+        g = torch.Generator().manual_seed(1)
+        for k in [k for k in w if k.endswith("mlp.router")]:
+            w[k] = (w[k].float() * 0.3).to(torch.bfloat16)
+            w[k + ".b"] = (1.5 * torch.randperm(w[k].shape[0], generator=g)).to(torch.bfloat16)
+    return cfg, w
 
 
 def tokens(name, n, seed=0):

@@ -42,7 +42,7 @@ def test_whole_portions_and_decoding(name, dtype):
 
 
 @pytest.mark.parametrize("dtype", DTYPES, ids=IDS)
-@pytest.mark.parametrize("name", ["odd", "even"])
+@pytest.mark.parametrize("name", ["odd", "even", "between"])
 def test_mixed_batches_and_reuse(name, dtype):
     """Unequal requests in one batch, portions beside single tokens, requests that pause, and a pool so small that
     blocks and slots change hands; every request must come out as it does alone."""
