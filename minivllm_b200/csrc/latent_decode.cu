@@ -31,6 +31,7 @@ constexpr int kLdUnits = kLdMaxRank / 16 / kLdWarps;   // 16-column units of the
 constexpr int kLdBox = kLdKeys * 128;       // bytes of a box of 32 keys, 64 columns
 constexpr int kLdAhead = 128;                // tiles whose cache rows are known ahead
 constexpr int kLdFewKeys = 128;
+constexpr int kLdQPieces = (kLdHeads * kLdMaxRow / 8 + kLdThreads - 1) / kLdThreads;   // 16-byte pieces of the queries per thread
 constexpr int kLdSStride = kLdKeys + 4;    // floats per score row
 constexpr int kLdPStride = kLdKeys + 8;    // bf16 per weight row
 
@@ -83,8 +84,9 @@ __device__ __forceinline__ void ld_prefix(const LdParams& p, int* s_start, int* 
 }
 __device__ __forceinline__ int ld_cut(int total, int c, int ctas) { return static_cast<int>(static_cast<int64_t>(total) * c / ctas); }
 
-// kSteps: 16-column steps of a quarter of a row that the query fragments have registers for.
-template <int kSteps>
+// kSteps: 16-column steps of a quarter of a row that the query fragments have registers for.  kRank, kRow: sizes known at
+// compile time (0: any), which leaves the tile loop without spilled addresses.
+template <int kSteps, int kRank = 0, int kRow = 0>
 __global__ void __launch_bounds__(kLdWorkers * kLdThreads, 1)
 latent_decode_kernel(const __grid_constant__ CUtensorMap tmap, const LdParams p) {
   extern __shared__ unsigned char raw[];
@@ -93,7 +95,7 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmap, const LdParams p)
   __shared__ __align__(8) uint64_t s_bar[kLdWorkers][2];
   __shared__ int s_abort, s_rows[kLdWorkers][kLdAhead][4];
   const int wk = threadIdx.x / kLdThreads, tid = threadIdx.x % kLdThreads, warp = tid >> 5, lane = tid & 31;
-  const int R = p.rank + p.rot_dim, row_bytes = R * 2 + 16;
+  const int rank = kRank ? kRank : p.rank, R = kRow ? kRow : p.rank + p.rot_dim, row_bytes = R * 2 + 16;
   const int boxes = (R + 63) / 64;
   const uint32_t base = (smem_u32(raw) + 1023u) & ~1023u;
   const uint32_t kv_s = base + wk * 2 * boxes * kLdBox;      // [2][box][32][128B], swizzled
@@ -146,18 +148,40 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmap, const LdParams p)
         tc::tma_load_3d_elected(kv_s + (buf * boxes + x) * kLdBox + r * p.box_rows * 128, &tmap, x * 64,
                                 s_row[(g - g0) % kLdAhead][r], 0, bar0 + 8 * buf);
   };
-  look(g0, kLdAhead);
+  // A sequence's queries: all pieces requested at once, and before they are needed.
+  auto load_q = [&](int b) {
+    int t = tid, chunks = R / 8;
+    asm volatile("" : "+r"(t), "+r"(chunks));     // computed here and not kept in registers across the tiles
+    uint4 raw[kLdQPieces];
+#pragma unroll
+    for (int k = 0; k < kLdQPieces; ++k) {
+      const int i = t + k * kLdThreads, h = i / chunks, col = (i - h * chunks) * 8;
+      raw[k] = make_uint4(0, 0, 0, 0);
+      if (h < nh)
+        raw[k] = *reinterpret_cast<const uint4*>(col < rank ? p.q_lat + b * p.q_lat_stride + (h0 + h) * p.q_lat_head_stride + col
+                                                              : p.q_rot + b * p.q_rot_stride + (h0 + h) * p.q_rot_head_stride + col - rank);
+    }
+#pragma unroll
+    for (int k = 0; k < kLdQPieces; ++k) {
+      const int i = t + k * kLdThreads, h = i / chunks, col = (i - h * chunks) * 8;
+      if (h < kLdHeads) *reinterpret_cast<uint4*>(sq + h * row_bytes + col * 2) = raw[k];
+    }
+  };
+  int b = find(g0), first_g = g0;
+  look(g0, 2);
   sync();
   load(g0, 0);
   load(g0 + 1, 1);
+  look(g0 + 2, kLdAhead - 2);      // while the first tiles are on their way
+  load_q(b);
+  sync();
 
   const int steps = R / 16, per = (steps + kLdQuarters - 1) / kLdQuarters;
   const int kt = warp & 1, quarter = warp >> 1;       // score role: 16 keys, a quarter of the row
   const int k_first = quarter * per;
-  const int units = p.rank / 16;
+  const int units = rank / 16;
   uint32_t qf[kSteps][4];
   float acc[kLdUnits][8];
-  int b = find(g0), first_g = g0;
   float m_row[2], l_lane[2];     // softmax rows of this warp: running maximum, this lane's part of the sum
   bool fresh = true;
   int nkeys = 0;
@@ -167,15 +191,6 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmap, const LdParams p)
     if (fresh) {
       first_g = g;
       nkeys = s_keys[b];
-      const int chunks = R / 8;
-      for (int i = tid; i < kLdHeads * chunks; i += kLdThreads) {
-        const int h = i / chunks, col = (i - h * chunks) * 8;
-        uint4 v = make_uint4(0, 0, 0, 0);
-        if (h < nh)
-          v = *reinterpret_cast<const uint4*>(col < p.rank ? p.q_lat + b * p.q_lat_stride + (h0 + h) * p.q_lat_head_stride + col
-                                                           : p.q_rot + b * p.q_rot_stride + (h0 + h) * p.q_rot_head_stride + col - p.rank);
-        *reinterpret_cast<uint4*>(sq + h * row_bytes + col * 2) = v;
-      }
 #pragma unroll
       for (int i = 0; i < 2; ++i) {
         m_row[i] = -INFINITY;
@@ -185,7 +200,6 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmap, const LdParams p)
       for (int i = 0; i < kLdUnits; ++i)
 #pragma unroll
         for (int j = 0; j < 8; ++j) acc[i][j] = 0.f;
-      sync();
       const uint32_t qa = q_s + ((lane & 7) + ((lane >> 3) & 1) * 8) * row_bytes + (lane >> 4) * 16 + k_first * 32;
 #pragma unroll
       for (int k = 0; k < kSteps; ++k) {
@@ -284,7 +298,7 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmap, const LdParams p)
       }
       sync();
       const int r = lane >> 2, col = (lane & 3) * 2;
-      float* piece = p.ws + ((static_cast<int64_t>(blockIdx.y) * ctas + c) * 2 + (first_g == g0 ? 0 : 1)) * ld_piece_floats(p.rank);
+      float* piece = p.ws + ((static_cast<int64_t>(blockIdx.y) * ctas + c) * 2 + (first_g == g0 ? 0 : 1)) * ld_piece_floats(rank);
       if (!whole && tid < kLdHeads) { piece[tid] = s_m[tid]; piece[kLdHeads + tid] = s_l[tid]; }
 #pragma unroll
       for (int hf = 0; hf < 2; ++hf) {
@@ -306,14 +320,19 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmap, const LdParams p)
             for (int t = 0; t < 2; ++t) {
               const int at = (warp + i * kLdWarps) * 16 + t * 8 + col;
               const float x = acc[i][t * 4 + hf * 2], y = acc[i][t * 4 + hf * 2 + 1];
-              if (!whole) *reinterpret_cast<float2*>(piece + 2 * kLdHeads + h * p.rank + at) = make_float2(x, y);
+              if (!whole) *reinterpret_cast<float2*>(piece + 2 * kLdHeads + h * rank + at) = make_float2(x, y);
               else if (h < nh)
                 *reinterpret_cast<__nv_bfloat162*>(p.out + b * p.out_stride + (h0 + h) * p.out_head_stride + at) =
                     __floats2bfloat162_rn(x * inv, y * inv);
             }
           }
       }
-      sync();         // s_m / s_l are read before the next sequence resets them
+      if (g + 1 < g1) {          // the next sequence's queries: every warp has its fragments of this one's
+        int nb = b + 1;
+        while (g + 1 >= s_start[nb + 1]) ++nb;
+        load_q(nb);
+      }
+      sync();         // queries of the next sequence are there, s_m and s_l are free
       fresh = true;
     }
   }
@@ -442,7 +461,7 @@ extern "C" int mv_latent_decode(void* out, int64_t out_stride, int64_t out_head_
     kernel<<<dim3(ctas, (heads + kLdHeads - 1) / kLdHeads), kLdWorkers * kLdThreads, smem, st>>>(tm, p);
     return check_launch("latent_decode");
   };
-  const int rc = rank + rot_dim <= 320 ? go(latent_decode_kernel<5>) : go(latent_decode_kernel<9>);
+  const int rc = rank == 512 && rot_dim == 64 ? go(latent_decode_kernel<9, 512, 576>) : rank + rot_dim <= 320 ? go(latent_decode_kernel<5>) : go(latent_decode_kernel<9>);
   if (rc) return rc;
   latent_combine_kernel<<<dim3(batch, heads), 128, 0, st>>>(p, ctas * kLdWorkers);
   return check_launch("latent_decode");
