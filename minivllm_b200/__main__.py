@@ -1,6 +1,6 @@
 """Command line: greedy or sampled generation from a model folder, token ids in and out (no tokenizer is bundled).
 
-    python -m minivllm_b200 --model DIR --prompt 5,17,3 [--prompt ...] [--max-tokens 64] [--temperature 0]
+    python -m minivllm_b200 --model DIR --prompt 12,7,30 [--prompt ...] [--max-tokens 64] [--temperature 0]
 """
 import argparse
 import json

@@ -4,12 +4,13 @@
 
 DIR holds config.json and model.safetensors.  Steps are read from standard input, one JSON object a line:
 
-    {"step": 0, "entries": [{"id": "a", "tokens": [5, 17, 3], "want": [0, 2]}], "end": []}
+    {"step": 4, "entries": [{"id": "x", "tokens": [12, 7], "want": [1]}, {"id": "y", "tokens": [30], "want": []}],
+     "end": ["y"]}                    (in one line)
 
-Each step's entries run as one batch through `LLMEngine.score_step`, i.e. the engine's own scheduler state, cache
+`want` names places among an entry's own tokens; `end` lists requests that are over.  Each step's entries run as one batch through `LLMEngine.score_step`, i.e. the engine's own scheduler state, cache
 blocks, state slots, model step and (for single tokens) decode graph.  The logits at the wanted places go to
 OUT/<step>.f32, little-endian 32-bit floats in the order of the entries, and a line `done <step>` follows every step.
-`--max-tokens` sizes the cache pool: the most tokens that live requests hold at a time, each rounded up to a block.
+`--max-tokens` sizes the cache pool, in tokens of all requests that are running at once, whole blocks each.
 """
 import argparse
 import json
@@ -25,7 +26,7 @@ def parse_args(argv=None):
     ap.add_argument("--model", required=True, help="folder with config.json and model.safetensors")
     ap.add_argument("--dtype", choices=("bfloat16", "float32"), default="bfloat16")
     ap.add_argument("--out", required=True, help="folder for <step>.f32")
-    ap.add_argument("--max-tokens", type=int, required=True, help="most tokens that live requests hold at any time")
+    ap.add_argument("--max-tokens", type=int, required=True, help="size of the cache pool in tokens")
     return ap.parse_args(argv)
 
 
