@@ -7,10 +7,11 @@ DIR holds config.json and model.safetensors.  Steps are read from standard input
     {"step": 4, "entries": [{"id": "x", "tokens": [12, 7], "want": [1]}, {"id": "y", "tokens": [30], "want": []}],
      "end": ["y"]}                    (in one line)
 
-`want` names places among an entry's own tokens; `end` lists requests that are over.  Each step's entries run as one batch through `LLMEngine.score_step`, i.e. the engine's own scheduler state, cache
-blocks, state slots, model step and (for single tokens) decode graph.  The logits at the wanted places go to
-OUT/<step>.f32, little-endian 32-bit floats in the order of the entries, and a line `done <step>` follows every step.
-`--max-tokens` sizes the cache pool, in tokens of all requests that are running at once, whole blocks each.
+`want` names places among an entry's own tokens; `end` lists requests that are over.  Each step's entries run as one
+batch through `LLMEngine.score_step`, i.e. the engine's own cache blocks, state slots, model step and (for single
+tokens) decode graph.  The logits at the wanted places go to OUT/<step>.f32, little-endian 32-bit floats in the order
+of the entries, and a line `done <step>` follows every step.  `--max-tokens` sizes the cache pool, in tokens of all
+requests that are running at once, whole blocks each.
 """
 import argparse
 import json
