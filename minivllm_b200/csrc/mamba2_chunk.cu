@@ -4,9 +4,9 @@
 // fp32 accumulators in registers.  With c_t the running sum of the log decays inside the chunk:
 //   Y = exp(c_t) (C S_prev) + (M X) + D X,   M[t, j] = exp(c_t - c_j) dt_j (C_t . B_j) for j <= t
 //   S = exp(c_last) S_prev + B^T (W X),       W_t = exp(c_last - c_t) dt_t
-// C, B and X are the bf16 outputs of the convolution and enter the products as they are.  W X, which enters the state,
-// goes in as two bf16 terms, the value and its rounding residue, so that S is advanced with 16 bits of it and kept in
-// fp32; M and the copy of S that is read out are single bf16 operands, as Y is a bf16 result.
+// C, B and X are the bf16 outputs of the convolution and enter the products as they are.  What the recurrence forms
+// itself (M, W X, S) is fp32 and enters a product as two bf16 terms, the value and its rounding residue, so that the
+// products carry 16 bits of it and nothing of the state is rounded to bf16.
 // Two CTAs per SM: one computes while the other waits for its loads.
 //
 // Bytes per token and head: (2 * P + 2 * N / heads_per_group) * 2 + 2; the state is touched once per sequence.
@@ -21,9 +21,9 @@ constexpr int kCsThreads = 256, kCsQ = 64;
 template <int N, int PB> struct CsShape {
   static constexpr int kXs = PB + 8, kBs = (N > PB ? N : PB) + 8, kMs = kCsQ + 8;  // row strides, elements (Y passes through C)
   static constexpr int kX = kCsQ * kXs, kB = kCsQ * kBs, kS = N * kXs;
-  static constexpr int kM2 = kCsQ * (kMs > kXs ? kMs : kXs);                      // M, later the residue of W X
+  static constexpr int kM2 = 2 * kCsQ * kMs;                                      // M (two terms), later the residue of W X
   static_assert(kM2 >= kX, "the residue of W X lies over M");
-  static constexpr int kElems = kX + 2 * kB + kM2 + kS;
+  static constexpr int kElems = kX + 2 * kB + kM2 + 2 * kS;
   static constexpr int kBytes = kElems * 2;
 };
 
@@ -37,6 +37,13 @@ struct CsParams {
 };
 
 using Mma = Mma16816<__nv_bfloat16>;
+__device__ __forceinline__ void split2(float a, float b, uint32_t& hi, uint32_t& lo) {
+  const __nv_bfloat162 h = __floats2bfloat162_rn(a, b);
+  const float2 f = __bfloat1622float2(h);
+  const __nv_bfloat162 r = __floats2bfloat162_rn(a - f.x, b - f.y);
+  hi = *reinterpret_cast<const uint32_t*>(&h);
+  lo = *reinterpret_cast<const uint32_t*>(&r);
+}
 template <int N, int PB>
 __global__ void __launch_bounds__(kCsThreads, 2) ssm_chunk_kernel(const CsParams p) {
   using Sh = CsShape<N, PB>;
@@ -71,15 +78,19 @@ __global__ void __launch_bounds__(kCsThreads, 2) ssm_chunk_kernel(const CsParams
         const int n = (sm0 + a) * 16 + r8 + (e >> 1) * 8, q = (sn0 + b) * 8 + c2 + (e & 1);
         S[a][b][e] = live && st0 > 0 && q < pw ? gS[static_cast<int64_t>(n) * p.P + q] : 0.f;
       }
-  auto store_S = [&] {      // S in bf16 to shared memory, for the product with C
+  auto store_S = [&] {      // both bf16 terms of S to shared memory, for the product with C
 #pragma unroll
     for (int a = 0; a < MPW; ++a)
 #pragma unroll
       for (int b = 0; b < SN; ++b)
 #pragma unroll
-        for (int half = 0; half < 2; ++half)
-          *reinterpret_cast<uint32_t*>(sS + ((sm0 + a) * 16 + r8 + half * 8) * Sh::kXs + (sn0 + b) * 8 + c2) =
-              pack2<__nv_bfloat16>(S[a][b][half * 2], S[a][b][half * 2 + 1]);
+        for (int half = 0; half < 2; ++half) {
+          uint32_t hi, lo;
+          split2(S[a][b][half * 2], S[a][b][half * 2 + 1], hi, lo);
+          const int at = ((sm0 + a) * 16 + r8 + half * 8) * Sh::kXs + (sn0 + b) * 8 + c2;
+          *reinterpret_cast<uint32_t*>(sS + at) = hi;
+          *reinterpret_cast<uint32_t*>(sS + Sh::kS + at) = lo;
+        }
   };
   store_S();
   const float a2 = -expf(__bfloat162float(p.A_log[h])) * 1.4426950408889634f;
@@ -162,7 +173,7 @@ __global__ void __launch_bounds__(kCsThreads, 2) ssm_chunk_kernel(const CsParams
 
     float acc[YN][4];
     const float ct0 = s_c[ym * 16 + r8], ct1 = s_c[ym * 16 + r8 + 8];
-    {  // G = C B^T for this warp's 16 x 32 block, then M
+    {  // G = C B^T for this warp's 16 x 32 block, then M in two terms
       const bool need = yn * 32 <= ym * 16 + 15;
       float G[4][4] = {};
       if (need) {
@@ -189,7 +200,10 @@ __global__ void __launch_bounds__(kCsThreads, 2) ssm_chunk_kernel(const CsParams
             const float ct = half ? ct1 : ct0;
             const float m0 = col <= row ? G[j][half * 2] * fast_exp2(ct - cj.x) * dj.x : 0.f;
             const float m1 = col + 1 <= row ? G[j][half * 2 + 1] * fast_exp2(ct - cj.y) * dj.y : 0.f;
-            *reinterpret_cast<uint32_t*>(sM + row * Sh::kMs + col) = pack2<__nv_bfloat16>(m0, m1);
+            uint32_t hi, lo;
+            split2(m0, m1, hi, lo);
+            *reinterpret_cast<uint32_t*>(sM + row * Sh::kMs + col) = hi;
+            *reinterpret_cast<uint32_t*>(sM + kCsQ * Sh::kMs + row * Sh::kMs + col) = lo;
           }
         }
       }
@@ -206,11 +220,13 @@ __global__ void __launch_bounds__(kCsThreads, 2) ssm_chunk_kernel(const CsParams
         uint32_t a[4], b[4];
         ldmatrix_x4(a, ca + k * 2);
 #pragma unroll
-        for (int i = 0; i < YN; i += 2) {
-          ldmatrix_x4_trans(b, sa + (k * Sh::kXs + i * 8) * 2);
-          Mma::run(acc[i], a, b[0], b[1]);
-          Mma::run(acc[i + 1], a, b[2], b[3]);
-        }
+        for (int term = 0; term < 2; ++term)
+#pragma unroll
+          for (int i = 0; i < YN; i += 2) {
+            ldmatrix_x4_trans(b, sa + (term * Sh::kS + k * Sh::kXs + i * 8) * 2);
+            Mma::run(acc[i], a, b[0], b[1]);
+            Mma::run(acc[i + 1], a, b[2], b[3]);
+          }
       }
       const float e0 = fast_exp2(ct0), e1 = fast_exp2(ct1);
 #pragma unroll
@@ -223,13 +239,16 @@ __global__ void __launch_bounds__(kCsThreads, 2) ssm_chunk_kernel(const CsParams
       const uint32_t ma = m_s + ((ym * 16 + l7 + l8 * 8) * Sh::kMs + l16 * 8) * 2;
       const uint32_t xa = x_s + ((l7 + l8 * 8) * Sh::kXs + yn * (PB / 2) + l16 * 8) * 2;
       for (int k = 0; k <= ym * 16; k += 16) {
-        uint32_t a[4], b[4];
-        ldmatrix_x4(a, ma + k * 2);
+        uint32_t hi[4], lo[4], b[4];
+        ldmatrix_x4(hi, ma + k * 2);
+        ldmatrix_x4(lo, ma + (kCsQ * Sh::kMs + k) * 2);
 #pragma unroll
         for (int i = 0; i < YN; i += 2) {
           ldmatrix_x4_trans(b, xa + (k * Sh::kXs + i * 8) * 2);
-          Mma::run(acc[i], a, b[0], b[1]);
-          Mma::run(acc[i + 1], a, b[2], b[3]);
+          Mma::run(acc[i], hi, b[0], b[1]);
+          Mma::run(acc[i + 1], hi, b[2], b[3]);
+          Mma::run(acc[i], lo, b[0], b[1]);
+          Mma::run(acc[i + 1], lo, b[2], b[3]);
         }
       }
       // Y goes to global memory through the buffer of C, whole rows at a time
