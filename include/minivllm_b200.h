@@ -23,6 +23,10 @@ extern "C" {
 /* Element types of activations, weights and of a non-quantised cache (each entry point says which it takes). */
 enum mv_dtype { MV_F16 = 0, MV_BF16 = 1, MV_F32 = 2 };
 
+/* What a gate g does to the value u beside it.  GELU_TANH: the tanh form of gelu.  CLAMPED (with a limit):
+ * g' sigmoid(1.702 g') (u' + 1) with g' = min(g, limit), u' = u clamped to +-limit. */
+enum mv_act { MV_ACT_NONE = -1, MV_ACT_SIGMOID = 0, MV_ACT_SILU = 1, MV_ACT_GELU_TANH = 2, MV_ACT_CLAMPED = 3 };
+
 enum mv_status {
   MV_OK = 0,
   MV_ERR_NULL = 1,        /* a required pointer is null */
@@ -417,17 +421,20 @@ int mv_silu_mul(void* out, const void* gate_up, int64_t gate_up_stride,
  * Steps between the sublayers of a decoder with an fp32 residual stream x (rows, width), updated in place, and RMS
  * norms over `groups` equal runs of channels.  dtype (MV_BF16 or MV_F32) is that of every void* operand; *_stride
  * are row strides in elements.  No counterpart in the reference.
- *   mv_embed_norm           x = embed[ids];  out = norm(x) * w_next
+ *   mv_embed_norm           x = embed[ids], or norm(embed[ids]) * w_post with w_post;  out = norm(x) * w_next, or x
+ *                           without w_next (in all of these)
  *   mv_gated_residual_norm  y' = y * sigmoid(gate + gate_bias) (gate may be null);
  *                           x += mult * norm(y') * w_post;  out = norm(x) * w_next
  *   mv_moe_residual_norm    the same with y = sum_k top_weights[t, k] * expert_rows[pos[t, k]]
  *                           + sigmoid(shared_gate[t]) * shared[t]   (shared may be null)
+ *   mv_pair_residual_norm   the same with y = (norm(a) * w_a + norm(b) * w_b) / 2, no gate
  *   mv_gated_group_norm     out = norm(y * silu(z)) * w
- *   mv_gate_mul             out = y * act(gate), act 0 = sigmoid, 1 = silu; a row of y is `heads` pieces
- *                           y_head_stride elements apart
+ *   mv_head_norm_gate       out = norm(y) * w * silu(z), norms over `heads` equal runs; w has one run's length
+ *   mv_gate_mul             out = gate applied to y (enum mv_act); a row of y is `heads` pieces y_head_stride
+ *                           elements apart
  */
 int mv_embed_norm(void* out, float* x, const int64_t* ids, const void* embed, int64_t vocab, const
-    void* w_next, int64_t rows, int width, int groups, float eps, int dtype, void* stream);
+    void* w_post, const void* w_next, int64_t rows, int width, int groups, float eps, int dtype, void* stream);
 int mv_gated_residual_norm(void* out, float* x, const void* y, int64_t y_stride, const void* gate,
     int64_t gate_stride, const void* gate_bias, const void* w_post, const void* w_next, float mult,
     int64_t rows, int width, int groups, float eps, int dtype, void* stream);
@@ -436,10 +443,16 @@ int mv_moe_residual_norm(void* out, float* x, const void* expert_rows, const int
     int64_t shared_gate_stride, const void* gate, int64_t gate_stride, const void* gate_bias, const
     void* w_post, const void* w_next, float mult, int64_t rows, int width, int groups, float eps,
     int dtype, void* stream);
+int mv_pair_residual_norm(void* out, float* x, const void* a, int64_t a_stride, const void* w_a, const
+    void* b, int64_t b_stride, const void* w_b, const void* w_post, const void* w_next, float mult,
+    int64_t rows, int width, int groups, float eps, int dtype, void* stream);
+int mv_head_norm_gate(void* out, const void* y, int64_t y_stride, const void* z, int64_t z_stride,
+    const void* w, int64_t rows, int width, int heads, float eps, int dtype, void* stream);
 int mv_gated_group_norm(void* out, const void* y, int64_t y_stride, const void* z, int64_t z_stride,
     const void* w, int64_t rows, int width, int groups, float eps, int dtype, void* stream);
 int mv_gate_mul(void* out, const void* y, int64_t y_stride, int64_t y_head_stride, int heads,
-    const void* gate, int64_t gate_stride, int act, int64_t rows, int cols, int dtype, void* stream);
+    const void* gate, int64_t gate_stride, int act, float limit, int64_t rows, int cols, int dtype, void*
+    stream);
 
 /*
  * Latent attention over a paged cache (num_blocks, block_size, rank + rot_dim) of rows [c | rotated key part].
@@ -486,29 +499,31 @@ int mv_ssm_scan(void* y, const void* xbc, const void* dt, int64_t dt_stride, con
 
 /*
  * Mixture of experts; the routing never leaves the device.
- *   mv_moe_route    idx, weight (tokens, top): largest logits + bias, softmax over them
+ *   mv_moe_route    idx, weight (tokens, top): largest logits + bias, softmax over them.  With `groups` > 1 the
+ *                   experts are that many equal runs, and only those of the `keep` runs with the largest maxima count
  *   mv_moe_sort     stable sort of the tokens * top entries by expert: pos[entry] = row, row_token[row] = token,
  *                   offsets (experts + 1) = row ranges
  *   mv_gather_rows  out[r] = x[row_token[r]]
- *   mv_grouped_rows rows of expert e times w[e]^T (out_dim, in_dim); gated: w[e] = [gate; up], silu(gate) * up
+ *   mv_grouped_rows rows of expert e times w[e]^T (out_dim, in_dim); with an activation (enum mv_act) w[e] =
+ *                   [gate; up] and the result is the gate applied to up
  * No counterpart in the reference.
  */
 int mv_moe_route(int32_t* idx, float* weight, const float* logits, int64_t logits_stride, const
-    float* bias, int64_t tokens, int experts, int top, void* stream);
+    float* bias, int64_t tokens, int experts, int top, int groups, int keep, void* stream);
 int64_t mv_moe_sort_workspace_bytes(int64_t tokens, int experts, int top);
 int mv_moe_sort(int32_t* pos, int32_t* row_token, int32_t* offsets, const int32_t* idx, int64_t
     tokens, int experts, int top, void* workspace, int64_t workspace_bytes, void* stream);
 int mv_gather_rows(void* out, const void* x, int64_t x_stride, const int32_t* row_token, int64_t
     rows, int width, int dtype, void* stream);
 int mv_grouped_rows(void* out, const void* x, const void* w, const int32_t* offsets, int experts,
-    int64_t rows, int in_dim, int out_dim, int gated, int dtype, void* stream);
+    int64_t rows, int in_dim, int out_dim, int act, float limit, int dtype, void* stream);
 
 /*
  * mv_grouped_rows on the tensor cores (tcgen05), bf16, in_dim a multiple of 8.  A bounded wait that runs out is
  * reported in *error_word, as by mv_prefill_varlen.
  */
 int mv_grouped_gemm(void* out, const void* x, const void* w, const int32_t* offsets, int experts,
-    int64_t rows, int in_dim, int out_dim, int gated, int* error_word, void* stream);
+    int64_t rows, int in_dim, int out_dim, int act, float limit, int* error_word, void* stream);
 
 /*
  * mv_latent_attention_rows for one query row per sequence on tensor cores, bf16: rank a multiple of 16 up to 512,
@@ -526,14 +541,15 @@ int mv_latent_decode(void* out, int64_t out_stride, int64_t out_head_stride, con
 
 /*
  * Prefill of latent attention with keys and values expanded per head, bf16, tcgen05.
- *   mv_latent_gather   out[cu_k[s] + j] = cache row of position j of sequence s (bf16 or fp32, rows of whole 16 bytes)
+ *   mv_latent_gather   out[cu_k[s] + j] = cache row of position first[s] + j of sequence s (first null: j; bf16 or fp32,
+ *                      rows of whole 16 bytes)
  *   mv_latent_prefill  q (tokens, heads * (dim + rot_dim)), k (keys, heads * dim), k_rot (keys, rot_dim) shared by the
  *                      heads, v (keys, heads * vdim); row strides in elements; sequence s has queries cu_q[s] .. at the
  *                      end of its keys cu_k[s] ..; sizes multiples of 8, 64-column boxes: at most three for dim and
  *                      rot_dim together, two for vdim; sink may be null.  Bounded waits report in *error_word.
  */
-int mv_latent_gather(void* out, const void* cache, const int32_t* cu_k, int num_seqs, int64_t keys,
-    const int32_t* block_tables, int64_t bt_stride, int max_blocks, int block_size, int64_t
+int mv_latent_gather(void* out, const void* cache, const int32_t* cu_k, const int32_t* first, int
+    num_seqs, int64_t keys, const int32_t* block_tables, int64_t bt_stride, int max_blocks, int block_size, int64_t
     num_blocks, int row, int dtype, void* stream);
 int mv_latent_prefill(void* out, int64_t out_stride, const void* q, int64_t q_stride, const void* k,
     int64_t k_stride, const void* k_rot, int64_t k_rot_stride, const void* v, int64_t v_stride,
@@ -558,6 +574,65 @@ int mv_ssm_step(void* y, const void* u, int64_t u_stride, const void* w, const v
     const void* conv_state, const void* dt, int64_t dt_stride, const void* dt_bias, const void*
     A_log, const void* D, int num_seqs, const int32_t* slots, const int32_t* start, float* state,
     int num_slots, int heads, int vdim, int state_dim, int groups, int dtype, void* stream);
+
+/*
+ * Grouped-query attention with a sliding window over a paged cache of rows [kv_heads * dim keys | kv_heads * vdim
+ * values].  Position i sees the keys j with 0 <= i - j < window; score = scale (q . k) + bias[h * bias_stride +
+ * min(i - j, distances - 1)] (fp32; null: none); exp(sink[h]) joins the denominator (null: none).
+ *   mv_kv_norm_store          q (in place) and k, each row of all heads: RMS norm with a weight per row; [k | v] goes to
+ *                             kv_out (tokens, row; may be null) and to cache[slot] (slot < 0 skips)
+ *   mv_window_attention_rows  any sizes up to vdim 1,024; token t belongs to the sequence of cu_q (null: row t)
+ *   mv_window_decode          one token per sequence, bf16, dim and vdim multiples of 8 up to 256; workspace_bytes is
+ *                             -1 when the sizes are not taken, most_keys = min(window, max_blocks * block_size)
+ *   mv_window_prefill         packed queries and keys as in mv_latent_prefill (a sequence's keys begin at or before the
+ *                             first one that its first query sees), bf16, dim up to 192, vdim up to 128, multiples of 8;
+ *                             mv_window_prefill_distances = largest `distances` taken (-1: sizes not taken)
+ * out is (tokens, heads * vdim).  No counterpart in the reference.
+ */
+int mv_kv_norm_store(void* q, const void* k, const void* v, int64_t stride, const void* q_weight, const
+    void* k_weight, void* kv_out, void* cache, const int64_t* slot_mapping, int64_t num_slots, int64_t
+    tokens, int q_rows, int k_rows, int v_rows, float eps, int dtype, void* stream);
+int mv_window_attention_rows(void* out, const void* q, int64_t q_stride, const void* cache, const
+    int32_t* block_tables, int64_t bt_stride, int max_blocks, int block_size, int64_t num_blocks,
+    const int32_t* cu_q, int num_seqs, const int64_t* positions, const float* bias, int64_t
+    bias_stride, int distances, const void* sink, int64_t tokens, int heads, int kv_heads, int dim,
+    int vdim, int64_t window, float scale, int dtype, void* stream);
+int64_t mv_window_decode_workspace_bytes(int batch, int heads, int kv_heads, int dim, int vdim, int64_t
+    most_keys);
+int mv_window_decode(void* out, const void* q, int64_t q_stride, const void* cache, const int32_t*
+    block_tables, int64_t bt_stride, int max_blocks, int block_size, int64_t num_blocks, const int64_t*
+    positions, const float* bias, int64_t bias_stride, int distances, const void* sink, int batch,
+    int heads, int kv_heads, int dim, int vdim, int64_t window, float scale, void* workspace, int64_t
+    workspace_bytes, void* stream);
+int mv_window_prefill_distances(int dim, int vdim);
+int mv_window_prefill(void* out, int64_t out_stride, const void* q, int64_t q_stride, const void* k,
+    int64_t k_stride, const void* v, int64_t v_stride, const int32_t* cu_q, const int32_t* cu_k, int
+    num_seqs, int64_t tokens, int64_t keys, int heads, int kv_heads, int dim, int vdim, int64_t window,
+    float scale, const float* bias, int64_t bias_stride, int distances, const void* sink, int*
+    error_word, void* stream);
+
+/*
+ * Matrix-state recurrences, fp32 state (num_slots, heads, dim, vdim) updated in place, one read-out per token; dim up
+ * to 256.  cu, slots and start as in mv_conv_silu.  With cu null (one token per sequence) the head's norm and the output
+ * gate follow in the same launch: out = rms_norm(o) * norm_w * silu(gate), norm_w (vdim); with cu they are ignored.
+ *   mv_gla_scan    S <- diag(sigmoid(z)^(1 / tau)) S + k v^T,  o = S^T (q_scale q);  rows of q, k, v share one stride
+ *   mv_delta_scan  S <- g S;  u = sigmoid(beta) (v - S^T k);  S <- S + k u^T;  o = S^T q, with q and k scaled to unit
+ *                  length per head (1e-6 added to the sum of squares), q by q_scale too, and
+ *                  g = exp(-exp(A_log) softplus(a + dt_bias)); rows of qkv are [q: kv_heads * dim | k | v: heads * vdim],
+ *                  after the convolution and silu, or with cu null before them (conv_state is read only)
+ * dtype MV_BF16 or MV_F32.  No counterpart in the reference.
+ */
+int mv_gla_scan(void* out, int64_t out_stride, const void* q, const void* k, const void* v, int64_t
+    stride, const void* z, int64_t z_stride, float tau, const int32_t* cu, int num_seqs, const
+    int32_t* slots, const int32_t* start, float* state, int num_slots, int heads, int dim, int vdim,
+    float q_scale, const void* gate, int64_t gate_stride, const void* norm_w, float eps, int dtype,
+    void* stream);
+int mv_delta_scan(void* out, int64_t out_stride, const void* qkv, int64_t stride, const void* beta,
+    const void* a, int64_t ba_stride, const void* A_log, const void* dt_bias, const int32_t* cu, int
+    num_seqs, const int32_t* slots, const int32_t* start, float* state, int num_slots, int heads,
+    int kv_heads, int dim, int vdim, float q_scale, const void* conv_w, int taps, const void*
+    conv_state, const void* gate, int64_t gate_stride, const void* norm_w, float eps, int dtype,
+    void* stream);
 
 #ifdef __cplusplus
 }

@@ -67,15 +67,19 @@ SIGNATURES = {
     "mv_add_rmsnorm": (_c_int, [_c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_i64, _c_i64, _c_ptr, _c_f32, _c_i64, _c_int,
                                 _c_int, _c_ptr]),
     "mv_silu_mul": (_c_int, [_c_ptr, _c_ptr, _c_i64, _c_i64, _c_int, _c_int, _c_ptr]),
-    "mv_embed_norm": (_c_int, [_c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_i64, _c_ptr, _c_i64, _c_int, _c_int, _c_f32,
+    "mv_embed_norm": (_c_int, [_c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_i64, _c_ptr, _c_ptr, _c_i64, _c_int, _c_int, _c_f32,
         _c_int, _c_ptr]),
     "mv_gated_residual_norm": (_c_int, [_c_ptr, _c_ptr, _c_ptr, _c_i64, _c_ptr, _c_i64, _c_ptr, _c_ptr, _c_ptr,
         _c_f32, _c_i64, _c_int, _c_int, _c_f32, _c_int, _c_ptr]),
     "mv_moe_residual_norm": (_c_int, [_c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_int, _c_ptr, _c_i64, _c_ptr,
         _c_i64, _c_ptr, _c_i64, _c_ptr, _c_ptr, _c_ptr, _c_f32, _c_i64, _c_int, _c_int, _c_f32, _c_int, _c_ptr]),
+    "mv_pair_residual_norm": (_c_int, [_c_ptr, _c_ptr, _c_ptr, _c_i64, _c_ptr, _c_ptr, _c_i64, _c_ptr, _c_ptr, _c_ptr,
+        _c_f32, _c_i64, _c_int, _c_int, _c_f32, _c_int, _c_ptr]),
+    "mv_head_norm_gate": (_c_int, [_c_ptr, _c_ptr, _c_i64, _c_ptr, _c_i64, _c_ptr, _c_i64, _c_int, _c_int, _c_f32,
+        _c_int, _c_ptr]),
     "mv_gated_group_norm": (_c_int, [_c_ptr, _c_ptr, _c_i64, _c_ptr, _c_i64, _c_ptr, _c_i64, _c_int, _c_int, _c_f32,
         _c_int, _c_ptr]),
-    "mv_gate_mul": (_c_int, [_c_ptr, _c_ptr, _c_i64, _c_i64, _c_int, _c_ptr, _c_i64, _c_int, _c_i64, _c_int, _c_int,
+    "mv_gate_mul": (_c_int, [_c_ptr, _c_ptr, _c_i64, _c_i64, _c_int, _c_ptr, _c_i64, _c_int, _c_f32, _c_i64, _c_int, _c_int,
         _c_ptr]),
     "mv_latent_prep": (_c_int, [_c_ptr, _c_i64, _c_ptr, _c_i64, _c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_i64, _c_ptr,
         _c_ptr, _c_ptr, _c_i64, _c_i64, _c_int, _c_int, _c_int, _c_int, _c_int, _c_f32, _c_int, _c_ptr]),
@@ -88,19 +92,19 @@ SIGNATURES = {
         _c_int, _c_int, _c_ptr]),
     "mv_ssm_scan": (_c_int, [_c_ptr, _c_ptr, _c_ptr, _c_i64, _c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_int, _c_ptr, _c_ptr,
         _c_ptr, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_ptr]),
-    "mv_moe_route": (_c_int, [_c_ptr, _c_ptr, _c_ptr, _c_i64, _c_ptr, _c_i64, _c_int, _c_int, _c_ptr]),
+    "mv_moe_route": (_c_int, [_c_ptr, _c_ptr, _c_ptr, _c_i64, _c_ptr, _c_i64, _c_int, _c_int, _c_int, _c_int, _c_ptr]),
     "mv_moe_sort_workspace_bytes": (_c_i64, [_c_i64, _c_int, _c_int]),
     "mv_moe_sort": (_c_int, [_c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_i64, _c_int, _c_int, _c_ptr, _c_i64, _c_ptr]),
     "mv_gather_rows": (_c_int, [_c_ptr, _c_ptr, _c_i64, _c_ptr, _c_i64, _c_int, _c_int, _c_ptr]),
-    "mv_grouped_rows": (_c_int, [_c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_int, _c_i64, _c_int, _c_int, _c_int, _c_int,
+    "mv_grouped_rows": (_c_int, [_c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_int, _c_i64, _c_int, _c_int, _c_int, _c_f32, _c_int,
         _c_ptr]),
-    "mv_grouped_gemm": (_c_int, [_c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_int, _c_i64, _c_int, _c_int, _c_int, _c_ptr,
+    "mv_grouped_gemm": (_c_int, [_c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_int, _c_i64, _c_int, _c_int, _c_int, _c_f32, _c_ptr,
         _c_ptr]),
     "mv_latent_decode_workspace_bytes": (_c_i64, [_c_int, _c_int, _c_int, _c_int]),
     "mv_latent_decode": (_c_int, [_c_ptr, _c_i64, _c_i64, _c_ptr, _c_i64, _c_i64, _c_ptr, _c_i64, _c_i64, _c_ptr,
         _c_ptr, _c_i64, _c_int, _c_int, _c_i64, _c_ptr, _c_ptr, _c_ptr, _c_int, _c_int, _c_int, _c_int, _c_f32,
         _c_ptr, _c_i64, _c_ptr, _c_ptr]),
-    "mv_latent_gather": (_c_int, [_c_ptr, _c_ptr, _c_ptr, _c_int, _c_i64, _c_ptr, _c_i64, _c_int, _c_int, _c_i64,
+    "mv_latent_gather": (_c_int, [_c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_int, _c_i64, _c_ptr, _c_i64, _c_int, _c_int, _c_i64,
         _c_int, _c_int, _c_ptr]),
     "mv_latent_prefill": (_c_int, [_c_ptr, _c_i64, _c_ptr, _c_i64, _c_ptr, _c_i64, _c_ptr, _c_i64, _c_ptr, _c_i64,
         _c_ptr, _c_ptr, _c_int, _c_i64, _c_i64, _c_int, _c_int, _c_int, _c_int, _c_f32, _c_ptr, _c_ptr, _c_ptr]),
@@ -109,6 +113,22 @@ SIGNATURES = {
         _c_int, _c_ptr, _c_ptr, _c_ptr, _c_int, _c_int, _c_int, _c_int, _c_int, _c_ptr]),
     "mv_ssm_step": (_c_int, [_c_ptr, _c_ptr, _c_i64, _c_ptr, _c_ptr, _c_int, _c_ptr, _c_ptr, _c_i64, _c_ptr, _c_ptr,
         _c_ptr, _c_int, _c_ptr, _c_ptr, _c_ptr, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_ptr]),
+    "mv_kv_norm_store": (_c_int, [_c_ptr, _c_ptr, _c_ptr, _c_i64, _c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_i64, _c_i64,
+        _c_int, _c_int, _c_int, _c_f32, _c_int, _c_ptr]),
+    "mv_window_attention_rows": (_c_int, [_c_ptr, _c_ptr, _c_i64, _c_ptr, _c_ptr, _c_i64, _c_int, _c_int, _c_i64, _c_ptr,
+        _c_int, _c_ptr, _c_ptr, _c_i64, _c_int, _c_ptr, _c_i64, _c_int, _c_int, _c_int, _c_int, _c_i64, _c_f32, _c_int,
+        _c_ptr]),
+    "mv_window_decode_workspace_bytes": (_c_i64, [_c_int, _c_int, _c_int, _c_int, _c_int, _c_i64]),
+    "mv_window_decode": (_c_int, [_c_ptr, _c_ptr, _c_i64, _c_ptr, _c_ptr, _c_i64, _c_int, _c_int, _c_i64, _c_ptr, _c_ptr,
+        _c_i64, _c_int, _c_ptr, _c_int, _c_int, _c_int, _c_int, _c_int, _c_i64, _c_f32, _c_ptr, _c_i64, _c_ptr]),
+    "mv_window_prefill_distances": (_c_int, [_c_int, _c_int]),
+    "mv_window_prefill": (_c_int, [_c_ptr, _c_i64, _c_ptr, _c_i64, _c_ptr, _c_i64, _c_ptr, _c_i64, _c_ptr, _c_ptr, _c_int,
+        _c_i64, _c_i64, _c_int, _c_int, _c_int, _c_int, _c_i64, _c_f32, _c_ptr, _c_i64, _c_int, _c_ptr, _c_ptr, _c_ptr]),
+    "mv_gla_scan": (_c_int, [_c_ptr, _c_i64, _c_ptr, _c_ptr, _c_ptr, _c_i64, _c_ptr, _c_i64, _c_f32, _c_ptr, _c_int, _c_ptr,
+        _c_ptr, _c_ptr, _c_int, _c_int, _c_int, _c_int, _c_f32, _c_ptr, _c_i64, _c_ptr, _c_f32, _c_int, _c_ptr]),
+    "mv_delta_scan": (_c_int, [_c_ptr, _c_i64, _c_ptr, _c_i64, _c_ptr, _c_ptr, _c_i64, _c_ptr, _c_ptr, _c_ptr, _c_int,
+        _c_ptr, _c_ptr, _c_ptr, _c_int, _c_int, _c_int, _c_int, _c_int, _c_f32, _c_ptr, _c_int, _c_ptr, _c_ptr, _c_i64,
+        _c_ptr, _c_f32, _c_int, _c_ptr]),
 }
 
 _lib = None

@@ -17,10 +17,12 @@ COMMON = ["api.cu", "metadata.cu", "sampling.cu"]
 GROUPS = {
     "qwen3": ["store_kvcache.cu", "paged_decode.cu", "paged_decode_int8.cu", "prefill_varlen.cu",
               "paged_decode_static.cu", "pre_attention.cu", "comm.cu"],
-    "sipazen": ["norms.cu", "latent_attention.cu", "latent_decode.cu", "latent_prefill.cu", "mamba2.cu",
+    "sipazen": ["norms.cu", "latent_attention.cu", "latent_decode.cu", "latent_prefill.cu", "short_conv.cu", "mamba2.cu",
                 "mamba2_chunk.cu", "moe.cu", "grouped_gemm.cu"],
+    "fozerax": ["norms.cu", "window_attention.cu", "latent_prefill.cu", "short_conv.cu", "gla.cu", "gated_delta.cu", "moe.cu",
+                "grouped_gemm.cu"],
 }
-SOURCES = COMMON + [s for g in GROUPS.values() for s in g]
+SOURCES = COMMON + list(dict.fromkeys(s for g in GROUPS.values() for s in g))
 NVCC_FLAGS = [
     "-gencode", "arch=compute_100a,code=sm_100a",
     "-O3", "-std=c++17", "-lineinfo",

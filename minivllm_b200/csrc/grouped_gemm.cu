@@ -4,7 +4,7 @@
 // The weights are the M side (128 output features = 128 TMEM lanes), the tokens the N side, so that a decode step
 // with a handful of tokens per expert wastes no tensor-core rows and streams each weight once, and a prefill step
 // uses the same kernel with 128-token tiles.  A unit of work is two 128-feature tiles times one token tile: the gate
-// and up rows of the same features (kGated: the epilogue writes silu(gate) * up), or 256 consecutive features.
+// and up rows of the same features (kGated: the epilogue applies the gate, glu_act), or 256 consecutive features.
 // Persistent CTAs walk the units of all experts in order; unit ranges come from the device-side offsets.
 //   warps 0-3  epilogue: accumulators -> registers -> global (a store instruction covers 32 consecutive features)
 //   warp 4     TMA producer: two weight tiles and a token tile per 64-deep slab, ring of kStages
@@ -34,6 +34,8 @@ struct GmParams {
   __nv_bfloat16* out;
   const int32_t* offsets;
   int experts, in_dim, out_dim, out_tiles;
+  int act;
+  float limit;
   int* error_word;
 };
 
@@ -190,10 +192,18 @@ grouped_gemm_kernel(const __grid_constant__ CUtensorMap tmap_w, const __grid_con
         tc::wait_ld();
         if (kGated) {
           if (o < p.out_dim) {
+            auto apply = [&](auto act) {
 #pragma unroll
-            for (int j = 0; j < kChunk; ++j) {
-              const float g = __uint_as_float(a[j]), v = __uint_as_float(c[j]);
-              if (j < lim) dst[static_cast<int64_t>(j) * p.out_dim] = __float2bfloat16_rn(__fdividef(g, 1.f + __expf(-g)) * v);
+              for (int j = 0; j < kChunk; ++j)
+                if (j < lim)
+                  dst[static_cast<int64_t>(j) * p.out_dim] = __float2bfloat16_rn(
+                      glu_act<__nv_bfloat16>(decltype(act)::value, __uint_as_float(a[j]), __uint_as_float(c[j]), p.limit));
+            };
+            switch (p.act) {
+              case MV_ACT_SILU: apply(std::integral_constant<int, MV_ACT_SILU>{}); break;
+              case MV_ACT_SIGMOID: apply(std::integral_constant<int, MV_ACT_SIGMOID>{}); break;
+              case MV_ACT_GELU_TANH: apply(std::integral_constant<int, MV_ACT_GELU_TANH>{}); break;
+              default: apply(std::integral_constant<int, MV_ACT_CLAMPED>{});
             }
           }
         } else {
@@ -238,8 +248,11 @@ static int launch_grouped(const CUtensorMap& tw, const void* x, int64_t rows, Gm
 }  // namespace mv
 
 extern "C" int mv_grouped_gemm(void* out, const void* x, const void* w, const int32_t* offsets, int experts,
-                               int64_t rows, int in_dim, int out_dim, int gated, int* error_word, void* stream) {
+                               int64_t rows, int in_dim, int out_dim, int act, float limit, int* error_word,
+                               void* stream) {
   using namespace mv;
+  if (act < MV_ACT_NONE || act > MV_ACT_CLAMPED) return fail(MV_ERR_SHAPE, "grouped_gemm: activation %d", act);
+  const bool gated = act != MV_ACT_NONE;
   if (rows < 0 || experts <= 0 || in_dim <= 0 || out_dim <= 0) return fail(MV_ERR_SHAPE, "grouped_gemm: %d x %d", out_dim, in_dim);
   if (in_dim % 8) return fail(MV_ERR_SHAPE, "grouped_gemm: in_dim %d is not a multiple of 8", in_dim);
   if (experts > kGmMaxExperts) return fail(MV_ERR_LIMIT, "grouped_gemm: %d experts (at most %d)", experts, kGmMaxExperts);
@@ -252,7 +265,7 @@ extern "C" int mv_grouped_gemm(void* out, const void* x, const void* w, const in
   const int rc = make_tmap_bf16(&tw, w, in_dim, wrows, 1, in_dim, wrows * in_dim, 128, 1, "grouped_gemm");
   if (rc) return rc;
   GmParams p{static_cast<__nv_bfloat16*>(out), offsets, experts, in_dim, out_dim,
-             gated ? (out_dim + 127) / 128 : (out_dim + 255) / 256, error_word};
+             gated ? (out_dim + 127) / 128 : (out_dim + 255) / 256, act, limit, error_word};
   auto st = static_cast<cudaStream_t>(stream);
   // token tile by the mean number of rows of an expert; an expert with more has several tiles
   const int64_t mean = (rows + experts - 1) / experts;

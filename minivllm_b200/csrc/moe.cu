@@ -17,7 +17,9 @@ constexpr int kRtMaxPer = 32;      // experts per lane: up to 1024 experts
 template <int kPer>
 __global__ void __launch_bounds__(kRtThreads)
 moe_route_kernel(int32_t* __restrict__ idx, float* __restrict__ weight, const float* __restrict__ logits,
-                 int64_t stride, const float* __restrict__ bias, int64_t tokens, int experts, int top) {
+                 int64_t stride, const float* __restrict__ bias, int64_t tokens, int experts, int top, int groups,
+                 int keep) {
+  __shared__ float s_best[kRtThreads / 32][32 * kPer];      // per group of experts: its largest logit
   const int lane = threadIdx.x & 31;
   const int64_t t = static_cast<int64_t>(blockIdx.x) * (kRtThreads / 32) + (threadIdx.x >> 5);
   if (t >= tokens) return;
@@ -28,6 +30,28 @@ moe_route_kernel(int32_t* __restrict__ idx, float* __restrict__ weight, const fl
     z[i] = e < experts ? logits[t * stride + e] + (bias ? bias[e] : 0.f) : -INFINITY;
   }
   uint32_t taken = 0;
+  if (groups > 1) {
+    // a group is dropped when `keep` groups come before it (larger maximum, ties: lower index)
+    float* best = s_best[threadIdx.x >> 5];
+    const int size = experts / groups;
+    for (int i = lane; i < groups; i += 32) {
+      float m = -INFINITY;
+      for (int e = i * size; e < (i + 1) * size; ++e) m = fmaxf(m, logits[t * stride + e] + (bias ? bias[e] : 0.f));
+      best[i] = m;
+    }
+    __syncwarp();
+#pragma unroll
+    for (int i = 0; i < kPer; ++i) {
+      const int e = i * 32 + lane;
+      if (e < experts) {
+        const int mine = e / size;
+        const float m = best[mine];
+        int before = 0;
+        for (int g = 0; g < groups; ++g) before += best[g] > m || (best[g] == m && g < mine);
+        if (before >= keep) taken |= 1u << i;
+      }
+    }
+  }
   float first = 0.f, sum = 0.f;
   for (int k = 0; k < top; ++k) {
     float best = -INFINITY;
@@ -188,12 +212,12 @@ gather_rows_kernel(T* __restrict__ out, const T* __restrict__ x, int64_t x_strid
 }
 
 // Grouped product, plain form: rows [offsets[e], offsets[e+1]) of x times w[e] (out_dim, in_dim) transposed.
-// kGated: w[e] holds 2 * out_dim rows (gate, then up) and the result is silu(gate) * up.
+// kGated: w[e] holds 2 * out_dim rows (gate, then up) and the result is the gate applied to up (glu_act).
 constexpr int kGgRows = 32, kGgCols = 64, kGgK = 32, kGgThreads = 256;
 template <typename T, bool kGated>
 __global__ void __launch_bounds__(kGgThreads)
 grouped_rows_kernel(T* __restrict__ out, const T* __restrict__ x, const T* __restrict__ w,
-                    const int32_t* __restrict__ offsets, int experts, int in_dim, int out_dim) {
+                    const int32_t* __restrict__ offsets, int experts, int in_dim, int out_dim, int act, float limit) {
   __shared__ float sx[kGgRows][kGgK + 1], sw[kGated ? 2 : 1][kGgCols][kGgK + 1];
   __shared__ int s_e, s_r0, s_r1;
   if (threadIdx.x == 0) {
@@ -251,7 +275,7 @@ grouped_rows_kernel(T* __restrict__ out, const T* __restrict__ x, const T* __res
     for (int j = 0; j < 4; ++j) {
       const int c = c0 + tc + 16 * j;
       if (c >= out_dim) continue;
-      const float v = kGated ? silu_f(acc[0][i][j]) * acc[kGated ? 1 : 0][i][j] : acc[0][i][j];
+      const float v = kGated ? glu_act<float>(act, acc[0][i][j], acc[kGated ? 1 : 0][i][j], limit) : acc[0][i][j];
       out[static_cast<int64_t>(r0 + r) * out_dim + c] = Elem<T>::from_f(v);
     }
   }
@@ -260,15 +284,18 @@ grouped_rows_kernel(T* __restrict__ out, const T* __restrict__ x, const T* __res
 }  // namespace mv
 
 extern "C" int mv_moe_route(int32_t* idx, float* weight, const float* logits, int64_t logits_stride, const float* bias,
-                            int64_t tokens, int experts, int top, void* stream) {
+                            int64_t tokens, int experts, int top, int groups, int keep, void* stream) {
   using namespace mv;
   if (tokens < 0 || experts <= 0 || top <= 0 || top > experts) return fail(MV_ERR_SHAPE, "moe_route: experts %d top %d", experts, top);
+  if (groups <= 0 || experts % groups || keep <= 0 || keep > groups || experts / groups * keep < top)
+    return fail(MV_ERR_SHAPE, "moe_route: %d groups of %d experts, %d kept, top %d", groups, experts, keep, top);
   if (experts > 32 * kRtMaxPer) return fail(MV_ERR_LIMIT, "moe_route: %d experts (at most %d)", experts, 32 * kRtMaxPer);
   if (tokens == 0) return MV_OK;
   if (!idx || !weight || !logits) return fail(MV_ERR_NULL, "moe_route: null pointer");
   const unsigned grid = static_cast<unsigned>((tokens + kRtThreads / 32 - 1) / (kRtThreads / 32));
   auto go = [&](auto kernel) {
-    kernel<<<grid, kRtThreads, 0, static_cast<cudaStream_t>(stream)>>>(idx, weight, logits, logits_stride, bias, tokens, experts, top);
+    kernel<<<grid, kRtThreads, 0, static_cast<cudaStream_t>(stream)>>>(idx, weight, logits, logits_stride, bias, tokens, experts, top,
+                                                                        keep < groups ? groups : 1, keep);
   };
   if (experts <= 64) go(moe_route_kernel<2>);
   else if (experts <= 256) go(moe_route_kernel<8>);
@@ -328,8 +355,9 @@ extern "C" int mv_gather_rows(void* out, const void* x, int64_t x_stride, const 
 }
 
 extern "C" int mv_grouped_rows(void* out, const void* x, const void* w, const int32_t* offsets, int experts,
-                               int64_t rows, int in_dim, int out_dim, int gated, int dtype, void* stream) {
+                               int64_t rows, int in_dim, int out_dim, int act, float limit, int dtype, void* stream) {
   using namespace mv;
+  if (act < MV_ACT_NONE || act > MV_ACT_CLAMPED) return fail(MV_ERR_SHAPE, "grouped_rows: activation %d", act);
   if (dtype != MV_BF16 && dtype != MV_F32) return fail(MV_ERR_DTYPE, "grouped_rows: dtype %d", dtype);
   if (rows < 0 || experts <= 0 || in_dim <= 0 || out_dim <= 0) return fail(MV_ERR_SHAPE, "grouped_rows: %d x %d", out_dim, in_dim);
   if (rows == 0) return MV_OK;
@@ -343,8 +371,8 @@ extern "C" int mv_grouped_rows(void* out, const void* x, const void* w, const in
     using T = decltype(tag);
     auto* o = static_cast<T*>(out);
     auto *a = static_cast<const T*>(x), *b = static_cast<const T*>(w);
-    if (gated) grouped_rows_kernel<T, true><<<grid, kGgThreads, 0, st>>>(o, a, b, offsets, experts, in_dim, out_dim);
-    else grouped_rows_kernel<T, false><<<grid, kGgThreads, 0, st>>>(o, a, b, offsets, experts, in_dim, out_dim);
+    if (act != MV_ACT_NONE) grouped_rows_kernel<T, true><<<grid, kGgThreads, 0, st>>>(o, a, b, offsets, experts, in_dim, out_dim, act, limit);
+    else grouped_rows_kernel<T, false><<<grid, kGgThreads, 0, st>>>(o, a, b, offsets, experts, in_dim, out_dim, act, limit);
     return check_launch("grouped_rows");
   };
   return dtype == MV_F32 ? run(float{}) : run(__nv_bfloat16{});

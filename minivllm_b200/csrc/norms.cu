@@ -14,15 +14,16 @@ constexpr int kNormThreads = 256;
 constexpr int kNormWarps = kNormThreads / 32;
 constexpr int kMaxTop = 256;     // choices per token
 
-enum { SRC_EMBED = 0, SRC_ROWS = 1, SRC_EXPERTS = 2 };
+enum { SRC_EMBED = 0, SRC_ROWS = 1, SRC_EXPERTS = 2, SRC_PAIR = 3 };
 
 template <typename T> struct ResidualParams {
-  T* out;                  // (rows, width): normalised residual
+  T* out;                  // (rows, width): normalised residual, or the residual itself without w_next
   float* x;                // (rows, width): residual stream, updated (SRC_EMBED: written)
   const T* y; int64_t y_stride;                 // SRC_ROWS: sublayer result;  SRC_EXPERTS: expert rows (sorted)
   const T* gate; int64_t gate_stride; const T* gate_bias;   // logits of the element gate (null: no gate)
-  const T* w_post;         // norm of the sublayer's result
-  const T* w_next;         // norm of the new residual
+  const T* y2; int64_t y2_stride; const T* w_y; const T* w_y2;   // SRC_PAIR: half the sum of norm(y) w_y and norm(y2) w_y2
+  const T* w_post;         // norm of the sublayer's result (SRC_EMBED: of the embedding row, may be null)
+  const T* w_next;         // norm of the new residual (null: none)
   const int64_t* ids; const T* embed; int64_t vocab;        // SRC_EMBED
   const int32_t* pos; const float* topw; int top;           // SRC_EXPERTS: row of (token, k) and its weight
   const T* shared; int64_t shared_stride; const T* sg; int64_t sg_stride;   // shared expert and its scalar gate
@@ -58,8 +59,47 @@ __global__ void __launch_bounds__(kNormThreads) residual_norm_kernel(const Resid
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
   const int64_t row = blockIdx.x;
   const GroupPlan gp(p.width, p.groups, V, warp);
+  const bool post = SRC != SRC_EMBED || p.w_post;
   float* x = p.x + row * p.width;
   float sgate = 0.f;
+  if (SRC == SRC_PAIR) {       // sums of squares of both rows
+    for (int g = gp.g0; g < p.groups; g += gp.cg) {
+      float a = 0.f, b = 0.f;
+      for (int i = gp.sub * 32 + lane; i < gp.chunks; i += gp.wpg * 32) {
+        const int c = g * gp.gs + i * V;
+        float u[V], v[V];
+        Vec<T, V>::load(p.y + row * p.y_stride + c, u);
+        Vec<T, V>::load(p.y2 + row * p.y2_stride + c, v);
+#pragma unroll
+        for (int e = 0; e < V; ++e) {
+          a = fmaf(u[e], u[e], a);
+          b = fmaf(v[e], v[e], b);
+        }
+      }
+      a = warp_sum(a);
+      b = warp_sum(b);
+      if (lane == 0) {
+        part[g * gp.wpg + gp.sub] = a;
+        part2[g * gp.wpg + gp.sub] = b;
+      }
+    }
+    __syncthreads();
+    for (int g = gp.g0; g < p.groups; g += gp.cg) {
+      const float ra = 0.5f * group_rs(part, g, gp.wpg, gp.gs, p.eps), rb = 0.5f * group_rs(part2, g, gp.wpg, gp.gs, p.eps);
+      for (int i = gp.sub * 32 + lane; i < gp.chunks; i += gp.wpg * 32) {
+        const int c = g * gp.gs + i * V;
+        float u[V], v[V], wu[V], wv[V];
+        Vec<T, V>::load(p.y + row * p.y_stride + c, u);
+        Vec<T, V>::load(p.y2 + row * p.y2_stride + c, v);
+        Vec<T, V>::load(p.w_y + c, wu);
+        Vec<T, V>::load(p.w_y2 + c, wv);
+#pragma unroll
+        for (int e = 0; e < V; ++e) u[e] = u[e] * ra * wu[e] + v[e] * rb * wv[e];
+        Vec<float, V>::store(s_row + c, u);      // read back by the thread that wrote it
+      }
+    }
+    __syncthreads();
+  }
   int64_t token = 0;
   if (SRC == SRC_EMBED) {
     token = p.ids[row];
@@ -83,10 +123,12 @@ __global__ void __launch_bounds__(kNormThreads) residual_norm_kernel(const Resid
       float v[V];
       if (SRC == SRC_EMBED) {
         Vec<T, V>::load(p.embed + token * p.width + c, v);
-        Vec<float, V>::store(x + c, v);
+        if (!post) Vec<float, V>::store(x + c, v);
       } else {
         if (SRC == SRC_ROWS) {
           Vec<T, V>::load(p.y + row * p.y_stride + c, v);
+        } else if (SRC == SRC_PAIR) {
+          Vec<float, V>::load(s_row + c, v);
         } else {
 #pragma unroll
           for (int e = 0; e < V; ++e) v[e] = 0.f;
@@ -127,7 +169,7 @@ __global__ void __launch_bounds__(kNormThreads) residual_norm_kernel(const Resid
   }
   __syncthreads();
   const float* fin = part;
-  if (SRC != SRC_EMBED) {
+  if (post) {
     for (int g = gp.g0; g < p.groups; g += gp.cg) {
       const float rs = group_rs(part, g, gp.wpg, gp.gs, p.eps);
       float acc = 0.f;
@@ -136,10 +178,10 @@ __global__ void __launch_bounds__(kNormThreads) residual_norm_kernel(const Resid
         float v[V], w[V], r[V];
         Vec<float, V>::load(s_row + c, v);
         Vec<T, V>::load(p.w_post + c, w);
-        Vec<float, V>::load(x + c, r);
+        if (SRC != SRC_EMBED) Vec<float, V>::load(x + c, r);
 #pragma unroll
         for (int e = 0; e < V; ++e) {
-          r[e] = fmaf(p.mult, v[e] * rs * w[e], r[e]);
+          r[e] = SRC == SRC_EMBED ? v[e] * rs * w[e] : fmaf(p.mult, v[e] * rs * w[e], r[e]);
           acc = fmaf(r[e], r[e], acc);
         }
         Vec<float, V>::store(x + c, r);
@@ -157,9 +199,11 @@ __global__ void __launch_bounds__(kNormThreads) residual_norm_kernel(const Resid
       const int c = g * gp.gs + i * V;
       float v[V], w[V];
       Vec<float, V>::load(s_row + c, v);
-      Vec<T, V>::load(p.w_next + c, w);
+      if (p.w_next) {
+        Vec<T, V>::load(p.w_next + c, w);
 #pragma unroll
-      for (int e = 0; e < V; ++e) v[e] = v[e] * rs * w[e];
+        for (int e = 0; e < V; ++e) v[e] = v[e] * rs * w[e];
+      }
       Vec<T, V>::store(p.out + row * p.width + c, v);
     }
   }
@@ -168,12 +212,12 @@ __global__ void __launch_bounds__(kNormThreads) residual_norm_kernel(const Resid
 // The same with the row in registers: at most eight groups, kCh pieces of eight channels per thread.  Everything a row
 // needs is requested at once; two block-wide sums follow.
 template <typename T, int SRC, int kCh>
-__global__ void __launch_bounds__(kNormThreads, SRC == SRC_EXPERTS ? (kCh == 1 ? 3 : 2) : 3) residual_norm_reg_kernel(const ResidualParams<T> p) {
-  __shared__ float part[kNormWarps], part2[kNormWarps];
+__global__ void __launch_bounds__(kNormThreads, SRC == SRC_EXPERTS ? (kCh == 1 ? 3 : 2) : SRC == SRC_PAIR && kCh == 2 ? 2 : 3) residual_norm_reg_kernel(const ResidualParams<T> p) {
+  __shared__ float part[kNormWarps], part2[kNormWarps], part3[SRC == SRC_PAIR ? 2 * kNormWarps : 1];
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
   const int64_t row = blockIdx.x;
   const GroupPlan gp(p.width, p.groups, 8, warp);
-  const bool on = gp.g0 < p.groups;
+  const bool on = gp.g0 < p.groups, post = SRC != SRC_EMBED || p.w_post;
   float* x = p.x + row * p.width;
   int col[kCh];
   bool has[kCh];
@@ -195,10 +239,10 @@ __global__ void __launch_bounds__(kNormThreads, SRC == SRC_EXPERTS ? (kCh == 1 ?
 #pragma unroll
   for (int k = 0; k < kCh; ++k)
     if (has[k]) {
-      wn[k].load(p.w_next + col[k]);
+      if (p.w_next) wn[k].load(p.w_next + col[k]);
+      if (post) wp[k].load(p.w_post + col[k]);
       if (SRC != SRC_EMBED) {
         Vec<float, 8>::load(x + col[k], r[k]);
-        wp[k].load(p.w_post + col[k]);
         if (p.gate) {
           gate[k].load(p.gate + row * p.gate_stride + col[k]);
           gb[k].load(p.gate_bias + col[k]);
@@ -248,6 +292,49 @@ __global__ void __launch_bounds__(kNormThreads, SRC == SRC_EXPERTS ? (kCh == 1 ?
 #pragma unroll
         for (int e = 0; e < 8; ++e) v[k][e] = fmaf(sgate, f[e], v[k][e]);
       }
+  } else if (SRC == SRC_PAIR) {
+    Raw8<T> a[kCh], b[kCh], wa[kCh], wb[kCh];
+#pragma unroll
+    for (int k = 0; k < kCh; ++k)
+      if (has[k]) {
+        a[k].load(p.y + row * p.y_stride + col[k]);
+        b[k].load(p.y2 + row * p.y2_stride + col[k]);
+        wa[k].load(p.w_y + col[k]);
+        wb[k].load(p.w_y2 + col[k]);
+      }
+    float sa = 0.f, sb = 0.f;
+#pragma unroll
+    for (int k = 0; k < kCh; ++k)
+      if (has[k]) {
+        float u[8], t[8];
+        a[k].get(u);
+        b[k].get(t);
+#pragma unroll
+        for (int e = 0; e < 8; ++e) {
+          sa = fmaf(u[e], u[e], sa);
+          sb = fmaf(t[e], t[e], sb);
+        }
+      }
+    sa = warp_sum(sa);
+    sb = warp_sum(sb);
+    if (lane == 0) {
+      part3[warp] = sa;
+      part3[kNormWarps + warp] = sb;
+    }
+    __syncthreads();
+    const float ra = on ? 0.5f * group_rs(part3, gp.g0, gp.wpg, gp.gs, p.eps) : 0.f;
+    const float rb = on ? 0.5f * group_rs(part3 + kNormWarps, gp.g0, gp.wpg, gp.gs, p.eps) : 0.f;
+#pragma unroll
+    for (int k = 0; k < kCh; ++k)
+      if (has[k]) {
+        float u[8], t[8], wu[8], wt[8];
+        a[k].get(u);
+        b[k].get(t);
+        wa[k].get(wu);
+        wb[k].get(wt);
+#pragma unroll
+        for (int e = 0; e < 8; ++e) v[k][e] = u[e] * ra * wu[e] + t[e] * rb * wt[e];
+      }
   } else {
 #pragma unroll
     for (int k = 0; k < kCh; ++k)
@@ -257,7 +344,7 @@ __global__ void __launch_bounds__(kNormThreads, SRC == SRC_EXPERTS ? (kCh == 1 ?
 #pragma unroll
   for (int k = 0; k < kCh; ++k)
     if (has[k]) {
-      if (SRC == SRC_EMBED) Vec<float, 8>::store(x + col[k], v[k]);
+      if (!post) Vec<float, 8>::store(x + col[k], v[k]);
       if (SRC != SRC_EMBED && p.gate) {
         float t[8], b[8];
         gate[k].get(t);
@@ -272,7 +359,7 @@ __global__ void __launch_bounds__(kNormThreads, SRC == SRC_EXPERTS ? (kCh == 1 ?
   if (lane == 0) part[warp] = acc;
   __syncthreads();
   const float* fin = part;
-  if (SRC != SRC_EMBED) {
+  if (post) {
     const float rs = on ? group_rs(part, gp.g0, gp.wpg, gp.gs, p.eps) : 0.f;
     acc = 0.f;
 #pragma unroll
@@ -282,7 +369,7 @@ __global__ void __launch_bounds__(kNormThreads, SRC == SRC_EXPERTS ? (kCh == 1 ?
         wp[k].get(w);
 #pragma unroll
         for (int e = 0; e < 8; ++e) {
-          v[k][e] = fmaf(p.mult, v[k][e] * rs * w[e], r[k][e]);
+          v[k][e] = SRC == SRC_EMBED ? v[k][e] * rs * w[e] : fmaf(p.mult, v[k][e] * rs * w[e], r[k][e]);
           acc = fmaf(v[k][e], v[k][e], acc);
         }
         Vec<float, 8>::store(x + col[k], v[k]);
@@ -296,16 +383,19 @@ __global__ void __launch_bounds__(kNormThreads, SRC == SRC_EXPERTS ? (kCh == 1 ?
 #pragma unroll
   for (int k = 0; k < kCh; ++k)
     if (has[k]) {
-      float w[8];
-      wn[k].get(w);
+      if (p.w_next) {
+        float w[8];
+        wn[k].get(w);
 #pragma unroll
-      for (int e = 0; e < 8; ++e) v[k][e] = v[k][e] * rs * w[e];
+        for (int e = 0; e < 8; ++e) v[k][e] = v[k][e] * rs * w[e];
+      }
       Vec<T, 8>::store(p.out + row * p.width + col[k], v[k]);
     }
 }
 
-// out = group_rms_norm(y * silu(z)) * w
-template <typename T, int V>
+// kGateFirst: out = group_rms_norm(y * silu(z)) * w.  Otherwise out = group_rms_norm(y) * w * silu(z), where w has one
+// group's length and is shared by the groups.
+template <typename T, int V, bool kGateFirst>
 __global__ void __launch_bounds__(kNormThreads)
 gated_group_norm_kernel(T* __restrict__ out, const T* __restrict__ y, int64_t y_stride, const T* __restrict__ z,
                         int64_t z_stride, const T* __restrict__ w, int width, int groups, float eps) {
@@ -320,10 +410,10 @@ gated_group_norm_kernel(T* __restrict__ out, const T* __restrict__ y, int64_t y_
       const int c = g * gp.gs + i * V;
       float v[V], t[V];
       Vec<T, V>::load(y + row * y_stride + c, v);
-      Vec<T, V>::load(z + row * z_stride + c, t);
+      if (kGateFirst) Vec<T, V>::load(z + row * z_stride + c, t);
 #pragma unroll
       for (int e = 0; e < V; ++e) {
-        v[e] *= silu_t<T>(t[e]);
+        if (kGateFirst) v[e] *= silu_t<T>(t[e]);
         acc = fmaf(v[e], v[e], acc);
       }
       Vec<float, V>::store(s_row + c, v);
@@ -338,19 +428,24 @@ gated_group_norm_kernel(T* __restrict__ out, const T* __restrict__ y, int64_t y_
       const int c = g * gp.gs + i * V;
       float v[V], t[V];
       Vec<float, V>::load(s_row + c, v);
-      Vec<T, V>::load(w + c, t);
+      Vec<T, V>::load(w + (kGateFirst ? c : c - g * gp.gs), t);
 #pragma unroll
       for (int e = 0; e < V; ++e) v[e] = v[e] * rs * t[e];
+      if (!kGateFirst) {
+        Vec<T, V>::load(z + row * z_stride + c, t);
+#pragma unroll
+        for (int e = 0; e < V; ++e) v[e] *= silu_t<T>(t[e]);
+      }
       Vec<T, V>::store(out + row * width + c, v);
     }
   }
 }
 
-// out = y * act(gate); row r of y is `heads` pieces of cols / heads elements, y_head_stride apart
+// out = act(gate, y), see glu_act; row r of y is `heads` pieces of cols / heads elements, y_head_stride apart
 template <typename T, int V>
 __global__ void __launch_bounds__(kNormThreads)
 gate_mul_kernel(T* __restrict__ out, const T* __restrict__ y, int64_t y_stride, int64_t y_head_stride, int head_cols,
-                const T* __restrict__ gate, int64_t gate_stride, int act, int64_t rows, int cols) {
+                const T* __restrict__ gate, int64_t gate_stride, int act, float limit, int64_t rows, int cols) {
   const int per = cols / V;
   const int64_t total = rows * per;
   for (int64_t i = static_cast<int64_t>(blockIdx.x) * kNormThreads + threadIdx.x; i < total;
@@ -361,7 +456,7 @@ gate_mul_kernel(T* __restrict__ out, const T* __restrict__ y, int64_t y_stride, 
     Vec<T, V>::load(y + row * y_stride + h * y_head_stride + (c - h * head_cols), v);
     Vec<T, V>::load(gate + row * gate_stride + c, g);
 #pragma unroll
-    for (int e = 0; e < V; ++e) v[e] *= act ? silu_t<T>(g[e]) : sigmoid_t<T>(g[e]);
+    for (int e = 0; e < V; ++e) v[e] = glu_act<T>(act, g[e], v[e], limit);
     Vec<T, V>::store(out + row * cols + c, v);
   }
 }
@@ -391,7 +486,7 @@ static int launch_residual_v(const ResidualParams<T>& p, int64_t rows, cudaStrea
   const int eb = sizeof(T);
   bool v8 = (p.width / p.groups) % 8 == 0 && aligned16(p.out) && aligned16(p.x) && aligned16(p.w_next) &&
             vec8_ok(p.y, p.y_stride, eb) && vec8_ok(p.gate, p.gate_stride, eb) && vec8_ok(p.gate_bias, 0, eb) &&
-            vec8_ok(p.w_post, 0, eb) && vec8_ok(p.embed, p.width, eb) && vec8_ok(p.shared, p.shared_stride, eb);
+            vec8_ok(p.y2, p.y2_stride, eb) && vec8_ok(p.w_y, 0, eb) && vec8_ok(p.w_y2, 0, eb) && vec8_ok(p.w_post, 0, eb) && vec8_ok(p.embed, p.width, eb) && vec8_ok(p.shared, p.shared_stride, eb);
   if (v8 && p.groups <= kNormWarps) {
     const int lanes = kNormWarps / p.groups * 32, per = (p.width / p.groups / 8 + lanes - 1) / lanes;
     if (per <= 2) {
@@ -411,17 +506,18 @@ static int check_norm(const char* what, int width, int groups, int dtype) {
 }  // namespace mv
 
 extern "C" int mv_embed_norm(void* out, float* x, const int64_t* ids, const void* embed, int64_t vocab,
-                             const void* w_next, int64_t rows, int width, int groups, float eps, int dtype,
+                             const void* w_post, const void* w_next, int64_t rows, int width, int groups, float eps, int dtype,
                              void* stream) {
   using namespace mv;
   int rc = check_norm("embed_norm", width, groups, dtype);
   if (rc || rows == 0) return rc;
-  if (!out || !x || !ids || !embed || !w_next) return fail(MV_ERR_NULL, "embed_norm: null pointer");
+  if (!out || !x || !ids || !embed) return fail(MV_ERR_NULL, "embed_norm: null pointer");
   auto run = [&](auto tag) {
     using T = decltype(tag);
     ResidualParams<T> p{};
     p.out = static_cast<T*>(out); p.x = x; p.ids = ids; p.embed = static_cast<const T*>(embed); p.vocab = vocab;
-    p.w_next = static_cast<const T*>(w_next); p.width = width; p.groups = groups; p.eps = eps;
+    p.w_post = static_cast<const T*>(w_post); p.w_next = static_cast<const T*>(w_next);
+    p.width = width; p.groups = groups; p.eps = eps;
     return launch_residual_v<T, SRC_EMBED>(p, rows, static_cast<cudaStream_t>(stream));
   };
   return dtype == MV_F32 ? run(float{}) : run(__nv_bfloat16{});
@@ -434,7 +530,7 @@ extern "C" int mv_gated_residual_norm(void* out, float* x, const void* y, int64_
   using namespace mv;
   int rc = check_norm("gated_residual_norm", width, groups, dtype);
   if (rc || rows == 0) return rc;
-  if (!out || !x || !y || !w_post || !w_next || (gate && !gate_bias))
+  if (!out || !x || !y || !w_post || (gate && !gate_bias))
     return fail(MV_ERR_NULL, "gated_residual_norm: null pointer");
   auto run = [&](auto tag) {
     using T = decltype(tag);
@@ -448,6 +544,27 @@ extern "C" int mv_gated_residual_norm(void* out, float* x, const void* y, int64_
   return dtype == MV_F32 ? run(float{}) : run(__nv_bfloat16{});
 }
 
+extern "C" int mv_pair_residual_norm(void* out, float* x, const void* a, int64_t a_stride, const void* w_a, const void* b,
+                                     int64_t b_stride, const void* w_b, const void* w_post, const void* w_next,
+                                     float mult, int64_t rows, int width, int groups, float eps, int dtype,
+                                     void* stream) {
+  using namespace mv;
+  int rc = check_norm("pair_residual_norm", width, groups, dtype);
+  if (rc || rows == 0) return rc;
+  if (!out || !x || !a || !w_a || !b || !w_b || !w_post) return fail(MV_ERR_NULL, "pair_residual_norm: null pointer");
+  auto run = [&](auto tag) {
+    using T = decltype(tag);
+    ResidualParams<T> p{};
+    p.out = static_cast<T*>(out); p.x = x; p.y = static_cast<const T*>(a); p.y_stride = a_stride;
+    p.y2 = static_cast<const T*>(b); p.y2_stride = b_stride;
+    p.w_y = static_cast<const T*>(w_a); p.w_y2 = static_cast<const T*>(w_b);
+    p.w_post = static_cast<const T*>(w_post); p.w_next = static_cast<const T*>(w_next);
+    p.mult = mult; p.width = width; p.groups = groups; p.eps = eps;
+    return launch_residual_v<T, SRC_PAIR>(p, rows, static_cast<cudaStream_t>(stream));
+  };
+  return dtype == MV_F32 ? run(float{}) : run(__nv_bfloat16{});
+}
+
 extern "C" int mv_moe_residual_norm(void* out, float* x, const void* expert_rows, const int32_t* pos,
                                     const float* top_weights, int top, const void* shared, int64_t shared_stride,
                                     const void* shared_gate, int64_t shared_gate_stride, const void* gate,
@@ -457,7 +574,7 @@ extern "C" int mv_moe_residual_norm(void* out, float* x, const void* expert_rows
   using namespace mv;
   int rc = check_norm("moe_residual_norm", width, groups, dtype);
   if (rc || rows == 0) return rc;
-  if (!out || !x || !expert_rows || !pos || !top_weights || !w_post || !w_next || (gate && !gate_bias))
+  if (!out || !x || !expert_rows || !pos || !top_weights || !w_post || (gate && !gate_bias))
     return fail(MV_ERR_NULL, "moe_residual_norm: null pointer");
   if (top <= 0 || top > kMaxTop) return fail(MV_ERR_SHAPE, "moe_residual_norm: top %d", top);
   auto run = [&](auto tag) {
@@ -475,40 +592,51 @@ extern "C" int mv_moe_residual_norm(void* out, float* x, const void* expert_rows
   return dtype == MV_F32 ? run(float{}) : run(__nv_bfloat16{});
 }
 
-extern "C" int mv_gated_group_norm(void* out, const void* y, int64_t y_stride, const void* z, int64_t z_stride,
-                                   const void* w, int64_t rows, int width, int groups, float eps, int dtype,
-                                   void* stream) {
+static int gated_norm(const char* what, bool gate_first, void* out, const void* y, int64_t y_stride, const void* z, int64_t z_stride,
+                      const void* w, int64_t rows, int width, int groups, float eps, int dtype, void* stream) {
   using namespace mv;
-  int rc = check_norm("gated_group_norm", width, groups, dtype);
+  int rc = check_norm(what, width, groups, dtype);
   if (rc || rows == 0) return rc;
-  if (!out || !y || !z || !w) return fail(MV_ERR_NULL, "gated_group_norm: null pointer");
+  if (!out || !y || !z || !w) return fail(MV_ERR_NULL, "%s: null pointer", what);
   const size_t smem = norm_smem(width, groups);
   auto run = [&](auto tag) {
     using T = decltype(tag);
     const int eb = sizeof(T);
     auto go = [&](auto kernel) {
-      const int r = allow_smem(kernel, smem, "gated_group_norm");
+      const int r = allow_smem(kernel, smem, what);
       if (r) return r;
       kernel<<<static_cast<unsigned>(rows), kNormThreads, smem, static_cast<cudaStream_t>(stream)>>>(
           static_cast<T*>(out), static_cast<const T*>(y), y_stride, static_cast<const T*>(z), z_stride,
           static_cast<const T*>(w), width, groups, eps);
-      return check_launch("gated_group_norm");
+      return check_launch(what);
     };
     if ((width / groups) % 8 == 0 && vec8_ok(out, width, eb) && vec8_ok(y, y_stride, eb) && vec8_ok(z, z_stride, eb) &&
         aligned16(w))
-      return go(gated_group_norm_kernel<T, 8>);
-    return go(gated_group_norm_kernel<T, 1>);
+      return gate_first ? go(gated_group_norm_kernel<T, 8, true>) : go(gated_group_norm_kernel<T, 8, false>);
+    return gate_first ? go(gated_group_norm_kernel<T, 1, true>) : go(gated_group_norm_kernel<T, 1, false>);
   };
   return dtype == MV_F32 ? run(float{}) : run(__nv_bfloat16{});
 }
 
+extern "C" int mv_gated_group_norm(void* out, const void* y, int64_t y_stride, const void* z, int64_t z_stride,
+                                   const void* w, int64_t rows, int width, int groups, float eps, int dtype,
+                                   void* stream) {
+  return gated_norm("gated_group_norm", true, out, y, y_stride, z, z_stride, w, rows, width, groups, eps, dtype, stream);
+}
+
+extern "C" int mv_head_norm_gate(void* out, const void* y, int64_t y_stride, const void* z, int64_t z_stride,
+                                 const void* w, int64_t rows, int width, int heads, float eps, int dtype, void* stream) {
+  return gated_norm("head_norm_gate", false, out, y, y_stride, z, z_stride, w, rows, width, heads, eps, dtype, stream);
+}
+
 extern "C" int mv_gate_mul(void* out, const void* y, int64_t y_stride, int64_t y_head_stride, int heads,
-                           const void* gate, int64_t gate_stride, int act, int64_t rows, int cols, int dtype,
-                           void* stream) {
+                           const void* gate, int64_t gate_stride, int act, float limit, int64_t rows, int cols,
+                           int dtype, void* stream) {
   using namespace mv;
   int rc = check_norm("gate_mul", cols, heads, dtype);
   if (rc || rows == 0) return rc;
   if (!out || !y || !gate) return fail(MV_ERR_NULL, "gate_mul: null pointer");
+  if (act < 0 || act > MV_ACT_CLAMPED) return fail(MV_ERR_SHAPE, "gate_mul: activation %d", act);
   auto run = [&](auto tag) {
     using T = decltype(tag);
     const int eb = sizeof(T), hc = cols / heads;
@@ -519,8 +647,8 @@ extern "C" int mv_gate_mul(void* out, const void* y, int64_t y_stride, int64_t y
     auto* o = static_cast<T*>(out);
     auto *a = static_cast<const T*>(y), *b = static_cast<const T*>(gate);
     auto st = static_cast<cudaStream_t>(stream);
-    if (v8) gate_mul_kernel<T, 8><<<grid, kNormThreads, 0, st>>>(o, a, y_stride, y_head_stride, hc, b, gate_stride, act, rows, cols);
-    else gate_mul_kernel<T, 1><<<grid, kNormThreads, 0, st>>>(o, a, y_stride, y_head_stride, hc, b, gate_stride, act, rows, cols);
+    if (v8) gate_mul_kernel<T, 8><<<grid, kNormThreads, 0, st>>>(o, a, y_stride, y_head_stride, hc, b, gate_stride, act, limit, rows, cols);
+    else gate_mul_kernel<T, 1><<<grid, kNormThreads, 0, st>>>(o, a, y_stride, y_head_stride, hc, b, gate_stride, act, limit, rows, cols);
     return check_launch("gate_mul");
   };
   return dtype == MV_F32 ? run(float{}) : run(__nv_bfloat16{});

@@ -76,6 +76,15 @@ template <typename T> __device__ __forceinline__ float sigmoid_t(float z) {
 template <typename T> __device__ __forceinline__ float silu_t(float z) {
   return sizeof(T) == 2 ? __fdividef(z, 1.f + __expf(-z)) : silu_f(z);
 }
+// What a gate does to the value beside it (mv_act): output gates and the activations of gated feed-forwards.
+template <typename T> __device__ __forceinline__ float glu_act(int act, float g, float u, float limit) {
+  if (act == MV_ACT_SILU) return silu_t<T>(g) * u;
+  if (act == MV_ACT_SIGMOID) return sigmoid_t<T>(g) * u;
+  if (act == MV_ACT_GELU_TANH)       // 0.5 (1 + tanh(a)) = sigmoid(2 a)
+    return g * sigmoid_t<T>(1.5957691216057308f * fmaf(0.044715f * g * g, g, g)) * u;
+  g = fminf(g, limit);
+  return g * sigmoid_t<T>(1.702f * g) * (fminf(fmaxf(u, -limit), limit) + 1.f);
+}
 __device__ __forceinline__ float softplus_f(float z) { return z > 20.f ? z : log1pf(expf(z)); }
 __device__ __forceinline__ float warp_sum(float v) {
 #pragma unroll

@@ -1,0 +1,599 @@
+// Grouped-query attention with a sliding window, a learned bias per distance and head, and a sink per head, over a paged
+// cache of rows [keys of all KV heads | values of all KV heads] (key and value sizes may differ).  Position i sees the
+// keys j with 0 <= i - j < window; score = scale (q . k) + bias[h][min(i - j, distances - 1)]; exp(sink[h]) joins the
+// denominator.  Bias and sink may be absent.
+//
+// kv_norm_store_kernel        RMS norm over all query rows and over all key rows of a token, scatter of [k | v]
+// window_attention_rows_kernel  any sizes, bf16 or fp32, token by token
+// window_decode_kernel        one token per sequence on mma.sync: HBM-bound on the rows inside the window
+// Portions of prompts run on tcgen05 in latent_prefill.cu.
+#include <algorithm>
+#include <type_traits>
+#include "mma.cuh"
+#include "vec.cuh"
+
+namespace mv {
+
+constexpr int kKnThreads = 256;
+
+template <typename T, int V>
+__global__ void __launch_bounds__(kKnThreads)
+kv_norm_store_kernel(T* __restrict__ q, const T* __restrict__ k, const T* __restrict__ v, int64_t stride,
+                     const T* __restrict__ q_weight, const T* __restrict__ k_weight, T* __restrict__ kv_out,
+                     T* __restrict__ cache, const int64_t* __restrict__ slot_mapping, int64_t num_slots, int qn, int kn,
+                     int vn, float eps) {
+  __shared__ float part[2][kKnThreads / 32];
+  const int64_t t = blockIdx.x;
+  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+  T* qr = q + t * stride;
+  const T *kr = k + t * stride, *vr = v + t * stride;
+  const int row = kn + vn;
+  T* lo = kv_out ? kv_out + t * row : nullptr;
+  T* co = nullptr;
+  if (cache) {
+    const int64_t slot = slot_mapping[t];
+    if (slot >= 0 && slot < num_slots) co = cache + slot * row;
+  }
+  // the first pieces stay in registers: rows of up to 2,048 queries and keys are read once
+  constexpr int kHold = 2;
+  float hold[kHold][V];
+  float a = 0.f, b = 0.f;
+  for (int i = tid, n = 0; i < (qn + kn) / V; i += kKnThreads, ++n) {
+    const int c = i * V;
+    float x[V];
+    Vec<T, V>::load(c < qn ? qr + c : kr + c - qn, x);
+    float s = 0.f;
+#pragma unroll
+    for (int e = 0; e < V; ++e) s = fmaf(x[e], x[e], s);
+    if (c < qn) a += s; else b += s;
+#pragma unroll
+    for (int h = 0; h < kHold; ++h)
+      if (h == n)
+#pragma unroll
+        for (int e = 0; e < V; ++e) hold[h][e] = x[e];
+  }
+  a = warp_sum(a);
+  b = warp_sum(b);
+  if (lane == 0) { part[0][warp] = a; part[1][warp] = b; }
+  for (int i = tid; i < vn / V; i += kKnThreads) {
+    float x[V];
+    Vec<T, V>::load(vr + i * V, x);
+    if (lo) Vec<T, V>::store(lo + kn + i * V, x);
+    if (co) Vec<T, V>::store(co + kn + i * V, x);
+  }
+  __syncthreads();
+  a = b = 0.f;
+  for (int w = 0; w < kKnThreads / 32; ++w) { a += part[0][w]; b += part[1][w]; }
+  const float rq = 1.f / sqrtf(a / static_cast<float>(qn) + eps), rk = 1.f / sqrtf(b / static_cast<float>(kn) + eps);
+  for (int i = tid, n = 0; i < (qn + kn) / V; i += kKnThreads, ++n) {
+    const int c = i * V;
+    const bool is_q = c < qn;
+    float x[V], w[V];
+    if (n >= kHold) Vec<T, V>::load(is_q ? qr + c : kr + c - qn, x);
+#pragma unroll
+    for (int h = 0; h < kHold; ++h)
+      if (h == n)
+#pragma unroll
+        for (int e = 0; e < V; ++e) x[e] = hold[h][e];
+    Vec<T, V>::load(is_q ? q_weight + c : k_weight + c - qn, w);
+#pragma unroll
+    for (int e = 0; e < V; ++e) x[e] = x[e] * (is_q ? rq : rk) * w[e];
+    if (is_q) {
+      Vec<T, V>::store(qr + c, x);
+    } else {
+      if (lo) Vec<T, V>::store(lo + c - qn, x);
+      if (co) Vec<T, V>::store(co + c - qn, x);
+    }
+  }
+}
+
+template <typename T> struct WindowParams {
+  T* out;                                    // (tokens, heads * vdim)
+  const T* q; int64_t q_stride;              // (tokens, heads * dim)
+  const T* cache;                            // (blocks, block_size, kv_heads * (dim + vdim))
+  const int32_t* tables; int64_t bt_stride; int max_blocks, block_size; int64_t num_blocks;
+  const int32_t* cu_q; int num_seqs;
+  const int64_t* positions;
+  const float* bias; int64_t bias_stride; int distances;       // bias[h * bias_stride + distance]
+  const T* sink;
+  int heads, kv_heads, dim, vdim;
+  int64_t window;
+  float scale;
+  // decode
+  int splits;
+  float *part_ml, *part_o;                   // (batch, splits, heads, 2) and (.., vdim)
+};
+
+constexpr int kWaThreads = 256, kWaHeads = 4, kWaKeys = 32, kWaPer = 4;    // vdim up to kWaThreads * kWaPer
+
+template <typename T>
+__global__ void __launch_bounds__(kWaThreads) window_attention_rows_kernel(const WindowParams<T> p) {
+  extern __shared__ __align__(16) float sm[];
+  const int group = p.heads / p.kv_heads, chunks = (group + kWaHeads - 1) / kWaHeads;
+  const int kv = blockIdx.y / chunks, g0 = (blockIdx.y - kv * chunks) * kWaHeads;
+  const int h0 = kv * group + g0, nh = min(kWaHeads, group - g0);
+  const int D = p.dim, VD = p.vdim, row = p.kv_heads * (D + VD);
+  float* sq = sm;                               // [kWaHeads][D]
+  float* sk = sq + kWaHeads * D;                // [kWaKeys][D + 1]
+  float* sv = sk + kWaKeys * (D + 1);           // [kWaKeys][VD]
+  float* ss = sv + kWaKeys * VD;                // [kWaHeads][kWaKeys]
+  __shared__ float s_m[kWaHeads], s_l[kWaHeads], s_c[kWaHeads];
+  const int t = blockIdx.x, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+  const int seq = seq_of_token(p.cu_q, p.num_seqs, t);
+  const int32_t* table = p.tables + static_cast<int64_t>(seq) * p.bt_stride;
+  const int64_t pos = p.positions[t];
+  const int nk = static_cast<int>(min(pos + 1, static_cast<int64_t>(p.max_blocks) * p.block_size));
+  const int first = static_cast<int>(max(pos - p.window + 1, static_cast<int64_t>(0)));
+  for (int i = tid; i < kWaHeads * D; i += kWaThreads) {
+    const int h = i / D, j = i - h * D;
+    sq[i] = h < nh ? Elem<T>::to_f(p.q[t * p.q_stride + static_cast<int64_t>(h0 + h) * D + j]) : 0.f;
+  }
+  // the sink is one more score without a value: it opens the running maximum and sum
+  if (tid < kWaHeads) {
+    s_m[tid] = tid < nh && p.sink ? Elem<T>::to_f(p.sink[h0 + tid]) : -INFINITY;
+    s_l[tid] = tid < nh && p.sink ? 1.f : 0.f;
+  }
+  float acc[kWaHeads][kWaPer];
+#pragma unroll
+  for (int h = 0; h < kWaHeads; ++h)
+#pragma unroll
+    for (int i = 0; i < kWaPer; ++i) acc[h][i] = 0.f;
+
+  for (int k0 = first; k0 < nk; k0 += kWaKeys) {
+    __syncthreads();
+    for (int k = warp; k < kWaKeys; k += kWaThreads / 32) {
+      const int at = k0 + k, blk = at / p.block_size;
+      const int32_t phys = at < nk && blk < p.max_blocks ? table[blk] : -1;
+      const bool ok = phys >= 0 && phys < p.num_blocks;
+      const T* src = p.cache + (static_cast<int64_t>(ok ? phys : 0) * p.block_size + (at - blk * p.block_size)) * row;
+      for (int i = lane; i < D; i += 32) sk[k * (D + 1) + i] = ok ? Elem<T>::to_f(src[kv * D + i]) : 0.f;
+      for (int i = lane; i < VD; i += 32) sv[k * VD + i] = ok ? Elem<T>::to_f(src[p.kv_heads * D + kv * VD + i]) : 0.f;
+      if (lane < kWaHeads) {
+        float b = ok ? 0.f : -INFINITY;
+        if (ok && p.bias && lane < nh)
+          b = p.bias[(h0 + lane) * p.bias_stride + min(static_cast<int>(pos) - at, p.distances - 1)];
+        ss[lane * kWaKeys + k] = b;
+      }
+    }
+    __syncthreads();
+    {  // two threads per (head, key)
+      const int pair = tid >> 1, h = pair / kWaKeys, k = pair % kWaKeys, half = tid & 1;
+      const float *a = sq + h * D, *b = sk + k * (D + 1);
+      float s = 0.f;
+      for (int i = half; i < D; i += 2) s = fmaf(a[i], b[i], s);
+      s += __shfl_xor_sync(0xffffffffu, s, 1);
+      if (half == 0) ss[h * kWaKeys + k] += s * p.scale;     // -inf stays -inf
+    }
+    __syncthreads();
+    if (warp < kWaHeads) {
+      const float s = ss[warp * kWaKeys + lane];
+      float mx = s;
+#pragma unroll
+      for (int o = 16; o; o >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, o));
+      const float m_old = s_m[warp], m_new = fmaxf(m_old, mx);
+      const float pr = m_new == -INFINITY ? 0.f : expf(s - m_new);
+      const float sum = warp_sum(pr);
+      ss[warp * kWaKeys + lane] = pr;
+      if (lane == 0) {
+        const float corr = m_new == -INFINITY ? 1.f : expf(m_old - m_new);
+        s_c[warp] = corr;
+        s_l[warp] = s_l[warp] * corr + sum;
+        s_m[warp] = m_new;
+      }
+    }
+    __syncthreads();
+#pragma unroll
+    for (int i = 0; i < kWaPer; ++i) {
+      const int d = tid + i * kWaThreads;
+      if (d < VD) {
+#pragma unroll
+        for (int h = 0; h < kWaHeads; ++h) acc[h][i] *= s_c[h];
+        for (int k = 0; k < kWaKeys; ++k) {
+          const float v = sv[k * VD + d];
+#pragma unroll
+          for (int h = 0; h < kWaHeads; ++h) acc[h][i] = fmaf(ss[h * kWaKeys + k], v, acc[h][i]);
+        }
+      }
+    }
+  }
+  __syncthreads();
+#pragma unroll
+  for (int h = 0; h < kWaHeads; ++h) {
+    if (h >= nh) break;
+    const float l = s_l[h], inv = l > 0.f ? 1.f / l : 0.f;
+#pragma unroll
+    for (int i = 0; i < kWaPer; ++i) {
+      const int d = tid + i * kWaThreads;
+      if (d < VD) p.out[(static_cast<int64_t>(t) * p.heads + h0 + h) * VD + d] = Elem<T>::from_f(acc[h][i] * inv);
+    }
+  }
+}
+
+// ------------------------------------------------------------------------------------------------ decode
+// One CTA per (piece of the window, KV head and tile of 16 query heads, sequence): four warps stream 16-key tiles of
+// their own through cp.async rings; the query heads are the rows of m16n8k16 products.  Attention weights enter their
+// product as value and rounding residue.
+constexpr int kWdWarps = 4, kWdThreads = 32 * kWdWarps, kWdStages = 3, kWdTile = 16;
+constexpr float kWdNeg = -1e30f;
+
+template <int KD, int VD> struct WdShape {
+  static constexpr int kK = kWdTile * KD * 2, kV = kWdTile * VD * 2, kStage = kK + kV, kWarp = kWdStages * kStage;
+  static constexpr int kRing = kWdWarps * kWarp, kStride = VD + 8;
+  static constexpr int kMerge = kWdWarps * 16 * (kStride + 2) * 4;
+  static constexpr int kSmem = kRing > kMerge ? kRing : kMerge;
+};
+
+template <int KD, int VD>
+__global__ void __launch_bounds__(kWdThreads, KD + VD > 256 ? 1 : 2)
+window_decode_kernel(const WindowParams<__nv_bfloat16> p) {
+  using T = __nv_bfloat16;
+  using S = WdShape<KD, VD>;
+  using Mma = Mma16816<T>;
+  constexpr int KSTEPS = KD / 16, NT = VD / 8, KC = KD / 8, VC = VD / 8;
+  extern __shared__ __align__(128) unsigned char smem[];
+  __shared__ uint32_t s_mask[kWdWarps][kWdStages];
+  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, g = lane >> 2, t = lane & 3;
+  const int group = p.heads / p.kv_heads, mtiles = (group + 15) / 16;
+  const int kv = blockIdx.y / mtiles, mt = blockIdx.y - kv * mtiles, b = blockIdx.z, split = blockIdx.x;
+  const int rows = min(16, group - mt * 16), h0 = kv * group + mt * 16;
+  const int64_t pos64 = p.positions[b];
+  const int pos = static_cast<int>(pos64);
+  const int nk = static_cast<int>(min(pos64 + 1, static_cast<int64_t>(p.max_blocks) * p.block_size));
+  const int lo = static_cast<int>(max(pos64 - p.window + 1, static_cast<int64_t>(0)));
+  const int span = max(nk - lo, 0);
+  const int len = ((span + p.splits - 1) / p.splits + kWdTile - 1) / kWdTile * kWdTile;
+  const int k_begin = lo + split * len, k_end = min(k_begin + len, nk);
+  const int tiles = k_end > k_begin ? (k_end - k_begin + kWdTile - 1) / kWdTile : 0;
+  const int my_tiles = tiles > warp ? (tiles - warp + kWdWarps - 1) / kWdWarps : 0;
+  const int32_t* table = p.tables + static_cast<int64_t>(b) * p.bt_stride;
+  const int64_t row_elems = static_cast<int64_t>(p.kv_heads) * (p.dim + p.vdim);
+  const T *k_base = p.cache + kv * p.dim, *v_base = p.cache + p.kv_heads * p.dim + kv * p.vdim;
+  const uint32_t ring = smem_u32(smem) + warp * S::kWarp;
+  const int kc_real = p.dim / 8, vc_real = p.vdim / 8;
+
+  auto issue = [&](int i) {
+    if (i < my_tiles) {
+      const int stage = i % kWdStages, tok0 = k_begin + (i * kWdWarps + warp) * kWdTile;
+      const int me = tok0 + (lane & 15), blk = me / p.block_size;
+      int64_t at = -1;
+      if (me < k_end && blk < p.max_blocks) {
+        const int32_t phys = __ldg(table + blk);
+        if (phys >= 0 && phys < p.num_blocks) at = (static_cast<int64_t>(phys) * p.block_size + (me - blk * p.block_size)) * row_elems;
+      }
+      const uint32_t live = __ballot_sync(0xffffffffu, at >= 0) & 0xffffu;
+      if (lane == 0) s_mask[warp][stage] = live;
+      const uint32_t kd = ring + stage * S::kStage, vd = kd + S::kK;
+#pragma unroll
+      for (int c0 = 0; c0 < kWdTile * KC; c0 += 32) {
+        const int r = (c0 + lane) / KC, c = (c0 + lane) % KC;
+        const int64_t src = __shfl_sync(0xffffffffu, at, r);
+        const bool ok = src >= 0 && c < kc_real;
+        cp_async16(kd + r * (KD * 2) + ((c ^ (r & 7)) << 4), ok ? k_base + src + c * 8 : p.cache, ok ? 16 : 0);
+      }
+#pragma unroll
+      for (int c0 = 0; c0 < kWdTile * VC; c0 += 32) {
+        const int r = (c0 + lane) / VC, c = (c0 + lane) % VC;
+        const int64_t src = __shfl_sync(0xffffffffu, at, r);
+        const bool ok = src >= 0 && c < vc_real;
+        cp_async16(vd + r * (VD * 2) + ((c ^ (r & 7)) << 4), ok ? v_base + src + c * 8 : p.cache, ok ? 16 : 0);
+      }
+    }
+    cp_async_commit();
+  };
+#pragma unroll
+  for (int i = 0; i < kWdStages - 1; ++i) issue(i);
+
+  uint32_t qa[KSTEPS][4];
+  {
+    const T* qb = p.q + b * p.q_stride + static_cast<int64_t>(h0) * p.dim;
+    const bool v0 = g < rows, v1 = g + 8 < rows;
+    const uint32_t* q0 = reinterpret_cast<const uint32_t*>(qb + static_cast<int64_t>(g) * p.dim);
+    const uint32_t* q1 = reinterpret_cast<const uint32_t*>(qb + static_cast<int64_t>(g + 8) * p.dim);
+    const int half = p.dim / 2;
+#pragma unroll
+    for (int ks = 0; ks < KSTEPS; ++ks) {
+      const int c = ks * 8 + t;
+      qa[ks][0] = v0 && c < half ? __ldg(q0 + c) : 0u;
+      qa[ks][1] = v1 && c < half ? __ldg(q1 + c) : 0u;
+      qa[ks][2] = v0 && c + 4 < half ? __ldg(q0 + c + 4) : 0u;
+      qa[ks][3] = v1 && c + 4 < half ? __ldg(q1 + c + 4) : 0u;
+    }
+  }
+  const float scale2 = p.scale * 1.4426950408889634f;
+  const float* bias0 = p.bias ? p.bias + (h0 + min(g, rows - 1)) * p.bias_stride : nullptr;
+  const float* bias1 = p.bias ? p.bias + (h0 + min(g + 8, rows - 1)) * p.bias_stride : nullptr;
+  const float far0 = bias0 ? bias0[p.distances - 1] * 1.4426950408889634f : 0.f;
+  const float far1 = bias1 ? bias1[p.distances - 1] * 1.4426950408889634f : 0.f;
+
+  float o[NT][4];
+#pragma unroll
+  for (int j = 0; j < NT; ++j) o[j][0] = o[j][1] = o[j][2] = o[j][3] = 0.f;
+  float m0 = kWdNeg, m1 = kWdNeg, l0 = 0.f, l1 = 0.f;
+  for (int i = 0; i < my_tiles; ++i) {
+    cp_async_wait<kWdStages - 2>();
+    __syncwarp();
+    const int stage = i % kWdStages, tok0 = k_begin + (i * kWdWarps + warp) * kWdTile;
+    const uint32_t kd = ring + stage * S::kStage, vd = kd + S::kK;
+    const uint32_t live = s_mask[warp][stage];
+    float s[2][4] = {};
+    {
+      const int row = (lane & 7) + ((lane >> 4) << 3), csel = (lane >> 3) & 1;
+#pragma unroll
+      for (int ks = 0; ks < KSTEPS; ++ks) {
+        uint32_t kb[4];
+        ldmatrix_x4(kb, kd + row * (KD * 2) + (((2 * ks + csel) ^ (row & 7)) << 4));
+        Mma::run(s[0], qa[ks], kb[0], kb[1]);
+        Mma::run(s[1], qa[ks], kb[2], kb[3]);
+      }
+    }
+    issue(i + kWdStages - 1);
+    const bool far = pos - tok0 - (kWdTile - 1) >= p.distances - 1;      // every key of the tile has the last bias
+    float mx0 = kWdNeg, mx1 = kWdNeg;
+#pragma unroll
+    for (int n = 0; n < 2; ++n) {
+#pragma unroll
+      for (int e = 0; e < 2; ++e) {
+        const int col = n * 8 + 2 * t + e;
+        float b0 = far0, b1 = far1;
+        if (p.bias && !far) {
+          const int d = min(max(pos - tok0 - col, 0), p.distances - 1);
+          b0 = __ldg(bias0 + d) * 1.4426950408889634f;
+          b1 = __ldg(bias1 + d) * 1.4426950408889634f;
+        }
+        const bool ok = (live >> col) & 1u;
+        s[n][e] = ok ? fmaf(s[n][e], scale2, b0) : -INFINITY;
+        s[n][2 + e] = ok ? fmaf(s[n][2 + e], scale2, b1) : -INFINITY;
+      }
+      mx0 = fmaxf(mx0, fmaxf(s[n][0], s[n][1]));
+      mx1 = fmaxf(mx1, fmaxf(s[n][2], s[n][3]));
+    }
+    mx0 = fmaxf(mx0, __shfl_xor_sync(0xffffffffu, mx0, 1));
+    mx0 = fmaxf(mx0, __shfl_xor_sync(0xffffffffu, mx0, 2));
+    mx1 = fmaxf(mx1, __shfl_xor_sync(0xffffffffu, mx1, 1));
+    mx1 = fmaxf(mx1, __shfl_xor_sync(0xffffffffu, mx1, 2));
+    const float mn0 = fmaxf(m0, mx0), mn1 = fmaxf(m1, mx1), a0 = fast_exp2(m0 - mn0), a1 = fast_exp2(m1 - mn1);
+    m0 = mn0;
+    m1 = mn1;
+    float ps0 = 0.f, ps1 = 0.f;
+#pragma unroll
+    for (int n = 0; n < 2; ++n) {
+      s[n][0] = fast_exp2(s[n][0] - mn0); s[n][1] = fast_exp2(s[n][1] - mn0);
+      s[n][2] = fast_exp2(s[n][2] - mn1); s[n][3] = fast_exp2(s[n][3] - mn1);
+      ps0 += s[n][0] + s[n][1];
+      ps1 += s[n][2] + s[n][3];
+    }
+    l0 = l0 * a0 + ps0;
+    l1 = l1 * a1 + ps1;
+    uint32_t pa[4], pl[4];
+#pragma unroll
+    for (int n = 0; n < 2; ++n)
+#pragma unroll
+      for (int hh = 0; hh < 2; ++hh) {
+        pa[2 * n + hh] = pack2<T>(s[n][2 * hh], s[n][2 * hh + 1]);
+        const float2 hi = Elem<T>::to_f2(*reinterpret_cast<const __nv_bfloat162*>(&pa[2 * n + hh]));
+        pl[2 * n + hh] = pack2<T>(s[n][2 * hh] - hi.x, s[n][2 * hh + 1] - hi.y);
+      }
+    if (__any_sync(0xffffffffu, a0 != 1.f || a1 != 1.f)) {
+#pragma unroll
+      for (int j = 0; j < NT; ++j) { o[j][0] *= a0; o[j][1] *= a0; o[j][2] *= a1; o[j][3] *= a1; }
+    }
+    {
+      const int row = (lane & 7) + (((lane >> 3) & 1) << 3), csel = lane >> 4;
+#pragma unroll
+      for (int jp = 0; jp < NT / 2; ++jp) {
+        uint32_t vb[4];
+        ldmatrix_x4_trans(vb, vd + row * (VD * 2) + (((2 * jp + csel) ^ (row & 7)) << 4));
+        Mma::run(o[2 * jp], pa, vb[0], vb[1]);
+        Mma::run(o[2 * jp + 1], pa, vb[2], vb[3]);
+        Mma::run(o[2 * jp], pl, vb[0], vb[1]);
+        Mma::run(o[2 * jp + 1], pl, vb[2], vb[3]);
+      }
+    }
+    __syncwarp();
+  }
+  cp_async_wait<0>();
+  l0 += __shfl_xor_sync(0xffffffffu, l0, 1);
+  l0 += __shfl_xor_sync(0xffffffffu, l0, 2);
+  l1 += __shfl_xor_sync(0xffffffffu, l1, 1);
+  l1 += __shfl_xor_sync(0xffffffffu, l1, 2);
+  __syncthreads();                       // the rings are idle
+  float* sO = reinterpret_cast<float*>(smem);
+  float* sML = sO + kWdWarps * 16 * S::kStride;
+  {
+    float* mine = sO + warp * 16 * S::kStride;
+#pragma unroll
+    for (int j = 0; j < NT; ++j) {
+      *reinterpret_cast<float2*>(mine + g * S::kStride + j * 8 + 2 * t) = make_float2(o[j][0], o[j][1]);
+      *reinterpret_cast<float2*>(mine + (g + 8) * S::kStride + j * 8 + 2 * t) = make_float2(o[j][2], o[j][3]);
+    }
+    if (t == 0) {
+      sML[(warp * 16 + g) * 2] = m0;
+      sML[(warp * 16 + g) * 2 + 1] = l0;
+      sML[(warp * 16 + g + 8) * 2] = m1;
+      sML[(warp * 16 + g + 8) * 2 + 1] = l1;
+    }
+  }
+  __syncthreads();
+  for (int i = tid; i < rows * p.vdim; i += kWdThreads) {
+    const int r = i / p.vdim, d = i - r * p.vdim, h = h0 + r;
+    float M = kWdNeg;
+#pragma unroll
+    for (int w = 0; w < kWdWarps; ++w) M = fmaxf(M, sML[(w * 16 + r) * 2]);
+    const float sk = p.sink ? __bfloat162float(p.sink[h]) * 1.4426950408889634f : kWdNeg;
+    if (p.splits == 1 && p.sink) M = fmaxf(M, sk);
+    float acc = 0.f, L = p.splits == 1 && p.sink ? fast_exp2(sk - M) : 0.f;
+#pragma unroll
+    for (int w = 0; w < kWdWarps; ++w) {
+      const float f = fast_exp2(sML[(w * 16 + r) * 2] - M);
+      acc = fmaf(f, sO[(w * 16 + r) * S::kStride + d], acc);
+      L = fmaf(f, sML[(w * 16 + r) * 2 + 1], L);
+    }
+    if (p.splits == 1) {
+      p.out[(static_cast<int64_t>(b) * p.heads + h) * p.vdim + d] = __float2bfloat16_rn(L > 0.f ? acc / L : 0.f);
+    } else {
+      const int64_t pi = (static_cast<int64_t>(b) * p.splits + split) * p.heads + h;
+      p.part_o[pi * p.vdim + d] = acc;
+      if (d == 0) {
+        p.part_ml[pi * 2] = M;
+        p.part_ml[pi * 2 + 1] = L;
+      }
+    }
+  }
+}
+
+// Joins the pieces of a sequence and head, and adds the sink.
+__global__ void __launch_bounds__(128) window_join_kernel(const WindowParams<__nv_bfloat16> p) {
+  const int h = blockIdx.x, b = blockIdx.y;
+  const int64_t first = static_cast<int64_t>(b) * p.splits * p.heads + h;
+  float M = p.sink ? __bfloat162float(p.sink[h]) * 1.4426950408889634f : kWdNeg;
+  float L = p.sink ? 1.f : 0.f;
+  const float opened = M;
+  for (int s = 0; s < p.splits; ++s) M = fmaxf(M, p.part_ml[(first + static_cast<int64_t>(s) * p.heads) * 2]);
+  L *= fast_exp2(opened - M);
+  for (int s = 0; s < p.splits; ++s) {
+    const float* ml = p.part_ml + (first + static_cast<int64_t>(s) * p.heads) * 2;
+    L = fmaf(fast_exp2(ml[0] - M), ml[1], L);
+  }
+  for (int d = threadIdx.x; d < p.vdim; d += 128) {
+    float acc = 0.f;
+    for (int s = 0; s < p.splits; ++s) {
+      const int64_t pi = first + static_cast<int64_t>(s) * p.heads;
+      acc = fmaf(fast_exp2(p.part_ml[pi * 2] - M), p.part_o[pi * p.vdim + d], acc);
+    }
+    p.out[(static_cast<int64_t>(b) * p.heads + h) * p.vdim + d] = __float2bfloat16_rn(L > 0.f ? acc / L : 0.f);
+  }
+}
+
+template <int KD, int VD> static int launch_window_decode(const WindowParams<__nv_bfloat16>& p, int batch, cudaStream_t st) {
+  const int smem = WdShape<KD, VD>::kSmem;
+  const cudaError_t e = cudaFuncSetAttribute(window_decode_kernel<KD, VD>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
+  if (e != cudaSuccess) return fail(MV_ERR_CUDA, "window_decode: %s", cudaGetErrorString(e));
+  const int mtiles = (p.heads / p.kv_heads + 15) / 16;
+  window_decode_kernel<KD, VD><<<dim3(p.splits, p.kv_heads * mtiles, batch), kWdThreads, smem, st>>>(p);
+  int rc = check_launch("window_decode");
+  if (rc || p.splits == 1) return rc;
+  window_join_kernel<<<dim3(p.heads, batch), 128, 0, st>>>(p);
+  return check_launch("window_join");
+}
+
+// Pieces per sequence: enough CTAs to fill the GPU twice, none of less than 64 keys.  Depends on shapes only.
+static int window_splits(int batch, int heads, int kv_heads, int64_t most_keys) {
+  const int64_t units = static_cast<int64_t>(batch) * kv_heads * ((heads / kv_heads + 15) / 16);
+  const int64_t want = (2 * kNumSMs + units - 1) / std::max<int64_t>(units, 1);
+  return static_cast<int>(std::max<int64_t>(1, std::min<int64_t>({want, most_keys / 64, 64})));
+}
+
+static int check_window(const char* what, int heads, int kv_heads, int dim, int vdim, int64_t window, int block_size) {
+  if (heads <= 0 || kv_heads <= 0 || heads % kv_heads || dim <= 0 || vdim <= 0 || window <= 0 || block_size <= 0)
+    return fail(MV_ERR_SHAPE, "%s: heads %d over %d, dim %d, vdim %d, window %lld", what, heads, kv_heads, dim, vdim, static_cast<long long>(window));
+  return MV_OK;
+}
+
+}  // namespace mv
+
+extern "C" int mv_kv_norm_store(void* q, const void* k, const void* v, int64_t stride, const void* q_weight,
+                                const void* k_weight, void* kv_out, void* cache, const int64_t* slot_mapping,
+                                int64_t num_slots, int64_t tokens, int q_rows, int k_rows, int v_rows, float eps, int dtype,
+                                void* stream) {
+  using namespace mv;
+  if (dtype != MV_BF16 && dtype != MV_F32) return fail(MV_ERR_DTYPE, "kv_norm_store: dtype %d", dtype);
+  if (tokens < 0 || q_rows <= 0 || k_rows <= 0 || v_rows <= 0) return fail(MV_ERR_SHAPE, "kv_norm_store: %d, %d, %d rows", q_rows, k_rows, v_rows);
+  if (tokens == 0) return MV_OK;
+  if (!q || !k || !v || !q_weight || !k_weight || (cache && !slot_mapping)) return fail(MV_ERR_NULL, "kv_norm_store: null pointer");
+  auto run = [&](auto tag) {
+    using T = decltype(tag);
+    const int eb = sizeof(T);
+    auto go = [&](auto kernel) {
+      kernel<<<static_cast<unsigned>(tokens), kKnThreads, 0, static_cast<cudaStream_t>(stream)>>>(
+          static_cast<T*>(q), static_cast<const T*>(k), static_cast<const T*>(v), stride, static_cast<const T*>(q_weight),
+          static_cast<const T*>(k_weight), static_cast<T*>(kv_out), static_cast<T*>(cache), slot_mapping, num_slots, q_rows,
+          k_rows, v_rows, eps);
+      return check_launch("kv_norm_store");
+    };
+    if (q_rows % 8 == 0 && k_rows % 8 == 0 && v_rows % 8 == 0 && vec8_ok(q, stride, eb) && vec8_ok(k, stride, eb) &&
+        vec8_ok(v, stride, eb) && aligned16(q_weight) && aligned16(k_weight) && aligned16(kv_out) && aligned16(cache))
+      return go(kv_norm_store_kernel<T, 8>);
+    return go(kv_norm_store_kernel<T, 1>);
+  };
+  return dtype == MV_F32 ? run(float{}) : run(__nv_bfloat16{});
+}
+
+extern "C" int mv_window_attention_rows(void* out, const void* q, int64_t q_stride, const void* cache,
+                                        const int32_t* block_tables, int64_t bt_stride, int max_blocks, int block_size,
+                                        int64_t num_blocks, const int32_t* cu_q, int num_seqs, const int64_t* positions,
+                                        const float* bias, int64_t bias_stride, int distances, const void* sink,
+                                        int64_t tokens, int heads, int kv_heads, int dim, int vdim, int64_t window,
+                                        float scale, int dtype, void* stream) {
+  using namespace mv;
+  if (dtype != MV_BF16 && dtype != MV_F32) return fail(MV_ERR_DTYPE, "window_attention_rows: dtype %d", dtype);
+  const int rc = check_window("window_attention_rows", heads, kv_heads, dim, vdim, window, block_size);
+  if (rc) return rc;
+  if (vdim > kWaThreads * kWaPer) return fail(MV_ERR_LIMIT, "window_attention_rows: vdim %d (at most %d)", vdim, kWaThreads * kWaPer);
+  if (bias && distances <= 0) return fail(MV_ERR_SHAPE, "window_attention_rows: %d distances", distances);
+  if (tokens <= 0) return tokens < 0 ? fail(MV_ERR_SHAPE, "window_attention_rows: tokens") : static_cast<int>(MV_OK);
+  if (!out || !q || !cache || !block_tables || !positions) return fail(MV_ERR_NULL, "window_attention_rows: null pointer");
+  const size_t smem = sizeof(float) * (static_cast<size_t>(kWaHeads) * dim + static_cast<size_t>(kWaKeys) * (dim + 1 + vdim) + kWaHeads * kWaKeys);
+  if (smem > 227 * 1024) return fail(MV_ERR_LIMIT, "window_attention_rows: dim %d, vdim %d", dim, vdim);
+  auto run = [&](auto tag) {
+    using T = decltype(tag);
+    const cudaError_t e = cudaFuncSetAttribute(window_attention_rows_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem));
+    if (e != cudaSuccess) return fail(MV_ERR_CUDA, "window_attention_rows: %s", cudaGetErrorString(e));
+    WindowParams<T> p{};
+    p.out = static_cast<T*>(out); p.q = static_cast<const T*>(q); p.q_stride = q_stride; p.cache = static_cast<const T*>(cache);
+    p.tables = block_tables; p.bt_stride = bt_stride; p.max_blocks = max_blocks; p.block_size = block_size; p.num_blocks = num_blocks;
+    p.cu_q = cu_q; p.num_seqs = num_seqs; p.positions = positions; p.bias = bias; p.bias_stride = bias_stride; p.distances = distances;
+    p.sink = static_cast<const T*>(sink); p.heads = heads; p.kv_heads = kv_heads; p.dim = dim; p.vdim = vdim; p.window = window; p.scale = scale;
+    const int chunks = (heads / kv_heads + kWaHeads - 1) / kWaHeads;
+    window_attention_rows_kernel<T><<<dim3(static_cast<unsigned>(tokens), kv_heads * chunks), kWaThreads, smem, static_cast<cudaStream_t>(stream)>>>(p);
+    return check_launch("window_attention_rows");
+  };
+  return dtype == MV_F32 ? run(float{}) : run(__nv_bfloat16{});
+}
+
+// Bytes of scratch, or -1 when the kernel does not take the sizes.
+extern "C" int64_t mv_window_decode_workspace_bytes(int batch, int heads, int kv_heads, int dim, int vdim, int64_t most_keys) {
+  using namespace mv;
+  if (batch < 0 || batch > 65535 || heads <= 0 || kv_heads <= 0 || heads % kv_heads || dim <= 0 || vdim <= 0 || dim % 8 || vdim % 8 ||
+      dim > 256 || vdim > 256 || most_keys <= 0)
+    return -1;
+  const int splits = window_splits(batch, heads, kv_heads, most_keys);
+  return splits == 1 ? 0 : static_cast<int64_t>(batch) * splits * heads * (vdim + 2) * 4;
+}
+
+extern "C" int mv_window_decode(void* out, const void* q, int64_t q_stride, const void* cache, const int32_t* block_tables,
+                                int64_t bt_stride, int max_blocks, int block_size, int64_t num_blocks,
+                                const int64_t* positions, const float* bias, int64_t bias_stride, int distances,
+                                const void* sink, int batch, int heads, int kv_heads, int dim, int vdim, int64_t window,
+                                float scale, void* workspace, int64_t workspace_bytes, void* stream) {
+  using namespace mv;
+  const int rc = check_window("window_decode", heads, kv_heads, dim, vdim, window, block_size);
+  if (rc) return rc;
+  const int64_t most = std::min<int64_t>(window, static_cast<int64_t>(max_blocks) * block_size);
+  const int64_t need = mv_window_decode_workspace_bytes(batch, heads, kv_heads, dim, vdim, std::max<int64_t>(most, 1));
+  if (need < 0) return fail(MV_ERR_LIMIT, "window_decode: dim %d, vdim %d, batch %d", dim, vdim, batch);
+  if (bias && distances <= 0) return fail(MV_ERR_SHAPE, "window_decode: %d distances", distances);
+  if (batch == 0) return MV_OK;
+  if (!out || !q || !cache || !block_tables || !positions) return fail(MV_ERR_NULL, "window_decode: null pointer");
+  if (!aligned16(cache) || (reinterpret_cast<uintptr_t>(q) & 3u) || q_stride % 2) return fail(MV_ERR_ALIGN, "window_decode: alignment");
+  if (need > 0 && (!workspace || workspace_bytes < need)) return fail(MV_ERR_WORKSPACE, "window_decode: workspace");
+  WindowParams<__nv_bfloat16> p{};
+  p.out = static_cast<__nv_bfloat16*>(out); p.q = static_cast<const __nv_bfloat16*>(q); p.q_stride = q_stride;
+  p.cache = static_cast<const __nv_bfloat16*>(cache);
+  p.tables = block_tables; p.bt_stride = bt_stride; p.max_blocks = max_blocks; p.block_size = block_size; p.num_blocks = num_blocks;
+  p.positions = positions; p.bias = bias; p.bias_stride = bias_stride; p.distances = bias ? distances : 1;
+  p.sink = static_cast<const __nv_bfloat16*>(sink); p.heads = heads; p.kv_heads = kv_heads; p.dim = dim; p.vdim = vdim;
+  p.window = window; p.scale = scale;
+  p.splits = window_splits(batch, heads, kv_heads, std::max<int64_t>(most, 1));
+  p.part_ml = static_cast<float*>(workspace);
+  p.part_o = p.part_ml ? p.part_ml + static_cast<int64_t>(batch) * p.splits * heads * 2 : nullptr;
+  auto st = static_cast<cudaStream_t>(stream);
+  auto go = [&](auto kd) {
+    constexpr int KD = decltype(kd)::value;
+    if (vdim <= 64) return launch_window_decode<KD, 64>(p, batch, st);
+    if (vdim <= 128) return launch_window_decode<KD, 128>(p, batch, st);
+    return launch_window_decode<KD, 256>(p, batch, st);
+  };
+  if (dim <= 64) return go(std::integral_constant<int, 64>{});
+  if (dim <= 128) return go(std::integral_constant<int, 128>{});
+  return go(std::integral_constant<int, 256>{});
+}

@@ -123,9 +123,8 @@ class ModelRunner:
     # ------------------------------------------------------------------ memory ---
     def kv_block_bytes(self):
         c = self.model_cfg
-        latent = cache.latent_block_bytes(self.model, self.block_size, self.dtype)
         if not self.kv_layers:
-            return latent
+            return cache.paged_block_bytes(self.model, self.block_size, self.dtype)
         rows = self.block_size * 2 * c.num_layers * (c.num_kv_heads // self.world_size)
         if self.kv_int8:
             return rows * (c.head_dim + 2)             # int8 codes + one fp16 scale per row
@@ -244,6 +243,7 @@ class ModelRunner:
                     positions=meta["positions"], last_token_index=rows, num_decode=nd,
                     portion_keys=sum(s.num_cached_tokens + n for s, n in zip(seqs[nd:], counts[nd:])),
                     portion_fresh=all(s.num_cached_tokens == 0 for s in seqs[nd:]),
+                    portion_spans=[(s.num_cached_tokens, n) for s, n in zip(seqs[nd:], counts[nd:])],
                     portion_cu_q=cu_q[nd:] - cu_q[nd], portion_cu_k=cu_k[nd:] - cu_k[nd],
                     state_slots=meta["slots"], state_starts=meta["starts"])
         return input_ids, order

@@ -17,6 +17,22 @@ _DTYPES = {"BF16": torch.bfloat16, "F16": torch.float16, "F32": torch.float32, "
            "BOOL": torch.bool}
 
 
+class Scope:
+    """A source under a name prefix."""
+
+    def __init__(self, source, prefix):
+        self.source, self.prefix = source, prefix
+
+    def __call__(self, name, shape):
+        return self.source(self.prefix + name, shape)
+
+    def shape(self, name, default):
+        return self.source.shape(self.prefix + name, default)
+
+    def scoped(self, prefix):
+        return Scope(self.source, self.prefix + prefix)
+
+
 class WeightSource:
     def __init__(self, dtype, device):
         self.dtype, self.device = dtype, torch.device(device)
@@ -32,8 +48,12 @@ class WeightSource:
         self.used.add(name)
         return t.to(device=self.device, dtype=self.dtype if t.is_floating_point() else t.dtype).contiguous()
 
+    def shape(self, name, default):
+        """Shape of a tensor that fixes a size by itself; `default` where the source has no tensors of its own."""
+        return tuple(default)
+
     def scoped(self, prefix):
-        return lambda name, shape: self(prefix + name, shape)
+        return Scope(self, prefix)
 
     def check_all_used(self):
         """Nothing by default; a file or dict reports tensors that no part of the model asked for."""
@@ -48,6 +68,11 @@ class DictWeights(WeightSource):
         if name not in self.tensors:
             raise KeyError(f"no tensor named '{name}'")
         return self.tensors[name]
+
+    def shape(self, name, default):
+        if name not in self.tensors:
+            raise KeyError(f"no tensor named '{name}'")
+        return tuple(self.tensors[name].shape)
 
     def check_all_used(self):
         left = sorted(set(self.tensors) - self.used)

@@ -88,12 +88,13 @@ def latent_decode(q_lat, q_rot, cache, block_tables, positions, sink, scale, wor
     return out
 
 
-def latent_gather(cache, cu_k, keys, block_tables):
-    """Packed latent rows (keys, row) of the sequences of cu_k, from position 0, out of the paged cache."""
+def latent_gather(cache, cu_k, keys, block_tables, first=None):
+    """Packed rows (keys, row) of the sequences of cu_k, from position `first` of each (0), out of the paged cache."""
     row = cache.shape[2]
     out = torch.empty((keys, row), dtype=cache.dtype, device=cache.device)
     _cabi.check(_cabi.lib().mv_latent_gather(
-        out.data_ptr(), cache.data_ptr(), cu_k.data_ptr(), cu_k.numel() - 1, keys, block_tables.data_ptr(),
+        out.data_ptr(), cache.data_ptr(), cu_k.data_ptr(), first.data_ptr() if first is not None else None,
+        cu_k.numel() - 1, keys, block_tables.data_ptr(),
         block_tables.stride(0), block_tables.shape[1], cache.shape[1], cache.shape[0], row,
         _cabi.layer_dtype_code(cache.dtype), _cabi.stream_ptr()))
     return out
@@ -127,10 +128,10 @@ class LatentAttention(nn.Module):
         self.ukv_w = param(torch.cat([load("uk", (H * d, rank)), load("uv", (H * vd, rank))]))
         self.o_w = param(load("o", (width, H * vd)))
         self.cos_t, self.sin_t = rope_table(m["rot"]["base"], self.rope_dims, max_position, self.o_w.device)
-        self.latent_cache = None        # (blocks, block_size, rank + rot_dim), assigned by the model runner
+        self.paged_cache = None        # (blocks, block_size, rank + rot_dim), assigned by the model runner
 
     @property
-    def latent_row(self):
+    def paged_row(self):
         return self.rank + self.rot_dim
 
     @property
@@ -154,9 +155,9 @@ class LatentAttention(nn.Module):
         q_lat = torch.bmm(q[:, :, :d].transpose(0, 1), self.uk_w).transpose(0, 1)            # (tokens, heads, rank)
         o = None
         if cu_q is None:
-            o = latent_decode(q_lat, q[:, :, d:], self.latent_cache, block_tables, positions, self.sink, self.scale)
+            o = latent_decode(q_lat, q[:, :, d:], self.paged_cache, block_tables, positions, self.sink, self.scale)
         if o is None:
-            o = latent_attention_rows(q_lat, q[:, :, d:], self.latent_cache, block_tables, cu_q, positions, self.sink,
+            o = latent_attention_rows(q_lat, q[:, :, d:], self.paged_cache, block_tables, cu_q, positions, self.sink,
                                       self.scale)
         return torch.bmm(o.transpose(0, 1), self.uv_w.transpose(1, 2)).transpose(0, 1)
 
@@ -176,7 +177,7 @@ class LatentAttention(nn.Module):
             cu_k = ctx.portion_cu_q
         else:
             cu_k = ctx.portion_cu_k
-            lat = latent_gather(self.latent_cache, cu_k, ctx.portion_keys, tables)
+            lat = latent_gather(self.paged_cache, cu_k, ctx.portion_keys, tables)
         kv = F.linear(lat[:, :rank], self.ukv_w)
         return latent_prefill(q2, kv, lat[:, rank:], ctx.portion_cu_q, cu_k, H, d, r, self.vdim, self.scale, self.sink)
 
@@ -187,7 +188,7 @@ class LatentAttention(nn.Module):
         H, d, r = self.heads, self.dim, self.rot_dim
         q, g, nd = p["q"], p["g"], ctx.num_decode
         lat = latent_prep(q, p["dkv"], self.c_norm, ctx.positions, self.cos_t, self.sin_t, H, d, r, self.rope_dims,
-                          self.rank, self.eps, self.latent_cache, ctx.slot_mapping)
+                          self.rank, self.eps, self.paged_cache, ctx.slot_mapping)
         o = torch.empty((h.shape[0], H * self.vdim), dtype=h.dtype, device=h.device)
         if nd:
             y = self._absorbed(q[:nd].unflatten(1, (H, d + r)), ctx.block_tables[:nd], None, ctx.positions[:nd])

@@ -9,9 +9,10 @@ import torch.nn.functional as F
 
 
 class StackedLinear(nn.Module):
-    """parts: {name: (out, in) weight}.  Calling it with (rows, in) returns {name: (rows, out) view}."""
+    """parts: {name: (out, in) weight}, biases: {name: (out,)} for some of them.  Calling it with (rows, in) returns
+    {name: (rows, out) view}."""
 
-    def __init__(self, parts):
+    def __init__(self, parts, biases=None):
         super().__init__()
         rows, self.spans, at = [], {}, 0
         for name, w in parts.items():
@@ -23,9 +24,15 @@ class StackedLinear(nn.Module):
                 rows.append(w.new_zeros(pad, w.shape[1]))
             at += n + pad
         self.weight = nn.Parameter(torch.cat(rows) if len(rows) > 1 else rows[0], requires_grad=False)
+        self.bias = None
+        if biases:
+            b = self.weight.new_zeros(at)
+            for name, t in biases.items():
+                b[self.spans[name][0]:self.spans[name][1]] = t
+            self.bias = nn.Parameter(b, requires_grad=False)
 
     def forward(self, h):
-        y = F.linear(h, self.weight)
+        y = F.linear(h, self.weight, self.bias)
         return {name: y[:, a:b] for name, (a, b) in self.spans.items()}
 
 

@@ -1,5 +1,5 @@
 """State-space mixer (Mamba-2 / SSD): stacked input projection, causal depthwise convolution with silu, the
-selective recurrence, gated group norm and output projection (csrc/mamba2.cu).
+selective recurrence, gated group norm and output projection (csrc/mamba2.cu, csrc/short_conv.cu).
 
 The per-sequence state (last convolution inputs, fp32 recurrent state) lives in slots assigned by the engine; the
 model runner allocates what `slot_state_spec` describes and fills `slot_state`.
@@ -12,25 +12,7 @@ from .. import _cabi
 from ..utils.context import get_context
 from .group_norm import gated_group_norm
 from .linear import StackedLinear
-
-
-def conv_silu(u, weight, bias, cu, slots, starts, state):
-    """u (tokens, channels) any row stride -> (tokens, channels); see mv_conv_silu."""
-    _cabi.require_cuda(u, weight, slots, starts)
-    tokens, channels = u.shape
-    out = torch.empty((tokens, channels), dtype=u.dtype, device=u.device)
-    _cabi.check(_cabi.lib().mv_conv_silu(
-        out.data_ptr(), u.data_ptr(), u.stride(0), weight.data_ptr(), bias.data_ptr(), weight.shape[1], channels,
-        cu.data_ptr() if cu is not None else None, slots.numel(), tokens, slots.data_ptr(), starts.data_ptr(),
-        state.data_ptr(), state.shape[0], _cabi.layer_dtype_code(u.dtype), _cabi.stream_ptr()))
-    return out
-
-
-def conv_state_update(state, u, taps, cu, slots, starts):
-    _cabi.check(_cabi.lib().mv_conv_state_update(
-        state.data_ptr(), u.data_ptr(), u.stride(0), taps, u.shape[1], cu.data_ptr() if cu is not None else None,
-        slots.numel(), slots.data_ptr(), starts.data_ptr(), state.shape[0], _cabi.layer_dtype_code(u.dtype),
-        _cabi.stream_ptr()))
+from .short_conv import conv_silu, conv_state_update
 
 
 def ssm_scan(xbc, dt, dt_bias, A_log, D, cu, slots, starts, state, heads, vdim, state_dim, groups, out=None,

@@ -11,7 +11,7 @@ package: they carry what the metadata kernels build on the GPU once per step
 (the reference rebuilds positions on the host in every layer,
 src/myvllm/models/qwen3.py:196-212) and default to None.
 """
-from dataclasses import dataclass, fields
+from dataclasses import dataclass, field, fields
 from typing import Optional
 
 import torch
@@ -38,8 +38,10 @@ class Context:
     portion_cu_k: Optional[torch.Tensor] = None
     portion_keys: int = 0                            # cu_seqlens_k's total over those sequences
     portion_fresh: bool = False                      # none of them has tokens behind it
+    portion_spans: Optional[list] = None             # (tokens behind it, tokens of this step) of each, on the host
     state_slots: Optional[torch.Tensor] = None       # (num_seqs,) int32 slot of each sequence
     state_starts: Optional[torch.Tensor] = None      # (num_seqs,) int32 tokens behind this step (-1: padding row)
+    memo: dict = field(default_factory=dict)         # what layers derive from the above once per step
 
 
 class _Holder:
