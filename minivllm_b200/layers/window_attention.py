@@ -26,7 +26,7 @@ def distance_buckets(count, buckets, bias_max):
     """Bucket of the distances 0 .. count - 1: the first half of the buckets one each, then geometrically up to
     bias_max."""
     half = buckets // 2
-    if half < 1 or bias_max <= half:
+    if half < 1 or (count > half and bias_max <= half):
         raise ValueError(f"distance bias: {buckets} buckets up to {bias_max}")
     far = lambda n: half + math.floor(math.log(n / half) / math.log(bias_max / half) * (buckets - half))
     return [n if n < half else min(buckets - 1, far(n)) for n in range(count)]
@@ -34,7 +34,7 @@ def distance_buckets(count, buckets, bias_max):
 
 def distance_bias(rel, bias_max, window):
     """rel (buckets, heads) -> (heads, distances) fp32; larger distances have the last one's bias."""
-    count = min(window, math.ceil(bias_max) + 1)
+    count = min(window, max(math.ceil(bias_max), rel.shape[0] // 2) + 1)
     idx = torch.tensor(distance_buckets(count, rel.shape[0], bias_max), device=rel.device)
     return rel.float()[idx].t().contiguous()
 

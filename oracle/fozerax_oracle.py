@@ -203,3 +203,59 @@ def forward(config, weights, token_ids, dtype=torch.float64, per_layer=None):
         if per_layer is not None:
             per_layer.append(x)
     return rms_norm(x, w["final.norm"], eps) @ w["head"].T
+
+
+def random_weights(config, seed=0, rank=5, buckets=10):
+    """Checkpoint tensors of a configuration from a seed, bfloat16, with every mechanism visible in the output
+    (projections of unit gain, norms around one, sinks around zero, biases of the size of the scores, decays between slow
+    and fast, router logits far apart)."""
+    g = torch.Generator().manual_seed(seed)
+
+    def mat(o, i, gain=1.0):
+        return torch.randn(o, i, generator=g) * (gain / math.sqrt(i))
+
+    def around(n, mean, spread):
+        return mean + spread * torch.randn(n, generator=g)
+
+    W = config["width"]
+    w = {"embed": torch.randn(config["vocab"], W, generator=g), "embed.norm": around(W, 1.0, 0.1),
+         "head": mat(config["vocab"], W), "final.norm": around(W, 1.0, 0.1)}
+    for i, layer in enumerate(config["layers"]):
+        l, m = f"l{i}.", layer["mixer"]
+        p = l + "mix."
+        w[l + "norm1"] = around(W, 1.0, 0.1)
+        if layer["type"] == "gla":
+            H, K, V = m["heads"], m["dim"], m["vdim"]
+            w.update({p + "q": mat(H * K, W), p + "k": mat(H * K, W), p + "v": mat(H * V, W), p + "g": mat(H * V, W),
+                      p + "o": mat(W, H * V), p + "norm": around(V, 1.0, 0.1), p + "a1": mat(rank, W),
+                      p + "a2": mat(H * K, rank), p + "a2.b": around(H * K, 2.0, 2.0)})
+        else:
+            a, b = m["left"], m["right"]
+            H, G, d, vd = a["heads"], a["kv_heads"], a["dim"], a["vdim"]
+            q = p + "left."
+            for n, rows in (("q", H * d), ("k", G * d), ("v", G * vd)):
+                w[q + n], w[q + n + ".b"] = mat(rows, W), around(rows, 0.0, 0.3)
+            w.update({q + "q.norm": around(H * d, 1.5, 0.2), q + "k.norm": around(G * d, 1.5, 0.2),
+                      q + "rel": torch.randn(buckets, H, generator=g), q + "sink": around(H, 1.0, 0.5),
+                      q + "o": mat(W, H * vd), q + "out": around(W, 1.0, 0.1)})
+            H, G, K, V = b["heads"], b["kv_heads"], b["dim"], b["vdim"]
+            q = p + "right."
+            for n, rows in (("q", G * K), ("k", G * K), ("v", H * V)):
+                w[q + n], w[q + n + ".conv"] = mat(rows, W), mat(rows, b["conv"])
+            w.update({q + "b": mat(H, W), q + "a": mat(H, W), q + "A_log": around(H, -1.0, 1.0),
+                      q + "dt_bias": around(H, -2.0, 1.0), q + "norm": around(V, 1.0, 0.1), q + "g": mat(H * V, W),
+                      q + "o": mat(W, H * V), q + "out": around(W, 1.0, 0.1)})
+        e = layer.get("mlp")
+        if not e:
+            continue
+        w[l + "norm2"] = around(W, 1.0, 0.1)
+        p = l + "mlp."
+        names = [("", e["ff"])] if e["kind"] == "dense" else \
+            [(f"e{j}.", e["expert"]["ff"]) for j in range(e["router"]["experts"])]
+        if e["kind"] == "moe":
+            w[p + "router"] = mat(e["router"]["experts"], W, 3.0)
+            if e.get("shared"):
+                names.append(("shared.", e["shared"]["ff"]))
+        for name, ff in names:
+            w[p + name + "gate"], w[p + name + "up"], w[p + name + "down"] = mat(ff, W, 1.5), mat(ff, W, 1.5), mat(W, ff)
+    return {k: v.to(torch.bfloat16) for k, v in w.items()}
