@@ -634,6 +634,23 @@ int mv_delta_scan(void* out, int64_t out_stride, const void* qkv, int64_t stride
     conv_state, const void* gate, int64_t gate_stride, const void* norm_w, float eps, int dtype,
     void* stream);
 
+/*
+ * The same recurrences for packed portions in chunks of 64 tokens on tensor cores, bf16: dim a multiple of 8 up to 128,
+ * vdim a multiple of 8, rows on 16-byte boundaries.  tokens = cu[num_seqs]; workspace_bytes is -1 when the sizes are not
+ * taken.
+ */
+int64_t mv_gla_chunk_workspace_bytes(int64_t tokens, int num_seqs, int heads, int dim, int vdim);
+int mv_gla_chunk_scan(void* out, int64_t out_stride, const void* q, const void* k, const void* v,
+    int64_t stride, const void* z, int64_t z_stride, float tau, const int32_t* cu, int num_seqs,
+    int64_t tokens, const int32_t* slots, const int32_t* start, float* state, int num_slots, int
+    heads, int dim, int vdim, float q_scale, void* workspace, int64_t workspace_bytes, void* stream);
+int64_t mv_delta_chunk_workspace_bytes(int64_t tokens, int num_seqs, int heads, int dim, int vdim);
+int mv_delta_chunk_scan(void* out, int64_t out_stride, const void* qkv, int64_t stride, const void*
+    beta, const void* a, int64_t ba_stride, const void* A_log, const void* dt_bias, const int32_t* cu,
+    int num_seqs, int64_t tokens, const int32_t* slots, const int32_t* start, float* state, int
+    num_slots, int heads, int kv_heads, int dim, int vdim, float q_scale, void* workspace, int64_t
+    workspace_bytes, void* stream);
+
 #ifdef __cplusplus
 }
 #endif

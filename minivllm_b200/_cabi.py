@@ -129,6 +129,12 @@ SIGNATURES = {
     "mv_delta_scan": (_c_int, [_c_ptr, _c_i64, _c_ptr, _c_i64, _c_ptr, _c_ptr, _c_i64, _c_ptr, _c_ptr, _c_ptr, _c_int,
         _c_ptr, _c_ptr, _c_ptr, _c_int, _c_int, _c_int, _c_int, _c_int, _c_f32, _c_ptr, _c_int, _c_ptr, _c_ptr, _c_i64,
         _c_ptr, _c_f32, _c_int, _c_ptr]),
+    "mv_gla_chunk_workspace_bytes": (_c_i64, [_c_i64, _c_int, _c_int, _c_int, _c_int]),
+    "mv_gla_chunk_scan": (_c_int, [_c_ptr, _c_i64, _c_ptr, _c_ptr, _c_ptr, _c_i64, _c_ptr, _c_i64, _c_f32, _c_ptr, _c_int,
+        _c_i64, _c_ptr, _c_ptr, _c_ptr, _c_int, _c_int, _c_int, _c_int, _c_f32, _c_ptr, _c_i64, _c_ptr]),
+    "mv_delta_chunk_workspace_bytes": (_c_i64, [_c_i64, _c_int, _c_int, _c_int, _c_int]),
+    "mv_delta_chunk_scan": (_c_int, [_c_ptr, _c_i64, _c_ptr, _c_i64, _c_ptr, _c_ptr, _c_i64, _c_ptr, _c_ptr, _c_ptr, _c_int,
+        _c_i64, _c_ptr, _c_ptr, _c_ptr, _c_int, _c_int, _c_int, _c_int, _c_int, _c_f32, _c_ptr, _c_i64, _c_ptr]),
 }
 
 _lib = None

@@ -19,8 +19,8 @@ GROUPS = {
               "paged_decode_static.cu", "pre_attention.cu", "comm.cu"],
     "sipazen": ["norms.cu", "latent_attention.cu", "latent_decode.cu", "latent_prefill.cu", "short_conv.cu", "mamba2.cu",
                 "mamba2_chunk.cu", "moe.cu", "grouped_gemm.cu"],
-    "fozerax": ["norms.cu", "window_attention.cu", "latent_prefill.cu", "short_conv.cu", "gla.cu", "gated_delta.cu", "moe.cu",
-                "grouped_gemm.cu"],
+    "fozerax": ["norms.cu", "window_attention.cu", "latent_prefill.cu", "short_conv.cu", "gla.cu", "gla_chunk.cu", "gated_delta.cu",
+                "gated_delta_chunk.cu", "moe.cu", "grouped_gemm.cu"],
 }
 SOURCES = COMMON + list(dict.fromkeys(s for g in GROUPS.values() for s in g))
 NVCC_FLAGS = [

@@ -37,13 +37,6 @@ struct CsParams {
 };
 
 using Mma = Mma16816<__nv_bfloat16>;
-__device__ __forceinline__ void split2(float a, float b, uint32_t& hi, uint32_t& lo) {
-  const __nv_bfloat162 h = __floats2bfloat162_rn(a, b);
-  const float2 f = __bfloat1622float2(h);
-  const __nv_bfloat162 r = __floats2bfloat162_rn(a - f.x, b - f.y);
-  hi = *reinterpret_cast<const uint32_t*>(&h);
-  lo = *reinterpret_cast<const uint32_t*>(&r);
-}
 template <int N, int PB>
 __global__ void __launch_bounds__(kCsThreads, 2) ssm_chunk_kernel(const CsParams p) {
   using Sh = CsShape<N, PB>;

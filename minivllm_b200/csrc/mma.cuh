@@ -39,4 +39,13 @@ template <typename T> __device__ __forceinline__ uint32_t pack2(float lo, float 
   return *reinterpret_cast<uint32_t*>(&v);
 }
 
+// A pair of fp32 values as two bf16 terms each: the value and its rounding residue (16 bits together).
+__device__ __forceinline__ void split2(float a, float b, uint32_t& hi, uint32_t& lo) {
+  const __nv_bfloat162 h = __floats2bfloat162_rn(a, b);
+  const float2 f = __bfloat1622float2(h);
+  const __nv_bfloat162 r = __floats2bfloat162_rn(a - f.x, b - f.y);
+  hi = *reinterpret_cast<const uint32_t*>(&h);
+  lo = *reinterpret_cast<const uint32_t*>(&r);
+}
+
 }  // namespace mv

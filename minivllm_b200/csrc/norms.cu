@@ -6,6 +6,7 @@
 // HBM-bound.  A CTA owns a row and keeps it in shared memory as fp32; every group of channels belongs to a fixed
 // set of warps, so sums are formed in a fixed order whatever the batch.
 #include <algorithm>
+#include <type_traits>
 #include "vec.cuh"
 
 namespace mv {
@@ -441,6 +442,55 @@ gated_group_norm_kernel(T* __restrict__ out, const T* __restrict__ y, int64_t y_
   }
 }
 
+// The second form of the above for runs of whole 16-byte pieces, up to 1,024 channels: L lanes (a power of two) per run,
+// everything in registers.
+template <typename T, int L, int kCh>
+__global__ void __launch_bounds__(kNormThreads)
+head_norm_gate_kernel(T* __restrict__ out, const T* __restrict__ y, int64_t y_stride, const T* __restrict__ z,
+                      int64_t z_stride, const T* __restrict__ w, int64_t rows, int heads, int gs, float eps) {
+  const int lane = threadIdx.x & (L - 1);
+  const int64_t items = rows * heads, step = static_cast<int64_t>(gridDim.x) * (kNormThreads / L);
+  for (int64_t i0 = static_cast<int64_t>(blockIdx.x) * (kNormThreads / L); i0 < items; i0 += step) {
+    const int64_t i = i0 + threadIdx.x / L, row = i / heads;
+    const int h = static_cast<int>(i - row * heads);
+    const bool on = i < items;
+    Raw8<T> a[kCh], b[kCh];
+    float acc = 0.f;
+#pragma unroll
+    for (int k = 0; k < kCh; ++k) {
+      const int c = (k * L + lane) * 8;
+      if (on && c < gs) {
+        a[k].load(y + row * y_stride + static_cast<int64_t>(h) * gs + c);
+        b[k].load(z + row * z_stride + static_cast<int64_t>(h) * gs + c);
+      }
+    }
+#pragma unroll
+    for (int k = 0; k < kCh; ++k)
+      if (on && (k * L + lane) * 8 < gs) {
+        float v[8];
+        a[k].get(v);
+#pragma unroll
+        for (int e = 0; e < 8; ++e) acc = fmaf(v[e], v[e], acc);
+      }
+#pragma unroll
+    for (int o = L / 2; o; o >>= 1) acc += __shfl_xor_sync(0xffffffffu, acc, o);
+    const float rs = 1.f / sqrtf(acc / static_cast<float>(gs) + eps);
+#pragma unroll
+    for (int k = 0; k < kCh; ++k) {
+      const int c = (k * L + lane) * 8;
+      if (on && c < gs) {
+        float v[8], t[8], g[8];
+        a[k].get(v);
+        b[k].get(g);
+        Vec<T, 8>::load(w + c, t);
+#pragma unroll
+        for (int e = 0; e < 8; ++e) v[e] = v[e] * rs * t[e] * silu_t<T>(g[e]);
+        Vec<T, 8>::store(out + row * (static_cast<int64_t>(heads) * gs) + static_cast<int64_t>(h) * gs + c, v);
+      }
+    }
+  }
+}
+
 // out = act(gate, y), see glu_act; row r of y is `heads` pieces of cols / heads elements, y_head_stride apart
 template <typename T, int V>
 __global__ void __launch_bounds__(kNormThreads)
@@ -610,8 +660,26 @@ static int gated_norm(const char* what, bool gate_first, void* out, const void* 
           static_cast<const T*>(w), width, groups, eps);
       return check_launch(what);
     };
-    if ((width / groups) % 8 == 0 && vec8_ok(out, width, eb) && vec8_ok(y, y_stride, eb) && vec8_ok(z, z_stride, eb) &&
-        aligned16(w))
+    const bool v8 = (width / groups) % 8 == 0 && vec8_ok(out, width, eb) && vec8_ok(y, y_stride, eb) && vec8_ok(z, z_stride, eb) &&
+        aligned16(w);
+    if (v8 && !gate_first && width / groups <= 1024) {
+      const int gs = width / groups;
+      auto lanes = [&](auto l, auto ch) {
+        constexpr int L = decltype(l)::value;
+        const int64_t blocks = (rows * groups + kNormThreads / L - 1) / (kNormThreads / L);
+        head_norm_gate_kernel<T, L, decltype(ch)::value><<<static_cast<unsigned>(std::min<int64_t>(blocks, kNumSMs * 32)), kNormThreads, 0,
+                                                           static_cast<cudaStream_t>(stream)>>>(
+            static_cast<T*>(out), static_cast<const T*>(y), y_stride, static_cast<const T*>(z), z_stride, static_cast<const T*>(w),
+            rows, groups, gs, eps);
+        return check_launch(what);
+      };
+      using std::integral_constant;
+      if (gs <= 64) return lanes(integral_constant<int, 8>{}, integral_constant<int, 1>{});
+      if (gs <= 128) return lanes(integral_constant<int, 16>{}, integral_constant<int, 1>{});
+      if (gs <= 256) return lanes(integral_constant<int, 32>{}, integral_constant<int, 1>{});
+      return lanes(integral_constant<int, 32>{}, integral_constant<int, 4>{});
+    }
+    if (v8)
       return gate_first ? go(gated_group_norm_kernel<T, 8, true>) : go(gated_group_norm_kernel<T, 8, false>);
     return gate_first ? go(gated_group_norm_kernel<T, 1, true>) : go(gated_group_norm_kernel<T, 1, false>);
   };

@@ -9,15 +9,18 @@
 // products run as fma.rn.f32x2 and a float4 of k or q from shared memory serves two of them.  The sums over K meet in a
 // reduce-scatter over the KP lanes: afterwards every lane holds one column's result.
 //
+// Decays near one enter as alpha - 1 (S + (alpha - 1) S): the rounding of alpha itself would add up over thousands of
+// tokens.
+//
 // The delta rule's scalar decay is kept out of the matrix: S = G * S', G the product of the decays, folded into S' when
 // it becomes small.
 //
 // scan_kernel   prompts: one CTA per (sequence, head, block of value columns).  While a tile of tokens is worked on,
 //               each warp has the next tile's token of its own in registers; it turns it into what the recurrence wants
 //               (unit norms, decays, step sizes) in shared memory at the end of the tile.
-// step_kernel   one token per sequence: convolution (delta rule), one step of the state, the head's norm and the output
-//               gate in one launch.  HBM-bound: 8 * heads * K * V bytes per sequence; the state's loads are issued
-//               before anything else.
+// step_quad_kernel, step_kernel (vdim not a multiple of four)
+//               one token per sequence: convolution (delta rule), one step of the state, the head's norm and the output
+//               gate in one launch.  HBM-bound: 8 * heads * K * V bytes per sequence.
 #pragma once
 #include <algorithm>
 #include <type_traits>
@@ -96,11 +99,11 @@ template <typename Sh> struct ScanState {
 #pragma unroll
         for (int v = 0; v < Sh::VT; v += 4) {
           if (vec) {
-            const float4 x = r < K && v < cols ? *reinterpret_cast<const float4*>(src + static_cast<int64_t>(r) * V + v) : make_float4(0.f, 0.f, 0.f, 0.f);
+            const float4 x = r < K && v < cols ? *reinterpret_cast<const float4*>(src + r * V + v) : make_float4(0.f, 0.f, 0.f, 0.f);
             t[v] = x.x; t[v + 1] = x.y; t[v + 2] = x.z; t[v + 3] = x.w;
           } else {
 #pragma unroll
-            for (int w = 0; w < 4; ++w) t[v + w] = r < K && v + w < cols ? src[static_cast<int64_t>(r) * V + v + w] : 0.f;
+            for (int w = 0; w < 4; ++w) t[v + w] = r < K && v + w < cols ? src[r * V + v + w] : 0.f;
           }
         }
 #pragma unroll
@@ -120,16 +123,16 @@ template <typename Sh> struct ScanState {
 #pragma unroll
           for (int w = 0; w < 4; ++w) t[w] = G * (e & 1 ? s[2 * i + e / 2][v + w].y : s[2 * i + e / 2][v + w].x);
           if (vec) {
-            if (v < cols) *reinterpret_cast<float4*>(dst + static_cast<int64_t>(r) * V + v) = make_float4(t[0], t[1], t[2], t[3]);
+            if (v < cols) *reinterpret_cast<float4*>(dst + r * V + v) = make_float4(t[0], t[1], t[2], t[3]);
           } else {
 #pragma unroll
             for (int w = 0; w < 4; ++w)
-              if (v + w < cols) dst[static_cast<int64_t>(r) * V + v + w] = t[w];
+              if (v + w < cols) dst[r * V + v + w] = t[w];
           }
         }
       }
   }
-  // One token of gated linear attention.  sk, sq, sa: K values in shared memory; v: this lane's columns.
+  // One token of gated linear attention.  sk, sq, sa: K values in shared memory (sa: alpha - 1); v: this lane's columns.
   // o receives the read-out of the columns first_held(kp) .. + HELD.
   __device__ __forceinline__ void gla(const float* sk, const float* sq, const float* sa, const float* sv, int kp, float (&o)[Sh::HELD]) {
     float2 acc[Sh::VT];
@@ -149,8 +152,8 @@ template <typename Sh> struct ScanState {
       const float4 a4 = *reinterpret_cast<const float4*>(sa + (i * Sh::KP + kp) * 4);
 #pragma unroll
       for (int v = 0; v < Sh::VT; ++v) {
-        s[2 * i][v] = fma_f32x2(make_float2(k4.x, k4.y), vv[v], mul_f32x2(make_float2(a4.x, a4.y), s[2 * i][v]));
-        s[2 * i + 1][v] = fma_f32x2(make_float2(k4.z, k4.w), vv[v], mul_f32x2(make_float2(a4.z, a4.w), s[2 * i + 1][v]));
+        s[2 * i][v] = fma_f32x2(make_float2(k4.x, k4.y), vv[v], fma_f32x2(make_float2(a4.x, a4.y), s[2 * i][v], s[2 * i][v]));
+        s[2 * i + 1][v] = fma_f32x2(make_float2(k4.z, k4.w), vv[v], fma_f32x2(make_float2(a4.z, a4.w), s[2 * i + 1][v], s[2 * i + 1][v]));
         acc[v] = fma_f32x2(make_float2(q4.x, q4.y), s[2 * i][v], acc[v]);
         acc[v] = fma_f32x2(make_float2(q4.z, q4.w), s[2 * i + 1][v], acc[v]);
       }
@@ -162,11 +165,11 @@ template <typename Sh> struct ScanState {
 #pragma unroll
     for (int j = 0; j < Sh::HELD; ++j) o[j] = val[j];
   }
-  // One token of the gated delta rule.  ks, qs: factors of the stored k and q; kq: their product k . q, scaled.
+  // One token of the gated delta rule.  gm1: g - 1; ks, qs: factors of the stored k and q; kq: their product k . q, scaled.
   // Lanes with the bit KP / 2 of kp set receive the read-outs.
-  __device__ __forceinline__ void delta(const float* sk, const float* sq, const float* sv, float g, float beta, float ks,
+  __device__ __forceinline__ void delta(const float* sk, const float* sq, const float* sv, float gm1, float beta, float ks,
                                         float qs, float kq, int kp, float (&o)[Sh::HELD]) {
-    float Gn = G * g;
+    float Gn = fmaf(G, gm1, G);
     if (Gn < 1e-6f) {
 #pragma unroll
       for (int i = 0; i < Sh::KT / 2; ++i)
@@ -232,10 +235,10 @@ template <int KIND, typename F> int scan_dispatch(int K, F&& f) {
 }
 constexpr int kScanMaxK = 256;
 
-// 32-bit forms of the gates that enter the recurrences.
-__device__ __forceinline__ float channel_decay(float z, float inv_tau) { return expf(-softplus_f(-z) * inv_tau); }
-__device__ __forceinline__ float head_decay(float a, float A_log, float dt_bias) { return expf(-expf(A_log) * softplus_f(a + dt_bias)); }
-constexpr float kUnitEps = 1e-6f;
+// Logarithms of the decays, in 32-bit.
+__device__ __forceinline__ float channel_log_decay(float z, float inv_tau) { return -softplus_f(-z) * inv_tau; }
+__device__ __forceinline__ float head_log_decay(float a, float A_log, float dt_bias) { return -expf(A_log) * softplus_f(a + dt_bias); }
+constexpr float kUnitEps = 1e-6f;       // of q and k scaled to unit length
 
 constexpr int kScanMaxWarps = 8, kScanCols = 128;      // columns per CTA at most
 
@@ -321,7 +324,7 @@ __global__ void __launch_bounds__(32 * W, 16 / W) scan_kernel(const ScanParams<T
       } else {
         vecs[j] = kf;
         vecs[K + j] = qf * p.q_scale;
-        vecs[2 * K + j] = channel_decay(Elem<T>::to_f(rz[m]), p.inv_tau);
+        vecs[2 * K + j] = expm1f(channel_log_decay(Elem<T>::to_f(rz[m]), p.inv_tau));
       }
     }
 #pragma unroll
@@ -338,7 +341,7 @@ __global__ void __launch_bounds__(32 * W, 16 / W) scan_kernel(const ScanParams<T
       }
       if (lane == 0) {
         float* par = s_par + (buf * TT + warp) * 4;
-        par[0] = head_decay(Elem<T>::to_f(rb[1]), A_log, dt_bias);
+        par[0] = expm1f(head_log_decay(Elem<T>::to_f(rb[1]), A_log, dt_bias));
         par[1] = sigmoid_f(Elem<T>::to_f(rb[0]));
         par[2] = kq * ks * qs;
       }
@@ -377,30 +380,14 @@ __global__ void __launch_bounds__(32 * W, 16 / W) scan_kernel(const ScanParams<T
   if (live && work) S.store(gS, kp, p.K, p.V, pw - c0, vec);
 }
 
-template <typename Sh, typename T>
-__global__ void __launch_bounds__(256, 2) step_kernel(const ScanParams<T> p) {
-  constexpr bool kDelta = Sh::KIND == SK_DELTA;
-  constexpr int K = Sh::K;
-  extern __shared__ __align__(16) float sm[];
-  const int vpad = (p.V + Sh::CW - 1) / Sh::CW * Sh::CW;
-  float *s_k = sm, *s_q = s_k + K, *s_a = s_q + K, *s_v = s_a + (kDelta ? 0 : K), *s_o = s_v + vpad;
-  const int s = blockIdx.x, h = blockIdx.y, tid = threadIdx.x, nthr = blockDim.x;
-  const int warp = tid >> 5, lane = tid & 31, kp = lane & (Sh::KP - 1), vp = lane / Sh::KP, warps = nthr >> 5;
+// The vectors of a token for the step kernels: K (padded) values of k and q, gated linear attention's alpha - 1, V (padded)
+// values of v; the delta rule's go through the convolution.
+template <int KIND, typename T>
+__device__ __forceinline__ void step_vectors(const ScanParams<T>& p, int s, int h, int slot, int st0, int K, int vpad, float* s_k,
+                                             float* s_q, float* s_a, float* s_v) {
+  constexpr bool kDelta = KIND == SK_DELTA;
   const int kh = h / (p.heads / p.kv_heads);
-  const int slot = p.slots[s], st0 = p.start[s];
-  T* out = p.out + static_cast<int64_t>(s) * p.out_stride + static_cast<int64_t>(h) * p.V;
-  if (slot < 0 || slot >= p.num_slots || st0 < 0) {
-    for (int i = tid; i < p.V; i += nthr) out[i] = Elem<T>::from_f(0.f);
-    return;
-  }
-  const bool vec = p.V % 4 == 0;
-  float* gS = p.state + (static_cast<int64_t>(slot) * p.heads + h) * p.K * p.V;
-  ScanState<Sh> S;
-  const int c_first = warp * Sh::CW + vp * Sh::VT;
-  if (st0 > 0) S.load(gS + c_first, kp, p.K, p.V, p.V - c_first, vec);
-  else S.zero();
-  // the token's vectors
-  for (int i = tid; i < K + K + vpad; i += nthr) {
+  for (int i = threadIdx.x; i < K + K + vpad; i += blockDim.x) {
     const int part = i < K ? 0 : i < 2 * K ? 1 : 2, j = part == 0 ? i : part == 1 ? i - K : i - 2 * K;
     const bool ok = j < (part == 2 ? p.V : p.K);
     float x = 0.f;
@@ -423,35 +410,72 @@ __global__ void __launch_bounds__(256, 2) step_kernel(const ScanParams<T> p) {
     }
     (part == 0 ? s_k : part == 1 ? s_q : s_v)[j] = x;
     if (!kDelta && part == 0)
-      s_a[j] = ok ? channel_decay(Elem<T>::to_f(p.z[static_cast<int64_t>(s) * p.z_stride + h * p.K + j]), p.inv_tau) : 0.f;
+      s_a[j] = ok ? expm1f(channel_log_decay(Elem<T>::to_f(p.z[static_cast<int64_t>(s) * p.z_stride + h * p.K + j]), p.inv_tau)) : 0.f;
   }
-  float g = 0.f, beta = 0.f, ks = 1.f, qs = 1.f, kq = 0.f;
-  if (kDelta) {
-    g = head_decay(Elem<T>::to_f(p.a[static_cast<int64_t>(s) * p.gate_stride + h]), Elem<T>::to_f(p.A_log[h]), Elem<T>::to_f(p.dt_bias[h]));
-    beta = sigmoid_f(Elem<T>::to_f(p.beta[static_cast<int64_t>(s) * p.gate_stride + h]));
+}
+
+// The delta rule's scalars of a token: g - 1, beta, the factors of k and q and their scaled product.  Every warp for itself.
+struct StepFactors { float gm1, beta, ks, qs, kq; };
+template <typename T>
+__device__ __forceinline__ StepFactors step_factors(const ScanParams<T>& p, int s, int h, int K, const float* s_k, const float* s_q) {
+  StepFactors f;
+  const int64_t at = static_cast<int64_t>(s) * p.gate_stride + h;
+  f.gm1 = expm1f(head_log_decay(Elem<T>::to_f(p.a[at]), Elem<T>::to_f(p.A_log[h]), Elem<T>::to_f(p.dt_bias[h])));
+  f.beta = sigmoid_f(Elem<T>::to_f(p.beta[at]));
+  float kk = 0.f, qq = 0.f, kq = 0.f;
+  for (int j = threadIdx.x & 31; j < K; j += 32) {
+    const float a = s_k[j], b = s_q[j];
+    kk = fmaf(a, a, kk);
+    qq = fmaf(b, b, qq);
+    kq = fmaf(a, b, kq);
   }
+  f.ks = 1.f / sqrtf(warp_sum(kk) + kUnitEps);
+  f.qs = p.q_scale / sqrtf(warp_sum(qq) + kUnitEps);
+  f.kq = warp_sum(kq) * f.ks * f.qs;
+  return f;
+}
+
+// Norm of the head's read-out and output gate.
+template <typename T>
+__device__ __forceinline__ void step_output(const ScanParams<T>& p, int s, int h, const float* s_o, T* out) {
+  float acc = 0.f;
+  for (int j = threadIdx.x & 31; j < p.V; j += 32) acc = fmaf(s_o[j], s_o[j], acc);
+  const float rs = 1.f / sqrtf(warp_sum(acc) / static_cast<float>(p.V) + p.eps);
+  const T* gate = p.gate + static_cast<int64_t>(s) * p.out_gate_stride + static_cast<int64_t>(h) * p.V;
+  for (int j = threadIdx.x; j < p.V; j += blockDim.x)
+    out[j] = Elem<T>::from_f(s_o[j] * rs * Elem<T>::to_f(p.norm_w[j]) * silu_t<T>(Elem<T>::to_f(gate[j])));
+}
+
+// Any sizes: the state in the prompt kernel's layout.
+template <typename Sh, typename T>
+__global__ void __launch_bounds__(256, 1) step_kernel(const ScanParams<T> p) {
+  constexpr bool kDelta = Sh::KIND == SK_DELTA;
+  constexpr int K = Sh::K;
+  extern __shared__ __align__(16) float sm[];
+  const int vpad = (p.V + Sh::CW - 1) / Sh::CW * Sh::CW;
+  float *s_k = sm, *s_q = s_k + K, *s_a = s_q + K, *s_v = s_a + (kDelta ? 0 : K), *s_o = s_v + vpad;
+  const int s = blockIdx.x, h = blockIdx.y, tid = threadIdx.x;
+  const int warp = tid >> 5, lane = tid & 31, kp = lane & (Sh::KP - 1), vp = lane / Sh::KP, warps = blockDim.x >> 5;
+  const int slot = p.slots[s], st0 = p.start[s];
+  T* out = p.out + static_cast<int64_t>(s) * p.out_stride + static_cast<int64_t>(h) * p.V;
+  if (slot < 0 || slot >= p.num_slots || st0 < 0) {
+    for (int i = tid; i < p.V; i += blockDim.x) out[i] = Elem<T>::from_f(0.f);
+    return;
+  }
+  const bool vec = p.V % 4 == 0;
+  float* gS = p.state + (static_cast<int64_t>(slot) * p.heads + h) * p.K * p.V;
+  step_vectors<Sh::KIND>(p, s, h, slot, st0, K, vpad, s_k, s_q, s_a, s_v);
   __syncthreads();
-  if (kDelta) {        // unit norms, every warp for itself
-    float kk = 0.f, qq = 0.f;
-    for (int j = lane; j < K; j += 32) {
-      const float a = s_k[j], b = s_q[j];
-      kk = fmaf(a, a, kk);
-      qq = fmaf(b, b, qq);
-      kq = fmaf(a, b, kq);
-    }
-    ks = 1.f / sqrtf(warp_sum(kk) + kUnitEps);
-    qs = p.q_scale / sqrtf(warp_sum(qq) + kUnitEps);
-    kq = warp_sum(kq) * ks * qs;
-  }
+  StepFactors f{};
+  if (kDelta) f = step_factors(p, s, h, K, s_k, s_q);
   const bool writes = (!kDelta || (kp & (Sh::KP / 2))) && (kp & (Sh::LOW - 1)) == 0;
+  ScanState<Sh> S;
   for (int cb = warp; cb * Sh::CW < p.V; cb += warps) {
     const int c0 = cb * Sh::CW + vp * Sh::VT;
-    if (cb != warp) {
-      if (st0 > 0) S.load(gS + c0, kp, p.K, p.V, p.V - c0, vec);
-      else S.zero();
-    }
+    if (st0 > 0) S.load(gS + c0, kp, p.K, p.V, p.V - c0, vec);
+    else S.zero();
     float o[Sh::HELD];
-    if constexpr (kDelta) S.delta(s_k, s_q, s_v + c0, g, beta, ks, qs, kq, kp, o);
+    if constexpr (kDelta) S.delta(s_k, s_q, s_v + c0, f.gm1, f.beta, f.ks, f.qs, f.kq, kp, o);
     else S.gla(s_k, s_q, s_a, s_v + c0, kp, o);
     if (writes)
 #pragma unroll
@@ -459,12 +483,123 @@ __global__ void __launch_bounds__(256, 2) step_kernel(const ScanParams<T> p) {
     S.store(gS + c0, kp, p.K, p.V, p.V - c0, vec);
   }
   __syncthreads();
-  float acc = 0.f;
-  for (int j = lane; j < p.V; j += 32) acc = fmaf(s_o[j], s_o[j], acc);
-  const float rs = 1.f / sqrtf(warp_sum(acc) / static_cast<float>(p.V) + p.eps);
-  const T* gate = p.gate + static_cast<int64_t>(s) * p.out_gate_stride + static_cast<int64_t>(h) * p.V;
-  for (int j = tid; j < p.V; j += nthr)
-    out[j] = Elem<T>::from_f(s_o[j] * rs * Elem<T>::to_f(p.norm_w[j]) * silu_t<T>(Elem<T>::to_f(gate[j])));
+  step_output(p, s, h, s_o, out);
+}
+
+// vdim a multiple of four: a thread has four columns of every rows-th row of S, so that a warp reads whole lines, and the
+// first kStHold of its rows in registers, requested before anything else.  The delta rule passes over S twice (read-outs,
+// update); rows that are not held are read again, from L2.
+constexpr int kStHold = 8, kStThreads4 = 512;
+template <int KIND, typename T>
+__global__ void __launch_bounds__(kStThreads4, 2) step_quad_kernel(const ScanParams<T> p, int vpad) {
+  constexpr bool kDelta = KIND == SK_DELTA;
+  extern __shared__ __align__(16) float sm[];
+  const int K = (p.K + 3) & ~3, nthr = blockDim.x, tid = threadIdx.x, s = blockIdx.x, h = blockIdx.y;
+  const int PQ = p.V / 4, rows = nthr / PQ, q = tid % PQ, r = tid / PQ;
+  const bool on = r < rows;
+  float *s_k = sm, *s_q = s_k + K, *s_a = s_q + K, *s_v = s_a + (kDelta ? 0 : K), *s_o = s_v + vpad;
+  float4* red = reinterpret_cast<float4*>(s_o + vpad);           // [rows][PQ], twice for the delta rule
+  const int slot = p.slots[s], st0 = p.start[s];
+  T* out = p.out + static_cast<int64_t>(s) * p.out_stride + static_cast<int64_t>(h) * p.V;
+  if (slot < 0 || slot >= p.num_slots || st0 < 0) {
+    for (int i = tid; i < p.V; i += nthr) out[i] = Elem<T>::from_f(0.f);
+    return;
+  }
+  float4* gS = reinterpret_cast<float4*>(p.state + (static_cast<int64_t>(slot) * p.heads + h) * p.K * p.V) + q;
+  const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
+  float4 x[kStHold];
+  auto fetch = [&](int n0) {
+#pragma unroll
+    for (int i = 0; i < kStHold; ++i) {
+      const int n = n0 + i * rows + r;
+      x[i] = on && n < p.K && st0 > 0 ? gS[n * PQ] : zero;
+    }
+  };
+  fetch(0);                              // in flight while the vectors are made
+  step_vectors<KIND>(p, s, h, slot, st0, K, vpad, s_k, s_q, s_a, s_v);
+  __syncthreads();
+  const float4 v = on ? *reinterpret_cast<const float4*>(s_v + q * 4) : zero;
+  float4 aq = zero, ak = zero;
+  auto add = [](float w, const float4& y, float4& acc) {
+    acc.x = fmaf(w, y.x, acc.x); acc.y = fmaf(w, y.y, acc.y); acc.z = fmaf(w, y.z, acc.z); acc.w = fmaf(w, y.w, acc.w);
+  };
+  const int span = kStHold * rows;
+  if constexpr (!kDelta) {
+    for (int n0 = 0; n0 < p.K; n0 += span) {
+      if (n0) fetch(n0);
+#pragma unroll
+      for (int i = 0; i < kStHold; ++i) {
+        const int n = n0 + i * rows + r;
+        if (on && n < p.K) {
+          const float a = s_a[n], k = s_k[n];
+          const float4 old = x[i];
+          add(a, old, x[i]);
+          add(k, v, x[i]);
+          gS[n * PQ] = x[i];
+          add(s_q[n], x[i], aq);
+        }
+      }
+    }
+    if (on) red[r * PQ + q] = aq;
+    __syncthreads();
+    for (int i = tid; i < p.V; i += nthr) {
+      float o = 0.f;
+      for (int k = 0; k < rows; ++k) o += reinterpret_cast<const float*>(red)[k * p.V + i];
+      s_o[i] = o;
+    }
+  } else {
+    const StepFactors f = step_factors(p, s, h, K, s_k, s_q);
+    for (int n0 = 0; n0 < p.K; n0 += span) {
+      if (n0 == 0) {
+#pragma unroll
+        for (int i = 0; i < kStHold; ++i) {
+          const int n = i * rows + r;
+          if (on && n < p.K) { add(s_k[n], x[i], ak); add(s_q[n], x[i], aq); }
+        }
+      } else {
+#pragma unroll
+        for (int i = 0; i < kStHold; ++i) {
+          const int n = n0 + i * rows + r;
+          if (on && n < p.K && st0 > 0) {
+            const float4 y = gS[n * PQ];
+            add(s_k[n], y, ak);
+            add(s_q[n], y, aq);
+          }
+        }
+      }
+    }
+    if (on) { red[r * PQ + q] = ak; red[(rows + r) * PQ + q] = aq; }
+    __syncthreads();
+    float4 u = zero;
+    if (on) {
+      float4 dk = zero;
+      for (int k = 0; k < rows; ++k) add(1.f, red[k * PQ + q], dk);
+      const float gk = (1.f + f.gm1) * f.ks;
+      u = make_float4(f.beta * fmaf(-gk, dk.x, v.x), f.beta * fmaf(-gk, dk.y, v.y), f.beta * fmaf(-gk, dk.z, v.z), f.beta * fmaf(-gk, dk.w, v.w));
+      if (r == 0) {
+        float4 dq = zero;
+        for (int k = 0; k < rows; ++k) add(1.f, red[(rows + k) * PQ + q], dq);
+        const float gq = (1.f + f.gm1) * f.qs;
+        *reinterpret_cast<float4*>(s_o + q * 4) = make_float4(fmaf(gq, dq.x, u.x * f.kq), fmaf(gq, dq.y, u.y * f.kq),
+                                                              fmaf(gq, dq.z, u.z * f.kq), fmaf(gq, dq.w, u.w * f.kq));
+      }
+    }
+    for (int n0 = 0; n0 < p.K; n0 += span) {
+      if (n0) fetch(n0);
+#pragma unroll
+      for (int i = 0; i < kStHold; ++i) {
+        const int n = n0 + i * rows + r;
+        if (on && n < p.K) {
+          const float4 old = x[i];
+          add(f.gm1, old, x[i]);
+          add(f.ks * s_k[n], u, x[i]);
+          gS[n * PQ] = x[i];
+        }
+      }
+    }
+  }
+  __syncthreads();
+  step_output(p, s, h, s_o, out);
 }
 
 template <typename Sh, typename T, int W>
@@ -489,6 +624,16 @@ template <int KIND, typename T> static int run_scan(const ScanParams<T>& p, int 
 }
 
 template <int KIND, typename T> static int run_step(const ScanParams<T>& p, int num_seqs, cudaStream_t st) {
+  if (p.V % 4 == 0 && p.V <= 4 * kStThreads4) {
+    const int quads = p.V / 4, K = (p.K + 3) & ~3;
+    const int threads = std::min(kStThreads4, std::max(128, (quads * ((p.K + kStHold - 1) / kStHold) + 31) / 32 * 32));
+    const int fit = std::max(threads, (quads + 31) / 32 * 32), rows = fit / quads;
+    const size_t smem = sizeof(float) * ((KIND == SK_DELTA ? 2 : 3) * K + 2 * p.V + (KIND == SK_DELTA ? 2 : 1) * static_cast<size_t>(rows) * p.V);
+    if (smem <= 48 * 1024) {
+      step_quad_kernel<KIND, T><<<dim3(num_seqs, p.heads), fit, smem, st>>>(p, p.V);
+      return check_launch("state_step");
+    }
+  }
   return scan_dispatch<KIND>(p.K, [&](auto sh) {
     using Sh = decltype(sh);
     const int blocks = (p.V + Sh::CW - 1) / Sh::CW, warps = std::min(8, blocks);

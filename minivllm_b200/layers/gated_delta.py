@@ -1,5 +1,6 @@
 """Gated delta rule: short convolutions on q, k and v, unit-length q and k per head, a scalar decay and a step size per
-head, the recurrence on a matrix state in 32-bit, a norm per head and an output gate (csrc/gated_delta.cu).
+head, the recurrence on a matrix state in 32-bit, a norm per head and an output gate (csrc/gated_delta.cu; portions of
+prompts in chunks on tensor cores, csrc/gated_delta_chunk.cu).
 """
 import torch
 import torch.nn as nn
@@ -7,23 +8,36 @@ import torch.nn.functional as F
 
 from .. import _cabi
 from ..utils.context import get_context
+from .gla import CHUNK_FROM
 from .group_norm import head_norm_gate
 from .linear import StackedLinear
 from .short_conv import conv_silu, conv_state_update
 
 
 def delta_scan(qkv, beta, a, A_log, dt_bias, cu, slots, starts, state, heads, kv_heads, dim, vdim, conv_w=None,
-               conv_state=None, gate=None, norm_w=None, eps=0.0, out=None):
+               conv_state=None, gate=None, norm_w=None, eps=0.0, out=None, chunked=None):
     """qkv (tokens, 2 * kv_heads * dim + heads * vdim), beta and a (tokens, heads) with one row stride.  Advances `state`
     (slots, heads, dim, vdim) fp32 and returns (tokens, heads * vdim): the read-outs of packed portions (cu; qkv after
     its convolution), or with cu None (one token per sequence) the normed and gated rows, the convolution included
-    (conv_state is only read).  See mv_delta_scan."""
+    (conv_state is only read).  See mv_delta_scan.  bf16 portions take the chunked kernels when those have the sizes."""
     _cabi.require_cuda(qkv, beta, a, state, gate, norm_w, conv_w, conv_state)
     if beta.stride(0) != a.stride(0):
         raise ValueError("beta and a must share a row stride")
     out = torch.empty((qkv.shape[0], heads * vdim), dtype=qkv.dtype, device=qkv.device) if out is None else out
+    L, tokens = _cabi.lib(), qkv.shape[0]
+    need = L.mv_delta_chunk_workspace_bytes(tokens, slots.numel(), heads, dim, vdim) if cu is not None else -1
+    if chunked is None:
+        chunked = need >= 0 and qkv.dtype == torch.bfloat16 and tokens >= CHUNK_FROM * slots.numel()
+    if chunked:
+        ws = torch.empty(max(need, 1), dtype=torch.uint8, device=qkv.device)
+        _cabi.check(L.mv_delta_chunk_scan(
+            out.data_ptr(), out.stride(0), qkv.data_ptr(), qkv.stride(0), beta.data_ptr(), a.data_ptr(), a.stride(0),
+            A_log.data_ptr(), dt_bias.data_ptr(), cu.data_ptr(), slots.numel(), tokens, slots.data_ptr(), starts.data_ptr(),
+            state.data_ptr(), state.shape[0], heads, kv_heads, dim, vdim, dim ** -0.5, ws.data_ptr(), ws.numel(),
+            _cabi.stream_ptr()))
+        return out
     ptr = lambda t: t.data_ptr() if t is not None else None
-    _cabi.check(_cabi.lib().mv_delta_scan(
+    _cabi.check(L.mv_delta_scan(
         out.data_ptr(), out.stride(0), qkv.data_ptr(), qkv.stride(0), beta.data_ptr(), a.data_ptr(), a.stride(0),
         A_log.data_ptr(), dt_bias.data_ptr(), ptr(cu), slots.numel(), slots.data_ptr(), starts.data_ptr(),
         state.data_ptr(), state.shape[0], heads, kv_heads, dim, vdim, dim ** -0.5, ptr(conv_w),

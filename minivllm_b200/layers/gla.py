@@ -1,5 +1,5 @@
 """Gated linear attention: a decay per key channel from a low-rank projection, the recurrence on a matrix state in
-32-bit, a norm per head and an output gate (csrc/gla.cu).
+32-bit, a norm per head and an output gate (csrc/gla.cu; portions of prompts in chunks on tensor cores, csrc/gla_chunk.cu).
 """
 import torch
 import torch.nn as nn
@@ -10,18 +10,32 @@ from ..utils.context import get_context
 from .group_norm import head_norm_gate
 from .linear import StackedLinear
 
+CHUNK_FROM = 16          # mean tokens per portion from which the chunked kernels are used
 DEFAULT_RANK = 16        # of seeded weights; a checkpoint's tensors have their own
 
 
-def gla_scan(q, k, v, z, tau, cu, slots, starts, state, heads, dim, vdim, gate=None, norm_w=None, eps=0.0, out=None):
+def gla_scan(q, k, v, z, tau, cu, slots, starts, state, heads, dim, vdim, gate=None, norm_w=None, eps=0.0, out=None,
+             chunked=None):
     """q, k, v, gate: views of one row-major product; z (tokens, heads * dim).  Advances `state` (slots, heads, dim,
     vdim) fp32 and returns (tokens, heads * vdim): the read-outs of packed portions (cu), or with cu None (one token per
-    sequence) the normed and gated rows.  See mv_gla_scan."""
+    sequence) the normed and gated rows.  See mv_gla_scan.  bf16 portions take the chunked kernels when those have the
+    sizes."""
     _cabi.require_cuda(q, k, v, z, state, gate, norm_w)
     if not q.stride(0) == k.stride(0) == v.stride(0):
         raise ValueError("q, k and v must share a row stride")
     out = torch.empty((q.shape[0], heads * vdim), dtype=q.dtype, device=q.device) if out is None else out
-    _cabi.check(_cabi.lib().mv_gla_scan(
+    L, tokens = _cabi.lib(), q.shape[0]
+    need = L.mv_gla_chunk_workspace_bytes(tokens, slots.numel(), heads, dim, vdim) if cu is not None else -1
+    if chunked is None:
+        chunked = need >= 0 and q.dtype == torch.bfloat16 and tokens >= CHUNK_FROM * slots.numel()
+    if chunked:
+        ws = torch.empty(max(need, 1), dtype=torch.uint8, device=q.device)
+        _cabi.check(L.mv_gla_chunk_scan(
+            out.data_ptr(), out.stride(0), q.data_ptr(), k.data_ptr(), v.data_ptr(), q.stride(0), z.data_ptr(), z.stride(0),
+            tau, cu.data_ptr(), slots.numel(), tokens, slots.data_ptr(), starts.data_ptr(), state.data_ptr(), state.shape[0],
+            heads, dim, vdim, dim ** -0.5, ws.data_ptr(), ws.numel(), _cabi.stream_ptr()))
+        return out
+    _cabi.check(L.mv_gla_scan(
         out.data_ptr(), out.stride(0), q.data_ptr(), k.data_ptr(), v.data_ptr(), q.stride(0), z.data_ptr(), z.stride(0),
         tau, cu.data_ptr() if cu is not None else None, slots.numel(), slots.data_ptr(), starts.data_ptr(),
         state.data_ptr(), state.shape[0], heads, dim, vdim, dim ** -0.5, gate.data_ptr() if gate is not None else None,

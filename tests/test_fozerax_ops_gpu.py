@@ -301,7 +301,7 @@ def _run_portions(fn, lens, cuts):
 
 
 SCAN_SIZES = [(2, 14, 10), (1, 37, 41), (3, 64, 64), (2, 128, 128), (1, 96, 36), (2, 32, 200), (1, 130, 20), (1, 256, 64), (4, 8, 8), (1, 1, 3),
-              (2, 48, 132), (1, 200, 300)]
+              (2, 48, 132), (1, 200, 300), (2, 96, 40), (1, 128, 256), (2, 16, 136)]
 
 
 @pytest.mark.parametrize("dtype", DTYPES, ids=IDS)
@@ -339,7 +339,7 @@ def test_gla_scan(heads, K, V, dtype):
 
         _run_portions(step, lens, cuts)
         for s in range(len(lens)):
-            _close(state[slots[s]], ref[s][1], 3e-6, "state")
+            _close(state[slots[s]], ref[s][1], 3e-6 if dtype == torch.float32 else 1e-4, "state")
         assert bool(state[[1, 3, 5]].isnan().all())
 
 
@@ -391,6 +391,50 @@ def test_delta_scan(heads, K, V, dtype):
         for s in range(len(lens)):
             _close(state[slots[s]], ref[s][1], 5e-6 if dtype == torch.float32 else 1.2e-2, "state")
         assert bool(state[[1, 3, 5]].isnan().all())
+
+
+@pytest.mark.parametrize("K,V", [(64, 64), (128, 128), (32, 24), (96, 72), (128, 256), (8, 200)])
+def test_chunked_scans(K, V):
+    """The chunked kernels against the oracle: lengths around the chunk size, cuts inside chunks, one sequence and several,
+    channels that forget at once; nothing of the state is rounded to 16 bits."""
+    from minivllm_b200.layers import gated_delta as D
+    from minivllm_b200.layers import gla as L
+    bf, d = torch.bfloat16, lambda t: t.double()
+    H, kv, tau = 2, 1, 2.0
+    for lens in ([1, 63, 64, 65, 130, 2], [200]):
+        z = [(_rnd(5 + s, n, H, K, scale=3.0) + 3.0).to(bf) for s, n in enumerate(lens)]
+        for x in z:
+            x[:, :, 0] = -70.0                   # alpha of 2^-50
+            x[:, :, 1::5] = 12.0                 # alpha close to one
+        g = [torch.cat([_rnd(20 + s, n, 2 * H * K), _rnd(40 + s, n, H * V)], 1).to(bf) for s, n in enumerate(lens)]
+        u = [torch.cat([_rnd(60 + s, n, 2 * kv * K), _rnd(80 + s, n, H * V)], 1).to(bf) for s, n in enumerate(lens)]
+        ba = [torch.cat([_rnd(100 + s, n, H, scale=2.0), _rnd(120 + s, n, H)], 1).to(bf) for s, n in enumerate(lens)]
+        A_log, dt_bias = torch.tensor([-3.0, 3.0]).to(bf), torch.tensor([-1.0, 0.5]).to(bf)
+        ref_g, ref_d = [], []
+        for s, n in enumerate(lens):
+            q, k, v = d(g[s]).split([H * K, H * K, H * V], 1)
+            ref_g.append(oracle.gla_scan(q.view(n, H, K) * K ** -0.5, k.view(n, H, K), v.view(n, H, V), oracle.channel_decay(d(z[s]), tau)))
+            q, k, v = d(u[s]).split([kv * K, kv * K, H * V], 1)
+            spread = lambda t: t.view(n, kv, K).repeat_interleave(H // kv, 1)
+            ref_d.append(oracle.delta_scan(oracle.unit(spread(q)) * K ** -0.5, oracle.unit(spread(k)), v.view(n, H, V),
+                                           oracle.sigmoid(d(ba[s][:, :H])), oracle.head_decay(d(ba[s][:, H:]), d(A_log), d(dt_bias))))
+        for cuts in ([400], [70, 3, 64, 1], [37]):
+            Sg, Sd = (torch.full((len(lens), H, K, V), float("nan"), device="cuda") for _ in range(2))
+
+            def step(spans):
+                cat = lambda x: torch.cat([x[s][a:b] for s, a, b in spans]).cuda()
+                sl, st, cu = _i32([s for s, _, _ in spans]), _i32([a for _, a, _ in spans]), _cu([b - a for _, a, b in spans])
+                q, k, v = cat(g).split([H * K, H * K, H * V], 1)
+                got = L.gla_scan(q, k, v, cat([x.flatten(1) for x in z]), tau, cu, sl, st, Sg, H, K, V, chunked=True)
+                _close(got, torch.cat([ref_g[s][0][a:b].flatten(1) for s, a, b in spans]), 6e-3, f"gla, {lens}, {spans}")
+                b = cat(ba)
+                got = D.delta_scan(cat(u), b[:, :H], b[:, H:], A_log.cuda(), dt_bias.cuda(), cu, sl, st, Sd, H, kv, K, V, chunked=True)
+                _close(got, torch.cat([ref_d[s][0][a:b].flatten(1) for s, a, b in spans]), 6e-3, f"delta, {lens}, {spans}")
+
+            _run_portions(step, lens, cuts)
+            for s in range(len(lens)):
+                _close(Sg[s], ref_g[s][1], 5e-5, "gla, state")
+                _close(Sd[s], ref_d[s][1], 5e-5, "delta, state")
 
 
 def test_padding_rows_leave_the_state_alone():
