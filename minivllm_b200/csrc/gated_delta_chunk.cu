@@ -257,7 +257,7 @@ __global__ void __launch_bounds__(256, 1) delta_chunk_kernel(const DeltaChunkPar
   issue(0);
   const bool work = warp * 16 < pw;
   ChunkState<K> S;
-  S.load(gS, p0 + warp * 16, work ? min(p.V, p0 + pw) : 0, p.K, lane, live && st0 > 0);
+  S.load(gS, p0 + warp * 16, p0 + pw, p.V, p.K, lane, work && live && st0 > 0);
   const LaneAt at(lane);
   for (int c = 0; c < chunks; ++c) {
     cp_async_wait<0>();
@@ -351,7 +351,7 @@ __global__ void __launch_bounds__(256, 1) delta_chunk_kernel(const DeltaChunkPar
               p.out + row0 * p.out_stride + static_cast<int64_t>(h) * p.V + p0 + warp * 16, p.out_stride,
               min(kChunk, n_tok - c * kChunk), pw - warp * 16, lane);
   }
-  if (live && work) S.store(gS, p0 + warp * 16, min(p.V, p0 + pw), p.K, lane);
+  if (live && work) S.store(gS, p0 + warp * 16, p0 + pw, p.V, p.K, lane);
 }
 
 }  // namespace mv

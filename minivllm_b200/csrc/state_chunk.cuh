@@ -66,24 +66,25 @@ struct LaneAt {
 // The 16 columns of a warp: tile n holds channels 8 n .. 8 n + 7 (accumulator columns), rows are value columns.
 template <int K> struct ChunkState {
   float s[K / 8][4];
-  __device__ __forceinline__ void load(const float* gS, int v0, int V, int K_real, int lane, bool on) {
+  // gS: the head's (K, V) state; columns v0 .. v0 + 15 below v_end
+  __device__ __forceinline__ void load(const float* gS, int v0, int v_end, int V, int K_real, int lane, bool on) {
     const int g = lane >> 2, c2 = (lane & 3) * 2;
 #pragma unroll
     for (int n = 0; n < K / 8; ++n)
 #pragma unroll
       for (int e = 0; e < 4; ++e) {
         const int ch = n * 8 + c2 + (e & 1), v = v0 + g + (e >> 1) * 8;
-        s[n][e] = on && ch < K_real && v < V ? gS[static_cast<int64_t>(ch) * V + v] : 0.f;
+        s[n][e] = on && ch < K_real && v < v_end ? gS[static_cast<int64_t>(ch) * V + v] : 0.f;
       }
   }
-  __device__ __forceinline__ void store(float* gS, int v0, int V, int K_real, int lane) const {
+  __device__ __forceinline__ void store(float* gS, int v0, int v_end, int V, int K_real, int lane) const {
     const int g = lane >> 2, c2 = (lane & 3) * 2;
 #pragma unroll
     for (int n = 0; n < K / 8; ++n)
 #pragma unroll
       for (int e = 0; e < 4; ++e) {
         const int ch = n * 8 + c2 + (e & 1), v = v0 + g + (e >> 1) * 8;
-        if (ch < K_real && v < V) gS[static_cast<int64_t>(ch) * V + v] = s[n][e];
+        if (ch < K_real && v < v_end) gS[static_cast<int64_t>(ch) * V + v] = s[n][e];
       }
   }
 };
