@@ -34,15 +34,16 @@ __device__ __forceinline__ unsigned char* delta_scratch(const DeltaChunkParams& 
 
 template <int K> struct DeltaPrepShape {
   static constexpr int kRow = K + 8, kA = 68, kT = 65;
-  static constexpr int kBytes = 2 * kChunk * kRow * 2 + kChunk * (kA + kT) * 4;
+  static constexpr int kTiles = 2 * kChunk * kRow * 2, kMats = kChunk * (kA + kT) * 4;
+  static constexpr int kBytes = kTiles > kMats ? kTiles : kMats;      // the matrices lie over the tiles of K and Q
 };
 
 template <int K>
-__global__ void __launch_bounds__(kDpThreads) delta_prepare_kernel(const DeltaChunkParams p) {
+__global__ void __launch_bounds__(kDpThreads, 4) delta_prepare_kernel(const DeltaChunkParams p) {
   using Sh = DeltaPrepShape<K>;
   extern __shared__ __align__(16) unsigned char smem[];
   __nv_bfloat16 *sK = reinterpret_cast<__nv_bfloat16*>(smem), *sQ = sK + kChunk * Sh::kRow;
-  float *sA = reinterpret_cast<float*>(sQ + kChunk * Sh::kRow), *sT = sA + kChunk * Sh::kA;      // A by column, T by row
+  float *sA = reinterpret_cast<float*>(smem), *sT = sA + kChunk * Sh::kA;      // A by column, T by row
   __shared__ float s_ks[kChunk], s_qs[kChunk], s_c[kChunk], s_b[kChunk];
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, kh = blockIdx.y;
   int seq, chunk;
@@ -213,11 +214,11 @@ template <int K> struct DeltaChunkShape {
 };
 
 template <int K>
-__global__ void __launch_bounds__(256, 1) delta_chunk_kernel(const DeltaChunkParams p, int pb) {
+__global__ void __launch_bounds__(kChunkThreads, 1) delta_chunk_kernel(const DeltaChunkParams p, int pb) {
   using Sh = DeltaChunkShape<K>;
   extern __shared__ __align__(16) unsigned char smem[];
   const int s = blockIdx.x, h = blockIdx.y, p0 = blockIdx.z * pb, pw = min(pb, p.V - p0);
-  const int tid = threadIdx.x, threads = blockDim.x, warp = tid >> 5, lane = tid & 31, c2 = (lane & 3) * 2;
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, c2 = (lane & 3) * 2;
   const int kh = h / (p.heads / p.kv_heads), vrow = pb + 8;
   const int first = p.cu[s], n_tok = p.cu[s + 1] - first;
   if (n_tok <= 0) return;
@@ -234,7 +235,7 @@ __global__ void __launch_bounds__(256, 1) delta_chunk_kernel(const DeltaChunkPar
     const uint32_t st = base + (c & 1) * stage_bytes;
     const int64_t row0 = static_cast<int64_t>(first) + c * kChunk;
     const int nt = min(kChunk, n_tok - c * kChunk);
-    for (int i = tid; i < kChunk * (K / 8); i += threads) {
+    for (int i = tid; i < kChunk * (K / 8); i += kChunkThreads) {
       const int r = i / (K / 8), cc = (i % (K / 8)) * 8;
       const bool ok = r < nt && cc < p.K;
       const int64_t off = ok ? (row0 + r) * p.stride + cc : 0;
@@ -242,16 +243,16 @@ __global__ void __launch_bounds__(256, 1) delta_chunk_kernel(const DeltaChunkPar
       cp_async16(st + Sh::kK + (r * Sh::kRow + cc) * 2, q + off, ok ? 16 : 0);
     }
     const uint32_t vd = st + 2 * Sh::kK;
-    for (int i = tid; i < kChunk * (pb / 8); i += threads) {
+    for (int i = tid; i < kChunk * (pb / 8); i += kChunkThreads) {
       const int r = i / (pb / 8), cc = (i % (pb / 8)) * 8;
       const bool ok = r < nt && cc < pw;
       cp_async16(vd + (r * vrow + cc) * 2, ok ? v + (row0 + r) * p.stride + cc : v, ok ? 16 : 0);
     }
     const unsigned char* src = delta_scratch(p, chunk0 + c, h);
     const uint32_t td = vd + kChunk * vrow * 2;
-    load_lower(td, reinterpret_cast<const __nv_bfloat16*>(src), tid, threads);
-    load_lower(td + Sh::kTile, reinterpret_cast<const __nv_bfloat16*>(src) + kDcTile, tid, threads);
-    for (int i = tid; i < kDcPar / 4; i += threads) cp_async16(td + 2 * Sh::kTile + i * 16, src + 2 * kDcTile * 2 + i * 16, 16);
+    load_lower(td, reinterpret_cast<const __nv_bfloat16*>(src), tid, kChunkThreads);
+    load_lower(td + Sh::kTile, reinterpret_cast<const __nv_bfloat16*>(src) + kDcTile, tid, kChunkThreads);
+    for (int i = tid; i < kDcPar / 4; i += kChunkThreads) cp_async16(td + 2 * Sh::kTile + i * 16, src + 2 * kDcTile * 2 + i * 16, 16);
     cp_async_commit();
   };
   issue(0);
@@ -276,17 +277,17 @@ __global__ void __launch_bounds__(256, 1) delta_chunk_kernel(const DeltaChunkPar
       const uint32_t ka = st + (at.row_b * Sh::kRow + kb * 16 + at.col_b) * 2;
 #pragma unroll
       for (int np = 0; np < 4; ++np) {
-        uint32_t b[4];
+        uint32_t b[4], d[4];
         ldmatrix_x4(b, ka + np * 16 * Sh::kRow * 2);
+        ldmatrix_x4(d, ka + Sh::kK + np * 16 * Sh::kRow * 2);
         Mma::run(P[2 * np], hi, b[0], b[1]);
         Mma::run(P[2 * np + 1], hi, b[2], b[3]);
+        Mma::run(O[2 * np], hi, d[0], d[1]);
+        Mma::run(O[2 * np + 1], hi, d[2], d[3]);
         Mma::run(P[2 * np], lo, b[0], b[1]);
         Mma::run(P[2 * np + 1], lo, b[2], b[3]);
-        ldmatrix_x4(b, ka + Sh::kK + np * 16 * Sh::kRow * 2);
-        Mma::run(O[2 * np], hi, b[0], b[1]);
-        Mma::run(O[2 * np + 1], hi, b[2], b[3]);
-        Mma::run(O[2 * np], lo, b[0], b[1]);
-        Mma::run(O[2 * np + 1], lo, b[2], b[3]);
+        Mma::run(O[2 * np], lo, d[0], d[1]);
+        Mma::run(O[2 * np + 1], lo, d[2], d[3]);
       }
     }
 #pragma unroll
@@ -337,13 +338,18 @@ __global__ void __launch_bounds__(256, 1) delta_chunk_kernel(const DeltaChunkPar
       split_a(U[2 * ib], U[2 * ib + 1], hi, lo);
       const uint32_t ka = st + ((ib * 16 + at.row_t) * Sh::kRow + at.col_t) * 2;
 #pragma unroll
-      for (int np = 0; np < K / 16; ++np) {
-        uint32_t b[4];
+      for (int np = 0; np < K / 16; np += 2) {
+        uint32_t b[4], d[4];
         ldmatrix_x4_trans(b, ka + np * 32);
+        ldmatrix_x4_trans(d, ka + np * 32 + 32);
         Mma::run(S.s[2 * np], hi, b[0], b[1]);
         Mma::run(S.s[2 * np + 1], hi, b[2], b[3]);
+        Mma::run(S.s[2 * np + 2], hi, d[0], d[1]);
+        Mma::run(S.s[2 * np + 3], hi, d[2], d[3]);
         Mma::run(S.s[2 * np], lo, b[0], b[1]);
         Mma::run(S.s[2 * np + 1], lo, b[2], b[3]);
+        Mma::run(S.s[2 * np + 2], lo, d[0], d[1]);
+        Mma::run(S.s[2 * np + 3], lo, d[2], d[3]);
       }
     }
     const int64_t row0 = static_cast<int64_t>(first) + c * kChunk;
@@ -392,7 +398,7 @@ extern "C" int mv_delta_chunk_scan(void* out, int64_t out_stride, const void* qk
     const int pb = chunk_columns(static_cast<int64_t>(num_seqs) * heads, vdim), smem = 2 * DeltaChunkShape<K>::stage(pb);
     e = cudaFuncSetAttribute(delta_chunk_kernel<K>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
     if (e != cudaSuccess) return fail(MV_ERR_CUDA, "delta_chunk_scan: %s", cudaGetErrorString(e));
-    delta_chunk_kernel<K><<<dim3(num_seqs, heads, (vdim + pb - 1) / pb), pb * 2, smem, st>>>(p, pb);
+    delta_chunk_kernel<K><<<dim3(num_seqs, heads, (vdim + pb - 1) / pb), kChunkThreads, smem, st>>>(p, pb);
     return check_launch("delta_chunk");
   });
 }

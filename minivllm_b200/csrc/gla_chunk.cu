@@ -1,9 +1,10 @@
 // Gated linear attention in chunks of 64 tokens.  With b_t the running sums of the channels' log2 decays inside the chunk:
 //   O = (q 2^b) S_0 + A V,      A[t, j] = sum_k q_t k_j 2^(b_t - b_j), j <= t
 //   S = 2^b_last S_0 + (k 2^(b_last - b))^T V
-// gla_prepare_kernel  per chunk and head: b, both decayed operands, A.  Every power of two is at most one: A's 16 x 16
-//                     blocks below the diagonal are products of factors taken against b at the start of the block's rows,
-//                     on tensor cores in two terms each; the blocks on the diagonal are summed channel by channel in fp32.
+// gla_prepare_kernel  per chunk and head: b, both decayed operands, A.  A's 16 x 16 blocks are products of factors taken
+//                     against b at one token, on tensor cores in two terms each.  Below the diagonal that is the last token
+//                     before the block's rows, and every power of two is at most one.  On the diagonal it is the block's
+//                     middle; a block in which some channel forgets more than 2^-60 is summed channel by channel instead.
 // gla_chunk_kernel    per sequence, head and block of value columns: see state_chunk.cuh
 // V enters as the projection left it; the decayed operands, A and S in two terms.
 #include "state_chunk.cuh"
@@ -110,10 +111,31 @@ __global__ void __launch_bounds__(kGpThreads) gla_prepare_kernel(const GlaChunkP
     gA[(t * kChunk + j) / 2] = hi;
     gA[kChunk * kChunk / 2 + (t * kChunk + j) / 2] = lo;
   };
-  if (warp < 6) {              // one block below the diagonal per warp: (1,0) (2,0) (2,1) (3,0) (3,1) (3,2)
-    const int bi = warp == 0 ? 1 : warp < 3 ? 2 : 3, bj = warp - bi * (bi - 1) / 2;
-    const int g = lane >> 2, c2 = (lane & 3) * 2;
-    const float* ref = sB + (bi * 16 - 1) * Sh::kB;
+  const int g = lane >> 2, c2 = (lane & 3) * 2;
+  // blocks 0 .. 5 below the diagonal, (1,0) (2,0) (2,1) (3,0) (3,1) (3,2), then the four on it
+#pragma unroll 1
+  for (int blk = warp; blk < 10; blk += kGpThreads / 32) {
+    const bool diag = blk >= 6;
+    const int bi = diag ? blk - 6 : blk == 0 ? 1 : blk < 3 ? 2 : 3, bj = diag ? bi : blk - bi * (bi - 1) / 2;
+    const float* ref = sB + (diag ? bi * 16 + 7 : bi * 16 - 1) * Sh::kB;
+    if (diag) {
+      float least = 0.f;
+      for (int c = lane; c < K; c += 32)
+        least = fminf(least, sB[(bi * 16 + 15) * Sh::kB + c] - (bi ? sB[(bi * 16 - 1) * Sh::kB + c] : 0.f));
+      if (__any_sync(0xffffffffu, least < -60.f)) {
+        for (int i = lane; i < 16 * 8; i += 32) {        // two neighbouring keys of one token
+          const int t = bi * 16 + (i >> 3), j = bi * 16 + (i & 7) * 2;
+          float x = 0.f, y = 0.f;
+          for (int c = 0; j <= t && c < K; ++c) {
+            const float q = __bfloat162float(sQ[t * Sh::kRow + c]), bt = sB[t * Sh::kB + c];
+            x = fmaf(q * __bfloat162float(sK[j * Sh::kRow + c]), fast_exp2(bt - sB[j * Sh::kB + c]), x);
+            if (j + 1 <= t) y = fmaf(q * __bfloat162float(sK[(j + 1) * Sh::kRow + c]), fast_exp2(bt - sB[(j + 1) * Sh::kB + c]), y);
+          }
+          put(t, j, x * p.q_scale, y * p.q_scale);
+        }
+        continue;
+      }
+    }
     float acc[2][4] = {};
 #pragma unroll 2
     for (int kb = 0; kb < K; kb += 16) {
@@ -140,31 +162,10 @@ __global__ void __launch_bounds__(kGpThreads) gla_prepare_kernel(const GlaChunkP
 #pragma unroll
     for (int n = 0; n < 2; ++n)
 #pragma unroll
-      for (int half = 0; half < 2; ++half)
-        put(bi * 16 + g + half * 8, bj * 16 + n * 8 + c2, acc[n][2 * half] * p.q_scale, acc[n][2 * half + 1] * p.q_scale);
-  }
-  // the blocks on the diagonal: a thread has two neighbouring keys of one token
-  for (int i = tid; i < 4 * 16 * 8; i += kGpThreads) {
-    const int blk = i >> 7, t = blk * 16 + ((i >> 3) & 15), j = blk * 16 + (i & 7) * 2;
-    float x = 0.f, y = 0.f;
-    if (j <= t) {
-      const bool second = j + 1 <= t;
-      for (int c = 0; c < K; c += 2) {
-        const float2 q = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(sQ + t * Sh::kRow + c));
-        const float2 bt = *reinterpret_cast<const float2*>(sB + t * Sh::kB + c);
-        const float2 k0 = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(sK + j * Sh::kRow + c));
-        const float2 b0 = *reinterpret_cast<const float2*>(sB + j * Sh::kB + c);
-        x = fmaf(q.x * k0.x, fast_exp2(bt.x - b0.x), x);
-        x = fmaf(q.y * k0.y, fast_exp2(bt.y - b0.y), x);
-        if (second) {
-          const float2 k1 = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(sK + (j + 1) * Sh::kRow + c));
-          const float2 b1 = *reinterpret_cast<const float2*>(sB + (j + 1) * Sh::kB + c);
-          y = fmaf(q.x * k1.x, fast_exp2(bt.x - b1.x), y);
-          y = fmaf(q.y * k1.y, fast_exp2(bt.y - b1.y), y);
-        }
+      for (int half = 0; half < 2; ++half) {
+        const int t = bi * 16 + g + half * 8, j = bj * 16 + n * 8 + c2;
+        put(t, j, j <= t ? acc[n][2 * half] * p.q_scale : 0.f, j + 1 <= t ? acc[n][2 * half + 1] * p.q_scale : 0.f);
       }
-    }
-    put(t, j, x * p.q_scale, y * p.q_scale);
   }
 }
 
@@ -175,12 +176,12 @@ template <int K> struct GlaChunkShape {
 };
 
 template <int K>
-__global__ void __launch_bounds__(256, 1) gla_chunk_kernel(const GlaChunkParams p, int pb) {
+__global__ void __launch_bounds__(kChunkThreads, 1) gla_chunk_kernel(const GlaChunkParams p, int pb) {
   using Sh = GlaChunkShape<K>;
   using Sc = GlaScratch<K>;
   extern __shared__ __align__(16) unsigned char smem[];
   const int s = blockIdx.x, h = blockIdx.y, p0 = blockIdx.z * pb, pw = min(pb, p.V - p0);
-  const int tid = threadIdx.x, threads = blockDim.x, warp = tid >> 5, lane = tid & 31, c2 = (lane & 3) * 2;
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, c2 = (lane & 3) * 2;
   const int vrow = pb + 8;
   const int first = p.cu[s], n_tok = p.cu[s + 1] - first;
   if (n_tok <= 0) return;
@@ -198,18 +199,18 @@ __global__ void __launch_bounds__(256, 1) gla_chunk_kernel(const GlaChunkParams 
     const int nt = min(kChunk, n_tok - c * kChunk);
     const __nv_bfloat16* src =
         reinterpret_cast<const __nv_bfloat16*>(p.scratch + (static_cast<int64_t>(chunk0 + c) * p.heads + h) * Sc::kBytes);
-    for (int i = tid; i < 4 * kChunk * (K / 8); i += threads) {
+    for (int i = tid; i < 4 * kChunk * (K / 8); i += kChunkThreads) {
       const int r = i / (K / 8), cc = (i % (K / 8)) * 8;
       cp_async16(st + (r * Sh::kRow + cc) * 2, src + r * K + cc, 16);
     }
     const uint32_t vd = st + 4 * Sh::kVec, ad = vd + kChunk * vrow * 2;
-    for (int i = tid; i < kChunk * (pb / 8); i += threads) {
+    for (int i = tid; i < kChunk * (pb / 8); i += kChunkThreads) {
       const int r = i / (pb / 8), cc = (i % (pb / 8)) * 8;
       const bool ok = r < nt && cc < pw;
       cp_async16(vd + (r * vrow + cc) * 2, ok ? v + (row0 + r) * p.stride + cc : p.v, ok ? 16 : 0);
     }
-    load_lower(ad, src + Sc::kA, tid, threads);
-    for (int i = tid; i < K / 4; i += threads) cp_async16(ad + Sh::kTile + i * 16, src + Sc::kDecay + i * 8, 16);
+    load_lower(ad, src + Sc::kA, tid, kChunkThreads);
+    for (int i = tid; i < K / 4; i += kChunkThreads) cp_async16(ad + Sh::kTile + i * 16, src + Sc::kDecay + i * 8, 16);
     cp_async_commit();
   };
   issue(0);
@@ -236,16 +237,25 @@ __global__ void __launch_bounds__(256, 1) gla_chunk_kernel(const GlaChunkParams 
       split_a(S.s[2 * kb], S.s[2 * kb + 1], hi, lo);
       const uint32_t qa = st + (at.row_b * Sh::kRow + kb * 16 + at.col_b) * 2;
 #pragma unroll
-      for (int np = 0; np < 4; ++np) {
-        uint32_t b[4];
-        ldmatrix_x4(b, qa + np * 16 * Sh::kRow * 2);
+      for (int np = 0; np < 4; np += 2) {
+        uint32_t b[4], d[4];
+        const uint32_t q0 = qa + np * 16 * Sh::kRow * 2, q1 = q0 + 16 * Sh::kRow * 2;
+        ldmatrix_x4(b, q0);
+        ldmatrix_x4(d, q1);
         Mma::run(O[2 * np], hi, b[0], b[1]);
         Mma::run(O[2 * np + 1], hi, b[2], b[3]);
+        Mma::run(O[2 * np + 2], hi, d[0], d[1]);
+        Mma::run(O[2 * np + 3], hi, d[2], d[3]);
         Mma::run(O[2 * np], lo, b[0], b[1]);
         Mma::run(O[2 * np + 1], lo, b[2], b[3]);
-        ldmatrix_x4(b, qa + Sh::kVec + np * 16 * Sh::kRow * 2);
+        Mma::run(O[2 * np + 2], lo, d[0], d[1]);
+        Mma::run(O[2 * np + 3], lo, d[2], d[3]);
+        ldmatrix_x4(b, q0 + Sh::kVec);
+        ldmatrix_x4(d, q1 + Sh::kVec);
         Mma::run(O[2 * np], hi, b[0], b[1]);
         Mma::run(O[2 * np + 1], hi, b[2], b[3]);
+        Mma::run(O[2 * np + 2], hi, d[0], d[1]);
+        Mma::run(O[2 * np + 3], hi, d[2], d[3]);
       }
     }
 #pragma unroll
@@ -256,19 +266,18 @@ __global__ void __launch_bounds__(256, 1) gla_chunk_kernel(const GlaChunkParams 
       S.s[n][0] *= d.x; S.s[n][1] *= d.y; S.s[n][2] *= d.x; S.s[n][3] *= d.y;
     }
 #pragma unroll
-    for (int ib = 0; ib < 4; ++ib) {
-      const uint32_t ka = st + 2 * Sh::kVec + ((ib * 16 + at.row_t) * Sh::kRow + at.col_t) * 2;
+    for (int term = 0; term < 2; ++term)
 #pragma unroll
-      for (int np = 0; np < K / 16; ++np) {
-        uint32_t b[4];
-        ldmatrix_x4_trans(b, ka + np * 32);
-        Mma::run(S.s[2 * np], va[ib], b[0], b[1]);
-        Mma::run(S.s[2 * np + 1], va[ib], b[2], b[3]);
-        ldmatrix_x4_trans(b, ka + Sh::kVec + np * 32);
-        Mma::run(S.s[2 * np], va[ib], b[0], b[1]);
-        Mma::run(S.s[2 * np + 1], va[ib], b[2], b[3]);
+      for (int ib = 0; ib < 4; ++ib) {
+        const uint32_t ka = st + (2 + term) * Sh::kVec + ((ib * 16 + at.row_t) * Sh::kRow + at.col_t) * 2;
+#pragma unroll
+        for (int np = 0; np < K / 16; ++np) {
+          uint32_t b[4];
+          ldmatrix_x4_trans(b, ka + np * 32);
+          Mma::run(S.s[2 * np], va[ib], b[0], b[1]);
+          Mma::run(S.s[2 * np + 1], va[ib], b[2], b[3]);
+        }
       }
-    }
     const int64_t row0 = static_cast<int64_t>(first) + c * kChunk;
     store_out(O, reinterpret_cast<__nv_bfloat16*>(stage + 4 * Sh::kVec) + warp * 16, vrow,
               p.out + row0 * p.out_stride + static_cast<int64_t>(h) * p.V + p0 + warp * 16, p.out_stride,
@@ -322,7 +331,7 @@ extern "C" int mv_gla_chunk_scan(void* out, int64_t out_stride, const void* q, c
     const int pb = chunk_columns(static_cast<int64_t>(num_seqs) * heads, vdim), smem = 2 * GlaChunkShape<K>::stage(pb);
     e = cudaFuncSetAttribute(gla_chunk_kernel<K>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
     if (e != cudaSuccess) return fail(MV_ERR_CUDA, "gla_chunk_scan: %s", cudaGetErrorString(e));
-    gla_chunk_kernel<K><<<dim3(num_seqs, heads, (vdim + pb - 1) / pb), pb * 2, smem, st>>>(p, pb);
+    gla_chunk_kernel<K><<<dim3(num_seqs, heads, (vdim + pb - 1) / pb), kChunkThreads, smem, st>>>(p, pb);
     return check_launch("gla_chunk");
   });
 }

@@ -98,25 +98,37 @@ __device__ __forceinline__ void split_a(const float (&x)[4], const float (&y)[4]
 }
 
 // acc += A B^T for a lower-triangular 64 x 64 B in two terms (rows of kCkRow elements, the second 64 rows after the
-// first), A's 16-column block ib.
+// first), A's 16-column block ib.  Here and below two tiles' products alternate, so that a product rarely waits for the
+// one before it.
 template <bool kTwoA>
 __device__ __forceinline__ void mma_lower(float (&acc)[8][4], const uint32_t (&hi)[4], const uint32_t (&lo)[4], uint32_t b_smem,
                                           int ib, const LaneAt& at) {
 #pragma unroll
-  for (int np = 0; np < 4; ++np) {
-    if (np < ib) continue;
-    uint32_t b[4];
-    const uint32_t addr = b_smem + ((np * 16 + at.row_b) * kCkRow + ib * 16 + at.col_b) * 2;
-    ldmatrix_x4(b, addr);
-    Mma::run(acc[2 * np], hi, b[0], b[1]);
-    Mma::run(acc[2 * np + 1], hi, b[2], b[3]);
+  for (int n0 = 0; n0 < 4; n0 += 2) {
+    uint32_t b[2][4];
+    const uint32_t addr = b_smem + ((n0 * 16 + at.row_b) * kCkRow + ib * 16 + at.col_b) * 2;
+#pragma unroll
+    for (int j = 0; j < 2; ++j)
+      if (n0 + j >= ib) {
+        ldmatrix_x4(b[j], addr + j * 16 * kCkRow * 2);
+        Mma::run(acc[2 * (n0 + j)], hi, b[j][0], b[j][1]);
+        Mma::run(acc[2 * (n0 + j) + 1], hi, b[j][2], b[j][3]);
+      }
     if (kTwoA) {
-      Mma::run(acc[2 * np], lo, b[0], b[1]);
-      Mma::run(acc[2 * np + 1], lo, b[2], b[3]);
+#pragma unroll
+      for (int j = 0; j < 2; ++j)
+        if (n0 + j >= ib) {
+          Mma::run(acc[2 * (n0 + j)], lo, b[j][0], b[j][1]);
+          Mma::run(acc[2 * (n0 + j) + 1], lo, b[j][2], b[j][3]);
+        }
     }
-    ldmatrix_x4(b, addr + kChunk * kCkRow * 2);
-    Mma::run(acc[2 * np], hi, b[0], b[1]);
-    Mma::run(acc[2 * np + 1], hi, b[2], b[3]);
+#pragma unroll
+    for (int j = 0; j < 2; ++j)
+      if (n0 + j >= ib) {
+        ldmatrix_x4(b[j], addr + (j * 16 + kChunk) * kCkRow * 2);
+        Mma::run(acc[2 * (n0 + j)], hi, b[j][0], b[j][1]);
+        Mma::run(acc[2 * (n0 + j) + 1], hi, b[j][2], b[j][3]);
+      }
   }
 }
 
@@ -145,6 +157,7 @@ __device__ __forceinline__ void store_out(const float (&o)[8][4], __nv_bfloat16*
   }
 }
 
+constexpr int kChunkThreads = 256;       // of the second kernel; warps without columns of their own only fetch tiles
 // Value columns per CTA of the second kernel: all of them, or fewer when there are few (sequence, head) pairs.
 inline int chunk_columns(int64_t pairs, int V) {
   int pb = std::min(128, (V + 15) / 16 * 16);
