@@ -111,7 +111,7 @@ def test_experts_with_a_clamp(experts, top, width, ff, tokens, dtype):
                 _close(got[int(pos[t, k])], want, 1e-5 if dtype == torch.float32 else 1.6e-2, f"token {t}")
 
 
-@pytest.mark.parametrize("experts,top,count,keep", [(12, 4, 4, 3), (9, 2, 3, 2), (8, 1, 8, 1), (8, 4, 2, 1), (6, 3, 1, 1), (6, 3, 3, 3),
+@pytest.mark.parametrize("experts,top,count,keep", [(10, 3, 5, 3), (9, 2, 3, 2), (8, 1, 8, 1), (8, 4, 2, 1), (6, 3, 1, 1), (6, 3, 3, 3),
                                                     (64, 6, 8, 3), (96, 5, 48, 7), (300, 8, 10, 4)])
 def test_routing_in_groups(experts, top, count, keep):
     from minivllm_b200.layers import moe
@@ -134,7 +134,7 @@ def test_routing_in_groups(experts, top, count, keep):
 # ------------------------------------------------------------------------------------------------ windowed attention
 def test_distance_bias_table():
     from minivllm_b200.layers import window_attention as WA
-    for buckets, bias_max, window in ((10, 23, 11), (32, 120, 1 << 30), (16, 64, 40), (7, 12, 100), (8, 5, 64), (32, 200, 17)):
+    for buckets, bias_max, window in ((10, 23, 11), (32, 110, 1 << 30), (16, 64, 40), (7, 12, 100), (8, 5, 64), (32, 200, 17)):
         rel = _rnd(buckets, buckets, 3)
         got = WA.distance_bias(rel, bias_max, window)
         far = min(window, 3 * bias_max)
