@@ -25,7 +25,7 @@ enum mv_dtype { MV_F16 = 0, MV_BF16 = 1, MV_F32 = 2 };
 
 /* What a gate g does to the value u beside it.  GELU_TANH: the tanh form of gelu.  CLAMPED (with a limit):
  * g' sigmoid(1.702 g') (u' + 1) with g' = min(g, limit), u' = u clamped to +-limit. */
-enum mv_act { MV_ACT_NONE = -1, MV_ACT_SIGMOID = 0, MV_ACT_SILU = 1, MV_ACT_GELU_TANH = 2, MV_ACT_CLAMPED = 3 };
+enum mv_act { MV_ACT_NONE = -1, MV_ACT_SIGMOID = 0, MV_ACT_SILU = 1, MV_ACT_GELU_TANH = 2, MV_ACT_CLAMPED = 3, MV_ACT_RELU = 4 };
 
 enum mv_status {
   MV_OK = 0,
@@ -429,7 +429,8 @@ int mv_silu_mul(void* out, const void* gate_up, int64_t gate_up_stride,
  *                           + sigmoid(shared_gate[t]) * shared[t]   (shared may be null)
  *   mv_pair_residual_norm   the same with y = (norm(a) * w_a + norm(b) * w_b) / 2, no gate
  *   mv_gated_group_norm     out = norm(y * silu(z)) * w
- *   mv_head_norm_gate       out = norm(y) * w * silu(z), norms over `heads` equal runs; w has one run's length
+ *   mv_head_norm_gate       out = norm(y / den) * w * act(z), norms over `heads` equal runs; den (rows, heads) may be null;
+ *                           w has one run's length, or the row's with full_weight; act MV_ACT_SILU or MV_ACT_SIGMOID
  *   mv_gate_mul             out = gate applied to y (enum mv_act); a row of y is `heads` pieces y_head_stride
  *                           elements apart
  */
@@ -446,8 +447,8 @@ int mv_moe_residual_norm(void* out, float* x, const void* expert_rows, const int
 int mv_pair_residual_norm(void* out, float* x, const void* a, int64_t a_stride, const void* w_a, const
     void* b, int64_t b_stride, const void* w_b, const void* w_post, const void* w_next, float mult,
     int64_t rows, int width, int groups, float eps, int dtype, void* stream);
-int mv_head_norm_gate(void* out, const void* y, int64_t y_stride, const void* z, int64_t z_stride,
-    const void* w, int64_t rows, int width, int heads, float eps, int dtype, void* stream);
+int mv_head_norm_gate(void* out, const void* y, int64_t y_stride, const float* den, const void* z, int64_t z_stride,
+    const void* w, int full_weight, int act, int64_t rows, int width, int heads, float eps, int dtype, void* stream);
 int mv_gated_group_norm(void* out, const void* y, int64_t y_stride, const void* z, int64_t z_stride,
     const void* w, int64_t rows, int width, int groups, float eps, int dtype, void* stream);
 int mv_gate_mul(void* out, const void* y, int64_t y_stride, int64_t y_head_stride, int heads,
@@ -481,12 +482,16 @@ int mv_latent_attention_rows(void* out, int64_t out_stride, int64_t out_head_str
  * State-space mixer over a packed batch.  Sequence s has tokens cu[s] .. cu[s + 1] (cu null: one token each), slot
  * slots[s] and start[s] earlier tokens; start 0 reads the slot as zeros, start < 0 marks a padding row.
  *   mv_conv_silu          out (tokens, channels) = silu(causal depthwise convolution of u with w (channels, taps))
+ *   mv_conv_add           the same without silu, added to u
  *   mv_conv_state_update  state (num_slots, taps - 1, channels): the last inputs, oldest first
  *   mv_ssm_scan           xbc = [x: heads * vdim | B: groups * state_dim | C: the same] per token, dt before
  *                         bias and softplus; state (num_slots, heads, state_dim, vdim) fp32, updated
  * dtype MV_BF16 or MV_F32.  No counterpart in the reference.
  */
 int mv_conv_silu(void* out, const void* u, int64_t u_stride, const void* w, const void* bias, int
+    taps, int channels, const int32_t* cu, int num_seqs, int64_t tokens, const int32_t* slots, const
+    int32_t* start, const void* state, int num_slots, int dtype, void* stream);
+int mv_conv_add(void* out, const void* u, int64_t u_stride, const void* w, const void* bias, int
     taps, int channels, const int32_t* cu, int num_seqs, int64_t tokens, const int32_t* slots, const
     int32_t* start, const void* state, int num_slots, int dtype, void* stream);
 int mv_conv_state_update(void* state, const void* u, int64_t u_stride, int taps, int channels, const
@@ -587,29 +592,41 @@ int mv_ssm_step(void* y, const void* u, int64_t u_stride, const void* w, const v
  *   mv_window_prefill         packed queries and keys as in mv_latent_prefill (a sequence's keys begin at or before the
  *                             first one that its first query sees), bf16, dim up to 192, vdim up to 128, multiples of 8;
  *                             mv_window_prefill_distances = largest `distances` taken (-1: sizes not taken)
- * out is (tokens, heads * vdim).  No counterpart in the reference.
+ *   mv_qkv_rope_store         q (in place) and k: RMS norm per head with a weight (dim), then pairs of neighbouring columns
+ *                             2i, 2i + 1 of the first `dims` turned by the angle in row positions[t], column i of cos_t and
+ *                             sin_t (table_rows, dims / 2); q of head h times temp[h] (null: 1).  v: its pairs turned by
+ *                             vcos_t, vsin_t (table_rows, vdim / 2; null: as it is).  [k | v] goes to kv_out and cache as
+ *                             above; kv_heads 0: queries only.  dim and vdim up to 1,024
+ * cos_t, sin_t (table_rows, vdim / 2) of the attention entries: the result of position i is turned in the same pairs by the
+ * opposite of row i's angles (null: not).  out is (tokens, heads * vdim).  No counterpart in the reference.
  */
 int mv_kv_norm_store(void* q, const void* k, const void* v, int64_t stride, const void* q_weight, const
     void* k_weight, void* kv_out, void* cache, const int64_t* slot_mapping, int64_t num_slots, int64_t
     tokens, int q_rows, int k_rows, int v_rows, float eps, int dtype, void* stream);
+int mv_qkv_rope_store(void* q, const void* k, const void* v, int64_t stride, const void* q_weight, const
+    void* k_weight, const void* temp, const float* cos_t, const float* sin_t, int dims, const float*
+    vcos_t, const float* vsin_t, int64_t table_rows, const int64_t* positions, void* kv_out, void* cache,
+    const int64_t* slot_mapping, int64_t num_slots, int64_t tokens, int heads, int kv_heads, int dim,
+    int vdim, float eps, int dtype, void* stream);
 int mv_window_attention_rows(void* out, const void* q, int64_t q_stride, const void* cache, const
     int32_t* block_tables, int64_t bt_stride, int max_blocks, int block_size, int64_t num_blocks,
     const int32_t* cu_q, int num_seqs, const int64_t* positions, const float* bias, int64_t
-    bias_stride, int distances, const void* sink, int64_t tokens, int heads, int kv_heads, int dim,
-    int vdim, int64_t window, float scale, int dtype, void* stream);
+    bias_stride, int distances, const void* sink, const float* cos_t, const float* sin_t, int64_t
+    table_rows, int64_t tokens, int heads, int kv_heads, int dim, int vdim, int64_t window, float
+    scale, int dtype, void* stream);
 int64_t mv_window_decode_workspace_bytes(int batch, int heads, int kv_heads, int dim, int vdim, int64_t
     most_keys);
 int mv_window_decode(void* out, const void* q, int64_t q_stride, const void* cache, const int32_t*
     block_tables, int64_t bt_stride, int max_blocks, int block_size, int64_t num_blocks, const int64_t*
-    positions, const float* bias, int64_t bias_stride, int distances, const void* sink, int batch,
-    int heads, int kv_heads, int dim, int vdim, int64_t window, float scale, void* workspace, int64_t
-    workspace_bytes, void* stream);
+    positions, const float* bias, int64_t bias_stride, int distances, const void* sink, const float*
+    cos_t, const float* sin_t, int64_t table_rows, int batch, int heads, int kv_heads, int dim, int vdim,
+    int64_t window, float scale, void* workspace, int64_t workspace_bytes, void* stream);
 int mv_window_prefill_distances(int dim, int vdim);
 int mv_window_prefill(void* out, int64_t out_stride, const void* q, int64_t q_stride, const void* k,
     int64_t k_stride, const void* v, int64_t v_stride, const int32_t* cu_q, const int32_t* cu_k, int
     num_seqs, int64_t tokens, int64_t keys, int heads, int kv_heads, int dim, int vdim, int64_t window,
-    float scale, const float* bias, int64_t bias_stride, int distances, const void* sink, int*
-    error_word, void* stream);
+    float scale, const float* bias, int64_t bias_stride, int distances, const void* sink, const float*
+    cos_t, const float* sin_t, int64_t table_rows, const int64_t* positions, int* error_word, void* stream);
 
 /*
  * Matrix-state recurrences, fp32 state (num_slots, heads, dim, vdim) updated in place, one read-out per token; dim up
@@ -650,6 +667,54 @@ int mv_delta_chunk_scan(void* out, int64_t out_stride, const void* qkv, int64_t 
     int num_seqs, int64_t tokens, const int32_t* slots, const int32_t* start, float* state, int
     num_slots, int heads, int kv_heads, int dim, int vdim, float q_scale, void* workspace, int64_t
     workspace_bytes, void* stream);
+
+/*
+ * Matrix memory with exponential gates and a running maximum (mLSTM), fp32 state S (num_slots, heads, dim, vdim), n (num_slots,
+ * heads, dim), m (num_slots, heads), updated in place; cu, slots and start as in mv_conv_silu.  Per head and token, with
+ * i = cap tanh((zi + i_b) / cap), f = logsigmoid(cap tanh((zf + f_b) / cap)):
+ *   m' = max(f + m, i);  S <- exp(f + m - m') S + exp(i - m') k v^T;  n likewise with k;  m <- m'
+ *   o = S^T q / (max(|n . q|, exp(-m)) + 1e-6), q scaled by q_scale
+ * gates (tokens, 2 * heads) fp32 holds [zi | zf], rows of q, k, v share one stride; dim up to 256.
+ *   mv_mlstm_gates       portions: chain (tokens, heads, 4) = i, f, m before and after the token; m advances
+ *   mv_mlstm_scan        portions, token by token: out = S^T q, den (tokens, heads) fp32 = its denominator
+ *   mv_mlstm_chunk_scan  the same in chunks of 64 tokens on tensor cores, bf16: dim a multiple of 8 up to 128, vdim a multiple
+ *                        of 8, rows on 16-byte boundaries; tokens = cu[num_seqs]; workspace_bytes is -1 when the sizes are
+ *                        not taken
+ *   mv_mlstm_step        one token per sequence: out = rms_norm(o) * norm_w * sigmoid(gate), norm_w (heads * vdim)
+ * dtype MV_BF16 or MV_F32.  No counterpart in the reference.
+ */
+int mv_mlstm_gates(float* chain, const float* gates, int64_t gates_stride, const void* i_b, const void* f_b,
+    float cap, const int32_t* cu, int num_seqs, const int32_t* slots, const int32_t* start, float* m_state,
+    int num_slots, int heads, int dtype, void* stream);
+int mv_mlstm_scan(void* out, int64_t out_stride, float* den, const void* q, const void* k, const void* v,
+    int64_t stride, const float* chain, const int32_t* cu, int num_seqs, const int32_t* slots, const
+    int32_t* start, float* S, float* n, int num_slots, int heads, int dim, int vdim, float q_scale, int
+    dtype, void* stream);
+int64_t mv_mlstm_chunk_workspace_bytes(int64_t tokens, int num_seqs, int heads, int dim, int vdim);
+int mv_mlstm_chunk_scan(void* out, int64_t out_stride, float* den, const void* q, const void* k, const void*
+    v, int64_t stride, const float* chain, const int32_t* cu, int num_seqs, int64_t tokens, const int32_t*
+    slots, const int32_t* start, float* S, float* n, int num_slots, int heads, int dim, int vdim, float
+    q_scale, void* workspace, int64_t workspace_bytes, void* stream);
+int mv_mlstm_step(void* out, int64_t out_stride, const void* q, const void* k, const void* v, int64_t stride,
+    const float* gates, int64_t gates_stride, const void* i_b, const void* f_b, float cap, int num_seqs,
+    const int32_t* slots, const int32_t* start, float* S, float* n, float* m, int num_slots, int heads, int
+    dim, int vdim, float q_scale, const void* gate, int64_t gate_stride, const void* norm_w, float eps, int
+    dtype, void* stream);
+
+/*
+ * Between two sublayers of a decoder with several residual streams x (rows, streams, width) fp32, at most 16.  The new streams
+ * x_t = sum_s mix[s, t] x_s + w_out[t] y (all from the old ones; with ids: every stream = the embedding row), then
+ * u = sum_s w_in[s] x_s (null: plain sum) and h = layer norm of u with norm_w and norm_b (norm_b null: RMS norm).
+ * Rows below conv_rows are one-token sequences with slots and starts as in mv_conv_silu: with taps > 0, out = h + causal
+ * convolution of h with taps_t (taps, width), whose inputs conv_state (num_slots, taps - 1, width) keeps and which moves on.
+ * Without taps out = h.  The h of the other rows goes to raw, from its first row on.  dtype MV_BF16 or MV_F32 of all but x.
+ * No counterpart in the reference.
+ */
+int mv_stream_step(void* out, void* raw, float* x, const int64_t* ids, const void* embed, int64_t vocab, const
+    void* y, int64_t y_stride, const void* mix, const void* w_out, const void* w_in, const void* norm_w,
+    const void* norm_b, const void* taps_t, int taps, void* conv_state, const int32_t* slots, const int32_t*
+    start, int num_slots, int64_t conv_rows, int64_t rows, int width, int streams, float eps, int dtype,
+    void* stream);
 
 #ifdef __cplusplus
 }

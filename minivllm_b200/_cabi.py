@@ -75,8 +75,8 @@ SIGNATURES = {
         _c_i64, _c_ptr, _c_i64, _c_ptr, _c_ptr, _c_ptr, _c_f32, _c_i64, _c_int, _c_int, _c_f32, _c_int, _c_ptr]),
     "mv_pair_residual_norm": (_c_int, [_c_ptr, _c_ptr, _c_ptr, _c_i64, _c_ptr, _c_ptr, _c_i64, _c_ptr, _c_ptr, _c_ptr,
         _c_f32, _c_i64, _c_int, _c_int, _c_f32, _c_int, _c_ptr]),
-    "mv_head_norm_gate": (_c_int, [_c_ptr, _c_ptr, _c_i64, _c_ptr, _c_i64, _c_ptr, _c_i64, _c_int, _c_int, _c_f32,
-        _c_int, _c_ptr]),
+    "mv_head_norm_gate": (_c_int, [_c_ptr, _c_ptr, _c_i64, _c_ptr, _c_ptr, _c_i64, _c_ptr, _c_int, _c_int, _c_i64, _c_int, _c_int,
+        _c_f32, _c_int, _c_ptr]),
     "mv_gated_group_norm": (_c_int, [_c_ptr, _c_ptr, _c_i64, _c_ptr, _c_i64, _c_ptr, _c_i64, _c_int, _c_int, _c_f32,
         _c_int, _c_ptr]),
     "mv_gate_mul": (_c_int, [_c_ptr, _c_ptr, _c_i64, _c_i64, _c_int, _c_ptr, _c_i64, _c_int, _c_f32, _c_i64, _c_int, _c_int,
@@ -87,6 +87,8 @@ SIGNATURES = {
         _c_int, _c_int, _c_i64, _c_ptr, _c_int, _c_ptr, _c_ptr, _c_i64, _c_int, _c_int, _c_int, _c_f32, _c_int,
         _c_ptr]),
     "mv_conv_silu": (_c_int, [_c_ptr, _c_ptr, _c_i64, _c_ptr, _c_ptr, _c_int, _c_int, _c_ptr, _c_int, _c_i64,
+        _c_ptr, _c_ptr, _c_ptr, _c_int, _c_int, _c_ptr]),
+    "mv_conv_add": (_c_int, [_c_ptr, _c_ptr, _c_i64, _c_ptr, _c_ptr, _c_int, _c_int, _c_ptr, _c_int, _c_i64,
         _c_ptr, _c_ptr, _c_ptr, _c_int, _c_int, _c_ptr]),
     "mv_conv_state_update": (_c_int, [_c_ptr, _c_ptr, _c_i64, _c_int, _c_int, _c_ptr, _c_int, _c_ptr, _c_ptr,
         _c_int, _c_int, _c_ptr]),
@@ -116,14 +118,16 @@ SIGNATURES = {
     "mv_kv_norm_store": (_c_int, [_c_ptr, _c_ptr, _c_ptr, _c_i64, _c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_i64, _c_i64,
         _c_int, _c_int, _c_int, _c_f32, _c_int, _c_ptr]),
     "mv_window_attention_rows": (_c_int, [_c_ptr, _c_ptr, _c_i64, _c_ptr, _c_ptr, _c_i64, _c_int, _c_int, _c_i64, _c_ptr,
-        _c_int, _c_ptr, _c_ptr, _c_i64, _c_int, _c_ptr, _c_i64, _c_int, _c_int, _c_int, _c_int, _c_i64, _c_f32, _c_int,
-        _c_ptr]),
+        _c_int, _c_ptr, _c_ptr, _c_i64, _c_int, _c_ptr, _c_ptr, _c_ptr, _c_i64, _c_i64, _c_int, _c_int, _c_int, _c_int, _c_i64,
+        _c_f32, _c_int, _c_ptr]),
     "mv_window_decode_workspace_bytes": (_c_i64, [_c_int, _c_int, _c_int, _c_int, _c_int, _c_i64]),
     "mv_window_decode": (_c_int, [_c_ptr, _c_ptr, _c_i64, _c_ptr, _c_ptr, _c_i64, _c_int, _c_int, _c_i64, _c_ptr, _c_ptr,
-        _c_i64, _c_int, _c_ptr, _c_int, _c_int, _c_int, _c_int, _c_int, _c_i64, _c_f32, _c_ptr, _c_i64, _c_ptr]),
+        _c_i64, _c_int, _c_ptr, _c_ptr, _c_ptr, _c_i64, _c_int, _c_int, _c_int, _c_int, _c_int, _c_i64, _c_f32, _c_ptr, _c_i64,
+        _c_ptr]),
     "mv_window_prefill_distances": (_c_int, [_c_int, _c_int]),
     "mv_window_prefill": (_c_int, [_c_ptr, _c_i64, _c_ptr, _c_i64, _c_ptr, _c_i64, _c_ptr, _c_i64, _c_ptr, _c_ptr, _c_int,
-        _c_i64, _c_i64, _c_int, _c_int, _c_int, _c_int, _c_i64, _c_f32, _c_ptr, _c_i64, _c_int, _c_ptr, _c_ptr, _c_ptr]),
+        _c_i64, _c_i64, _c_int, _c_int, _c_int, _c_int, _c_i64, _c_f32, _c_ptr, _c_i64, _c_int, _c_ptr, _c_ptr, _c_ptr, _c_i64,
+        _c_ptr, _c_ptr, _c_ptr]),
     "mv_gla_scan": (_c_int, [_c_ptr, _c_i64, _c_ptr, _c_ptr, _c_ptr, _c_i64, _c_ptr, _c_i64, _c_f32, _c_ptr, _c_int, _c_ptr,
         _c_ptr, _c_ptr, _c_int, _c_int, _c_int, _c_int, _c_f32, _c_ptr, _c_i64, _c_ptr, _c_f32, _c_int, _c_ptr]),
     "mv_delta_scan": (_c_int, [_c_ptr, _c_i64, _c_ptr, _c_i64, _c_ptr, _c_ptr, _c_i64, _c_ptr, _c_ptr, _c_ptr, _c_int,
@@ -135,6 +139,23 @@ SIGNATURES = {
     "mv_delta_chunk_workspace_bytes": (_c_i64, [_c_i64, _c_int, _c_int, _c_int, _c_int]),
     "mv_delta_chunk_scan": (_c_int, [_c_ptr, _c_i64, _c_ptr, _c_i64, _c_ptr, _c_ptr, _c_i64, _c_ptr, _c_ptr, _c_ptr, _c_int,
         _c_i64, _c_ptr, _c_ptr, _c_ptr, _c_int, _c_int, _c_int, _c_int, _c_int, _c_f32, _c_ptr, _c_i64, _c_ptr]),
+        "mv_qkv_rope_store": (_c_int, [_c_ptr, _c_ptr, _c_ptr, _c_i64, _c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_int,
+        _c_ptr, _c_ptr, _c_i64, _c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_i64, _c_i64, _c_int, _c_int, _c_int, _c_int,
+        _c_f32, _c_int, _c_ptr]),
+        "mv_mlstm_gates": (_c_int, [_c_ptr, _c_ptr, _c_i64, _c_ptr, _c_ptr, _c_f32, _c_ptr, _c_int, _c_ptr, _c_ptr,
+        _c_ptr, _c_int, _c_int, _c_int, _c_ptr]),
+        "mv_mlstm_scan": (_c_int, [_c_ptr, _c_i64, _c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_i64, _c_ptr, _c_ptr, _c_int,
+        _c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_int, _c_int, _c_int, _c_int, _c_f32, _c_int, _c_ptr]),
+        "mv_mlstm_chunk_workspace_bytes": (_c_i64, [_c_i64, _c_int, _c_int, _c_int, _c_int]),
+        "mv_mlstm_chunk_scan": (_c_int, [_c_ptr, _c_i64, _c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_i64, _c_ptr, _c_ptr,
+        _c_int, _c_i64, _c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_int, _c_int, _c_int, _c_int, _c_f32, _c_ptr, _c_i64,
+        _c_ptr]),
+        "mv_mlstm_step": (_c_int, [_c_ptr, _c_i64, _c_ptr, _c_ptr, _c_ptr, _c_i64, _c_ptr, _c_i64, _c_ptr, _c_ptr,
+        _c_f32, _c_int, _c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_int, _c_int, _c_int, _c_int, _c_f32, _c_ptr,
+        _c_i64, _c_ptr, _c_f32, _c_int, _c_ptr]),
+        "mv_stream_step": (_c_int, [_c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_i64, _c_ptr, _c_i64, _c_ptr, _c_ptr,
+        _c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_int, _c_ptr, _c_ptr, _c_ptr, _c_int, _c_i64, _c_i64, _c_int, _c_int,
+        _c_f32, _c_int, _c_ptr]),
 }
 
 _lib = None

@@ -21,6 +21,7 @@ GROUPS = {
                 "mamba2_chunk.cu", "moe.cu", "grouped_gemm.cu"],
     "fozerax": ["norms.cu", "window_attention.cu", "latent_prefill.cu", "short_conv.cu", "gla.cu", "gla_chunk.cu", "gated_delta.cu",
                 "gated_delta_chunk.cu", "moe.cu", "grouped_gemm.cu"],
+    "dafotar": ["norms.cu", "streams.cu", "short_conv.cu", "window_attention.cu", "latent_prefill.cu", "mlstm.cu", "mlstm_chunk.cu"],
 }
 SOURCES = COMMON + list(dict.fromkeys(s for g in GROUPS.values() for s in g))
 NVCC_FLAGS = [

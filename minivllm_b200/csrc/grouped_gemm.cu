@@ -203,6 +203,7 @@ grouped_gemm_kernel(const __grid_constant__ CUtensorMap tmap_w, const __grid_con
               case MV_ACT_SILU: apply(std::integral_constant<int, MV_ACT_SILU>{}); break;
               case MV_ACT_SIGMOID: apply(std::integral_constant<int, MV_ACT_SIGMOID>{}); break;
               case MV_ACT_GELU_TANH: apply(std::integral_constant<int, MV_ACT_GELU_TANH>{}); break;
+              case MV_ACT_RELU: apply(std::integral_constant<int, MV_ACT_RELU>{}); break;
               default: apply(std::integral_constant<int, MV_ACT_CLAMPED>{});
             }
           }
@@ -251,7 +252,7 @@ extern "C" int mv_grouped_gemm(void* out, const void* x, const void* w, const in
                                int64_t rows, int in_dim, int out_dim, int act, float limit, int* error_word,
                                void* stream) {
   using namespace mv;
-  if (act < MV_ACT_NONE || act > MV_ACT_CLAMPED) return fail(MV_ERR_SHAPE, "grouped_gemm: activation %d", act);
+  if (act < MV_ACT_NONE || act > MV_ACT_RELU) return fail(MV_ERR_SHAPE, "grouped_gemm: activation %d", act);
   const bool gated = act != MV_ACT_NONE;
   if (rows < 0 || experts <= 0 || in_dim <= 0 || out_dim <= 0) return fail(MV_ERR_SHAPE, "grouped_gemm: %d x %d", out_dim, in_dim);
   if (in_dim % 8) return fail(MV_ERR_SHAPE, "grouped_gemm: in_dim %d is not a multiple of 8", in_dim);

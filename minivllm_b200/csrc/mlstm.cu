@@ -1,0 +1,135 @@
+// Matrix memory with exponential gates (mLSTM) over a packed batch, the state in slots: the chain of running maxima here, the
+// recurrence token by token in state_scan.cuh.
+#include "state_scan.cuh"
+
+namespace mv {
+
+// One warp per (sequence, head): m' = max(f + m, i) token by token.  A run of tokens acts on m as m -> max(m + F, A), F the sum
+// of the f's, and runs compose, so that the warp takes 128 tokens at a time, four per lane.
+constexpr int kMgRun = 4;
+
+template <typename T> __global__ void __launch_bounds__(32) mlstm_gates_kernel(const ScanParams<T> p, float4* __restrict__ chain) {
+  const int s = blockIdx.x, h = blockIdx.y, lane = threadIdx.x;
+  const int first = p.cu[s], n_tok = p.cu[s + 1] - first;
+  if (n_tok <= 0) return;
+  const int slot = p.slots[s], st0 = p.start[s];
+  const bool live = slot >= 0 && slot < p.num_slots && st0 >= 0;
+  float* gm = p.m_state + static_cast<int64_t>(live ? slot : 0) * p.heads + h;
+  float m = live && st0 > 0 ? *gm : 0.f;
+  const float ib = Elem<T>::to_f(p.i_b[h]), fb = Elem<T>::to_f(p.f_b[h]);
+  float zi[kMgRun], zf[kMgRun];
+  auto fetch = [&](int t0) {
+#pragma unroll
+    for (int e = 0; e < kMgRun; ++e) {
+      const int t = t0 + lane * kMgRun + e;
+      const float* z = p.gates + static_cast<int64_t>(first + (t < n_tok ? t : 0)) * p.gates_stride + h;
+      zi[e] = z[0];
+      zf[e] = z[p.heads];
+    }
+  };
+  fetch(0);
+  for (int t0 = 0; t0 < n_tok; t0 += 32 * kMgRun) {
+    float i[kMgRun], f[kMgRun], F = 0.f, A = -INFINITY;
+#pragma unroll
+    for (int e = 0; e < kMgRun; ++e) {
+      const bool on = t0 + lane * kMgRun + e < n_tok;
+      i[e] = on ? mem_log_input(zi[e] + ib, p.cap) : -INFINITY;
+      f[e] = on ? mem_log_forget(zf[e] + fb, p.cap) : 0.f;
+      A = fmaxf(A + f[e], i[e]);
+      F += f[e];
+    }
+    if (t0 + 32 * kMgRun < n_tok) fetch(t0 + 32 * kMgRun);
+#pragma unroll
+    for (int o = 1; o < 32; o <<= 1) {
+      const float Fb = __shfl_up_sync(0xffffffffu, F, o), Ab = __shfl_up_sync(0xffffffffu, A, o);
+      if (lane >= o) {
+        A = fmaxf(Ab + F, A);
+        F += Fb;
+      }
+    }
+    const float Fb = __shfl_up_sync(0xffffffffu, F, 1), Ab = __shfl_up_sync(0xffffffffu, A, 1);
+    float after[kMgRun], at = lane == 0 ? m : fmaxf(m + Fb, Ab);
+#pragma unroll
+    for (int e = 0; e < kMgRun; ++e) after[e] = at = fmaxf(f[e] + at, i[e]);
+    // what a token continues is what the token before it left, to the last bit
+    float before = __shfl_up_sync(0xffffffffu, at, 1);
+    if (lane == 0) before = m;
+#pragma unroll
+    for (int e = 0; e < kMgRun; ++e) {
+      const int t = t0 + lane * kMgRun + e;
+      if (t < n_tok) chain[static_cast<int64_t>(first + t) * p.heads + h] = make_float4(i[e], f[e], before, after[e]);
+      before = after[e];
+    }
+    m = __shfl_sync(0xffffffffu, at, 31);
+  }
+  if (live && lane == 0) *gm = m;
+}
+
+template <typename F> static int by_dtype(int dtype, F&& f) { return dtype == MV_F32 ? f(float{}) : f(__nv_bfloat16{}); }
+
+}  // namespace mv
+
+extern "C" int mv_mlstm_gates(float* chain, const float* gates, int64_t gates_stride, const void* i_b, const void* f_b,
+                              float cap, const int32_t* cu, int num_seqs, const int32_t* slots, const int32_t* start,
+                              float* m_state, int num_slots, int heads, int dtype, void* stream) {
+  using namespace mv;
+  const int rc = check_scan("mlstm_gates", dtype, num_seqs, heads, heads, 1, 1);
+  if (rc || num_seqs == 0) return rc;
+  if (!(cap > 0.f)) return fail(MV_ERR_SHAPE, "mlstm_gates: cap %f", cap);
+  if (!chain || !gates || !i_b || !f_b || !cu || !slots || !start || !m_state) return fail(MV_ERR_NULL, "mlstm_gates: null pointer");
+  if (!aligned16(chain)) return fail(MV_ERR_ALIGN, "mlstm_gates: chain");
+  return by_dtype(dtype, [&](auto tag) {
+    using T = decltype(tag);
+    ScanParams<T> p{};
+    p.gates = gates; p.gates_stride = gates_stride; p.i_b = static_cast<const T*>(i_b); p.f_b = static_cast<const T*>(f_b); p.cap = cap;
+    p.cu = cu; p.slots = slots; p.start = start; p.m_state = m_state; p.num_slots = num_slots; p.heads = heads;
+    mlstm_gates_kernel<T><<<dim3(num_seqs, heads), 32, 0, static_cast<cudaStream_t>(stream)>>>(p, reinterpret_cast<float4*>(chain));
+    return check_launch("mlstm_gates");
+  });
+}
+
+extern "C" int mv_mlstm_scan(void* out, int64_t out_stride, float* den, const void* q, const void* k, const void* v,
+                             int64_t stride, const float* chain, const int32_t* cu, int num_seqs, const int32_t* slots,
+                             const int32_t* start, float* S, float* n, int num_slots, int heads, int dim, int vdim,
+                             float q_scale, int dtype, void* stream) {
+  using namespace mv;
+  const int rc = check_scan("mlstm_scan", dtype, num_seqs, heads, heads, dim, vdim);
+  if (rc || num_seqs == 0) return rc;
+  if (!out || !den || !q || !k || !v || !chain || !cu || !slots || !start || !S || !n) return fail(MV_ERR_NULL, "mlstm_scan: null pointer");
+  if (!aligned16(S) || !aligned16(chain)) return fail(MV_ERR_ALIGN, "mlstm_scan: state");
+  return by_dtype(dtype, [&](auto tag) {
+    using T = decltype(tag);
+    auto c = [](const void* x) { return static_cast<const T*>(x); };
+    ScanParams<T> p{};
+    p.out = static_cast<T*>(out); p.out_stride = out_stride; p.q = c(q); p.k = c(k); p.v = c(v); p.stride = stride;
+    p.chain = reinterpret_cast<const float4*>(chain); p.den = den; p.n_state = n;
+    p.cu = cu; p.slots = slots; p.start = start; p.state = S; p.num_slots = num_slots;
+    p.heads = heads; p.kv_heads = heads; p.K = dim; p.V = vdim; p.q_scale = q_scale;
+    return run_scan<SK_MLSTM, T>(p, num_seqs, static_cast<cudaStream_t>(stream));
+  });
+}
+
+extern "C" int mv_mlstm_step(void* out, int64_t out_stride, const void* q, const void* k, const void* v, int64_t stride,
+                             const float* gates, int64_t gates_stride, const void* i_b, const void* f_b, float cap,
+                             int num_seqs, const int32_t* slots, const int32_t* start, float* S, float* n, float* m,
+                             int num_slots, int heads, int dim, int vdim, float q_scale, const void* gate,
+                             int64_t gate_stride, const void* norm_w, float eps, int dtype, void* stream) {
+  using namespace mv;
+  const int rc = check_scan("mlstm_step", dtype, num_seqs, heads, heads, dim, vdim);
+  if (rc || num_seqs == 0) return rc;
+  if (!(cap > 0.f)) return fail(MV_ERR_SHAPE, "mlstm_step: cap %f", cap);
+  if (!out || !q || !k || !v || !gates || !i_b || !f_b || !slots || !start || !S || !n || !m || !gate || !norm_w)
+    return fail(MV_ERR_NULL, "mlstm_step: null pointer");
+  if (!aligned16(S)) return fail(MV_ERR_ALIGN, "mlstm_step: state");
+  return by_dtype(dtype, [&](auto tag) {
+    using T = decltype(tag);
+    auto c = [](const void* x) { return static_cast<const T*>(x); };
+    ScanParams<T> p{};
+    p.out = static_cast<T*>(out); p.out_stride = out_stride; p.q = c(q); p.k = c(k); p.v = c(v); p.stride = stride;
+    p.gates = gates; p.gates_stride = gates_stride; p.i_b = c(i_b); p.f_b = c(f_b); p.cap = cap; p.n_state = n; p.m_state = m;
+    p.slots = slots; p.start = start; p.state = S; p.num_slots = num_slots;
+    p.heads = heads; p.kv_heads = heads; p.K = dim; p.V = vdim; p.q_scale = q_scale;
+    p.gate = c(gate); p.out_gate_stride = gate_stride; p.norm_w = c(norm_w); p.eps = eps;
+    return run_step<SK_MLSTM, T>(p, num_seqs, static_cast<cudaStream_t>(stream));
+  });
+}

@@ -357,7 +357,7 @@ extern "C" int mv_gather_rows(void* out, const void* x, int64_t x_stride, const 
 extern "C" int mv_grouped_rows(void* out, const void* x, const void* w, const int32_t* offsets, int experts,
                                int64_t rows, int in_dim, int out_dim, int act, float limit, int dtype, void* stream) {
   using namespace mv;
-  if (act < MV_ACT_NONE || act > MV_ACT_CLAMPED) return fail(MV_ERR_SHAPE, "grouped_rows: activation %d", act);
+  if (act < MV_ACT_NONE || act > MV_ACT_RELU) return fail(MV_ERR_SHAPE, "grouped_rows: activation %d", act);
   if (dtype != MV_BF16 && dtype != MV_F32) return fail(MV_ERR_DTYPE, "grouped_rows: dtype %d", dtype);
   if (rows < 0 || experts <= 0 || in_dim <= 0 || out_dim <= 0) return fail(MV_ERR_SHAPE, "grouped_rows: %d x %d", out_dim, in_dim);
   if (rows == 0) return MV_OK;

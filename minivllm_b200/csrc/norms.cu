@@ -394,12 +394,18 @@ __global__ void __launch_bounds__(kNormThreads, SRC == SRC_EXPERTS ? (kCh == 1 ?
     }
 }
 
-// kGateFirst: out = group_rms_norm(y * silu(z)) * w.  Otherwise out = group_rms_norm(y) * w * silu(z), where w has one
-// group's length and is shared by the groups.
+// What follows a norm per head: the read-outs' denominators (rows, heads), null: none; the norm's weight for the whole row
+// instead of one that the heads share; the gate's activation.
+struct HeadNorm {
+  const float* den;
+  bool full_weight, sigmoid;
+};
+
+// kGateFirst: out = group_rms_norm(y * silu(z)) * w.  Otherwise out = group_rms_norm(y / den) * w * act(z).
 template <typename T, int V, bool kGateFirst>
 __global__ void __launch_bounds__(kNormThreads)
 gated_group_norm_kernel(T* __restrict__ out, const T* __restrict__ y, int64_t y_stride, const T* __restrict__ z,
-                        int64_t z_stride, const T* __restrict__ w, int width, int groups, float eps) {
+                        int64_t z_stride, const T* __restrict__ w, int width, int groups, float eps, const HeadNorm hn) {
   extern __shared__ __align__(16) float s_row[];
   float* part = s_row + ((width + 3) & ~3);
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
@@ -407,6 +413,7 @@ gated_group_norm_kernel(T* __restrict__ out, const T* __restrict__ y, int64_t y_
   const GroupPlan gp(width, groups, V, warp);
   for (int g = gp.g0; g < groups; g += gp.cg) {
     float acc = 0.f;
+    const float den = !kGateFirst && hn.den ? 1.f / hn.den[row * groups + g] : 1.f;
     for (int i = gp.sub * 32 + lane; i < gp.chunks; i += gp.wpg * 32) {
       const int c = g * gp.gs + i * V;
       float v[V], t[V];
@@ -414,7 +421,7 @@ gated_group_norm_kernel(T* __restrict__ out, const T* __restrict__ y, int64_t y_
       if (kGateFirst) Vec<T, V>::load(z + row * z_stride + c, t);
 #pragma unroll
       for (int e = 0; e < V; ++e) {
-        if (kGateFirst) v[e] *= silu_t<T>(t[e]);
+        v[e] *= kGateFirst ? silu_t<T>(t[e]) : den;
         acc = fmaf(v[e], v[e], acc);
       }
       Vec<float, V>::store(s_row + c, v);
@@ -429,13 +436,13 @@ gated_group_norm_kernel(T* __restrict__ out, const T* __restrict__ y, int64_t y_
       const int c = g * gp.gs + i * V;
       float v[V], t[V];
       Vec<float, V>::load(s_row + c, v);
-      Vec<T, V>::load(w + (kGateFirst ? c : c - g * gp.gs), t);
+      Vec<T, V>::load(w + (kGateFirst || hn.full_weight ? c : c - g * gp.gs), t);
 #pragma unroll
       for (int e = 0; e < V; ++e) v[e] = v[e] * rs * t[e];
       if (!kGateFirst) {
         Vec<T, V>::load(z + row * z_stride + c, t);
 #pragma unroll
-        for (int e = 0; e < V; ++e) v[e] *= silu_t<T>(t[e]);
+        for (int e = 0; e < V; ++e) v[e] *= hn.sigmoid ? sigmoid_t<T>(t[e]) : silu_t<T>(t[e]);
       }
       Vec<T, V>::store(out + row * width + c, v);
     }
@@ -447,13 +454,15 @@ gated_group_norm_kernel(T* __restrict__ out, const T* __restrict__ y, int64_t y_
 template <typename T, int L, int kCh>
 __global__ void __launch_bounds__(kNormThreads)
 head_norm_gate_kernel(T* __restrict__ out, const T* __restrict__ y, int64_t y_stride, const T* __restrict__ z,
-                      int64_t z_stride, const T* __restrict__ w, int64_t rows, int heads, int gs, float eps) {
+                      int64_t z_stride, const T* __restrict__ w, int64_t rows, int heads, int gs, float eps, const HeadNorm hn) {
   const int lane = threadIdx.x & (L - 1);
   const int64_t items = rows * heads, step = static_cast<int64_t>(gridDim.x) * (kNormThreads / L);
   for (int64_t i0 = static_cast<int64_t>(blockIdx.x) * (kNormThreads / L); i0 < items; i0 += step) {
     const int64_t i = i0 + threadIdx.x / L, row = i / heads;
     const int h = static_cast<int>(i - row * heads);
     const bool on = i < items;
+    const float den = on && hn.den ? 1.f / hn.den[i] : 1.f;
+    const T* wh = w + (hn.full_weight ? static_cast<int64_t>(h) * gs : 0);
     Raw8<T> a[kCh], b[kCh];
     float acc = 0.f;
 #pragma unroll
@@ -470,11 +479,11 @@ head_norm_gate_kernel(T* __restrict__ out, const T* __restrict__ y, int64_t y_st
         float v[8];
         a[k].get(v);
 #pragma unroll
-        for (int e = 0; e < 8; ++e) acc = fmaf(v[e], v[e], acc);
+        for (int e = 0; e < 8; ++e) acc = fmaf(v[e] * den, v[e] * den, acc);
       }
 #pragma unroll
     for (int o = L / 2; o; o >>= 1) acc += __shfl_xor_sync(0xffffffffu, acc, o);
-    const float rs = 1.f / sqrtf(acc / static_cast<float>(gs) + eps);
+    const float rs = den / sqrtf(acc / static_cast<float>(gs) + eps);
 #pragma unroll
     for (int k = 0; k < kCh; ++k) {
       const int c = (k * L + lane) * 8;
@@ -482,9 +491,9 @@ head_norm_gate_kernel(T* __restrict__ out, const T* __restrict__ y, int64_t y_st
         float v[8], t[8], g[8];
         a[k].get(v);
         b[k].get(g);
-        Vec<T, 8>::load(w + c, t);
+        Vec<T, 8>::load(wh + c, t);
 #pragma unroll
-        for (int e = 0; e < 8; ++e) v[e] = v[e] * rs * t[e] * silu_t<T>(g[e]);
+        for (int e = 0; e < 8; ++e) v[e] = v[e] * rs * t[e] * (hn.sigmoid ? sigmoid_t<T>(g[e]) : silu_t<T>(g[e]));
         Vec<T, 8>::store(out + row * (static_cast<int64_t>(heads) * gs) + static_cast<int64_t>(h) * gs + c, v);
       }
     }
@@ -643,7 +652,7 @@ extern "C" int mv_moe_residual_norm(void* out, float* x, const void* expert_rows
 }
 
 static int gated_norm(const char* what, bool gate_first, void* out, const void* y, int64_t y_stride, const void* z, int64_t z_stride,
-                      const void* w, int64_t rows, int width, int groups, float eps, int dtype, void* stream) {
+                      const void* w, int64_t rows, int width, int groups, float eps, int dtype, void* stream, mv::HeadNorm hn = {}) {
   using namespace mv;
   int rc = check_norm(what, width, groups, dtype);
   if (rc || rows == 0) return rc;
@@ -657,7 +666,7 @@ static int gated_norm(const char* what, bool gate_first, void* out, const void* 
       if (r) return r;
       kernel<<<static_cast<unsigned>(rows), kNormThreads, smem, static_cast<cudaStream_t>(stream)>>>(
           static_cast<T*>(out), static_cast<const T*>(y), y_stride, static_cast<const T*>(z), z_stride,
-          static_cast<const T*>(w), width, groups, eps);
+          static_cast<const T*>(w), width, groups, eps, hn);
       return check_launch(what);
     };
     const bool v8 = (width / groups) % 8 == 0 && vec8_ok(out, width, eb) && vec8_ok(y, y_stride, eb) && vec8_ok(z, z_stride, eb) &&
@@ -670,7 +679,7 @@ static int gated_norm(const char* what, bool gate_first, void* out, const void* 
         head_norm_gate_kernel<T, L, decltype(ch)::value><<<static_cast<unsigned>(std::min<int64_t>(blocks, kNumSMs * 32)), kNormThreads, 0,
                                                            static_cast<cudaStream_t>(stream)>>>(
             static_cast<T*>(out), static_cast<const T*>(y), y_stride, static_cast<const T*>(z), z_stride, static_cast<const T*>(w),
-            rows, groups, gs, eps);
+            rows, groups, gs, eps, hn);
         return check_launch(what);
       };
       using std::integral_constant;
@@ -692,9 +701,12 @@ extern "C" int mv_gated_group_norm(void* out, const void* y, int64_t y_stride, c
   return gated_norm("gated_group_norm", true, out, y, y_stride, z, z_stride, w, rows, width, groups, eps, dtype, stream);
 }
 
-extern "C" int mv_head_norm_gate(void* out, const void* y, int64_t y_stride, const void* z, int64_t z_stride,
-                                 const void* w, int64_t rows, int width, int heads, float eps, int dtype, void* stream) {
-  return gated_norm("head_norm_gate", false, out, y, y_stride, z, z_stride, w, rows, width, heads, eps, dtype, stream);
+extern "C" int mv_head_norm_gate(void* out, const void* y, int64_t y_stride, const float* den, const void* z, int64_t z_stride,
+                                 const void* w, int full_weight, int act, int64_t rows, int width, int heads, float eps,
+                                 int dtype, void* stream) {
+  if (act != MV_ACT_SILU && act != MV_ACT_SIGMOID) return mv::fail(MV_ERR_SHAPE, "head_norm_gate: activation %d", act);
+  return gated_norm("head_norm_gate", false, out, y, y_stride, z, z_stride, w, rows, width, heads, eps, dtype, stream,
+                    {den, full_weight != 0, act == MV_ACT_SIGMOID});
 }
 
 extern "C" int mv_gate_mul(void* out, const void* y, int64_t y_stride, int64_t y_head_stride, int heads,
@@ -704,7 +716,7 @@ extern "C" int mv_gate_mul(void* out, const void* y, int64_t y_stride, int64_t y
   int rc = check_norm("gate_mul", cols, heads, dtype);
   if (rc || rows == 0) return rc;
   if (!out || !y || !gate) return fail(MV_ERR_NULL, "gate_mul: null pointer");
-  if (act < 0 || act > MV_ACT_CLAMPED) return fail(MV_ERR_SHAPE, "gate_mul: activation %d", act);
+  if (act < 0 || act > MV_ACT_RELU) return fail(MV_ERR_SHAPE, "gate_mul: activation %d", act);
   auto run = [&](auto tag) {
     using T = decltype(tag);
     const int eb = sizeof(T), hc = cols / heads;

@@ -1,8 +1,8 @@
-// Short causal depthwise convolution followed by silu, over a packed batch, with the last inputs of every sequence in
-// slots that the engine assigns.  Sequence s of the batch has tokens cu[s] .. cu[s+1] and `start[s]` tokens behind it;
+// Short causal depthwise convolution over a packed batch, followed by silu or added to its own input, with the last inputs of
+// every sequence in slots that the engine assigns.  Sequence s of the batch has tokens cu[s] .. cu[s+1] and `start[s]` tokens behind it;
 // start 0 means that the slot's contents belong to somebody else and count as zero.
 //
-// conv_silu_kernel      every token and channel of the step (reads the slot, does not change it); conv_silu_vec_kernel
+// conv_kernel           every token and channel of the step (reads the slot, does not change it); conv_vec_kernel
 //                       is the same with eight channels per thread and the taps in registers
 // conv_state_kernel     writes the slot's inputs for the next step
 #include <algorithm>
@@ -12,6 +12,12 @@ namespace mv {
 
 constexpr int kCvThreads = 128;
 constexpr int kCvTokens = 8;    // tokens per CTA
+enum { CV_SILU = 0, CV_ADD = 1 };
+
+// What becomes of a convolution's result; v: the newest input.
+template <typename T, int OP> __device__ __forceinline__ float conv_result(float acc, float v) {
+  return OP == CV_SILU ? silu_t<T>(acc) : acc + v;
+}
 
 // Input of the convolution `back` tokens before token j of the portion (0 before the start of the sequence).
 template <typename T>
@@ -21,9 +27,9 @@ __device__ __forceinline__ float conv_input(const T* u, int64_t u_stride, int64_
   return state && hist + j >= 0 ? Elem<T>::to_f(state[static_cast<int64_t>(hist + j) * channels + c]) : 0.f;
 }
 
-template <typename T>
+template <typename T, int OP>
 __global__ void __launch_bounds__(kCvThreads)
-conv_silu_kernel(T* __restrict__ out, const T* __restrict__ u, int64_t u_stride, const T* __restrict__ w,
+conv_kernel(T* __restrict__ out, const T* __restrict__ u, int64_t u_stride, const T* __restrict__ w,
                  const T* __restrict__ bias, int taps, int channels, const int32_t* __restrict__ cu, int num_seqs,
                  int64_t tokens, const int32_t* __restrict__ slots, const int32_t* __restrict__ start,
                  const T* __restrict__ state, int num_slots) {
@@ -49,14 +55,14 @@ conv_silu_kernel(T* __restrict__ out, const T* __restrict__ u, int64_t u_stride,
     float acc = b;
     for (int k = 0; k < taps; ++k)
       acc = fmaf(Elem<T>::to_f(wc[k]), conv_input(u, u_stride, first, j - hist + k, c, st, hist, channels), acc);
-    out[t * channels + c] = Elem<T>::from_f(silu_t<T>(acc));
+    out[t * channels + c] = Elem<T>::from_f(conv_result<T, OP>(acc, conv_input(u, u_stride, first, j, c, st, hist, channels)));
   }
 }
 
 // Eight channels per thread, up to kCvRun consecutive tokens, the last taps - 1 inputs kept in registers.
-template <typename T, int TAPS>
+template <typename T, int TAPS, int OP>
 __global__ void __launch_bounds__(kCvThreads)
-conv_silu_vec_kernel(T* __restrict__ out, const T* __restrict__ u, int64_t u_stride, const T* __restrict__ w,
+conv_vec_kernel(T* __restrict__ out, const T* __restrict__ u, int64_t u_stride, const T* __restrict__ w,
                      const T* __restrict__ bias, int channels, const int32_t* __restrict__ cu, int num_seqs,
                      int64_t tokens, const int32_t* __restrict__ slots, const int32_t* __restrict__ start,
                      const T* __restrict__ state, int num_slots, int run) {
@@ -119,7 +125,7 @@ conv_silu_vec_kernel(T* __restrict__ out, const T* __restrict__ u, int64_t u_str
           float a = b[e];
 #pragma unroll
           for (int k = 0; k < TAPS; ++k) a = fmaf(wt[k][e], v[n + k][e], a);
-          r[e] = silu_t<T>(a);
+          r[e] = conv_result<T, OP>(a, v[n + HIST][e]);
         }
         Vec<T, 8>::store(out + (t + n) * channels + c, r);
       }
@@ -137,7 +143,7 @@ conv_silu_vec_kernel(T* __restrict__ out, const T* __restrict__ u, int64_t u_str
       float a = b[e];
 #pragma unroll
       for (int k = 0; k < HIST; ++k) a = fmaf(wt[k][e], win[k][e], a);
-      r[e] = silu_t<T>(fmaf(wt[HIST][e], v[e], a));
+      r[e] = conv_result<T, OP>(fmaf(wt[HIST][e], v[e], a), v[e]);
 #pragma unroll
       for (int k = 0; k + 1 < HIST; ++k) win[k][e] = win[k + 1][e];
       win[HIST - 1][e] = v[e];
@@ -176,15 +182,16 @@ static int check_conv(const char* what, int dtype, int num_seqs, int channels, i
   return MV_OK;
 }
 
-extern "C" int mv_conv_silu(void* out, const void* u, int64_t u_stride, const void* w, const void* bias, int taps,
-                            int channels, const int32_t* cu, int num_seqs, int64_t tokens, const int32_t* slots,
-                            const int32_t* start, const void* state, int num_slots, int dtype, void* stream) {
+template <int OP>
+static int run_conv(const char* what, void* out, const void* u, int64_t u_stride, const void* w, const void* bias, int taps,
+                    int channels, const int32_t* cu, int num_seqs, int64_t tokens, const int32_t* slots,
+                    const int32_t* start, const void* state, int num_slots, int dtype, void* stream) {
   using namespace mv;
-  const int rc = check_conv("conv_silu", dtype, num_seqs, channels, taps);
+  const int rc = check_conv(what, dtype, num_seqs, channels, taps);
   if (rc || tokens == 0 || num_seqs == 0) return rc;
-  if (!out || !u || !w || !slots || !start || (taps > 1 && !state)) return fail(MV_ERR_NULL, "conv_silu: null pointer");
+  if (!out || !u || !w || !slots || !start || (taps > 1 && !state)) return fail(MV_ERR_NULL, "%s: null pointer", what);
   const dim3 grid((channels + kCvThreads - 1) / kCvThreads, static_cast<unsigned>((tokens + kCvTokens - 1) / kCvTokens));
-  if (grid.y > 65535) return fail(MV_ERR_LIMIT, "conv_silu: %lld tokens", static_cast<long long>(tokens));
+  if (grid.y > 65535) return fail(MV_ERR_LIMIT, "%s: %lld tokens", what, static_cast<long long>(tokens));
   auto run = [&](auto tag) {
     using T = decltype(tag);
     const int eb = sizeof(T);
@@ -195,16 +202,28 @@ extern "C" int mv_conv_silu(void* out, const void* u, int64_t u_stride, const vo
         kernel<<<vg, kCvThreads, 0, static_cast<cudaStream_t>(stream)>>>(
             static_cast<T*>(out), static_cast<const T*>(u), u_stride, static_cast<const T*>(w), static_cast<const T*>(bias),
             channels, cu, num_seqs, tokens, slots, start, static_cast<const T*>(state), num_slots, len);
-        return check_launch("conv_silu");
+        return check_launch(what);
       };
-      return taps == 2 ? go(conv_silu_vec_kernel<T, 2>) : taps == 3 ? go(conv_silu_vec_kernel<T, 3>) : go(conv_silu_vec_kernel<T, 4>);
+      return taps == 2 ? go(conv_vec_kernel<T, 2, OP>) : taps == 3 ? go(conv_vec_kernel<T, 3, OP>) : go(conv_vec_kernel<T, 4, OP>);
     }
-    conv_silu_kernel<T><<<grid, kCvThreads, 0, static_cast<cudaStream_t>(stream)>>>(
+    conv_kernel<T, OP><<<grid, kCvThreads, 0, static_cast<cudaStream_t>(stream)>>>(
         static_cast<T*>(out), static_cast<const T*>(u), u_stride, static_cast<const T*>(w), static_cast<const T*>(bias),
         taps, channels, cu, num_seqs, tokens, slots, start, static_cast<const T*>(state), num_slots);
-    return check_launch("conv_silu");
+    return check_launch(what);
   };
   return dtype == MV_F32 ? run(float{}) : run(__nv_bfloat16{});
+}
+
+extern "C" int mv_conv_silu(void* out, const void* u, int64_t u_stride, const void* w, const void* bias, int taps,
+                            int channels, const int32_t* cu, int num_seqs, int64_t tokens, const int32_t* slots,
+                            const int32_t* start, const void* state, int num_slots, int dtype, void* stream) {
+  return run_conv<mv::CV_SILU>("conv_silu", out, u, u_stride, w, bias, taps, channels, cu, num_seqs, tokens, slots, start, state, num_slots, dtype, stream);
+}
+
+extern "C" int mv_conv_add(void* out, const void* u, int64_t u_stride, const void* w, const void* bias, int taps,
+                           int channels, const int32_t* cu, int num_seqs, int64_t tokens, const int32_t* slots,
+                           const int32_t* start, const void* state, int num_slots, int dtype, void* stream) {
+  return run_conv<mv::CV_ADD>("conv_add", out, u, u_stride, w, bias, taps, channels, cu, num_seqs, tokens, slots, start, state, num_slots, dtype, stream);
 }
 
 extern "C" int mv_conv_state_update(void* state, const void* u, int64_t u_stride, int taps, int channels,

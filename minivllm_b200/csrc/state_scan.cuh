@@ -1,6 +1,8 @@
 // Recurrences on a matrix state S (K x V, fp32) per sequence and head, read out once per token:
 //   gated linear attention   S <- diag(alpha) S + k v^T,                             o = S^T q
 //   gated delta rule         S <- g S;  u = beta (v - S^T k);  S <- S + k u^T,       o = S^T q
+//   matrix memory (mLSTM)    S <- alpha S + w k v^T;  n <- alpha n + w k,            o = S^T q / (max(|n . q|, e^-m') + 1e-6)
+//     with alpha = e^(f + m - m'), w = e^(i - m'), m' = max(f + m, i) the running maximum of the gates' logarithms
 // Everything is computed in 32-bit, token by token, with the state in registers, so a result does not depend on how a
 // prompt is cut.
 //
@@ -18,6 +20,8 @@
 // scan_kernel   prompts: one CTA per (sequence, head, block of value columns).  While a tile of tokens is worked on,
 //               each warp has the next tile's token of its own in registers; it turns it into what the recurrence wants
 //               (unit norms, decays, step sizes) in shared memory at the end of the tile.
+//               Matrix memory: the chain of maxima comes from mlstm.cu; the first warp of the first block of columns keeps n
+//               and leaves the denominators to the norm that follows.
 // step_quad_kernel, step_kernel (vdim not a multiple of four)
 //               one token per sequence: convolution (delta rule), one step of the state, the head's norm and the output
 //               gate in one launch.  HBM-bound: 8 * heads * K * V bytes per sequence.
@@ -28,7 +32,7 @@
 
 namespace mv {
 
-enum { SK_GLA = 0, SK_DELTA = 1 };
+enum { SK_GLA = 0, SK_DELTA = 1, SK_MLSTM = 2 };
 
 constexpr int log2_c(int n) { return n <= 1 ? 0 : 1 + log2_c(n / 2); }
 
@@ -228,8 +232,8 @@ template <int KIND, typename F> int scan_dispatch(int K, F&& f) {
   if (K <= 64) return f(ScanShape<KIND, 8, 8, 8>{});
   if (K <= 96) return f(ScanShape<KIND, 8, 12, 4>{});
   if (K <= 128) {
-    if constexpr (KIND == SK_GLA) return f(ScanShape<KIND, 16, 8, 8>{});
-    else return f(ScanShape<KIND, 8, 16, 4>{});
+    if constexpr (KIND == SK_DELTA) return f(ScanShape<KIND, 8, 16, 4>{});
+    else return f(ScanShape<KIND, 16, 8, 8>{});
   }
   return f(ScanShape<KIND, 16, 16, 4>{});
 }
@@ -239,6 +243,11 @@ constexpr int kScanMaxK = 256;
 __device__ __forceinline__ float channel_log_decay(float z, float inv_tau) { return -softplus_f(-z) * inv_tau; }
 __device__ __forceinline__ float head_log_decay(float a, float A_log, float dt_bias) { return -expf(A_log) * softplus_f(a + dt_bias); }
 constexpr float kUnitEps = 1e-6f;       // of q and k scaled to unit length
+constexpr float kMemFloor = 1e-6f;      // matrix memory: added to the denominator
+
+// Matrix memory: logarithms of the input and the forget gate from their logits.
+__device__ __forceinline__ float mem_log_input(float z, float cap) { return cap * tanhf(z / cap); }
+__device__ __forceinline__ float mem_log_forget(float z, float cap) { return -softplus_f(-cap * tanhf(z / cap)); }
 
 constexpr int kScanMaxWarps = 8, kScanCols = 128;      // columns per CTA at most
 
@@ -249,6 +258,10 @@ template <typename T> struct ScanParams {
   float inv_tau;
   const T *beta, *a; int64_t gate_stride;              // delta rule: (heads) logits of the step size and of the decay
   const T *A_log, *dt_bias;
+  const float* gates; int64_t gates_stride;            // matrix memory: (heads) logits of the input gate, (heads) of the forget gate
+  const T *i_b, *f_b; float cap;
+  float *n_state, *m_state;                            //   (num_slots, heads, K), (num_slots, heads)
+  const float4* chain; float* den;                     //   prompts: (tokens, heads) i, f, m, m' and denominators
   const int32_t *cu, *slots, *start;
   float* state; int num_slots, heads, kv_heads, K, V;
   float q_scale;
@@ -259,7 +272,7 @@ template <typename T> struct ScanParams {
 
 template <typename Sh, typename T, int W>
 __global__ void __launch_bounds__(32 * W, 16 / W) scan_kernel(const ScanParams<T> p, int cols_cta) {
-  constexpr bool kDelta = Sh::KIND == SK_DELTA;
+  constexpr bool kDelta = Sh::KIND == SK_DELTA, kMem = Sh::KIND == SK_MLSTM;
   constexpr int K = Sh::K, KL = K / 32, VL = kScanCols / 32, TT = W;      // a tile: one token per warp
   constexpr int VEC = kDelta ? 2 : 3;
   extern __shared__ __align__(16) float sm[];
@@ -280,7 +293,15 @@ __global__ void __launch_bounds__(32 * W, 16 / W) scan_kernel(const ScanParams<T
   if (work && live && st0 > 0) S.load(gS, kp, p.K, p.V, pw - c0, vec);
   else S.zero();
 
-  T rk[KL], rq[KL], rz[kDelta ? 1 : KL], rv[VL], rb[2];
+  T rk[KL], rq[KL], rz[kDelta || kMem ? 1 : KL], rv[VL], rb[2];
+  float4 rc = make_float4(0.f, 0.f, 0.f, 0.f);
+  float n[kMem ? KL : 1];                // matrix memory: this lane's entries of n
+  const bool keeps_n = kMem && blockIdx.z == 0 && warp == 0;
+  float* gN = kMem ? p.n_state + (static_cast<int64_t>(live ? slot : 0) * p.heads + h) * p.K : nullptr;
+  if constexpr (kMem) {
+#pragma unroll
+    for (int m = 0; m < KL; ++m) n[m] = keeps_n && live && st0 > 0 && m * 32 + lane < p.K ? gN[m * 32 + lane] : 0.f;
+  }
   float A_log = 0.f, dt_bias = 0.f;
   if (kDelta) {
     A_log = Elem<T>::to_f(p.A_log[h]);
@@ -296,13 +317,14 @@ __global__ void __launch_bounds__(32 * W, 16 / W) scan_kernel(const ScanParams<T
       const bool ok = on && j < p.K;
       rk[m] = ok ? p.k[row * p.stride + kh * p.K + j] : zero_t;
       rq[m] = ok ? p.q[row * p.stride + kh * p.K + j] : zero_t;
-      if (!kDelta) rz[m] = ok ? p.z[row * p.z_stride + h * p.K + j] : zero_t;
+      if constexpr (!kDelta && !kMem) rz[m] = ok ? p.z[row * p.z_stride + h * p.K + j] : zero_t;
     }
 #pragma unroll
     for (int m = 0; m < VL; ++m) {
       const int j = m * 32 + lane;
       rv[m] = on && j < pw ? p.v[row * p.stride + static_cast<int64_t>(h) * p.V + p0 + j] : zero_t;
     }
+    if (kMem && on) rc = p.chain[row * p.heads + h];
     if (kDelta) {
       rb[0] = on ? p.beta[row * p.gate_stride + h] : zero_t;
       rb[1] = on ? p.a[row * p.gate_stride + h] : zero_t;
@@ -311,16 +333,22 @@ __global__ void __launch_bounds__(32 * W, 16 / W) scan_kernel(const ScanParams<T
   auto prepare = [&](int buf) {
     float* vecs = s_vec + (buf * TT + warp) * VEC * K;
     float kk = 0.f, qq = 0.f, kq = 0.f;
+    const float alpha_m1 = kMem ? expm1f(rc.y + rc.z - rc.w) : 0.f, write = kMem ? expf(rc.x - rc.w) : 0.f;
+    if (kMem && lane == 0) s_par[(buf * TT + warp) * 4] = expf(-rc.w);
 #pragma unroll
     for (int m = 0; m < KL; ++m) {
       const int j = m * 32 + lane;
       const float kf = Elem<T>::to_f(rk[m]), qf = Elem<T>::to_f(rq[m]);
-      if (kDelta) {
+      if constexpr (kDelta) {
         kk = fmaf(kf, kf, kk);
         qq = fmaf(qf, qf, qq);
         kq = fmaf(kf, qf, kq);
         vecs[j] = kf;
         vecs[K + j] = qf;
+      } else if constexpr (kMem) {
+        vecs[j] = kf * write;
+        vecs[K + j] = qf * p.q_scale;
+        vecs[2 * K + j] = alpha_m1;
       } else {
         vecs[j] = kf;
         vecs[K + j] = qf * p.q_scale;
@@ -372,20 +400,61 @@ __global__ void __launch_bounds__(32 * W, 16 / W) scan_kernel(const ScanParams<T
         for (int j = 0; j < Sh::HELD; ++j)
           if (j < held) out[j] = Elem<T>::from_f(o[j]);
         out += p.out_stride;
+        if constexpr (kMem) {
+          if (!keeps_n) continue;
+          float dot = 0.f;
+#pragma unroll
+          for (int m = 0; m < KL; ++m) {
+            const int j = m * 32 + lane;
+            n[m] = fmaf(vecs[2 * K], n[m], n[m]) + vecs[j];
+            dot = fmaf(n[m], vecs[K + j], dot);
+          }
+          dot = warp_sum(dot);
+          if (lane == 0)
+            p.den[static_cast<int64_t>(first + t0 + t) * p.heads + h] = fmaxf(fabsf(dot), s_par[(buf * TT + t) * 4]) + kMemFloor;
+        }
       }
     }
     if (more) prepare(buf ^ 1);
     __syncthreads();
   }
   if (live && work) S.store(gS, kp, p.K, p.V, pw - c0, vec);
+  if constexpr (kMem) {
+    if (keeps_n && live)
+#pragma unroll
+      for (int m = 0; m < KL; ++m)
+        if (m * 32 + lane < p.K) gN[m * 32 + lane] = n[m];
+  }
+}
+
+// Matrix memory: factors of the old state and of the new entry of a token, and its running maximum.  Every thread for itself.
+struct MemFactors { float alpha_m1, write, m; };
+template <typename T> __device__ __forceinline__ MemFactors mem_factors(const ScanParams<T>& p, int s, int h, int slot, int st0) {
+  const float* z = p.gates + static_cast<int64_t>(s) * p.gates_stride + h;
+  const float i = mem_log_input(z[0] + Elem<T>::to_f(p.i_b[h]), p.cap), f = mem_log_forget(z[p.heads] + Elem<T>::to_f(p.f_b[h]), p.cap);
+  const float old = st0 > 0 ? p.m_state[static_cast<int64_t>(slot) * p.heads + h] : 0.f;
+  const float m = fmaxf(f + old, i);
+  return {expm1f(f + old - m), expf(i - m), m};
+}
+// The state's n and m one token on, and the terms of n . q; between two barriers.
+template <typename T>
+__device__ __forceinline__ void mem_advance(const ScanParams<T>& p, int h, int slot, int st0, const MemFactors& f, const float* s_k,
+                                            const float* s_q, float* s_nq) {
+  float* gN = p.n_state + (static_cast<int64_t>(slot) * p.heads + h) * p.K;
+  for (int j = threadIdx.x; j < p.K; j += blockDim.x) {
+    const float old = st0 > 0 ? gN[j] : 0.f, n = fmaf(f.alpha_m1, old, old) + s_k[j];
+    gN[j] = n;
+    s_nq[j] = n * s_q[j];
+  }
+  if (threadIdx.x == 0) p.m_state[static_cast<int64_t>(slot) * p.heads + h] = f.m;
 }
 
 // The vectors of a token for the step kernels: K (padded) values of k and q, gated linear attention's alpha - 1, V (padded)
-// values of v; the delta rule's go through the convolution.
+// values of v; the delta rule's go through the convolution, matrix memory's k takes its factor.
 template <int KIND, typename T>
 __device__ __forceinline__ void step_vectors(const ScanParams<T>& p, int s, int h, int slot, int st0, int K, int vpad, float* s_k,
-                                             float* s_q, float* s_a, float* s_v) {
-  constexpr bool kDelta = KIND == SK_DELTA;
+                                             float* s_q, float* s_a, float* s_v, const MemFactors& mem) {
+  constexpr bool kDelta = KIND == SK_DELTA, kMem = KIND == SK_MLSTM;
   const int kh = h / (p.heads / p.kv_heads);
   for (int i = threadIdx.x; i < K + K + vpad; i += blockDim.x) {
     const int part = i < K ? 0 : i < 2 * K ? 1 : 2, j = part == 0 ? i : part == 1 ? i - K : i - 2 * K;
@@ -406,10 +475,13 @@ __device__ __forceinline__ void step_vectors(const ScanParams<T>& p, int s, int 
         x = Elem<T>::to_f(Elem<T>::from_f(silu_t<T>(acc)));       // rounded as the prompt path stores it
       } else if (part == 1) {
         x *= p.q_scale;
+      } else if (kMem && part == 0) {
+        x *= mem.write;
       }
     }
     (part == 0 ? s_k : part == 1 ? s_q : s_v)[j] = x;
-    if (!kDelta && part == 0)
+    if (kMem && part == 0) s_a[j] = mem.alpha_m1;
+    if (!kDelta && !kMem && part == 0)
       s_a[j] = ok ? expm1f(channel_log_decay(Elem<T>::to_f(p.z[static_cast<int64_t>(s) * p.z_stride + h * p.K + j]), p.inv_tau)) : 0.f;
   }
 }
@@ -435,25 +507,36 @@ __device__ __forceinline__ StepFactors step_factors(const ScanParams<T>& p, int 
   return f;
 }
 
-// Norm of the head's read-out and output gate.
-template <typename T>
-__device__ __forceinline__ void step_output(const ScanParams<T>& p, int s, int h, const float* s_o, T* out) {
+// Norm of the head's read-out and output gate; matrix memory divides first (s_nq: the terms of n . q).
+template <int KIND, typename T>
+__device__ __forceinline__ void step_output(const ScanParams<T>& p, int s, int h, const float* s_o, T* out, const float* s_nq,
+                                            const MemFactors& mem) {
+  constexpr bool kMem = KIND == SK_MLSTM;
+  float inv = 1.f;
+  if (kMem) {
+    float dot = 0.f;
+    for (int j = threadIdx.x & 31; j < p.K; j += 32) dot += s_nq[j];
+    inv = 1.f / (fmaxf(fabsf(warp_sum(dot)), expf(-mem.m)) + kMemFloor);
+  }
   float acc = 0.f;
-  for (int j = threadIdx.x & 31; j < p.V; j += 32) acc = fmaf(s_o[j], s_o[j], acc);
-  const float rs = 1.f / sqrtf(warp_sum(acc) / static_cast<float>(p.V) + p.eps);
+  for (int j = threadIdx.x & 31; j < p.V; j += 32) acc = fmaf(s_o[j] * inv, s_o[j] * inv, acc);
+  const float rs = inv / sqrtf(warp_sum(acc) / static_cast<float>(p.V) + p.eps);
   const T* gate = p.gate + static_cast<int64_t>(s) * p.out_gate_stride + static_cast<int64_t>(h) * p.V;
-  for (int j = threadIdx.x; j < p.V; j += blockDim.x)
-    out[j] = Elem<T>::from_f(s_o[j] * rs * Elem<T>::to_f(p.norm_w[j]) * silu_t<T>(Elem<T>::to_f(gate[j])));
+  const T* w = p.norm_w + (kMem ? static_cast<int64_t>(h) * p.V : 0);
+  for (int j = threadIdx.x; j < p.V; j += blockDim.x) {
+    const float g = Elem<T>::to_f(gate[j]);
+    out[j] = Elem<T>::from_f(s_o[j] * rs * Elem<T>::to_f(w[j]) * (kMem ? sigmoid_t<T>(g) : silu_t<T>(g)));
+  }
 }
 
 // Any sizes: the state in the prompt kernel's layout.
 template <typename Sh, typename T>
 __global__ void __launch_bounds__(256, 1) step_kernel(const ScanParams<T> p) {
-  constexpr bool kDelta = Sh::KIND == SK_DELTA;
+  constexpr bool kDelta = Sh::KIND == SK_DELTA, kMem = Sh::KIND == SK_MLSTM;
   constexpr int K = Sh::K;
   extern __shared__ __align__(16) float sm[];
   const int vpad = (p.V + Sh::CW - 1) / Sh::CW * Sh::CW;
-  float *s_k = sm, *s_q = s_k + K, *s_a = s_q + K, *s_v = s_a + (kDelta ? 0 : K), *s_o = s_v + vpad;
+  float *s_k = sm, *s_q = s_k + K, *s_a = s_q + K, *s_v = s_a + (kDelta ? 0 : K), *s_o = s_v + vpad, *s_nq = s_o + vpad;
   const int s = blockIdx.x, h = blockIdx.y, tid = threadIdx.x;
   const int warp = tid >> 5, lane = tid & 31, kp = lane & (Sh::KP - 1), vp = lane / Sh::KP, warps = blockDim.x >> 5;
   const int slot = p.slots[s], st0 = p.start[s];
@@ -464,8 +547,11 @@ __global__ void __launch_bounds__(256, 1) step_kernel(const ScanParams<T> p) {
   }
   const bool vec = p.V % 4 == 0;
   float* gS = p.state + (static_cast<int64_t>(slot) * p.heads + h) * p.K * p.V;
-  step_vectors<Sh::KIND>(p, s, h, slot, st0, K, vpad, s_k, s_q, s_a, s_v);
+  MemFactors mem{};
+  if constexpr (kMem) mem = mem_factors(p, s, h, slot, st0);
+  step_vectors<Sh::KIND>(p, s, h, slot, st0, K, vpad, s_k, s_q, s_a, s_v, mem);
   __syncthreads();
+  if constexpr (kMem) mem_advance(p, h, slot, st0, mem, s_k, s_q, s_nq);
   StepFactors f{};
   if (kDelta) f = step_factors(p, s, h, K, s_k, s_q);
   const bool writes = (!kDelta || (kp & (Sh::KP / 2))) && (kp & (Sh::LOW - 1)) == 0;
@@ -483,7 +569,7 @@ __global__ void __launch_bounds__(256, 1) step_kernel(const ScanParams<T> p) {
     S.store(gS + c0, kp, p.K, p.V, p.V - c0, vec);
   }
   __syncthreads();
-  step_output(p, s, h, s_o, out);
+  step_output<Sh::KIND>(p, s, h, s_o, out, s_nq, mem);
 }
 
 // vdim a multiple of four: a thread has four columns of every rows-th row of S, so that a warp reads whole lines, and the
@@ -492,13 +578,14 @@ __global__ void __launch_bounds__(256, 1) step_kernel(const ScanParams<T> p) {
 constexpr int kStHold = 8, kStThreads4 = 512;
 template <int KIND, typename T>
 __global__ void __launch_bounds__(kStThreads4, 2) step_quad_kernel(const ScanParams<T> p, int vpad) {
-  constexpr bool kDelta = KIND == SK_DELTA;
+  constexpr bool kDelta = KIND == SK_DELTA, kMem = KIND == SK_MLSTM;
   extern __shared__ __align__(16) float sm[];
   const int K = (p.K + 3) & ~3, nthr = blockDim.x, tid = threadIdx.x, s = blockIdx.x, h = blockIdx.y;
   const int PQ = p.V / 4, rows = nthr / PQ, q = tid % PQ, r = tid / PQ;
   const bool on = r < rows;
   float *s_k = sm, *s_q = s_k + K, *s_a = s_q + K, *s_v = s_a + (kDelta ? 0 : K), *s_o = s_v + vpad;
-  float4* red = reinterpret_cast<float4*>(s_o + vpad);           // [rows][PQ], twice for the delta rule
+  float* s_nq = s_o + vpad;                                      // matrix memory
+  float4* red = reinterpret_cast<float4*>(s_nq + (kMem ? K : 0));        // [rows][PQ], twice for the delta rule
   const int slot = p.slots[s], st0 = p.start[s];
   T* out = p.out + static_cast<int64_t>(s) * p.out_stride + static_cast<int64_t>(h) * p.V;
   if (slot < 0 || slot >= p.num_slots || st0 < 0) {
@@ -516,8 +603,11 @@ __global__ void __launch_bounds__(kStThreads4, 2) step_quad_kernel(const ScanPar
     }
   };
   fetch(0);                              // in flight while the vectors are made
-  step_vectors<KIND>(p, s, h, slot, st0, K, vpad, s_k, s_q, s_a, s_v);
+  MemFactors mem{};
+  if constexpr (kMem) mem = mem_factors(p, s, h, slot, st0);
+  step_vectors<KIND>(p, s, h, slot, st0, K, vpad, s_k, s_q, s_a, s_v, mem);
   __syncthreads();
+  if constexpr (kMem) mem_advance(p, h, slot, st0, mem, s_k, s_q, s_nq);
   const float4 v = on ? *reinterpret_cast<const float4*>(s_v + q * 4) : zero;
   float4 aq = zero, ak = zero;
   auto add = [](float w, const float4& y, float4& acc) {
@@ -599,7 +689,7 @@ __global__ void __launch_bounds__(kStThreads4, 2) step_quad_kernel(const ScanPar
     }
   }
   __syncthreads();
-  step_output(p, s, h, s_o, out);
+  step_output<KIND>(p, s, h, s_o, out, s_nq, mem);
 }
 
 template <typename Sh, typename T, int W>
@@ -628,7 +718,7 @@ template <int KIND, typename T> static int run_step(const ScanParams<T>& p, int 
     const int quads = p.V / 4, K = (p.K + 3) & ~3;
     const int threads = std::min(kStThreads4, std::max(128, (quads * ((p.K + kStHold - 1) / kStHold) + 31) / 32 * 32));
     const int fit = std::max(threads, (quads + 31) / 32 * 32), rows = fit / quads;
-    const size_t smem = sizeof(float) * ((KIND == SK_DELTA ? 2 : 3) * K + 2 * p.V + (KIND == SK_DELTA ? 2 : 1) * static_cast<size_t>(rows) * p.V);
+    const size_t smem = sizeof(float) * ((KIND == SK_DELTA ? 2 : KIND == SK_GLA ? 3 : 4) * K + 2 * p.V + (KIND == SK_DELTA ? 2 : 1) * static_cast<size_t>(rows) * p.V);
     if (smem <= 48 * 1024) {
       step_quad_kernel<KIND, T><<<dim3(num_seqs, p.heads), fit, smem, st>>>(p, p.V);
       return check_launch("state_step");
@@ -637,7 +727,7 @@ template <int KIND, typename T> static int run_step(const ScanParams<T>& p, int 
   return scan_dispatch<KIND>(p.K, [&](auto sh) {
     using Sh = decltype(sh);
     const int blocks = (p.V + Sh::CW - 1) / Sh::CW, warps = std::min(8, blocks);
-    const size_t smem = sizeof(float) * ((KIND == SK_DELTA ? 2 : 3) * Sh::K + 2 * static_cast<size_t>(blocks) * Sh::CW);
+    const size_t smem = sizeof(float) * ((KIND == SK_DELTA ? 2 : KIND == SK_GLA ? 3 : 4) * Sh::K + 2 * static_cast<size_t>(blocks) * Sh::CW);
     if (smem > 48 * 1024) return fail(MV_ERR_LIMIT, "state_step: vdim %d", p.V);
     step_kernel<Sh, T><<<dim3(num_seqs, p.heads), 32 * warps, smem, st>>>(p);
     return check_launch("state_step");

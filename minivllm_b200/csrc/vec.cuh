@@ -82,6 +82,7 @@ template <typename T> __device__ __forceinline__ float glu_act(int act, float g,
   if (act == MV_ACT_SIGMOID) return sigmoid_t<T>(g) * u;
   if (act == MV_ACT_GELU_TANH)       // 0.5 (1 + tanh(a)) = sigmoid(2 a)
     return g * sigmoid_t<T>(1.5957691216057308f * fmaf(0.044715f * g * g, g, g)) * u;
+  if (act == MV_ACT_RELU) return fmaxf(g, 0.f) * u;
   g = fminf(g, limit);
   return g * sigmoid_t<T>(1.702f * g) * (fminf(fmaxf(u, -limit), limit) + 1.f);
 }

@@ -1,9 +1,11 @@
 // Grouped-query attention with a sliding window, a learned bias per distance and head, and a sink per head, over a paged
 // cache of rows [keys of all KV heads | values of all KV heads] (key and value sizes may differ).  Position i sees the
 // keys j with 0 <= i - j < window; score = scale (q . k) + bias[h][min(i - j, distances - 1)]; exp(sink[h]) joins the
-// denominator.  Bias and sink may be absent.
+// denominator.  Bias and sink may be absent.  With a rotation table the result of position i is turned by -i in pairs of
+// neighbouring columns (values that were turned by their own positions when they were stored).
 //
 // kv_norm_store_kernel        RMS norm over all query rows and over all key rows of a token, scatter of [k | v]
+// qkv_rope_store_kernel       RMS norm and rotation per query and key head, rotation of the values, scatter of [k | v]
 // window_attention_rows_kernel  any sizes, bf16 or fp32, token by token
 // window_decode_kernel        one token per sequence on mma.sync: HBM-bound on the rows inside the window
 // Portions of prompts run on tcgen05 in latent_prefill.cu.
@@ -87,6 +89,117 @@ kv_norm_store_kernel(T* __restrict__ q, const T* __restrict__ k, const T* __rest
   }
 }
 
+// Row of a rotation table; padding rows have positions below zero.
+__device__ __forceinline__ int64_t table_row(int64_t pos, int64_t rows) { return min(max(pos, static_cast<int64_t>(0)), rows - 1); }
+
+// The pairs of neighbouring columns c .. c + V - 1 of a row of `dims` rotated columns, turned by the table's angles.
+template <int V>
+__device__ __forceinline__ void turn_pairs(float (&x)[V], int c, int dims, const float* __restrict__ cos_row, const float* __restrict__ sin_row) {
+#pragma unroll
+  for (int e = 0; e < V; e += 2) {
+    if (c + e >= dims) return;
+    const float co = cos_row[(c + e) / 2], si = sin_row[(c + e) / 2], a = x[e], b = x[e + 1];
+    x[e] = a * co - b * si;
+    x[e + 1] = b * co + a * si;
+  }
+}
+// A pair turned by the opposite angle.
+__device__ __forceinline__ void turn_back(float& a, float& b, float co, float si) {
+  const float x = fmaf(a, co, b * si);
+  b = fmaf(b, co, -a * si);
+  a = x;
+}
+
+template <typename T> struct RopeStoreParams {
+  T *q; const T *k, *v; int64_t stride;        // (tokens, heads * dim), (tokens, kv_heads * dim), (tokens, kv_heads * vdim)
+  const T *q_weight, *k_weight, *temp;         // (dim), (dim), (heads) or null
+  const float *cos_t, *sin_t; int dims;        // (table_rows, dims / 2)
+  const float *vcos_t, *vsin_t;                // (table_rows, vdim / 2), null: values are stored as they are
+  int64_t table_rows;
+  const int64_t* positions;
+  T *kv_out, *cache; const int64_t* slot_mapping; int64_t num_slots;
+  int64_t tokens;
+  int heads, kv_heads, dim, vdim;
+  float eps;
+};
+
+// L lanes (a power of two) per head of a token, kCh pieces of V (8, or 2 for any sizes) columns per lane.  Items of a token: query heads, key heads,
+// value heads.
+template <typename T, int V, int L, int kCh>
+__global__ void __launch_bounds__(kKnThreads) qkv_rope_store_kernel(const RopeStoreParams<T> p) {
+  const int lane = threadIdx.x & (L - 1), per = p.heads + 2 * p.kv_heads, row = p.kv_heads * (p.dim + p.vdim);
+  const int64_t items = p.tokens * per, step = static_cast<int64_t>(gridDim.x) * (kKnThreads / L);
+  for (int64_t i0 = static_cast<int64_t>(blockIdx.x) * (kKnThreads / L); i0 < items; i0 += step) {
+    const int64_t i = i0 + threadIdx.x / L;
+    const bool on = i < items;                 // lanes of a warp stay together for the sums
+    const int64_t t = on ? i / per : 0;
+    const int item = on ? static_cast<int>(i - t * per) : 0;
+    const bool is_q = item < p.heads, is_v = item >= p.heads + p.kv_heads;
+    const int head = is_q ? item : is_v ? item - p.heads - p.kv_heads : item - p.heads, n = is_v ? p.vdim : p.dim;
+    const T* src = is_q ? p.q : is_v ? p.v : p.k;
+    src += t * p.stride + static_cast<int64_t>(head) * n;
+    const int64_t pos = table_row(p.positions[t], p.table_rows);
+    float x[kCh][V], acc = 0.f;
+#pragma unroll
+    for (int k = 0; k < kCh; ++k) {
+      const int c = (k * L + lane) * V;
+      if (on && c < n) {
+        if constexpr (V == 8) {
+          Vec<T, V>::load(src + c, x[k]);
+        } else {
+          x[k][0] = Elem<T>::to_f(src[c]);
+          x[k][1] = c + 1 < n ? Elem<T>::to_f(src[c + 1]) : 0.f;
+        }
+#pragma unroll
+        for (int e = 0; e < V; ++e) acc = fmaf(x[k][e], x[k][e], acc);
+      }
+    }
+#pragma unroll
+    for (int o = L / 2; o; o >>= 1) acc += __shfl_xor_sync(0xffffffffu, acc, o);
+    const float rs = is_v ? 1.f : 1.f / sqrtf(acc / static_cast<float>(n) + p.eps);
+    const T* weight = is_q ? p.q_weight : p.k_weight;
+    const float f = is_q && p.temp && on ? Elem<T>::to_f(p.temp[head]) : 1.f;
+    const float* co = is_v ? p.vcos_t : p.cos_t;
+    const float* si = is_v ? p.vsin_t : p.sin_t;
+    const int dims = is_v ? (co ? p.vdim : 0) : p.dims;
+    T *d0 = nullptr, *d1 = nullptr;
+    if (is_q) {
+      d0 = p.q + t * p.stride + static_cast<int64_t>(head) * n;
+    } else {
+      const int64_t at = is_v ? static_cast<int64_t>(p.kv_heads) * p.dim + static_cast<int64_t>(head) * n : static_cast<int64_t>(head) * n;
+      if (p.kv_out) d0 = p.kv_out + t * row + at;
+      if (p.cache) {
+        const int64_t slot = p.slot_mapping[t];
+        if (slot >= 0 && slot < p.num_slots) d1 = p.cache + slot * row + at;
+      }
+    }
+#pragma unroll
+    for (int k = 0; k < kCh; ++k) {
+      const int c = (k * L + lane) * V;
+      if (!on || c >= n) continue;
+      if (!is_v) {
+#pragma unroll
+        for (int e = 0; e < V; ++e)
+          if (V == 8 || c + e < n) x[k][e] = x[k][e] * rs * Elem<T>::to_f(weight[c + e]);
+      }
+      turn_pairs<V>(x[k], c, dims, co + pos * (dims / 2), si + pos * (dims / 2));
+#pragma unroll
+      for (int e = 0; e < V; ++e) x[k][e] *= f;
+#pragma unroll
+      for (int w = 0; w < 2; ++w) {
+        T* d = w == 0 ? d0 : d1;
+        if (!d) continue;
+        if constexpr (V == 8) {
+          Vec<T, V>::store(d + c, x[k]);
+        } else {
+          d[c] = Elem<T>::from_f(x[k][0]);
+          if (c + 1 < n) d[c + 1] = Elem<T>::from_f(x[k][1]);
+        }
+      }
+    }
+  }
+}
+
 template <typename T> struct WindowParams {
   T* out;                                    // (tokens, heads * vdim)
   const T* q; int64_t q_stride;              // (tokens, heads * dim)
@@ -99,6 +212,7 @@ template <typename T> struct WindowParams {
   int heads, kv_heads, dim, vdim;
   int64_t window;
   float scale;
+  const float *cos_t, *sin_t; int64_t table_rows;              // (table_rows, vdim / 2): results are turned back; null: not
   // decode
   int splits;
   float *part_ml, *part_o;                   // (batch, splits, heads, 2) and (.., vdim)
@@ -197,6 +311,7 @@ __global__ void __launch_bounds__(kWaThreads) window_attention_rows_kernel(const
     }
   }
   __syncthreads();
+  const int64_t turn = p.cos_t ? table_row(pos, p.table_rows) * (VD / 2) : 0;
 #pragma unroll
   for (int h = 0; h < kWaHeads; ++h) {
     if (h >= nh) break;
@@ -204,6 +319,13 @@ __global__ void __launch_bounds__(kWaThreads) window_attention_rows_kernel(const
 #pragma unroll
     for (int i = 0; i < kWaPer; ++i) {
       const int d = tid + i * kWaThreads;
+      if (p.cos_t && i * kWaThreads < VD) {      // the other column of the pair is the neighbouring thread's
+        const float other = __shfl_xor_sync(0xffffffffu, acc[h][i], 1);
+        if (d < VD) {
+          const float co = p.cos_t[turn + d / 2], si = p.sin_t[turn + d / 2];
+          acc[h][i] = fmaf(acc[h][i], co, d & 1 ? -other * si : other * si);
+        }
+      }
       if (d < VD) p.out[(static_cast<int64_t>(t) * p.heads + h0 + h) * VD + d] = Elem<T>::from_f(acc[h][i] * inv);
     }
   }
@@ -414,25 +536,34 @@ window_decode_kernel(const WindowParams<__nv_bfloat16> p) {
     }
   }
   __syncthreads();
-  for (int i = tid; i < rows * p.vdim; i += kWdThreads) {
-    const int r = i / p.vdim, d = i - r * p.vdim, h = h0 + r;
+  const int half = p.vdim / 2;           // a thread has pairs of neighbouring columns
+  const int64_t turn = p.cos_t ? table_row(pos64, p.table_rows) * half : 0;
+  for (int i = tid; i < rows * half; i += kWdThreads) {
+    const int r = i / half, d = (i - r * half) * 2, h = h0 + r;
     float M = kWdNeg;
 #pragma unroll
     for (int w = 0; w < kWdWarps; ++w) M = fmaxf(M, sML[(w * 16 + r) * 2]);
     const float sk = p.sink ? __bfloat162float(p.sink[h]) * 1.4426950408889634f : kWdNeg;
     if (p.splits == 1 && p.sink) M = fmaxf(M, sk);
-    float acc = 0.f, L = p.splits == 1 && p.sink ? fast_exp2(sk - M) : 0.f;
+    float2 acc = make_float2(0.f, 0.f);
+    float L = p.splits == 1 && p.sink ? fast_exp2(sk - M) : 0.f;
 #pragma unroll
     for (int w = 0; w < kWdWarps; ++w) {
       const float f = fast_exp2(sML[(w * 16 + r) * 2] - M);
-      acc = fmaf(f, sO[(w * 16 + r) * S::kStride + d], acc);
+      const float2 o2 = *reinterpret_cast<const float2*>(sO + (w * 16 + r) * S::kStride + d);
+      acc.x = fmaf(f, o2.x, acc.x);
+      acc.y = fmaf(f, o2.y, acc.y);
       L = fmaf(f, sML[(w * 16 + r) * 2 + 1], L);
     }
     if (p.splits == 1) {
-      p.out[(static_cast<int64_t>(b) * p.heads + h) * p.vdim + d] = __float2bfloat16_rn(L > 0.f ? acc / L : 0.f);
+      const float inv = L > 0.f ? 1.f / L : 0.f;
+      acc.x *= inv;
+      acc.y *= inv;
+      if (p.cos_t) turn_back(acc.x, acc.y, p.cos_t[turn + d / 2], p.sin_t[turn + d / 2]);
+      *reinterpret_cast<__nv_bfloat162*>(p.out + (static_cast<int64_t>(b) * p.heads + h) * p.vdim + d) = __floats2bfloat162_rn(acc.x, acc.y);
     } else {
       const int64_t pi = (static_cast<int64_t>(b) * p.splits + split) * p.heads + h;
-      p.part_o[pi * p.vdim + d] = acc;
+      *reinterpret_cast<float2*>(p.part_o + pi * p.vdim + d) = acc;
       if (d == 0) {
         p.part_ml[pi * 2] = M;
         p.part_ml[pi * 2 + 1] = L;
@@ -454,13 +585,21 @@ __global__ void __launch_bounds__(128) window_join_kernel(const WindowParams<__n
     const float* ml = p.part_ml + (first + static_cast<int64_t>(s) * p.heads) * 2;
     L = fmaf(fast_exp2(ml[0] - M), ml[1], L);
   }
-  for (int d = threadIdx.x; d < p.vdim; d += 128) {
-    float acc = 0.f;
+  const float inv = L > 0.f ? 1.f / L : 0.f;
+  const int64_t turn = p.cos_t ? table_row(p.positions[b], p.table_rows) * (p.vdim / 2) : 0;
+  for (int d = threadIdx.x * 2; d < p.vdim; d += 256) {
+    float2 acc = make_float2(0.f, 0.f);
     for (int s = 0; s < p.splits; ++s) {
       const int64_t pi = first + static_cast<int64_t>(s) * p.heads;
-      acc = fmaf(fast_exp2(p.part_ml[pi * 2] - M), p.part_o[pi * p.vdim + d], acc);
+      const float f = fast_exp2(p.part_ml[pi * 2] - M);
+      const float2 o2 = *reinterpret_cast<const float2*>(p.part_o + pi * p.vdim + d);
+      acc.x = fmaf(f, o2.x, acc.x);
+      acc.y = fmaf(f, o2.y, acc.y);
     }
-    p.out[(static_cast<int64_t>(b) * p.heads + h) * p.vdim + d] = __float2bfloat16_rn(L > 0.f ? acc / L : 0.f);
+    acc.x *= inv;
+    acc.y *= inv;
+    if (p.cos_t) turn_back(acc.x, acc.y, p.cos_t[turn + d / 2], p.sin_t[turn + d / 2]);
+    *reinterpret_cast<__nv_bfloat162*>(p.out + (static_cast<int64_t>(b) * p.heads + h) * p.vdim + d) = __floats2bfloat162_rn(acc.x, acc.y);
   }
 }
 
@@ -483,6 +622,9 @@ static int window_splits(int batch, int heads, int kv_heads, int64_t most_keys) 
   return static_cast<int>(std::max<int64_t>(1, std::min<int64_t>({want, most_keys / 64, 64})));
 }
 
+static bool check_turn(const float* cos_t, const float* sin_t, int64_t table_rows, int vdim) {
+  return !cos_t ? !sin_t : sin_t && table_rows > 0 && vdim % 2 == 0;
+}
 static int check_window(const char* what, int heads, int kv_heads, int dim, int vdim, int64_t window, int block_size) {
   if (heads <= 0 || kv_heads <= 0 || heads % kv_heads || dim <= 0 || vdim <= 0 || window <= 0 || block_size <= 0)
     return fail(MV_ERR_SHAPE, "%s: heads %d over %d, dim %d, vdim %d, window %lld", what, heads, kv_heads, dim, vdim, static_cast<long long>(window));
@@ -518,16 +660,57 @@ extern "C" int mv_kv_norm_store(void* q, const void* k, const void* v, int64_t s
   return dtype == MV_F32 ? run(float{}) : run(__nv_bfloat16{});
 }
 
+extern "C" int mv_qkv_rope_store(void* q, const void* k, const void* v, int64_t stride, const void* q_weight,
+                                 const void* k_weight, const void* temp, const float* cos_t, const float* sin_t, int dims,
+                                 const float* vcos_t, const float* vsin_t, int64_t table_rows, const int64_t* positions,
+                                 void* kv_out, void* cache, const int64_t* slot_mapping, int64_t num_slots, int64_t tokens,
+                                 int heads, int kv_heads, int dim, int vdim, float eps, int dtype, void* stream) {
+  using namespace mv;
+  if (dtype != MV_BF16 && dtype != MV_F32) return fail(MV_ERR_DTYPE, "qkv_rope_store: dtype %d", dtype);
+  if (tokens < 0 || heads <= 0 || kv_heads < 0 || dim <= 0 || vdim < 0 || (kv_heads && vdim <= 0) || dims < 0 || dims > dim || dims % 2 ||
+      (vcos_t && vdim % 2) || table_rows <= 0)
+    return fail(MV_ERR_SHAPE, "qkv_rope_store: heads %d over %d, dim %d (%d rotated), vdim %d", heads, kv_heads, dim, dims, vdim);
+  const int widest = kv_heads ? std::max(dim, vdim) : dim;
+  if (widest > 1024) return fail(MV_ERR_LIMIT, "qkv_rope_store: dim %d, vdim %d (at most 1024)", dim, vdim);
+  if (tokens == 0) return MV_OK;
+  if (!q || !q_weight || !positions || (dims && (!cos_t || !sin_t)) || !vcos_t != !vsin_t ||
+      (kv_heads && (!k || !v || !k_weight)) || (cache && !slot_mapping))
+    return fail(MV_ERR_NULL, "qkv_rope_store: null pointer");
+  auto run = [&](auto tag) {
+    using T = decltype(tag);
+    const int eb = sizeof(T);
+    auto c = [](const void* x) { return static_cast<const T*>(x); };
+    RopeStoreParams<T> p{static_cast<T*>(q), c(k), c(v), stride, c(q_weight), c(k_weight), c(temp), cos_t, sin_t, dims, vcos_t, vsin_t,
+                         table_rows, positions, static_cast<T*>(kv_out), static_cast<T*>(cache), slot_mapping, num_slots, tokens,
+                         heads, kv_heads, dim, vdim, eps};
+    auto go = [&](auto kernel, int lanes) {
+      const int64_t blocks = (tokens * (heads + 2 * kv_heads) + kKnThreads / lanes - 1) / (kKnThreads / lanes);
+      kernel<<<static_cast<unsigned>(std::min<int64_t>(blocks, kNumSMs * 64)), kKnThreads, 0, static_cast<cudaStream_t>(stream)>>>(p);
+      return check_launch("qkv_rope_store");
+    };
+    const bool v8 = dim % 8 == 0 && vdim % 8 == 0 && vec8_ok(q, stride, eb) && vec8_ok(k, stride, eb) && vec8_ok(v, stride, eb) &&
+                    aligned16(kv_out) && aligned16(cache);
+    if (v8 && widest <= 64) return go(qkv_rope_store_kernel<T, 8, 8, 1>, 8);
+    if (v8 && widest <= 128) return go(qkv_rope_store_kernel<T, 8, 16, 1>, 16);
+    if (v8 && widest <= 256) return go(qkv_rope_store_kernel<T, 8, 32, 1>, 32);
+    if (v8) return go(qkv_rope_store_kernel<T, 8, 32, 4>, 32);
+    return go(qkv_rope_store_kernel<T, 2, 32, 16>, 32);
+  };
+  return dtype == MV_F32 ? run(float{}) : run(__nv_bfloat16{});
+}
+
 extern "C" int mv_window_attention_rows(void* out, const void* q, int64_t q_stride, const void* cache,
                                         const int32_t* block_tables, int64_t bt_stride, int max_blocks, int block_size,
                                         int64_t num_blocks, const int32_t* cu_q, int num_seqs, const int64_t* positions,
                                         const float* bias, int64_t bias_stride, int distances, const void* sink,
-                                        int64_t tokens, int heads, int kv_heads, int dim, int vdim, int64_t window,
-                                        float scale, int dtype, void* stream) {
+                                        const float* cos_t, const float* sin_t, int64_t table_rows, int64_t tokens,
+                                        int heads, int kv_heads, int dim, int vdim, int64_t window, float scale, int dtype,
+                                        void* stream) {
   using namespace mv;
   if (dtype != MV_BF16 && dtype != MV_F32) return fail(MV_ERR_DTYPE, "window_attention_rows: dtype %d", dtype);
   const int rc = check_window("window_attention_rows", heads, kv_heads, dim, vdim, window, block_size);
   if (rc) return rc;
+  if (!check_turn(cos_t, sin_t, table_rows, vdim)) return fail(MV_ERR_SHAPE, "window_attention_rows: rotation of %d columns", vdim);
   if (vdim > kWaThreads * kWaPer) return fail(MV_ERR_LIMIT, "window_attention_rows: vdim %d (at most %d)", vdim, kWaThreads * kWaPer);
   if (bias && distances <= 0) return fail(MV_ERR_SHAPE, "window_attention_rows: %d distances", distances);
   if (tokens <= 0) return tokens < 0 ? fail(MV_ERR_SHAPE, "window_attention_rows: tokens") : static_cast<int>(MV_OK);
@@ -543,6 +726,7 @@ extern "C" int mv_window_attention_rows(void* out, const void* q, int64_t q_stri
     p.tables = block_tables; p.bt_stride = bt_stride; p.max_blocks = max_blocks; p.block_size = block_size; p.num_blocks = num_blocks;
     p.cu_q = cu_q; p.num_seqs = num_seqs; p.positions = positions; p.bias = bias; p.bias_stride = bias_stride; p.distances = distances;
     p.sink = static_cast<const T*>(sink); p.heads = heads; p.kv_heads = kv_heads; p.dim = dim; p.vdim = vdim; p.window = window; p.scale = scale;
+    p.cos_t = cos_t; p.sin_t = sin_t; p.table_rows = table_rows;
     const int chunks = (heads / kv_heads + kWaHeads - 1) / kWaHeads;
     window_attention_rows_kernel<T><<<dim3(static_cast<unsigned>(tokens), kv_heads * chunks), kWaThreads, smem, static_cast<cudaStream_t>(stream)>>>(p);
     return check_launch("window_attention_rows");
@@ -563,18 +747,20 @@ extern "C" int64_t mv_window_decode_workspace_bytes(int batch, int heads, int kv
 extern "C" int mv_window_decode(void* out, const void* q, int64_t q_stride, const void* cache, const int32_t* block_tables,
                                 int64_t bt_stride, int max_blocks, int block_size, int64_t num_blocks,
                                 const int64_t* positions, const float* bias, int64_t bias_stride, int distances,
-                                const void* sink, int batch, int heads, int kv_heads, int dim, int vdim, int64_t window,
-                                float scale, void* workspace, int64_t workspace_bytes, void* stream) {
+                                const void* sink, const float* cos_t, const float* sin_t, int64_t table_rows, int batch,
+                                int heads, int kv_heads, int dim, int vdim, int64_t window, float scale, void* workspace, int64_t workspace_bytes, void* stream) {
   using namespace mv;
   const int rc = check_window("window_decode", heads, kv_heads, dim, vdim, window, block_size);
   if (rc) return rc;
   const int64_t most = std::min<int64_t>(window, static_cast<int64_t>(max_blocks) * block_size);
   const int64_t need = mv_window_decode_workspace_bytes(batch, heads, kv_heads, dim, vdim, std::max<int64_t>(most, 1));
+  if (!check_turn(cos_t, sin_t, table_rows, vdim)) return fail(MV_ERR_SHAPE, "window_decode: rotation of %d columns", vdim);
   if (need < 0) return fail(MV_ERR_LIMIT, "window_decode: dim %d, vdim %d, batch %d", dim, vdim, batch);
   if (bias && distances <= 0) return fail(MV_ERR_SHAPE, "window_decode: %d distances", distances);
   if (batch == 0) return MV_OK;
   if (!out || !q || !cache || !block_tables || !positions) return fail(MV_ERR_NULL, "window_decode: null pointer");
-  if (!aligned16(cache) || (reinterpret_cast<uintptr_t>(q) & 3u) || q_stride % 2) return fail(MV_ERR_ALIGN, "window_decode: alignment");
+  if (!aligned16(cache) || (reinterpret_cast<uintptr_t>(q) & 3u) || (reinterpret_cast<uintptr_t>(out) & 3u) || q_stride % 2)
+    return fail(MV_ERR_ALIGN, "window_decode: alignment");
   if (need > 0 && (!workspace || workspace_bytes < need)) return fail(MV_ERR_WORKSPACE, "window_decode: workspace");
   WindowParams<__nv_bfloat16> p{};
   p.out = static_cast<__nv_bfloat16*>(out); p.q = static_cast<const __nv_bfloat16*>(q); p.q_stride = q_stride;
@@ -582,7 +768,7 @@ extern "C" int mv_window_decode(void* out, const void* q, int64_t q_stride, cons
   p.tables = block_tables; p.bt_stride = bt_stride; p.max_blocks = max_blocks; p.block_size = block_size; p.num_blocks = num_blocks;
   p.positions = positions; p.bias = bias; p.bias_stride = bias_stride; p.distances = bias ? distances : 1;
   p.sink = static_cast<const __nv_bfloat16*>(sink); p.heads = heads; p.kv_heads = kv_heads; p.dim = dim; p.vdim = vdim;
-  p.window = window; p.scale = scale;
+  p.window = window; p.scale = scale; p.cos_t = cos_t; p.sin_t = sin_t; p.table_rows = table_rows;
   p.splits = window_splits(batch, heads, kv_heads, std::max<int64_t>(most, 1));
   p.part_ml = static_cast<float*>(workspace);
   p.part_o = p.part_ml ? p.part_ml + static_cast<int64_t>(batch) * p.splits * heads * 2 : nullptr;

@@ -8,6 +8,7 @@ import json
 import os
 from dataclasses import dataclass
 
+from .dafotar import DafotarConfig, DafotarForCausalLM
 from .fozerax import FozeraxConfig, FozeraxForCausalLM
 from .qwen3 import Qwen3Config, Qwen3ForCausalLM
 from .sipazen import SipazenConfig, SipazenForCausalLM
@@ -27,6 +28,7 @@ FAMILIES = {f.name: f for f in (
     ModelFamily("Qwen3ForCausalLM", Qwen3Config, Qwen3ForCausalLM, "qwen3"),
     ModelFamily("Sipazen", SipazenConfig, SipazenForCausalLM, "sipazen", loads_folders=True),
     ModelFamily("Fozerax", FozeraxConfig, FozeraxForCausalLM, "fozerax", loads_folders=True),
+    ModelFamily("Dafotar", DafotarConfig, DafotarForCausalLM, "dafotar", loads_folders=True),
 )}
 DEFAULT_FAMILY = "Qwen3ForCausalLM"
 

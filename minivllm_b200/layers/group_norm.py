@@ -14,7 +14,7 @@ def _rows(t, name):
     return t.data_ptr(), t.stride(0)
 
 
-ACTS = {"sigmoid": 0, "silu": 1, "gelu_tanh": 2, "clamped": 3}      # enum mv_act
+ACTS = {"sigmoid": 0, "silu": 1, "gelu_tanh": 2, "clamped": 3, "relu": 4}      # enum mv_act
 
 
 def _ptr(t):
@@ -91,20 +91,25 @@ def gated_group_norm(y, z, weight, groups, eps):
     return out
 
 
-def head_norm_gate(y, z, weight, heads, eps, out=None):
-    """norm(y) * weight * silu(z), rows in `heads` runs of channels; weight has one run's length."""
-    _cabi.require_cuda(y, z, weight)
+def head_norm_gate(y, z, weight, heads, eps, out=None, den=None, act="silu"):
+    """norm(y / den) * weight * act(z), rows in `heads` runs of channels; den (rows, heads) fp32 or None; weight has one run's
+    length, or a row's; act silu or sigmoid."""
+    _cabi.require_cuda(y, z, weight, den)
     yp, ys = _rows(y, "y")
     zp, zs = _rows(z, "z")
     if out is None:
         out = torch.empty(y.shape, dtype=y.dtype, device=y.device)
-    _cabi.check(_cabi.lib().mv_head_norm_gate(out.data_ptr(), yp, ys, zp, zs, weight.data_ptr(), y.shape[0], y.shape[1],
-                                              heads, eps, _cabi.layer_dtype_code(y.dtype), _cabi.stream_ptr()))
+    full = weight.numel() == y.shape[1]
+    if not full and weight.numel() * heads != y.shape[1]:
+        raise ValueError("the norm's weight has neither a head's nor a row's length")
+    _cabi.check(_cabi.lib().mv_head_norm_gate(
+        out.data_ptr(), yp, ys, _ptr(den), zp, zs, weight.data_ptr(), int(full), ACTS[act], y.shape[0], y.shape[1], heads, eps,
+        _cabi.layer_dtype_code(y.dtype), _cabi.stream_ptr()))
     return out
 
 
 def gate_mul(y, gate, act="sigmoid", out=None, limit=0.0):
-    """A gate applied to y: y * act(gate) for sigmoid, silu and gelu_tanh; "clamped" with `limit` see enum mv_act.  y (rows, cols), or (rows, heads, cols / heads) with any row and head
+    """A gate applied to y: y * act(gate) for sigmoid, silu, gelu_tanh and relu; "clamped" with `limit` see enum mv_act.  y (rows, cols), or (rows, heads, cols / heads) with any row and head
     stride; gate (rows, cols).  Returns (rows, cols)."""
     _cabi.require_cuda(y, gate)
     rows, cols = gate.shape

@@ -58,8 +58,13 @@ def _bias_args(bias):
     return (bias.data_ptr(), bias.stride(0), bias.shape[1]) if bias is not None else (None, 0, 1)
 
 
+def _turn_args(turn):
+    """turn: (cos, sin) tables (positions, vdim / 2) by whose angles results are turned back, or None."""
+    return (turn[0].data_ptr(), turn[1].data_ptr(), turn[0].shape[0]) if turn is not None else (None, None, 0)
+
+
 def window_attention_rows(q, cache, block_tables, cu_q, positions, kv_heads, dim, vdim, window, scale, bias=None, sink=None,
-                          out=None):
+                          out=None, turn=None):
     """q (tokens, heads * dim) -> (tokens, heads * vdim); cu_q None: one token per row of block_tables."""
     _cabi.require_cuda(q, cache, block_tables, positions, bias, sink)
     tokens, heads = q.shape[0], q.shape[1] // dim
@@ -67,12 +72,13 @@ def window_attention_rows(q, cache, block_tables, cu_q, positions, kv_heads, dim
     _cabi.check(_cabi.lib().mv_window_attention_rows(
         out.data_ptr(), q.data_ptr(), q.stride(0), cache.data_ptr(), block_tables.data_ptr(), block_tables.stride(0),
         block_tables.shape[1], cache.shape[1], cache.shape[0], cu_q.data_ptr() if cu_q is not None else None,
-        block_tables.shape[0], positions.data_ptr(), *_bias_args(bias), sink.data_ptr() if sink is not None else None, tokens,
-        heads, kv_heads, dim, vdim, window, scale, _cabi.layer_dtype_code(q.dtype), _cabi.stream_ptr()))
+        block_tables.shape[0], positions.data_ptr(), *_bias_args(bias), sink.data_ptr() if sink is not None else None, *_turn_args(turn),
+        tokens, heads, kv_heads, dim, vdim, window, scale, _cabi.layer_dtype_code(q.dtype), _cabi.stream_ptr()))
     return out
 
 
-def window_decode(q, cache, block_tables, positions, kv_heads, dim, vdim, window, scale, bias=None, sink=None, out=None):
+def window_decode(q, cache, block_tables, positions, kv_heads, dim, vdim, window, scale, bias=None, sink=None, out=None,
+                  turn=None):
     """window_attention_rows for one row per sequence on tensor cores; None when the kernel does not take the sizes."""
     _cabi.require_cuda(q, cache, block_tables, positions, bias, sink)
     batch, heads = q.shape[0], q.shape[1] // dim
@@ -86,13 +92,15 @@ def window_decode(q, cache, block_tables, positions, kv_heads, dim, vdim, window
     _cabi.check(L.mv_window_decode(
         out.data_ptr(), q.data_ptr(), q.stride(0), cache.data_ptr(), block_tables.data_ptr(), block_tables.stride(0),
         block_tables.shape[1], cache.shape[1], cache.shape[0], positions.data_ptr(), *_bias_args(bias),
-        sink.data_ptr() if sink is not None else None, batch, heads, kv_heads, dim, vdim, window, scale, ws.data_ptr(),
+        sink.data_ptr() if sink is not None else None, *_turn_args(turn), batch, heads, kv_heads, dim, vdim, window, scale, ws.data_ptr(),
         ws.numel(), _cabi.stream_ptr()))
     return out
 
 
-def window_prefill(q, kv, cu_q, cu_k, kv_heads, dim, vdim, window, scale, bias=None, sink=None, out=None):
-    """q (tokens, heads * dim), kv (keys, kv_heads * (dim + vdim)) packed rows -> (tokens, heads * vdim)."""
+def window_prefill(q, kv, cu_q, cu_k, kv_heads, dim, vdim, window, scale, bias=None, sink=None, out=None, turn=None,
+                   positions=None):
+    """q (tokens, heads * dim), kv (keys, kv_heads * (dim + vdim)) packed rows -> (tokens, heads * vdim).  `turn` wants the
+    queries' positions."""
     _cabi.require_cuda(q, kv, cu_q, cu_k, bias, sink)
     heads = q.shape[1] // dim
     out = torch.empty((q.shape[0], heads * vdim), dtype=q.dtype, device=q.device) if out is None else out
@@ -100,7 +108,8 @@ def window_prefill(q, kv, cu_q, cu_k, kv_heads, dim, vdim, window, scale, bias=N
     _cabi.check(_cabi.lib().mv_window_prefill(
         out.data_ptr(), out.stride(0), q.data_ptr(), q.stride(0), kv.data_ptr(), kv.stride(0), v.data_ptr(), v.stride(0),
         cu_q.data_ptr(), cu_k.data_ptr(), cu_q.numel() - 1, q.shape[0], kv.shape[0], heads, kv_heads, dim, vdim, window, scale,
-        *_bias_args(bias), sink.data_ptr() if sink is not None else None, _error_word(q.device).data_ptr(),
+        *_bias_args(bias), sink.data_ptr() if sink is not None else None, *_turn_args(turn),
+        positions.data_ptr() if turn is not None else None, _error_word(q.device).data_ptr(),
         _cabi.stream_ptr()))
     return out
 
