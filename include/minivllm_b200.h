@@ -597,8 +597,8 @@ int mv_ssm_step(void* y, const void* u, int64_t u_stride, const void* w, const v
  *                             sin_t (table_rows, dims / 2); q of head h times temp[h] (null: 1).  v: its pairs turned by
  *                             vcos_t, vsin_t (table_rows, vdim / 2; null: as it is).  [k | v] goes to kv_out and cache as
  *                             above; kv_heads 0: queries only.  dim and vdim up to 1,024
- * cos_t, sin_t (table_rows, vdim / 2) of the attention entries: the result of position i is turned in the same pairs by the
- * opposite of row i's angles (null: not).  out is (tokens, heads * vdim).  No counterpart in the reference.
+ * turn (vdim / 2, table_rows, 2) of the attention entries: the result of position i is turned in the same pairs by the
+ * opposite of the angles whose (cos, sin) are at [pair, i] (null: not).  out is (tokens, heads * vdim).  No counterpart in the reference.
  */
 int mv_kv_norm_store(void* q, const void* k, const void* v, int64_t stride, const void* q_weight, const
     void* k_weight, void* kv_out, void* cache, const int64_t* slot_mapping, int64_t num_slots, int64_t
@@ -611,22 +611,21 @@ int mv_qkv_rope_store(void* q, const void* k, const void* v, int64_t stride, con
 int mv_window_attention_rows(void* out, const void* q, int64_t q_stride, const void* cache, const
     int32_t* block_tables, int64_t bt_stride, int max_blocks, int block_size, int64_t num_blocks,
     const int32_t* cu_q, int num_seqs, const int64_t* positions, const float* bias, int64_t
-    bias_stride, int distances, const void* sink, const float* cos_t, const float* sin_t, int64_t
-    table_rows, int64_t tokens, int heads, int kv_heads, int dim, int vdim, int64_t window, float
+    bias_stride, int distances, const void* sink, const float* turn, int64_t table_rows, int64_t tokens, int heads, int kv_heads, int dim, int vdim, int64_t window, float
     scale, int dtype, void* stream);
 int64_t mv_window_decode_workspace_bytes(int batch, int heads, int kv_heads, int dim, int vdim, int64_t
     most_keys);
 int mv_window_decode(void* out, const void* q, int64_t q_stride, const void* cache, const int32_t*
     block_tables, int64_t bt_stride, int max_blocks, int block_size, int64_t num_blocks, const int64_t*
     positions, const float* bias, int64_t bias_stride, int distances, const void* sink, const float*
-    cos_t, const float* sin_t, int64_t table_rows, int batch, int heads, int kv_heads, int dim, int vdim,
+    turn, int64_t table_rows, int batch, int heads, int kv_heads, int dim, int vdim,
     int64_t window, float scale, void* workspace, int64_t workspace_bytes, void* stream);
 int mv_window_prefill_distances(int dim, int vdim);
 int mv_window_prefill(void* out, int64_t out_stride, const void* q, int64_t q_stride, const void* k,
     int64_t k_stride, const void* v, int64_t v_stride, const int32_t* cu_q, const int32_t* cu_k, int
     num_seqs, int64_t tokens, int64_t keys, int heads, int kv_heads, int dim, int vdim, int64_t window,
     float scale, const float* bias, int64_t bias_stride, int distances, const void* sink, const float*
-    cos_t, const float* sin_t, int64_t table_rows, const int64_t* positions, int* error_word, void* stream);
+    turn, int64_t table_rows, const int64_t* positions, int* error_word, void* stream);
 
 /*
  * Matrix-state recurrences, fp32 state (num_slots, heads, dim, vdim) updated in place, one read-out per token; dim up
@@ -680,7 +679,8 @@ int mv_delta_chunk_scan(void* out, int64_t out_stride, const void* qkv, int64_t 
  *   mv_mlstm_chunk_scan  the same in chunks of 64 tokens on tensor cores, bf16: dim a multiple of 8 up to 128, vdim a multiple
  *                        of 8, rows on 16-byte boundaries; tokens = cu[num_seqs]; workspace_bytes is -1 when the sizes are
  *                        not taken
- *   mv_mlstm_step        one token per sequence: out = rms_norm(o) * norm_w * sigmoid(gate), norm_w (heads * vdim)
+ *   mv_mlstm_step        one token per sequence: out = rms_norm(o) * norm_w * sigmoid(gate), norm_w (heads * vdim); the gates'
+ *                        logits are x (tokens, width) times gates_w (2 * heads, width)
  * dtype MV_BF16 or MV_F32.  No counterpart in the reference.
  */
 int mv_mlstm_gates(float* chain, const float* gates, int64_t gates_stride, const void* i_b, const void* f_b,
@@ -696,8 +696,8 @@ int mv_mlstm_chunk_scan(void* out, int64_t out_stride, float* den, const void* q
     slots, const int32_t* start, float* S, float* n, int num_slots, int heads, int dim, int vdim, float
     q_scale, void* workspace, int64_t workspace_bytes, void* stream);
 int mv_mlstm_step(void* out, int64_t out_stride, const void* q, const void* k, const void* v, int64_t stride,
-    const float* gates, int64_t gates_stride, const void* i_b, const void* f_b, float cap, int num_seqs,
-    const int32_t* slots, const int32_t* start, float* S, float* n, float* m, int num_slots, int heads, int
+    const void* x, int64_t x_stride, const void* gates_w, int width, const void* i_b, const void* f_b, float
+    cap, int num_seqs, const int32_t* slots, const int32_t* start, float* S, float* n, float* m, int num_slots, int heads, int
     dim, int vdim, float q_scale, const void* gate, int64_t gate_stride, const void* norm_w, float eps, int
     dtype, void* stream);
 

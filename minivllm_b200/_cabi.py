@@ -117,17 +117,17 @@ SIGNATURES = {
         _c_ptr, _c_int, _c_ptr, _c_ptr, _c_ptr, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_ptr]),
     "mv_kv_norm_store": (_c_int, [_c_ptr, _c_ptr, _c_ptr, _c_i64, _c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_i64, _c_i64,
         _c_int, _c_int, _c_int, _c_f32, _c_int, _c_ptr]),
-    "mv_window_attention_rows": (_c_int, [_c_ptr, _c_ptr, _c_i64, _c_ptr, _c_ptr, _c_i64, _c_int, _c_int, _c_i64, _c_ptr,
-        _c_int, _c_ptr, _c_ptr, _c_i64, _c_int, _c_ptr, _c_ptr, _c_ptr, _c_i64, _c_i64, _c_int, _c_int, _c_int, _c_int, _c_i64,
-        _c_f32, _c_int, _c_ptr]),
+    "mv_window_attention_rows": (_c_int, [_c_ptr, _c_ptr, _c_i64, _c_ptr, _c_ptr, _c_i64, _c_int, _c_int, _c_i64,
+        _c_ptr, _c_int, _c_ptr, _c_ptr, _c_i64, _c_int, _c_ptr, _c_ptr, _c_i64, _c_i64, _c_int, _c_int, _c_int,
+        _c_int, _c_i64, _c_f32, _c_int, _c_ptr]),
     "mv_window_decode_workspace_bytes": (_c_i64, [_c_int, _c_int, _c_int, _c_int, _c_int, _c_i64]),
-    "mv_window_decode": (_c_int, [_c_ptr, _c_ptr, _c_i64, _c_ptr, _c_ptr, _c_i64, _c_int, _c_int, _c_i64, _c_ptr, _c_ptr,
-        _c_i64, _c_int, _c_ptr, _c_ptr, _c_ptr, _c_i64, _c_int, _c_int, _c_int, _c_int, _c_int, _c_i64, _c_f32, _c_ptr, _c_i64,
-        _c_ptr]),
+    "mv_window_decode": (_c_int, [_c_ptr, _c_ptr, _c_i64, _c_ptr, _c_ptr, _c_i64, _c_int, _c_int, _c_i64, _c_ptr,
+        _c_ptr, _c_i64, _c_int, _c_ptr, _c_ptr, _c_i64, _c_int, _c_int, _c_int, _c_int, _c_int, _c_i64, _c_f32,
+        _c_ptr, _c_i64, _c_ptr]),
     "mv_window_prefill_distances": (_c_int, [_c_int, _c_int]),
-    "mv_window_prefill": (_c_int, [_c_ptr, _c_i64, _c_ptr, _c_i64, _c_ptr, _c_i64, _c_ptr, _c_i64, _c_ptr, _c_ptr, _c_int,
-        _c_i64, _c_i64, _c_int, _c_int, _c_int, _c_int, _c_i64, _c_f32, _c_ptr, _c_i64, _c_int, _c_ptr, _c_ptr, _c_ptr, _c_i64,
-        _c_ptr, _c_ptr, _c_ptr]),
+    "mv_window_prefill": (_c_int, [_c_ptr, _c_i64, _c_ptr, _c_i64, _c_ptr, _c_i64, _c_ptr, _c_i64, _c_ptr, _c_ptr,
+        _c_int, _c_i64, _c_i64, _c_int, _c_int, _c_int, _c_int, _c_i64, _c_f32, _c_ptr, _c_i64, _c_int, _c_ptr,
+        _c_ptr, _c_i64, _c_ptr, _c_ptr, _c_ptr]),
     "mv_gla_scan": (_c_int, [_c_ptr, _c_i64, _c_ptr, _c_ptr, _c_ptr, _c_i64, _c_ptr, _c_i64, _c_f32, _c_ptr, _c_int, _c_ptr,
         _c_ptr, _c_ptr, _c_int, _c_int, _c_int, _c_int, _c_f32, _c_ptr, _c_i64, _c_ptr, _c_f32, _c_int, _c_ptr]),
     "mv_delta_scan": (_c_int, [_c_ptr, _c_i64, _c_ptr, _c_i64, _c_ptr, _c_ptr, _c_i64, _c_ptr, _c_ptr, _c_ptr, _c_int,
@@ -150,10 +150,10 @@ SIGNATURES = {
         "mv_mlstm_chunk_scan": (_c_int, [_c_ptr, _c_i64, _c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_i64, _c_ptr, _c_ptr,
         _c_int, _c_i64, _c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_int, _c_int, _c_int, _c_int, _c_f32, _c_ptr, _c_i64,
         _c_ptr]),
-        "mv_mlstm_step": (_c_int, [_c_ptr, _c_i64, _c_ptr, _c_ptr, _c_ptr, _c_i64, _c_ptr, _c_i64, _c_ptr, _c_ptr,
-        _c_f32, _c_int, _c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_int, _c_int, _c_int, _c_int, _c_f32, _c_ptr,
-        _c_i64, _c_ptr, _c_f32, _c_int, _c_ptr]),
-        "mv_stream_step": (_c_int, [_c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_i64, _c_ptr, _c_i64, _c_ptr, _c_ptr,
+        "mv_mlstm_step": (_c_int, [_c_ptr, _c_i64, _c_ptr, _c_ptr, _c_ptr, _c_i64, _c_ptr, _c_i64, _c_ptr, _c_int, _c_ptr,
+        _c_ptr, _c_f32, _c_int, _c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_int, _c_int, _c_int, _c_int, _c_f32,
+        _c_ptr, _c_i64, _c_ptr, _c_f32, _c_int, _c_ptr]),
+    "mv_stream_step": (_c_int, [_c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_i64, _c_ptr, _c_i64, _c_ptr, _c_ptr,
         _c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_int, _c_ptr, _c_ptr, _c_ptr, _c_int, _c_i64, _c_i64, _c_int, _c_int,
         _c_f32, _c_int, _c_ptr]),
 }

@@ -49,18 +49,18 @@ struct LfParams {
   int group;                                          // query heads per KV head
   int window, distances;                              // kWin; bias may be null
   const float* bias; int64_t bias_stride;
-  const float *cos_t, *sin_t; int64_t table_rows;     // kWin: (table_rows, vdim / 2), null: results stay as they are
+  const float2* turn; int64_t table_rows;             // kWin: (vdim / 2, table_rows) cos, sin; null: results stay as they are
   const int64_t* positions;                           // of the queries
 };
 
 enum { LB_Q = 0, LB_KFULL = 1, LB_KEMPTY = 3, LB_VFULL = 5, LB_VEMPTY = 7, LB_SFULL = 9, LB_PREADY = 11, LB_ODONE = 13,
        LB_DRAIN = 15, LB_COUNT = 16 };
 
-// A pair of columns (fp32 bits) turned by the angle's opposite.
-__device__ __forceinline__ void turn_back(uint32_t& a, uint32_t& b, float co, float si) {
+// A pair of columns (fp32 bits) turned by the opposite of an angle, given as (cos, sin).
+__device__ __forceinline__ void turn_back(uint32_t& a, uint32_t& b, float2 cs) {
   const float x = __uint_as_float(a), y = __uint_as_float(b);
-  a = __float_as_uint(fmaf(x, co, y * si));
-  b = __float_as_uint(fmaf(y, co, -x * si));
+  a = __float_as_uint(fmaf(x, cs.x, y * cs.y));
+  b = __float_as_uint(fmaf(y, cs.x, -x * cs.y));
 }
 
 template <int NQ, int NV, bool kWin>
@@ -360,9 +360,9 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap tm_qn, const __grid_co
       const float inv = l > 0.f ? f / l : 0.f;
       const int qrow = q0 + t * kLfTile + row;
       __nv_bfloat16* orow = p.out + static_cast<int64_t>(q_start + qrow) * p.out_stride + static_cast<int64_t>(head) * p.vdim;
-      const bool turn = kWin && p.cos_t && qrow < q_len;
-      int64_t angle = 0;
-      if (turn) angle = min(max(p.positions[q_start + qrow], static_cast<int64_t>(0)), p.table_rows - 1) * (p.vdim / 2);
+      const bool turn = kWin && p.turn && qrow < q_len;
+      const float2* angle = p.turn;      // neighbouring rows read neighbouring entries
+      if (turn) angle += min(max(p.positions[q_start + qrow], static_cast<int64_t>(0)), p.table_rows - 1);
 #pragma unroll
       for (int c = 0; c < 2 * NV; ++c) {
         uint32_t ov[32];
@@ -373,12 +373,9 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap tm_qn, const __grid_co
           for (int i = 0; i < 4; ++i) {
             if (c * 32 + i * 8 >= p.vdim) continue;
             if (turn) {
-              const float4 co = __ldg(reinterpret_cast<const float4*>(p.cos_t + angle + c * 16 + i * 4));
-              const float4 si = __ldg(reinterpret_cast<const float4*>(p.sin_t + angle + c * 16 + i * 4));
-              turn_back(ov[8 * i + 0], ov[8 * i + 1], co.x, si.x);
-              turn_back(ov[8 * i + 2], ov[8 * i + 3], co.y, si.y);
-              turn_back(ov[8 * i + 4], ov[8 * i + 5], co.z, si.z);
-              turn_back(ov[8 * i + 6], ov[8 * i + 7], co.w, si.w);
+#pragma unroll
+              for (int e = 0; e < 4; ++e)
+                turn_back(ov[8 * i + 2 * e], ov[8 * i + 2 * e + 1], __ldg(angle + (c * 16 + i * 4 + e) * p.table_rows));
             }
             uint4 w;
             w.x = pack2<__nv_bfloat16>(__uint_as_float(ov[8 * i + 0]) * inv, __uint_as_float(ov[8 * i + 1]) * inv);
@@ -480,7 +477,7 @@ extern "C" int mv_latent_prefill(void* out, int64_t out_stride, const void* q, i
   if (rc) return rc;
   if (!rot_dim) { tm[1] = tm[0]; tm[3] = tm[2]; }
   LfParams p{static_cast<__nv_bfloat16*>(out), out_stride, vdim, cu_q, cu_k, num_seqs, nd, dim, rot_dim,
-             scale * 1.4426950408889634f, static_cast<const __nv_bfloat16*>(sink), error_word, 1, 0, 0, nullptr, 0, nullptr, nullptr, 0, nullptr};
+             scale * 1.4426950408889634f, static_cast<const __nv_bfloat16*>(sink), error_word, 1, 0, 0, nullptr, 0, nullptr, 0, nullptr};
   auto st = static_cast<cudaStream_t>(stream);
   if (nq == 1) return nv == 1 ? launch_latent_prefill<1, 1>(tm, p, tokens, heads, st) : launch_latent_prefill<1, 2>(tm, p, tokens, heads, st);
   if (nq == 2) return nv == 1 ? launch_latent_prefill<2, 1>(tm, p, tokens, heads, st) : launch_latent_prefill<2, 2>(tm, p, tokens, heads, st);
@@ -501,13 +498,13 @@ extern "C" int mv_window_prefill(void* out, int64_t out_stride, const void* q, i
                                  int64_t k_stride, const void* v, int64_t v_stride, const int32_t* cu_q,
                                  const int32_t* cu_k, int num_seqs, int64_t tokens, int64_t keys, int heads, int kv_heads,
                                  int dim, int vdim, int64_t window, float scale, const float* bias, int64_t bias_stride,
-                                 int distances, const void* sink, const float* cos_t, const float* sin_t,
-                                 int64_t table_rows, const int64_t* positions, int* error_word, void* stream) {
+                                 int distances, const void* sink, const float* turn, int64_t table_rows,
+                                 const int64_t* positions, int* error_word, void* stream) {
   using namespace mv;
   const char* w = "window_prefill";
   if (num_seqs < 0 || tokens < 0 || keys < tokens || heads <= 0 || kv_heads <= 0 || heads % kv_heads || window <= 0 || distances <= 0)
     return fail(MV_ERR_SHAPE, "window_prefill: heads %d over %d, window %lld, %d distances", heads, kv_heads, static_cast<long long>(window), distances);
-  if (!cos_t != !sin_t || (cos_t && (table_rows <= 0 || !positions || !aligned16(cos_t) || !aligned16(sin_t))))
+  if (turn && (table_rows <= 0 || !positions || (reinterpret_cast<uintptr_t>(turn) & 7u)))
     return fail(MV_ERR_NULL, "window_prefill: rotation table");
   if (mv_window_prefill_distances(dim, vdim) < 0) return fail(MV_ERR_LIMIT, "window_prefill: dim %d vdim %d", dim, vdim);
   if (tokens == 0 || num_seqs == 0) return MV_OK;
@@ -525,7 +522,7 @@ extern "C" int mv_window_prefill(void* out, int64_t out_stride, const void* q, i
   const int win = static_cast<int>(std::min<int64_t>(window, 1 << 30));
   LfParams p{static_cast<__nv_bfloat16*>(out), out_stride, vdim, cu_q, cu_k, num_seqs, nq, dim, 0,
              scale * 1.4426950408889634f, static_cast<const __nv_bfloat16*>(sink), error_word, heads / kv_heads, win,
-             bias ? std::min(distances, win) : 1, bias, bias_stride, cos_t, sin_t, table_rows, positions};
+             bias ? std::min(distances, win) : 1, bias, bias_stride, reinterpret_cast<const float2*>(turn), table_rows, positions};
   auto st = static_cast<cudaStream_t>(stream);
   if (nq == 1) return nv == 1 ? launch_latent_prefill<1, 1, true>(tm, p, tokens, heads, st) : launch_latent_prefill<1, 2, true>(tm, p, tokens, heads, st);
   if (nq == 2) return nv == 1 ? launch_latent_prefill<2, 1, true>(tm, p, tokens, heads, st) : launch_latent_prefill<2, 2, true>(tm, p, tokens, heads, st);

@@ -1,8 +1,8 @@
 // Matrix memory with exponential gates (mLSTM) in chunks of 64 tokens.  With b_t the running sums of the forget gates' logarithms
-// inside the chunk, a_j = i_j - b_j, M_t = m_t - b_t and m_0 the maximum in front of the chunk, all of which the chain of mlstm.cu
-// fixes, every power below is at most one:
-//   O = alpha (Q S_0) + A V,     A[t, j] = q_t k_j e^(a_j - M_t), j <= t,     alpha_t = e^(m_0 - M_t)
-//   S = e^(m_0 - M_last) S_0 + (w K)^T V,     w_j = e^(a_j - M_last);     n the same with V = 1
+// inside the chunk, m_0 the maximum in front of it, a_j = i_j - m_0 - b_j and M_t = m_t - m_0 - b_t, all of which the chain of
+// mlstm.cu fixes, every power below is at most one:
+//   O = alpha (Q S_0) + A V,     A[t, j] = q_t k_j e^(a_j - M_t), j <= t,     alpha_t = e^(-M_t)
+//   S = e^(-M_last) S_0 + (w K)^T V,     w_j = e^(a_j - M_last);     n the same with V = 1
 //   denominator of t = max(|alpha_t q_t n_0 + sum_j A[t, j]|, e^-m_t) + 1e-6
 // mlstm_prepare_kernel  per chunk and head: the factors, A in two terms, its row sums, sum_j w_j k_j
 // mlstm_chunk_kernel    per sequence, head and block of value columns: see state_chunk.cuh.  The first block of columns also
@@ -59,18 +59,17 @@ __global__ void __launch_bounds__(kMpThreads) mlstm_prepare_kernel(const MemChun
     cp_async_commit();
   }
   if (warp == 0) {                       // two neighbouring tokens per lane, base-2 logarithms
-    float b[2], m[2], a[2], M[2], run = 0.f, m0 = 0.f;
+    float b[2], m[2], a[2], M[2], run = 0.f;
+    const float m0 = p.chain[first * p.heads + h].z;
 #pragma unroll
     for (int e = 0; e < 2; ++e) {
       const int t = lane * 2 + e;
       const float4 c = t < nt ? p.chain[(first + t) * p.heads + h] : make_float4(0.f, 0.f, 0.f, 0.f);
-      if (e == 0) m0 = c.z * kLog2e;
       run += c.y * kLog2e;
       b[e] = run;
-      a[e] = c.x * kLog2e;
-      m[e] = c.w * kLog2e;
+      a[e] = (c.x - m0) * kLog2e;
+      m[e] = c.w;
     }
-    m0 = __shfl_sync(0xffffffffu, m0, 0);
     float before = run;
 #pragma unroll
     for (int o = 1; o < 32; o <<= 1) {
@@ -81,7 +80,7 @@ __global__ void __launch_bounds__(kMpThreads) mlstm_prepare_kernel(const MemChun
 #pragma unroll
     for (int e = 0; e < 2; ++e) {
       a[e] -= before + b[e];
-      M[e] = m[e] - (before + b[e]);
+      M[e] = (m[e] - m0) * kLog2e - (before + b[e]);
     }
     const float last = __shfl_sync(0xffffffffu, (nt - 1) & 1 ? M[1] : M[0], (nt - 1) >> 1);
 #pragma unroll
@@ -92,10 +91,10 @@ __global__ void __launch_bounds__(kMpThreads) mlstm_prepare_kernel(const MemChun
       s_M[t] = on ? M[e] : 1e30f;          // rows past the end become zero
       s_w[t] = on ? fast_exp2(a[e] - last) : 0.f;
       vec[Vc::kWrite + t] = s_w[t];
-      vec[Vc::kAlpha + t] = on ? p.q_scale * fast_exp2(m0 - M[e]) : 0.f;
-      vec[Vc::kFloor + t] = on ? fast_exp2(-m[e]) : 1.f;
+      vec[Vc::kAlpha + t] = on ? p.q_scale * fast_exp2(-M[e]) : 0.f;
+      vec[Vc::kFloor + t] = on ? fast_exp2(-m[e] * kLog2e) : 1.f;
     }
-    if (lane == 0) vec[Vc::kDecay] = fast_exp2(m0 - last);
+    if (lane == 0) vec[Vc::kDecay] = fast_exp2(-last);
   }
   cp_async_wait<0>();
   __syncthreads();

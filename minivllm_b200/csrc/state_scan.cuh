@@ -12,7 +12,7 @@
 // reduce-scatter over the KP lanes: afterwards every lane holds one column's result.
 //
 // Decays near one enter as alpha - 1 (S + (alpha - 1) S): the rounding of alpha itself would add up over thousands of
-// tokens.
+// tokens.  For the same reason matrix memory forms f - (m' - m), which returns to S what the rounding of m' = f + m lost.
 //
 // The delta rule's scalar decay is kept out of the matrix: S = G * S', G the product of the decays, folded into S' when
 // it becomes small.
@@ -258,7 +258,8 @@ template <typename T> struct ScanParams {
   float inv_tau;
   const T *beta, *a; int64_t gate_stride;              // delta rule: (heads) logits of the step size and of the decay
   const T *A_log, *dt_bias;
-  const float* gates; int64_t gates_stride;            // matrix memory: (heads) logits of the input gate, (heads) of the forget gate
+  const float* gates; int64_t gates_stride;            // matrix memory, prompts: (heads) logits of the input gate, (heads) of the forget gate
+  const T *x, *gates_w; int64_t x_stride; int width;   //   one token: (width) input of the gates, (2 heads, width) weights
   const T *i_b, *f_b; float cap;
   float *n_state, *m_state;                            //   (num_slots, heads, K), (num_slots, heads)
   const float4* chain; float* den;                     //   prompts: (tokens, heads) i, f, m, m' and denominators
@@ -333,7 +334,7 @@ __global__ void __launch_bounds__(32 * W, 16 / W) scan_kernel(const ScanParams<T
   auto prepare = [&](int buf) {
     float* vecs = s_vec + (buf * TT + warp) * VEC * K;
     float kk = 0.f, qq = 0.f, kq = 0.f;
-    const float alpha_m1 = kMem ? expm1f(rc.y + rc.z - rc.w) : 0.f, write = kMem ? expf(rc.x - rc.w) : 0.f;
+    const float alpha_m1 = kMem ? expm1f(rc.y - (rc.w - rc.z)) : 0.f, write = kMem ? expf(rc.x - rc.w) : 0.f;
     if (kMem && lane == 0) s_par[(buf * TT + warp) * 4] = expf(-rc.w);
 #pragma unroll
     for (int m = 0; m < KL; ++m) {
@@ -427,14 +428,43 @@ __global__ void __launch_bounds__(32 * W, 16 / W) scan_kernel(const ScanParams<T
   }
 }
 
-// Matrix memory: factors of the old state and of the new entry of a token, and its running maximum.  Every thread for itself.
+// Matrix memory: factors of the old state and of the new entry of a token, and its running maximum, for every thread of the
+// block; the gates' logits are formed here.
 struct MemFactors { float alpha_m1, write, m; };
 template <typename T> __device__ __forceinline__ MemFactors mem_factors(const ScanParams<T>& p, int s, int h, int slot, int st0) {
-  const float* z = p.gates + static_cast<int64_t>(s) * p.gates_stride + h;
-  const float i = mem_log_input(z[0] + Elem<T>::to_f(p.i_b[h]), p.cap), f = mem_log_forget(z[p.heads] + Elem<T>::to_f(p.f_b[h]), p.cap);
+  __shared__ float2 part[32];
+  const T *x = p.x + static_cast<int64_t>(s) * p.x_stride, *wi = p.gates_w + static_cast<int64_t>(h) * p.width;
+  const T* wf = wi + static_cast<int64_t>(p.heads) * p.width;
+  float2 z = make_float2(0.f, 0.f);
+  auto add = [&](float a, float bi, float bf) {
+    z.x = fmaf(a, bi, z.x);
+    z.y = fmaf(a, bf, z.y);
+  };
+  const uintptr_t bits = reinterpret_cast<uintptr_t>(x) | reinterpret_cast<uintptr_t>(wi) | reinterpret_cast<uintptr_t>(wf);
+  if ((bits & 15u) == 0 && p.width % 8 == 0) {
+    for (int c = threadIdx.x * 8; c < p.width; c += blockDim.x * 8) {
+      float a[8], bi[8], bf[8];
+      Vec<T, 8>::load(x + c, a);
+      Vec<T, 8>::load(wi + c, bi);
+      Vec<T, 8>::load(wf + c, bf);
+#pragma unroll
+      for (int e = 0; e < 8; ++e) add(a[e], bi[e], bf[e]);
+    }
+  } else {
+    for (int c = threadIdx.x; c < p.width; c += blockDim.x) add(Elem<T>::to_f(x[c]), Elem<T>::to_f(wi[c]), Elem<T>::to_f(wf[c]));
+  }
+  z = make_float2(warp_sum(z.x), warp_sum(z.y));
+  if ((threadIdx.x & 31) == 0) part[threadIdx.x >> 5] = z;
+  __syncthreads();
+  z = make_float2(0.f, 0.f);
+  for (int w = 0; w < static_cast<int>(blockDim.x >> 5); ++w) {
+    z.x += part[w].x;
+    z.y += part[w].y;
+  }
+  const float i = mem_log_input(z.x + Elem<T>::to_f(p.i_b[h]), p.cap), f = mem_log_forget(z.y + Elem<T>::to_f(p.f_b[h]), p.cap);
   const float old = st0 > 0 ? p.m_state[static_cast<int64_t>(slot) * p.heads + h] : 0.f;
   const float m = fmaxf(f + old, i);
-  return {expm1f(f + old - m), expf(i - m), m};
+  return {expm1f(f - (m - old)), expf(i - m), m};
 }
 // The state's n and m one token on, and the terms of n . q; between two barriers.
 template <typename T>

@@ -103,10 +103,10 @@ __device__ __forceinline__ void turn_pairs(float (&x)[V], int c, int dims, const
     x[e + 1] = b * co + a * si;
   }
 }
-// A pair turned by the opposite angle.
-__device__ __forceinline__ void turn_back(float& a, float& b, float co, float si) {
-  const float x = fmaf(a, co, b * si);
-  b = fmaf(b, co, -a * si);
+// A pair turned by the opposite of an angle, given as (cos, sin).
+__device__ __forceinline__ void turn_back(float& a, float& b, float2 cs) {
+  const float x = fmaf(a, cs.x, b * cs.y);
+  b = fmaf(b, cs.x, -a * cs.y);
   a = x;
 }
 
@@ -212,7 +212,7 @@ template <typename T> struct WindowParams {
   int heads, kv_heads, dim, vdim;
   int64_t window;
   float scale;
-  const float *cos_t, *sin_t; int64_t table_rows;              // (table_rows, vdim / 2): results are turned back; null: not
+  const float2* turn; int64_t table_rows;                      // (vdim / 2, table_rows) cos, sin: results are turned back; null: not
   // decode
   int splits;
   float *part_ml, *part_o;                   // (batch, splits, heads, 2) and (.., vdim)
@@ -311,7 +311,7 @@ __global__ void __launch_bounds__(kWaThreads) window_attention_rows_kernel(const
     }
   }
   __syncthreads();
-  const int64_t turn = p.cos_t ? table_row(pos, p.table_rows) * (VD / 2) : 0;
+  const int64_t angle = p.turn ? table_row(pos, p.table_rows) : 0;
 #pragma unroll
   for (int h = 0; h < kWaHeads; ++h) {
     if (h >= nh) break;
@@ -319,11 +319,11 @@ __global__ void __launch_bounds__(kWaThreads) window_attention_rows_kernel(const
 #pragma unroll
     for (int i = 0; i < kWaPer; ++i) {
       const int d = tid + i * kWaThreads;
-      if (p.cos_t && i * kWaThreads < VD) {      // the other column of the pair is the neighbouring thread's
+      if (p.turn && i * kWaThreads < VD) {      // the other column of the pair is the neighbouring thread's
         const float other = __shfl_xor_sync(0xffffffffu, acc[h][i], 1);
         if (d < VD) {
-          const float co = p.cos_t[turn + d / 2], si = p.sin_t[turn + d / 2];
-          acc[h][i] = fmaf(acc[h][i], co, d & 1 ? -other * si : other * si);
+          const float2 cs = p.turn[d / 2 * p.table_rows + angle];
+          acc[h][i] = fmaf(acc[h][i], cs.x, d & 1 ? -other * cs.y : other * cs.y);
         }
       }
       if (d < VD) p.out[(static_cast<int64_t>(t) * p.heads + h0 + h) * VD + d] = Elem<T>::from_f(acc[h][i] * inv);
@@ -537,7 +537,7 @@ window_decode_kernel(const WindowParams<__nv_bfloat16> p) {
   }
   __syncthreads();
   const int half = p.vdim / 2;           // a thread has pairs of neighbouring columns
-  const int64_t turn = p.cos_t ? table_row(pos64, p.table_rows) * half : 0;
+  const int64_t angle = p.turn ? table_row(pos64, p.table_rows) : 0;
   for (int i = tid; i < rows * half; i += kWdThreads) {
     const int r = i / half, d = (i - r * half) * 2, h = h0 + r;
     float M = kWdNeg;
@@ -559,7 +559,7 @@ window_decode_kernel(const WindowParams<__nv_bfloat16> p) {
       const float inv = L > 0.f ? 1.f / L : 0.f;
       acc.x *= inv;
       acc.y *= inv;
-      if (p.cos_t) turn_back(acc.x, acc.y, p.cos_t[turn + d / 2], p.sin_t[turn + d / 2]);
+      if (p.turn) turn_back(acc.x, acc.y, p.turn[d / 2 * p.table_rows + angle]);
       *reinterpret_cast<__nv_bfloat162*>(p.out + (static_cast<int64_t>(b) * p.heads + h) * p.vdim + d) = __floats2bfloat162_rn(acc.x, acc.y);
     } else {
       const int64_t pi = (static_cast<int64_t>(b) * p.splits + split) * p.heads + h;
@@ -586,7 +586,7 @@ __global__ void __launch_bounds__(128) window_join_kernel(const WindowParams<__n
     L = fmaf(fast_exp2(ml[0] - M), ml[1], L);
   }
   const float inv = L > 0.f ? 1.f / L : 0.f;
-  const int64_t turn = p.cos_t ? table_row(p.positions[b], p.table_rows) * (p.vdim / 2) : 0;
+  const int64_t angle = p.turn ? table_row(p.positions[b], p.table_rows) : 0;
   for (int d = threadIdx.x * 2; d < p.vdim; d += 256) {
     float2 acc = make_float2(0.f, 0.f);
     for (int s = 0; s < p.splits; ++s) {
@@ -598,7 +598,7 @@ __global__ void __launch_bounds__(128) window_join_kernel(const WindowParams<__n
     }
     acc.x *= inv;
     acc.y *= inv;
-    if (p.cos_t) turn_back(acc.x, acc.y, p.cos_t[turn + d / 2], p.sin_t[turn + d / 2]);
+    if (p.turn) turn_back(acc.x, acc.y, p.turn[d / 2 * p.table_rows + angle]);
     *reinterpret_cast<__nv_bfloat162*>(p.out + (static_cast<int64_t>(b) * p.heads + h) * p.vdim + d) = __floats2bfloat162_rn(acc.x, acc.y);
   }
 }
@@ -622,8 +622,8 @@ static int window_splits(int batch, int heads, int kv_heads, int64_t most_keys) 
   return static_cast<int>(std::max<int64_t>(1, std::min<int64_t>({want, most_keys / 64, 64})));
 }
 
-static bool check_turn(const float* cos_t, const float* sin_t, int64_t table_rows, int vdim) {
-  return !cos_t ? !sin_t : sin_t && table_rows > 0 && vdim % 2 == 0;
+static bool check_turn(const float* turn, int64_t table_rows, int vdim) {
+  return !turn || (table_rows > 0 && vdim % 2 == 0 && (reinterpret_cast<uintptr_t>(turn) & 7u) == 0);
 }
 static int check_window(const char* what, int heads, int kv_heads, int dim, int vdim, int64_t window, int block_size) {
   if (heads <= 0 || kv_heads <= 0 || heads % kv_heads || dim <= 0 || vdim <= 0 || window <= 0 || block_size <= 0)
@@ -703,14 +703,13 @@ extern "C" int mv_window_attention_rows(void* out, const void* q, int64_t q_stri
                                         const int32_t* block_tables, int64_t bt_stride, int max_blocks, int block_size,
                                         int64_t num_blocks, const int32_t* cu_q, int num_seqs, const int64_t* positions,
                                         const float* bias, int64_t bias_stride, int distances, const void* sink,
-                                        const float* cos_t, const float* sin_t, int64_t table_rows, int64_t tokens,
-                                        int heads, int kv_heads, int dim, int vdim, int64_t window, float scale, int dtype,
-                                        void* stream) {
+                                        const float* turn, int64_t table_rows, int64_t tokens, int heads, int kv_heads,
+                                        int dim, int vdim, int64_t window, float scale, int dtype, void* stream) {
   using namespace mv;
   if (dtype != MV_BF16 && dtype != MV_F32) return fail(MV_ERR_DTYPE, "window_attention_rows: dtype %d", dtype);
   const int rc = check_window("window_attention_rows", heads, kv_heads, dim, vdim, window, block_size);
   if (rc) return rc;
-  if (!check_turn(cos_t, sin_t, table_rows, vdim)) return fail(MV_ERR_SHAPE, "window_attention_rows: rotation of %d columns", vdim);
+  if (!check_turn(turn, table_rows, vdim)) return fail(MV_ERR_SHAPE, "window_attention_rows: rotation of %d columns", vdim);
   if (vdim > kWaThreads * kWaPer) return fail(MV_ERR_LIMIT, "window_attention_rows: vdim %d (at most %d)", vdim, kWaThreads * kWaPer);
   if (bias && distances <= 0) return fail(MV_ERR_SHAPE, "window_attention_rows: %d distances", distances);
   if (tokens <= 0) return tokens < 0 ? fail(MV_ERR_SHAPE, "window_attention_rows: tokens") : static_cast<int>(MV_OK);
@@ -726,7 +725,7 @@ extern "C" int mv_window_attention_rows(void* out, const void* q, int64_t q_stri
     p.tables = block_tables; p.bt_stride = bt_stride; p.max_blocks = max_blocks; p.block_size = block_size; p.num_blocks = num_blocks;
     p.cu_q = cu_q; p.num_seqs = num_seqs; p.positions = positions; p.bias = bias; p.bias_stride = bias_stride; p.distances = distances;
     p.sink = static_cast<const T*>(sink); p.heads = heads; p.kv_heads = kv_heads; p.dim = dim; p.vdim = vdim; p.window = window; p.scale = scale;
-    p.cos_t = cos_t; p.sin_t = sin_t; p.table_rows = table_rows;
+    p.turn = reinterpret_cast<const float2*>(turn); p.table_rows = table_rows;
     const int chunks = (heads / kv_heads + kWaHeads - 1) / kWaHeads;
     window_attention_rows_kernel<T><<<dim3(static_cast<unsigned>(tokens), kv_heads * chunks), kWaThreads, smem, static_cast<cudaStream_t>(stream)>>>(p);
     return check_launch("window_attention_rows");
@@ -747,14 +746,14 @@ extern "C" int64_t mv_window_decode_workspace_bytes(int batch, int heads, int kv
 extern "C" int mv_window_decode(void* out, const void* q, int64_t q_stride, const void* cache, const int32_t* block_tables,
                                 int64_t bt_stride, int max_blocks, int block_size, int64_t num_blocks,
                                 const int64_t* positions, const float* bias, int64_t bias_stride, int distances,
-                                const void* sink, const float* cos_t, const float* sin_t, int64_t table_rows, int batch,
-                                int heads, int kv_heads, int dim, int vdim, int64_t window, float scale, void* workspace, int64_t workspace_bytes, void* stream) {
+                                const void* sink, const float* turn, int64_t table_rows, int batch, int heads,
+                                int kv_heads, int dim, int vdim, int64_t window, float scale, void* workspace, int64_t workspace_bytes, void* stream) {
   using namespace mv;
   const int rc = check_window("window_decode", heads, kv_heads, dim, vdim, window, block_size);
   if (rc) return rc;
   const int64_t most = std::min<int64_t>(window, static_cast<int64_t>(max_blocks) * block_size);
   const int64_t need = mv_window_decode_workspace_bytes(batch, heads, kv_heads, dim, vdim, std::max<int64_t>(most, 1));
-  if (!check_turn(cos_t, sin_t, table_rows, vdim)) return fail(MV_ERR_SHAPE, "window_decode: rotation of %d columns", vdim);
+  if (!check_turn(turn, table_rows, vdim)) return fail(MV_ERR_SHAPE, "window_decode: rotation of %d columns", vdim);
   if (need < 0) return fail(MV_ERR_LIMIT, "window_decode: dim %d, vdim %d, batch %d", dim, vdim, batch);
   if (bias && distances <= 0) return fail(MV_ERR_SHAPE, "window_decode: %d distances", distances);
   if (batch == 0) return MV_OK;
@@ -768,7 +767,7 @@ extern "C" int mv_window_decode(void* out, const void* q, int64_t q_stride, cons
   p.tables = block_tables; p.bt_stride = bt_stride; p.max_blocks = max_blocks; p.block_size = block_size; p.num_blocks = num_blocks;
   p.positions = positions; p.bias = bias; p.bias_stride = bias_stride; p.distances = bias ? distances : 1;
   p.sink = static_cast<const __nv_bfloat16*>(sink); p.heads = heads; p.kv_heads = kv_heads; p.dim = dim; p.vdim = vdim;
-  p.window = window; p.scale = scale; p.cos_t = cos_t; p.sin_t = sin_t; p.table_rows = table_rows;
+  p.window = window; p.scale = scale; p.turn = reinterpret_cast<const float2*>(turn); p.table_rows = table_rows;
   p.splits = window_splits(batch, heads, kv_heads, std::max<int64_t>(most, 1));
   p.part_ml = static_cast<float*>(workspace);
   p.part_o = p.part_ml ? p.part_ml + static_cast<int64_t>(batch) * p.splits * heads * 2 : nullptr;

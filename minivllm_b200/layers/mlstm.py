@@ -49,15 +49,16 @@ def mlstm_scan(q, k, v, chain, cu, slots, starts, S, n, heads, dim, vdim, chunke
     return out, den
 
 
-def mlstm_step(q, k, v, gates, i_b, f_b, cap, slots, starts, S, n, m, heads, dim, vdim, gate, norm_w, eps, out=None):
-    """One token per sequence: the normed and gated rows (tokens, heads * vdim).  See mv_mlstm_step."""
-    _cabi.require_cuda(q, k, v, gates, S, n, m, gate, norm_w)
+def mlstm_step(q, k, v, x, gates_w, i_b, f_b, cap, slots, starts, S, n, m, heads, dim, vdim, gate, norm_w, eps, out=None):
+    """One token per sequence: the normed and gated rows (tokens, heads * vdim).  The gates' logits are formed here, from x
+    (tokens, width) and gates_w (2 * heads, width).  See mv_mlstm_step."""
+    _cabi.require_cuda(q, k, v, x, gates_w, S, n, m, gate, norm_w)
     if not q.stride(0) == k.stride(0) == v.stride(0):
         raise ValueError("q, k and v must share a row stride")
     out = torch.empty((q.shape[0], heads * vdim), dtype=q.dtype, device=q.device) if out is None else out
     _cabi.check(_cabi.lib().mv_mlstm_step(
-        out.data_ptr(), out.stride(0), q.data_ptr(), k.data_ptr(), v.data_ptr(), q.stride(0), gates.data_ptr(), gates.stride(0),
-        i_b.data_ptr(), f_b.data_ptr(), cap, slots.numel(), slots.data_ptr(), starts.data_ptr(), S.data_ptr(), n.data_ptr(),
+        out.data_ptr(), out.stride(0), q.data_ptr(), k.data_ptr(), v.data_ptr(), q.stride(0), x.data_ptr(), x.stride(0),
+        gates_w.data_ptr(), x.shape[1], i_b.data_ptr(), f_b.data_ptr(), cap, slots.numel(), slots.data_ptr(), starts.data_ptr(), S.data_ptr(), n.data_ptr(),
         m.data_ptr(), S.shape[0], heads, dim, vdim, dim ** -0.5, gate.data_ptr(), gate.stride(0), norm_w.data_ptr(), eps,
         _cabi.layer_dtype_code(q.dtype), _cabi.stream_ptr()))
     return out
@@ -86,18 +87,19 @@ class MatrixMemory(nn.Module):
     def forward(self, h):
         """h (tokens, width) -> (tokens, width)."""
         ctx = get_context()
-        p, z = self.stacked(h), router_logits(h, self.gates_w)       # the gates' logits stay in 32-bit
+        p = self.stacked(h)
         q, k, v, g = p["q"], p["k"], p["v"], p["g"]
         slots, starts, nd = ctx.state_slots, ctx.state_starts, ctx.num_decode
         S, n, m = (self.slot_state[name] for name in ("S", "n", "m"))
         dims = (self.heads, self.dim, self.vdim)
         y = torch.empty((h.shape[0], self.heads * self.vdim), dtype=h.dtype, device=h.device)
         if nd:                           # sequences with one token come first
-            mlstm_step(q[:nd], k[:nd], v[:nd], z[:nd], self.i_b, self.f_b, self.cap, slots[:nd], starts[:nd], S, n, m, *dims,
+            mlstm_step(q[:nd], k[:nd], v[:nd], h[:nd], self.gates_w, self.i_b, self.f_b, self.cap, slots[:nd], starts[:nd], S, n, m, *dims,
                        g[:nd], self.norm_w, self.eps, out=y[:nd])
         if h.shape[0] > nd:
             cu, at = ctx.portion_cu_q, (slots[nd:], starts[nd:])
-            chain = mlstm_gates(z[nd:], self.i_b, self.f_b, self.cap, cu, *at, m, self.heads)
+            z = router_logits(h[nd:], self.gates_w)          # the gates' logits stay in 32-bit
+            chain = mlstm_gates(z, self.i_b, self.f_b, self.cap, cu, *at, m, self.heads)
             o, den = mlstm_scan(q[nd:], k[nd:], v[nd:], chain, cu, *at, S, n, *dims)
             head_norm_gate(o, g[nd:], self.norm_w, self.heads, self.eps, out=y[nd:], den=den, act="sigmoid")
         return F.linear(y, self.o_w)

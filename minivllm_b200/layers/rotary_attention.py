@@ -22,6 +22,17 @@ def pair_order(size, dims):
     return [i // 2 + (i % 2) * (dims // 2) for i in range(dims)] + list(range(dims, size))
 
 
+_turn_tables = {}
+
+
+def turn_table(base, dims, max_position, device):
+    """(dims / 2, max_position, 2) fp32: cos and sin of position * base^(-2i / dims), positions side by side."""
+    key = (float(base), int(dims), int(max_position), str(device))
+    if key not in _turn_tables:
+        _turn_tables[key] = torch.stack([t.t() for t in rope_table(base, dims, max_position, device)], 2).contiguous()
+    return _turn_tables[key]
+
+
 def _reorder(w, heads, order, dim=0):
     """Puts the columns of every head, along dimension `dim` of w, into `order`."""
     if order == list(range(len(order))):
@@ -121,6 +132,7 @@ class RotaryWindowAttention(nn.Module):
         tokens = q.shape[0]
         table = rope_table(self.base, self.dims, self.max_position, h.device) if self.dims else None
         vtable = rope_table(self.base, self.vdim, self.max_position, h.device)
+        turn = turn_table(self.base, self.vdim, self.max_position, h.device)
         tiles = tokens > nd and self._tiles(q.dtype)
         fresh = tiles and ctx.portion_fresh
         kv = qkv_rope_store(q, p.get("k"), p.get("v"), self.q_norm, self.k_norm, self.temp, self.eps, ctx.positions, table, self.dims,
@@ -131,13 +143,13 @@ class RotaryWindowAttention(nn.Module):
         o = torch.empty((tokens, self.heads * self.vdim), dtype=q.dtype, device=q.device)
         if nd:                           # sequences with one token come first
             args = (q[:nd], cache, ctx.block_tables[:nd])
-            if window_decode(*args, ctx.positions[:nd], *sizes, out=o[:nd], turn=vtable) is None:
-                window_attention_rows(*args, None, ctx.positions[:nd], *sizes, out=o[:nd], turn=vtable)
+            if window_decode(*args, ctx.positions[:nd], *sizes, out=o[:nd], turn=turn) is None:
+                window_attention_rows(*args, None, ctx.positions[:nd], *sizes, out=o[:nd], turn=turn)
         if tokens > nd:
             tables, cu_q, pos = ctx.block_tables[nd:], ctx.portion_cu_q, ctx.positions[nd:]
             if not tiles:
-                window_attention_rows(q[nd:], cache, tables, cu_q, pos, *sizes, out=o[nd:], turn=vtable)
+                window_attention_rows(q[nd:], cache, tables, cu_q, pos, *sizes, out=o[nd:], turn=turn)
             else:
                 rows, cu_k = self._portion_rows(ctx, fresh, kv[nd:] if fresh else None, tables)
-                window_prefill(q[nd:], rows, cu_q, cu_k, *sizes, out=o[nd:], turn=vtable, positions=pos)
+                window_prefill(q[nd:], rows, cu_q, cu_k, *sizes, out=o[nd:], turn=turn, positions=pos)
         return F.linear(o, self.o_w)

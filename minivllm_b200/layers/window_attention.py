@@ -59,8 +59,8 @@ def _bias_args(bias):
 
 
 def _turn_args(turn):
-    """turn: (cos, sin) tables (positions, vdim / 2) by whose angles results are turned back, or None."""
-    return (turn[0].data_ptr(), turn[1].data_ptr(), turn[0].shape[0]) if turn is not None else (None, None, 0)
+    """turn: (vdim / 2, positions, 2) fp32 (cos, sin) of the angles by which results are turned back, or None."""
+    return (turn.data_ptr(), turn.shape[1]) if turn is not None else (None, 0)
 
 
 def window_attention_rows(q, cache, block_tables, cu_q, positions, kv_heads, dim, vdim, window, scale, bias=None, sink=None,

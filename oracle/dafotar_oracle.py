@@ -195,11 +195,11 @@ def random_weights(config, seed=0):
         H, d, vd = m["heads"], m["dim"], m["vdim"]
         if layer["type"] == "mlstm":
             w.update({p + "q": mat(H * d, W), p + "k": mat(H * d, W), p + "v": mat(H * vd, W), p + "g": mat(H * vd, W),
-                      p + "o": mat(W, H * vd, 2.0), p + "norm": around(H * vd, 1.0, 0.1), p + "i": mat(H, W, 2.0),
-                      p + "i.b": around(H, 0.0, 2.0), p + "f": mat(H, W), p + "f.b": around(H, 3.0, 1.0)})
+                      p + "o": mat(W, H * vd), p + "norm": around(H * vd, 1.0, 0.1), p + "i": mat(H, W),
+                      p + "i.b": around(H, -1.0, 1.0), p + "f": mat(H, W), p + "f.b": around(H, 3.0, 1.0)})
         else:
-            w.update({p + "q": mat(H * d, W), p + "q.norm": around(d, 1.0, 0.2), p + "temp": around(H, 1.5, 0.4),
-                      p + "o": mat(W, H * vd, 2.0)})
+            w.update({p + "q": mat(H * d, W), p + "q.norm": around(d, 1.0, 0.2), p + "temp": around(H, 1.2, 0.3),
+                      p + "o": mat(W, H * vd, 1.5)})
             if "kv_from" not in m:
                 w.update({p + "k": mat(m["kv_heads"] * d, W), p + "v": mat(m["kv_heads"] * vd, W), p + "k.norm": around(d, 1.0, 0.2)})
         if layer.get("mlp"):
