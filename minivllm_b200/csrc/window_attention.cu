@@ -95,6 +95,18 @@ __device__ __forceinline__ int64_t table_row(int64_t pos, int64_t rows) { return
 // The pairs of neighbouring columns c .. c + V - 1 of a row of `dims` rotated columns, turned by the table's angles.
 template <int V>
 __device__ __forceinline__ void turn_pairs(float (&x)[V], int c, int dims, const float* __restrict__ cos_row, const float* __restrict__ sin_row) {
+  if (V == 8 && dims % 8 == 0) {         // rows of whole 16-byte pieces
+    if (c >= dims) return;
+    const float4 co = __ldg(reinterpret_cast<const float4*>(cos_row + c / 2)), si = __ldg(reinterpret_cast<const float4*>(sin_row + c / 2));
+    const float cs[4] = {co.x, co.y, co.z, co.w}, sn[4] = {si.x, si.y, si.z, si.w};
+#pragma unroll
+    for (int e = 0; e < V / 2; ++e) {
+      const float a = x[2 * e], b = x[2 * e + 1];
+      x[2 * e] = a * cs[e & 3] - b * sn[e & 3];
+      x[2 * e + 1] = b * cs[e & 3] + a * sn[e & 3];
+    }
+    return;
+  }
 #pragma unroll
   for (int e = 0; e < V; e += 2) {
     if (c + e >= dims) return;
@@ -128,12 +140,12 @@ template <typename T> struct RopeStoreParams {
 template <typename T, int V, int L, int kCh>
 __global__ void __launch_bounds__(kKnThreads) qkv_rope_store_kernel(const RopeStoreParams<T> p) {
   const int lane = threadIdx.x & (L - 1), per = p.heads + 2 * p.kv_heads, row = p.kv_heads * (p.dim + p.vdim);
-  const int64_t items = p.tokens * per, step = static_cast<int64_t>(gridDim.x) * (kKnThreads / L);
-  for (int64_t i0 = static_cast<int64_t>(blockIdx.x) * (kKnThreads / L); i0 < items; i0 += step) {
-    const int64_t i = i0 + threadIdx.x / L;
+  const uint32_t items = static_cast<uint32_t>(p.tokens * per), step = gridDim.x * (kKnThreads / L);      // the host checks the range
+  for (uint32_t i0 = blockIdx.x * (kKnThreads / L); i0 < items; i0 += step) {
+    const uint32_t i = i0 + threadIdx.x / L, row_i = i / static_cast<uint32_t>(per);
     const bool on = i < items;                 // lanes of a warp stay together for the sums
-    const int64_t t = on ? i / per : 0;
-    const int item = on ? static_cast<int>(i - t * per) : 0;
+    const int64_t t = on ? row_i : 0;
+    const int item = on ? static_cast<int>(i - row_i * per) : 0;
     const bool is_q = item < p.heads, is_v = item >= p.heads + p.kv_heads;
     const int head = is_q ? item : is_v ? item - p.heads - p.kv_heads : item - p.heads, n = is_v ? p.vdim : p.dim;
     const T* src = is_q ? p.q : is_v ? p.v : p.k;
@@ -178,9 +190,16 @@ __global__ void __launch_bounds__(kKnThreads) qkv_rope_store_kernel(const RopeSt
       const int c = (k * L + lane) * V;
       if (!on || c >= n) continue;
       if (!is_v) {
+        if constexpr (V == 8) {
+          float w[8];
+          Vec<T, 8>::load(weight + c, w);
 #pragma unroll
-        for (int e = 0; e < V; ++e)
-          if (V == 8 || c + e < n) x[k][e] = x[k][e] * rs * Elem<T>::to_f(weight[c + e]);
+          for (int e = 0; e < 8; ++e) x[k][e] *= rs * w[e];
+        } else {
+#pragma unroll
+          for (int e = 0; e < V; ++e)
+            if (c + e < n) x[k][e] = x[k][e] * rs * Elem<T>::to_f(weight[c + e]);
+        }
       }
       turn_pairs<V>(x[k], c, dims, co + pos * (dims / 2), si + pos * (dims / 2));
 #pragma unroll
@@ -672,6 +691,7 @@ extern "C" int mv_qkv_rope_store(void* q, const void* k, const void* v, int64_t 
     return fail(MV_ERR_SHAPE, "qkv_rope_store: heads %d over %d, dim %d (%d rotated), vdim %d", heads, kv_heads, dim, dims, vdim);
   const int widest = kv_heads ? std::max(dim, vdim) : dim;
   if (widest > 1024) return fail(MV_ERR_LIMIT, "qkv_rope_store: dim %d, vdim %d (at most 1024)", dim, vdim);
+  if (tokens * (heads + 2 * static_cast<int64_t>(kv_heads)) >= 1LL << 31) return fail(MV_ERR_LIMIT, "qkv_rope_store: %lld tokens", static_cast<long long>(tokens));
   if (tokens == 0) return MV_OK;
   if (!q || !q_weight || !positions || (dims && (!cos_t || !sin_t)) || !vcos_t != !vsin_t ||
       (kv_heads && (!k || !v || !k_weight)) || (cache && !slot_mapping))
@@ -689,7 +709,8 @@ extern "C" int mv_qkv_rope_store(void* q, const void* k, const void* v, int64_t 
       return check_launch("qkv_rope_store");
     };
     const bool v8 = dim % 8 == 0 && vdim % 8 == 0 && vec8_ok(q, stride, eb) && vec8_ok(k, stride, eb) && vec8_ok(v, stride, eb) &&
-                    aligned16(kv_out) && aligned16(cache);
+                    aligned16(kv_out) && aligned16(cache) && aligned16(q_weight) && aligned16(k_weight) && aligned16(cos_t) &&
+                    aligned16(sin_t) && aligned16(vcos_t) && aligned16(vsin_t);
     if (v8 && widest <= 64) return go(qkv_rope_store_kernel<T, 8, 8, 1>, 8);
     if (v8 && widest <= 128) return go(qkv_rope_store_kernel<T, 8, 16, 1>, 16);
     if (v8 && widest <= 256) return go(qkv_rope_store_kernel<T, 8, 32, 1>, 32);
