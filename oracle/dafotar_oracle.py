@@ -172,8 +172,8 @@ def forward(config, weights, token_ids, dtype=torch.float64, per_layer=None):
 
 def random_weights(config, seed=0):
     """Checkpoint tensors of a configuration from a seed, bfloat16, with every mechanism visible in the output
-    (projections of unit gain, norms around one, streams that differ, forget gates mostly open, input gates of either
-    sign)."""
+    (projections of unit gain, norms around one, streams that differ, forget gates mostly open, input gates around
+    minus one)."""
     g = torch.Generator().manual_seed(seed)
 
     def mat(o, i, gain=1.0):
