@@ -429,8 +429,9 @@ int mv_silu_mul(void* out, const void* gate_up, int64_t gate_up_stride,
  *                           + sigmoid(shared_gate[t]) * shared[t]   (shared may be null)
  *   mv_pair_residual_norm   the same with y = (norm(a) * w_a + norm(b) * w_b) / 2, no gate
  *   mv_gated_group_norm     out = norm(y * silu(z)) * w
- *   mv_head_norm_gate       out = norm(y / den) * w * act(z), norms over `heads` equal runs; den (rows, heads) may be null;
- *                           w has one run's length, or the row's with full_weight; act MV_ACT_SILU or MV_ACT_SIGMOID
+ *   mv_head_norm_gate       out = norm(y / den) * w * act(z) * mult, norms over `heads` equal runs; den (rows, heads) may be
+ *                           null; w has one run's length, or the row's with full_weight; act MV_ACT_SILU or MV_ACT_SIGMOID;
+ *                           out_stride 0: dense rows
  *   mv_gate_mul             out = gate applied to y (enum mv_act); a row of y is `heads` pieces y_head_stride
  *                           elements apart
  */
@@ -447,8 +448,9 @@ int mv_moe_residual_norm(void* out, float* x, const void* expert_rows, const int
 int mv_pair_residual_norm(void* out, float* x, const void* a, int64_t a_stride, const void* w_a, const
     void* b, int64_t b_stride, const void* w_b, const void* w_post, const void* w_next, float mult,
     int64_t rows, int width, int groups, float eps, int dtype, void* stream);
-int mv_head_norm_gate(void* out, const void* y, int64_t y_stride, const float* den, const void* z, int64_t z_stride,
-    const void* w, int full_weight, int act, int64_t rows, int width, int heads, float eps, int dtype, void* stream);
+int mv_head_norm_gate(void* out, int64_t out_stride, const void* y, int64_t y_stride, const float* den, const void* z,
+    int64_t z_stride, const void* w, int full_weight, int act, float mult, int64_t rows, int width, int heads, float eps,
+    int dtype, void* stream);
 int mv_gated_group_norm(void* out, const void* y, int64_t y_stride, const void* z, int64_t z_stride,
     const void* w, int64_t rows, int width, int groups, float eps, int dtype, void* stream);
 int mv_gate_mul(void* out, const void* y, int64_t y_stride, int64_t y_head_stride, int heads,
@@ -504,8 +506,9 @@ int mv_ssm_scan(void* y, const void* xbc, const void* dt, int64_t dt_stride, con
 
 /*
  * Mixture of experts; the routing never leaves the device.
- *   mv_moe_route    idx, weight (tokens, top): largest logits + bias, softmax over them.  With `groups` > 1 the
- *                   experts are that many equal runs, and only those of the `keep` runs with the largest maxima count
+ *   mv_moe_route    idx, weight (tokens, top): largest logits + bias, softmax over them (with over_all: over all
+ *                   experts), times scale.  With `groups` > 1 the experts are that many equal runs, and only those of the
+ *                   `keep` runs with the largest maxima can be chosen
  *   mv_moe_sort     stable sort of the tokens * top entries by expert: pos[entry] = row, row_token[row] = token,
  *                   offsets (experts + 1) = row ranges
  *   mv_gather_rows  out[r] = x[row_token[r]]
@@ -514,7 +517,7 @@ int mv_ssm_scan(void* y, const void* xbc, const void* dt, int64_t dt_stride, con
  * No counterpart in the reference.
  */
 int mv_moe_route(int32_t* idx, float* weight, const float* logits, int64_t logits_stride, const
-    float* bias, int64_t tokens, int experts, int top, int groups, int keep, void* stream);
+    float* bias, int64_t tokens, int experts, int top, int groups, int keep, int over_all, float scale, void* stream);
 int64_t mv_moe_sort_workspace_bytes(int64_t tokens, int experts, int top);
 int mv_moe_sort(int32_t* pos, int32_t* row_token, int32_t* offsets, const int32_t* idx, int64_t
     tokens, int experts, int top, void* workspace, int64_t workspace_bytes, void* stream);
@@ -595,8 +598,9 @@ int mv_ssm_step(void* y, const void* u, int64_t u_stride, const void* w, const v
  *   mv_qkv_rope_store         q (in place) and k: RMS norm per head with a weight (dim), then pairs of neighbouring columns
  *                             2i, 2i + 1 of the first `dims` turned by the angle in row positions[t], column i of cos_t and
  *                             sin_t (table_rows, dims / 2); q of head h times temp[h] (null: 1).  v: its pairs turned by
- *                             vcos_t, vsin_t (table_rows, vdim / 2; null: as it is).  [k | v] goes to kv_out and cache as
- *                             above; kv_heads 0: queries only.  dim and vdim up to 1,024
+ *                             vcos_t, vsin_t (table_rows, vdim / 2; null: as it is).  [k: kv_heads * dim | v: v_heads *
+ *                             vdim] goes to kv_out and cache as above; kv_heads and v_heads 0: queries only; heads 0: keys and
+ *                             values only; k_weight null: keys without a norm.  dim and vdim up to 1,024
  * turn (vdim / 2, table_rows, 2) of the attention entries: the result of position i is turned in the same pairs by the
  * opposite of the angles whose (cos, sin) are at [pair, i] (null: not).  out is (tokens, heads * vdim).  No counterpart in the reference.
  */
@@ -606,7 +610,7 @@ int mv_kv_norm_store(void* q, const void* k, const void* v, int64_t stride, cons
 int mv_qkv_rope_store(void* q, const void* k, const void* v, int64_t stride, const void* q_weight, const
     void* k_weight, const void* temp, const float* cos_t, const float* sin_t, int dims, const float*
     vcos_t, const float* vsin_t, int64_t table_rows, const int64_t* positions, void* kv_out, void* cache,
-    const int64_t* slot_mapping, int64_t num_slots, int64_t tokens, int heads, int kv_heads, int dim,
+    const int64_t* slot_mapping, int64_t num_slots, int64_t tokens, int heads, int kv_heads, int v_heads, int dim,
     int vdim, float eps, int dtype, void* stream);
 int mv_window_attention_rows(void* out, const void* q, int64_t q_stride, const void* cache, const
     int32_t* block_tables, int64_t bt_stride, int max_blocks, int block_size, int64_t num_blocks,
@@ -715,6 +719,100 @@ int mv_stream_step(void* out, void* raw, float* x, const int64_t* ids, const voi
     const void* norm_b, const void* taps_t, int taps, void* conv_state, const int32_t* slots, const int32_t*
     start, int num_slots, int64_t conv_rows, int64_t rows, int width, int streams, float eps, int dtype,
     void* stream);
+
+/*
+ * Grouped-query attention whose softmax weights are mixed across the heads, over the same kind of cache (key and value rows of
+ * kv_heads heads each), causal:
+ *   s = cap tanh(scale (q . k) / cap) - r1[h] ln(1 + r2[h] (i - j)),  w = softmax over j <= i,
+ *   w'_h = sum_g talk[h, g] w_g,  out_h = out_scale sum_j w'_h(j) v_j of h's own value head
+ * r1, r2 (heads) and talk (heads, heads) fp32.
+ *   mv_talk_decode          one token per sequence, bf16, dim and vdim multiples of 8 up to 256, cap up to 60; workspace_bytes is
+ *                           -1 when sizes or cap are not taken, most_keys = max_blocks * block_size
+ *   mv_talk_prefill         packed queries, keys and values (row strides in elements) as in mv_window_prefill, bf16, dim up to
+ *                           128, vdim up to 256, multiples of 8, cap up to 60 (mv_talk_prefill_takes): a (tokens, heads,
+ *                           kv_heads, vdim) = every head's w over the values of every value head
+ *   mv_talk_attention_rows  any sizes, a as above in fp32; cu_q as in mv_window_attention_rows
+ *   mv_head_mix             out_h = out_scale sum_g talk[h, g] a[g, value head of h]; a in fp32 or in the type of out
+ * No counterpart in the reference.
+ */
+int64_t mv_talk_decode_workspace_bytes(int batch, int heads, int kv_heads, int dim, int vdim, float cap, int64_t most_keys);
+int mv_talk_decode(void* out, int64_t out_stride, const void* q, int64_t q_stride, const void* cache, const int32_t*
+    block_tables, int64_t bt_stride, int max_blocks, int block_size, int64_t num_blocks, const int64_t* positions,
+    const float* r1, const float* r2, const float* talk, float cap, int batch, int heads, int kv_heads, int dim, int
+    vdim, float scale, float out_scale, void* workspace, int64_t workspace_bytes, void* stream);
+int mv_talk_prefill_takes(int dim, int vdim, float cap);
+int mv_talk_prefill(void* a, const void* q, int64_t q_stride, const void* k, int64_t k_stride, const void* v, int64_t
+    v_stride, const int32_t* cu_q, const int32_t* cu_k, int num_seqs, int64_t tokens, int64_t keys, const float* r1,
+    const float* r2, float cap, int heads, int kv_heads, int dim, int vdim, float scale, int* error_word, void* stream);
+int mv_talk_attention_rows(float* a, const void* q, int64_t q_stride, const void* cache, const int32_t* block_tables,
+    int64_t bt_stride, int max_blocks, int block_size, int64_t num_blocks, const int32_t* cu_q, int num_seqs, const
+    int64_t* positions, const float* r1, const float* r2, float cap, int64_t tokens, int heads, int kv_heads, int dim,
+    int vdim, float scale, int dtype, void* stream);
+int mv_head_mix(void* out, int64_t out_stride, const void* a, int a_dtype, const float* talk, float out_scale, int64_t
+    tokens, int heads, int kv_heads, int vdim, int dtype, void* stream);
+
+/*
+ * Differential attention in chunks: a head has two maps, with queries (heads, 2, dim) and keys (kv_heads, 2, dim) of their own
+ * and the same values; position i sees j <= i with floor(j / chunk) = floor(i / chunk).  Cache rows are [kv_heads * 2 * dim keys
+ * | kv_heads * vdim values].  out = rms_norm(a1 - lambda a2) mult sigmoid(gate), the norm over the head's vdim, without weight.
+ *   mv_diff_decode          one token per sequence, bf16, dim up to 128, vdim up to 256, multiples of 8; workspace_bytes is -1
+ *                           when the sizes are not taken, most_keys = min(chunk, max_blocks * block_size)
+ *   mv_diff_prefill         packed rows; a sequence's keys begin at the beginning of a chunk; scale > 0; bf16, dim and vdim up to
+ *                           128, multiples of 8 (mv_diff_prefill_takes)
+ *   mv_diff_attention_rows  any sizes: a (tokens, heads, 2, vdim) = a1 and a2 in fp32
+ *   mv_diff_norm_gate       the rest of it, from a
+ * No counterpart in the reference.
+ */
+int64_t mv_diff_decode_workspace_bytes(int batch, int heads, int kv_heads, int dim, int vdim, int64_t most_keys);
+int mv_diff_decode(void* out, const void* q, int64_t q_stride, const void* cache, const int32_t* block_tables, int64_t
+    bt_stride, int max_blocks, int block_size, int64_t num_blocks, const int64_t* positions, int64_t chunk, const void*
+    gate, int64_t gate_stride, float lambda, float mult, float eps, int batch, int heads, int kv_heads, int dim, int
+    vdim, float scale, void* workspace, int64_t workspace_bytes, void* stream);
+int mv_diff_prefill_takes(int dim, int vdim);
+int mv_diff_prefill(void* out, const void* q, int64_t q_stride, const void* k, int64_t k_stride, const void* v, int64_t
+    v_stride, const int32_t* cu_q, const int32_t* cu_k, int num_seqs, int64_t tokens, int64_t keys, int64_t chunk,
+    const void* gate, int64_t gate_stride, float lambda, float mult, float eps, int heads, int kv_heads,
+    int dim, int vdim, float scale, int* error_word, void* stream);
+int mv_diff_attention_rows(float* a, const void* q, int64_t q_stride, const void* cache, const int32_t* block_tables,
+    int64_t bt_stride, int max_blocks, int block_size, int64_t num_blocks, const int32_t* cu_q, int num_seqs, const
+    int64_t* positions, int64_t chunk, int64_t tokens, int heads, int kv_heads, int dim, int vdim, float scale, int
+    dtype, void* stream);
+int mv_diff_norm_gate(void* out, const float* a, const void* gate, int64_t gate_stride, float lambda, float mult, float
+    eps, int64_t tokens, int heads, int vdim, int dtype, void* stream);
+
+/*
+ * Time mixing on a matrix state: o = (S + diag(bonus) k v^T)^T r, then S <- diag(exp(-exp(z + w0))) S + k v^T; z (tokens, heads *
+ * dim) fp32, w0 and bonus (heads, dim); state, cu, slots and start as in mv_gla_scan.  With cu null the norm and the gate follow:
+ * out = rms_norm(o) * norm_w * silu(gate) * out_scale, norm_w (heads * vdim).  mv_time_chunk_scan: portions in chunks of 64 tokens
+ * on tensor cores, with the sizes and the workspace of mv_gla_chunk_scan.  No counterpart in the reference.
+ */
+int mv_time_scan(void* out, int64_t out_stride, const void* r, const void* k, const void* v, int64_t stride, const float*
+    z, int64_t z_stride, const void* w0, const void* bonus, const int32_t* cu, int num_seqs, const int32_t* slots, const
+    int32_t* start, float* state, int num_slots, int heads, int dim, int vdim, const void* gate, int64_t gate_stride,
+    const void* norm_w, float eps, float out_scale, int dtype, void* stream);
+int mv_time_chunk_scan(void* out, int64_t out_stride, const void* r, const void* k, const void* v, int64_t stride, const
+    float* z, int64_t z_stride, const void* w0, const void* bonus, const int32_t* cu, int num_seqs, int64_t tokens, const
+    int32_t* slots, const int32_t* start, float* state, int num_slots, int heads, int dim, int vdim, void* workspace,
+    int64_t workspace_bytes, void* stream);
+
+/*
+ * Between two sublayers of a decoder with one fp32 residual stream and an element-wise norm: out = tanh(alpha x') w + b, where
+ * x_out = x' is x_in plus y (rows, y_stride), or plus sum_k top_weights[t, k] y[pos[t, k]] (pos not null), or with ids the
+ * embedding row, to which sin(position inv_freq[i]) and cos of the same are added in columns 2i and 2i + 1 (inv_freq null: not).
+ * mixes > 0: mixed[m] (rows, width) = out + (before - out) mu[m], with the out of the sequence's token before (zeros for its
+ * first); kept (num_slots, width) holds the last one.  A sequence with one row in this step moves its kept row on; for longer
+ * ones mv_conv_state_update does it afterwards.  With mixes x_out and x_in must differ.  cu, slots and start as in mv_conv_silu.
+ *   mv_xielu      out = a z^2 + z / 2 for z > 0, else b (e^z - 1 - z) + z / 2
+ *   mv_tanh_rows  out = tanh(y), y in fp32
+ * dtype MV_BF16 or MV_F32 of all but x, y of mv_tanh_rows and top_weights.  No counterpart in the reference.
+ */
+int mv_tanh_step(void* out, float* x_out, const float* x_in, const int64_t* ids, const void* embed, int64_t vocab, const
+    int64_t* positions, const double* inv_freq, const void* y, int64_t y_stride, const int32_t* pos, const float*
+    top_weights, int top, float alpha, const void* w, const void* b, void* mixed, const void* mu, int mixes, void* kept,
+    const int32_t* slots, const int32_t* start, int num_slots, const int32_t* cu, int num_seqs, int64_t rows, int width,
+    int dtype, void* stream);
+int mv_xielu(void* out, const void* y, int64_t y_stride, float a, float b, int64_t rows, int cols, int dtype, void* stream);
+int mv_tanh_rows(void* out, const float* y, int64_t y_stride, int64_t rows, int cols, int dtype, void* stream);
 
 #ifdef __cplusplus
 }

@@ -75,8 +75,8 @@ SIGNATURES = {
         _c_i64, _c_ptr, _c_i64, _c_ptr, _c_ptr, _c_ptr, _c_f32, _c_i64, _c_int, _c_int, _c_f32, _c_int, _c_ptr]),
     "mv_pair_residual_norm": (_c_int, [_c_ptr, _c_ptr, _c_ptr, _c_i64, _c_ptr, _c_ptr, _c_i64, _c_ptr, _c_ptr, _c_ptr,
         _c_f32, _c_i64, _c_int, _c_int, _c_f32, _c_int, _c_ptr]),
-    "mv_head_norm_gate": (_c_int, [_c_ptr, _c_ptr, _c_i64, _c_ptr, _c_ptr, _c_i64, _c_ptr, _c_int, _c_int, _c_i64, _c_int, _c_int,
-        _c_f32, _c_int, _c_ptr]),
+    "mv_head_norm_gate": (_c_int, [_c_ptr, _c_i64, _c_ptr, _c_i64, _c_ptr, _c_ptr, _c_i64, _c_ptr, _c_int, _c_int,
+        _c_f32, _c_i64, _c_int, _c_int, _c_f32, _c_int, _c_ptr]),
     "mv_gated_group_norm": (_c_int, [_c_ptr, _c_ptr, _c_i64, _c_ptr, _c_i64, _c_ptr, _c_i64, _c_int, _c_int, _c_f32,
         _c_int, _c_ptr]),
     "mv_gate_mul": (_c_int, [_c_ptr, _c_ptr, _c_i64, _c_i64, _c_int, _c_ptr, _c_i64, _c_int, _c_f32, _c_i64, _c_int, _c_int,
@@ -94,7 +94,8 @@ SIGNATURES = {
         _c_int, _c_int, _c_ptr]),
     "mv_ssm_scan": (_c_int, [_c_ptr, _c_ptr, _c_ptr, _c_i64, _c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_int, _c_ptr, _c_ptr,
         _c_ptr, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_ptr]),
-    "mv_moe_route": (_c_int, [_c_ptr, _c_ptr, _c_ptr, _c_i64, _c_ptr, _c_i64, _c_int, _c_int, _c_int, _c_int, _c_ptr]),
+    "mv_moe_route": (_c_int, [_c_ptr, _c_ptr, _c_ptr, _c_i64, _c_ptr, _c_i64, _c_int, _c_int, _c_int, _c_int, _c_int,
+        _c_f32, _c_ptr]),
     "mv_moe_sort_workspace_bytes": (_c_i64, [_c_i64, _c_int, _c_int]),
     "mv_moe_sort": (_c_int, [_c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_i64, _c_int, _c_int, _c_ptr, _c_i64, _c_ptr]),
     "mv_gather_rows": (_c_int, [_c_ptr, _c_ptr, _c_i64, _c_ptr, _c_i64, _c_int, _c_int, _c_ptr]),
@@ -139,9 +140,9 @@ SIGNATURES = {
     "mv_delta_chunk_workspace_bytes": (_c_i64, [_c_i64, _c_int, _c_int, _c_int, _c_int]),
     "mv_delta_chunk_scan": (_c_int, [_c_ptr, _c_i64, _c_ptr, _c_i64, _c_ptr, _c_ptr, _c_i64, _c_ptr, _c_ptr, _c_ptr, _c_int,
         _c_i64, _c_ptr, _c_ptr, _c_ptr, _c_int, _c_int, _c_int, _c_int, _c_int, _c_f32, _c_ptr, _c_i64, _c_ptr]),
-        "mv_qkv_rope_store": (_c_int, [_c_ptr, _c_ptr, _c_ptr, _c_i64, _c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_int,
+    "mv_qkv_rope_store": (_c_int, [_c_ptr, _c_ptr, _c_ptr, _c_i64, _c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_int,
         _c_ptr, _c_ptr, _c_i64, _c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_i64, _c_i64, _c_int, _c_int, _c_int, _c_int,
-        _c_f32, _c_int, _c_ptr]),
+        _c_int, _c_f32, _c_int, _c_ptr]),
         "mv_mlstm_gates": (_c_int, [_c_ptr, _c_ptr, _c_i64, _c_ptr, _c_ptr, _c_f32, _c_ptr, _c_int, _c_ptr, _c_ptr,
         _c_ptr, _c_int, _c_int, _c_int, _c_ptr]),
         "mv_mlstm_scan": (_c_int, [_c_ptr, _c_i64, _c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_i64, _c_ptr, _c_ptr, _c_int,
@@ -156,6 +157,40 @@ SIGNATURES = {
     "mv_stream_step": (_c_int, [_c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_i64, _c_ptr, _c_i64, _c_ptr, _c_ptr,
         _c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_int, _c_ptr, _c_ptr, _c_ptr, _c_int, _c_i64, _c_i64, _c_int, _c_int,
         _c_f32, _c_int, _c_ptr]),
+    "mv_talk_decode_workspace_bytes": (_c_i64, [_c_int, _c_int, _c_int, _c_int, _c_int, _c_f32, _c_i64]),
+    "mv_talk_decode": (_c_int, [_c_ptr, _c_i64, _c_ptr, _c_i64, _c_ptr, _c_ptr, _c_i64, _c_int, _c_int, _c_i64,
+        _c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_f32, _c_int, _c_int, _c_int, _c_int, _c_int, _c_f32, _c_f32, _c_ptr,
+        _c_i64, _c_ptr]),
+    "mv_talk_prefill_takes": (_c_int, [_c_int, _c_int, _c_f32]),
+    "mv_talk_prefill": (_c_int, [_c_ptr, _c_ptr, _c_i64, _c_ptr, _c_i64, _c_ptr, _c_i64, _c_ptr, _c_ptr, _c_int,
+        _c_i64, _c_i64, _c_ptr, _c_ptr, _c_f32, _c_int, _c_int, _c_int, _c_int, _c_f32, _c_ptr, _c_ptr]),
+    "mv_talk_attention_rows": (_c_int, [_c_ptr, _c_ptr, _c_i64, _c_ptr, _c_ptr, _c_i64, _c_int, _c_int, _c_i64,
+        _c_ptr, _c_int, _c_ptr, _c_ptr, _c_ptr, _c_f32, _c_i64, _c_int, _c_int, _c_int, _c_int, _c_f32, _c_int,
+        _c_ptr]),
+    "mv_head_mix": (_c_int, [_c_ptr, _c_i64, _c_ptr, _c_int, _c_ptr, _c_f32, _c_i64, _c_int, _c_int, _c_int, _c_int,
+        _c_ptr]),
+    "mv_diff_decode_workspace_bytes": (_c_i64, [_c_int, _c_int, _c_int, _c_int, _c_int, _c_i64]),
+    "mv_diff_decode": (_c_int, [_c_ptr, _c_ptr, _c_i64, _c_ptr, _c_ptr, _c_i64, _c_int, _c_int, _c_i64, _c_ptr,
+        _c_i64, _c_ptr, _c_i64, _c_f32, _c_f32, _c_f32, _c_int, _c_int, _c_int, _c_int, _c_int, _c_f32, _c_ptr,
+        _c_i64, _c_ptr]),
+    "mv_diff_prefill_takes": (_c_int, [_c_int, _c_int]),
+    "mv_diff_prefill": (_c_int, [_c_ptr, _c_ptr, _c_i64, _c_ptr, _c_i64, _c_ptr, _c_i64, _c_ptr, _c_ptr, _c_int,
+        _c_i64, _c_i64, _c_i64, _c_ptr, _c_i64, _c_f32, _c_f32, _c_f32, _c_int, _c_int, _c_int, _c_int, _c_f32,
+        _c_ptr, _c_ptr]),
+    "mv_diff_attention_rows": (_c_int, [_c_ptr, _c_ptr, _c_i64, _c_ptr, _c_ptr, _c_i64, _c_int, _c_int, _c_i64,
+        _c_ptr, _c_int, _c_ptr, _c_i64, _c_i64, _c_int, _c_int, _c_int, _c_int, _c_f32, _c_int, _c_ptr]),
+    "mv_diff_norm_gate": (_c_int, [_c_ptr, _c_ptr, _c_ptr, _c_i64, _c_f32, _c_f32, _c_f32, _c_i64, _c_int, _c_int,
+        _c_int, _c_ptr]),
+    "mv_time_scan": (_c_int, [_c_ptr, _c_i64, _c_ptr, _c_ptr, _c_ptr, _c_i64, _c_ptr, _c_i64, _c_ptr, _c_ptr, _c_ptr,
+        _c_int, _c_ptr, _c_ptr, _c_ptr, _c_int, _c_int, _c_int, _c_int, _c_ptr, _c_i64, _c_ptr, _c_f32, _c_f32,
+        _c_int, _c_ptr]),
+    "mv_time_chunk_scan": (_c_int, [_c_ptr, _c_i64, _c_ptr, _c_ptr, _c_ptr, _c_i64, _c_ptr, _c_i64, _c_ptr, _c_ptr,
+        _c_ptr, _c_int, _c_i64, _c_ptr, _c_ptr, _c_ptr, _c_int, _c_int, _c_int, _c_int, _c_ptr, _c_i64, _c_ptr]),
+    "mv_tanh_step": (_c_int, [_c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_i64, _c_ptr, _c_ptr, _c_ptr, _c_i64, _c_ptr,
+        _c_ptr, _c_int, _c_f32, _c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_int, _c_ptr, _c_ptr, _c_ptr, _c_int, _c_ptr,
+        _c_int, _c_i64, _c_int, _c_int, _c_ptr]),
+    "mv_xielu": (_c_int, [_c_ptr, _c_ptr, _c_i64, _c_f32, _c_f32, _c_i64, _c_int, _c_int, _c_ptr]),
+    "mv_tanh_rows": (_c_int, [_c_ptr, _c_ptr, _c_i64, _c_i64, _c_int, _c_int, _c_ptr]),
 }
 
 _lib = None

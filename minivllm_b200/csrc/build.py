@@ -22,6 +22,8 @@ GROUPS = {
     "fozerax": ["norms.cu", "window_attention.cu", "latent_prefill.cu", "short_conv.cu", "gla.cu", "gla_chunk.cu", "gated_delta.cu",
                 "gated_delta_chunk.cu", "moe.cu", "grouped_gemm.cu"],
     "dafotar": ["norms.cu", "streams.cu", "short_conv.cu", "window_attention.cu", "latent_prefill.cu", "mlstm.cu", "mlstm_chunk.cu"],
+    "subivik": ["norms.cu", "tanh_norm.cu", "short_conv.cu", "window_attention.cu", "latent_prefill.cu", "talk_attention.cu",
+                "talk_prefill.cu", "time_mix.cu", "gla_chunk.cu", "moe.cu", "grouped_gemm.cu"],
 }
 SOURCES = COMMON + list(dict.fromkeys(s for g in GROUPS.values() for s in g))
 NVCC_FLAGS = [

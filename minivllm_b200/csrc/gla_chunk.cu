@@ -1,6 +1,8 @@
-// Gated linear attention in chunks of 64 tokens.  With b_t the running sums of the channels' log2 decays inside the chunk:
+// Gated linear attention and time mixing in chunks of 64 tokens.  With b_t the running sums of the channels' log2 decays inside the chunk:
 //   O = (q 2^b) S_0 + A V,      A[t, j] = sum_k q_t k_j 2^(b_t - b_j), j <= t
 //   S = 2^b_last S_0 + (k 2^(b_last - b))^T V
+// Time mixing (kTime) reads the state before the token's own decay: b_(t-1) in the place of b_t beside q, j < t in A, whose
+// diagonal is q_t . (u k_t).
 // gla_prepare_kernel  per chunk and head: b, both decayed operands, A.  A's 16 x 16 blocks are products of factors taken
 //                     against b at one token, on tensor cores in two terms each.  Below the diagonal that is the last token
 //                     before the block's rows, and every power of two is at most one.  On the diagonal it is the block's
@@ -18,6 +20,7 @@ struct GlaChunkParams {
   const __nv_bfloat16 *q, *k, *v; int64_t stride;
   const __nv_bfloat16* z; int64_t z_stride;
   float inv_tau, q_scale;
+  const float* zf; const __nv_bfloat16 *w0, *bonus;      // time mixing: z in fp32, its offset and the bonus (heads, K)
   const int32_t *cu, *slots, *start;
   int num_seqs;
   float* state; int num_slots, heads, K, V;
@@ -31,16 +34,17 @@ template <int K> struct GlaScratch {
 
 template <int K> struct GlaPrepShape {
   static constexpr int kRow = K + 8, kB = K + 4;
-  static constexpr int kBytes = 2 * kChunk * kRow * 2 + kChunk * kB * 4;
+  static constexpr int kBytes = 2 * kChunk * kRow * 2 + (kChunk + 1) * kB * 4 + kChunk * 4;
 };
 
-template <int K>
+template <int K, bool kTime>
 __global__ void __launch_bounds__(kGpThreads) gla_prepare_kernel(const GlaChunkParams p) {
   using Sh = GlaPrepShape<K>;
   using Sc = GlaScratch<K>;
   extern __shared__ __align__(16) unsigned char smem[];
   __nv_bfloat16 *sQ = reinterpret_cast<__nv_bfloat16*>(smem), *sK = sQ + kChunk * Sh::kRow;
-  float* sB = reinterpret_cast<float*>(sK + kChunk * Sh::kRow);
+  float* sB = reinterpret_cast<float*>(sK + kChunk * Sh::kRow) + Sh::kB;     // a row of zeros in front of token 0
+  float* sOwn = sB + kChunk * Sh::kB;                                        // A's diagonal, time mixing
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, h = blockIdx.y;
   int seq, chunk;
   if (!find_chunk(p.cu, p.num_seqs, blockIdx.x, seq, chunk)) return;     // uniform: the grid is an upper bound
@@ -60,9 +64,13 @@ __global__ void __launch_bounds__(kGpThreads) gla_prepare_kernel(const GlaChunkP
   }
   for (int i = tid; i < kChunk * K; i += kGpThreads) {
     const int r = i / K, c = i % K;
-    sB[r * Sh::kB + c] = r < nt && c < p.K
-        ? channel_log_decay(__bfloat162float(p.z[(first + r) * p.z_stride + h * p.K + c]), p.inv_tau) * kLog2e : 0.f;
+    const int64_t at = (first + r) * p.z_stride + h * p.K + c;
+    float b = 0.f;
+    if (r < nt && c < p.K)
+      b = kTime ? time_log_decay(p.zf[at] + __bfloat162float(p.w0[h * p.K + c])) : channel_log_decay(__bfloat162float(p.z[at]), p.inv_tau);
+    sB[r * Sh::kB + c] = b * kLog2e;
   }
+  for (int c = tid; c < Sh::kB; c += kGpThreads) sB[c - Sh::kB] = 0.f;
   __syncthreads();
   for (int i = tid; i < 4 * K; i += kGpThreads) {        // running sums of 16 tokens
     float* b = sB + (i / K) * 16 * Sh::kB + i % K;
@@ -87,16 +95,27 @@ __global__ void __launch_bounds__(kGpThreads) gla_prepare_kernel(const GlaChunkP
   }
   cp_async_wait<0>();
   __syncthreads();
+  if (kTime) {
+    for (int t = warp; t < kChunk; t += kGpThreads / 32) {
+      float own = 0.f;
+      for (int c = lane; c < p.K; c += 32)
+        own = fmaf(__bfloat162float(sQ[t * Sh::kRow + c]) * __bfloat162float(p.bonus[h * p.K + c]), __bfloat162float(sK[t * Sh::kRow + c]), own);
+      own = warp_sum(own);
+      if (lane == 0) sOwn[t] = own;
+    }
+    __syncthreads();
+  }
+  const float* sE = kTime ? sB - Sh::kB : sB;            // exponents beside q
   {
     uint32_t* o = reinterpret_cast<uint32_t*>(dst);
     for (int i = tid; i < kChunk * K / 2; i += kGpThreads) {
       const int r = i / (K / 2), c = (i % (K / 2)) * 2;
-      const float2 b = *reinterpret_cast<const float2*>(sB + r * Sh::kB + c);
+      const float2 b = *reinterpret_cast<const float2*>(sB + r * Sh::kB + c), e = *reinterpret_cast<const float2*>(sE + r * Sh::kB + c);
       const float2 last = *reinterpret_cast<const float2*>(sB + (kChunk - 1) * Sh::kB + c);
       const float2 q = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(sQ + r * Sh::kRow + c));
       const float2 k = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(sK + r * Sh::kRow + c));
       uint32_t hi, lo;
-      split2(q.x * p.q_scale * fast_exp2(b.x), q.y * p.q_scale * fast_exp2(b.y), hi, lo);
+      split2(q.x * p.q_scale * fast_exp2(e.x), q.y * p.q_scale * fast_exp2(e.y), hi, lo);
       o[i] = hi;
       o[Sc::kVec / 2 + i] = lo;
       split2(k.x * fast_exp2(last.x - b.x), k.y * fast_exp2(last.y - b.y), hi, lo);
@@ -125,11 +144,16 @@ __global__ void __launch_bounds__(kGpThreads) gla_prepare_kernel(const GlaChunkP
       if (__any_sync(0xffffffffu, least < -60.f)) {
         for (int i = lane; i < 16 * 8; i += 32) {        // two neighbouring keys of one token
           const int t = bi * 16 + (i >> 3), j = bi * 16 + (i & 7) * 2;
+          const int j_end = kTime ? t - 1 : t;
           float x = 0.f, y = 0.f;
-          for (int c = 0; j <= t && c < K; ++c) {
-            const float q = __bfloat162float(sQ[t * Sh::kRow + c]), bt = sB[t * Sh::kB + c];
+          for (int c = 0; j <= j_end && c < K; ++c) {
+            const float q = __bfloat162float(sQ[t * Sh::kRow + c]), bt = sE[t * Sh::kB + c];
             x = fmaf(q * __bfloat162float(sK[j * Sh::kRow + c]), fast_exp2(bt - sB[j * Sh::kB + c]), x);
-            if (j + 1 <= t) y = fmaf(q * __bfloat162float(sK[(j + 1) * Sh::kRow + c]), fast_exp2(bt - sB[(j + 1) * Sh::kB + c]), y);
+            if (j + 1 <= j_end) y = fmaf(q * __bfloat162float(sK[(j + 1) * Sh::kRow + c]), fast_exp2(bt - sB[(j + 1) * Sh::kB + c]), y);
+          }
+          if (kTime) {
+            if (j == t) x = sOwn[t];
+            if (j + 1 == t) y = sOwn[t];
           }
           put(t, j, x * p.q_scale, y * p.q_scale);
         }
@@ -144,7 +168,7 @@ __global__ void __launch_bounds__(kGpThreads) gla_prepare_kernel(const GlaChunkP
       for (int x = 0; x < 4; ++x) {
         // A: rows g, g + 8 of the block's tokens, channels c2 and c2 + 8;  B: n-tiles of eight keys each
         const int c = kb + c2 + (x >> 1) * 8, t = bi * 16 + g + (x & 1) * 8;
-        const float2 r = *reinterpret_cast<const float2*>(ref + c), b = *reinterpret_cast<const float2*>(sB + t * Sh::kB + c);
+        const float2 r = *reinterpret_cast<const float2*>(ref + c), b = *reinterpret_cast<const float2*>(sE + t * Sh::kB + c);
         const float2 q = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(sQ + t * Sh::kRow + c));
         split2(q.x * fast_exp2(b.x - r.x), q.y * fast_exp2(b.y - r.y), ah[x], al[x]);
         const int cj = kb + c2 + (x & 1) * 8, j = bj * 16 + g + (x >> 1) * 8;
@@ -164,7 +188,12 @@ __global__ void __launch_bounds__(kGpThreads) gla_prepare_kernel(const GlaChunkP
 #pragma unroll
       for (int half = 0; half < 2; ++half) {
         const int t = bi * 16 + g + half * 8, j = bj * 16 + n * 8 + c2;
-        put(t, j, j <= t ? acc[n][2 * half] * p.q_scale : 0.f, j + 1 <= t ? acc[n][2 * half + 1] * p.q_scale : 0.f);
+        float x = acc[n][2 * half], y = acc[n][2 * half + 1];
+        if (kTime) {
+          if (j == t) x = sOwn[t];
+          if (j + 1 == t) y = sOwn[t];
+        }
+        put(t, j, j <= t ? x * p.q_scale : 0.f, j + 1 <= t ? y * p.q_scale : 0.f);
       }
   }
 }
@@ -301,37 +330,60 @@ extern "C" int64_t mv_gla_chunk_workspace_bytes(int64_t tokens, int num_seqs, in
   return chunk_bound(tokens, num_seqs) * heads * gla_scratch_bytes(dim);
 }
 
+// Both recurrences; kTime: p.zf, p.w0 and p.bonus, else p.z and p.inv_tau.
+template <bool kTime>
+static int run_chunks(const char* what, const mv::GlaChunkParams& p, int64_t tokens, int64_t workspace_bytes, cudaStream_t st) {
+  using namespace mv;
+  const int num_seqs = p.num_seqs, heads = p.heads, dim = p.K, vdim = p.V;
+  if (num_seqs < 0 || tokens < 0 || heads <= 0 || heads > 65535 || !chunk_takes(dim, vdim))
+    return fail(MV_ERR_SHAPE, "%s: heads %d, dim %d, vdim %d", what, heads, dim, vdim);
+  if (num_seqs == 0 || tokens == 0) return MV_OK;
+  if (!p.out || !p.q || !p.k || !p.v || !(kTime ? p.zf && p.w0 && p.bonus : p.z != nullptr) || !p.cu || !p.slots || !p.start || !p.state)
+    return fail(MV_ERR_NULL, "%s: null pointer", what);
+  if (!vec8_ok(p.out, p.out_stride, 2) || !vec8_ok(p.q, p.stride, 2) || !vec8_ok(p.k, p.stride, 2) || !vec8_ok(p.v, p.stride, 2))
+    return fail(MV_ERR_ALIGN, "%s: rows must start on 16-byte boundaries", what);
+  const int64_t chunks = chunk_bound(tokens, num_seqs);
+  if (!p.scratch || !aligned16(p.scratch) || workspace_bytes < chunks * heads * gla_scratch_bytes(dim))
+    return fail(MV_ERR_WORKSPACE, "%s: workspace", what);
+  return chunk_dispatch(dim, [&](auto kk) {
+    constexpr int K = decltype(kk)::value;
+    constexpr int prep = GlaPrepShape<K>::kBytes;
+    cudaError_t e = cudaFuncSetAttribute(gla_prepare_kernel<K, kTime>, cudaFuncAttributeMaxDynamicSharedMemorySize, prep);
+    if (e != cudaSuccess) return fail(MV_ERR_CUDA, "%s: %s", what, cudaGetErrorString(e));
+    gla_prepare_kernel<K, kTime><<<dim3(static_cast<unsigned>(chunks), heads), kGpThreads, prep, st>>>(p);
+    int rc = check_launch(what);
+    if (rc) return rc;
+    const int pb = chunk_columns(static_cast<int64_t>(num_seqs) * heads, vdim), smem = 2 * GlaChunkShape<K>::stage(pb);
+    e = cudaFuncSetAttribute(gla_chunk_kernel<K>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
+    if (e != cudaSuccess) return fail(MV_ERR_CUDA, "%s: %s", what, cudaGetErrorString(e));
+    gla_chunk_kernel<K><<<dim3(num_seqs, heads, (vdim + pb - 1) / pb), kChunkThreads, smem, st>>>(p, pb);
+    return check_launch(what);
+  });
+}
+
 extern "C" int mv_gla_chunk_scan(void* out, int64_t out_stride, const void* q, const void* k, const void* v, int64_t stride,
                                  const void* z, int64_t z_stride, float tau, const int32_t* cu, int num_seqs,
                                  int64_t tokens, const int32_t* slots, const int32_t* start, float* state, int num_slots,
                                  int heads, int dim, int vdim, float q_scale, void* workspace, int64_t workspace_bytes,
                                  void* stream) {
   using namespace mv;
-  if (num_seqs < 0 || tokens < 0 || heads <= 0 || heads > 65535 || !(tau > 0.f) || !chunk_takes(dim, vdim))
-    return fail(MV_ERR_SHAPE, "gla_chunk_scan: heads %d, dim %d, vdim %d, tau %f", heads, dim, vdim, tau);
-  if (num_seqs == 0 || tokens == 0) return MV_OK;
-  if (!out || !q || !k || !v || !z || !cu || !slots || !start || !state) return fail(MV_ERR_NULL, "gla_chunk_scan: null pointer");
-  if (!vec8_ok(out, out_stride, 2) || !vec8_ok(q, stride, 2) || !vec8_ok(k, stride, 2) || !vec8_ok(v, stride, 2))
-    return fail(MV_ERR_ALIGN, "gla_chunk_scan: rows must start on 16-byte boundaries");
-  const int64_t chunks = chunk_bound(tokens, num_seqs);
-  if (!workspace || !aligned16(workspace) || workspace_bytes < chunks * heads * gla_scratch_bytes(dim))
-    return fail(MV_ERR_WORKSPACE, "gla_chunk_scan: workspace");
+  if (!(tau > 0.f)) return fail(MV_ERR_SHAPE, "gla_chunk_scan: tau %f", tau);
   auto c = [](const void* x) { return static_cast<const __nv_bfloat16*>(x); };
   const GlaChunkParams p{static_cast<__nv_bfloat16*>(out), out_stride, c(q), c(k), c(v), stride, c(z), z_stride, 1.f / tau, q_scale,
+                         nullptr, nullptr, nullptr,
                          cu, slots, start, num_seqs, state, num_slots, heads, dim, vdim, static_cast<unsigned char*>(workspace)};
-  auto st = static_cast<cudaStream_t>(stream);
-  return chunk_dispatch(dim, [&](auto kk) {
-    constexpr int K = decltype(kk)::value;
-    constexpr int prep = GlaPrepShape<K>::kBytes;
-    cudaError_t e = cudaFuncSetAttribute(gla_prepare_kernel<K>, cudaFuncAttributeMaxDynamicSharedMemorySize, prep);
-    if (e != cudaSuccess) return fail(MV_ERR_CUDA, "gla_chunk_scan: %s", cudaGetErrorString(e));
-    gla_prepare_kernel<K><<<dim3(static_cast<unsigned>(chunks), heads), kGpThreads, prep, st>>>(p);
-    int rc = check_launch("gla_prepare");
-    if (rc) return rc;
-    const int pb = chunk_columns(static_cast<int64_t>(num_seqs) * heads, vdim), smem = 2 * GlaChunkShape<K>::stage(pb);
-    e = cudaFuncSetAttribute(gla_chunk_kernel<K>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
-    if (e != cudaSuccess) return fail(MV_ERR_CUDA, "gla_chunk_scan: %s", cudaGetErrorString(e));
-    gla_chunk_kernel<K><<<dim3(num_seqs, heads, (vdim + pb - 1) / pb), kChunkThreads, smem, st>>>(p, pb);
-    return check_launch("gla_chunk");
-  });
+  return run_chunks<false>("gla_chunk_scan", p, tokens, workspace_bytes, static_cast<cudaStream_t>(stream));
+}
+
+extern "C" int mv_time_chunk_scan(void* out, int64_t out_stride, const void* r, const void* k, const void* v, int64_t stride,
+                                  const float* z, int64_t z_stride, const void* w0, const void* bonus, const int32_t* cu,
+                                  int num_seqs, int64_t tokens, const int32_t* slots, const int32_t* start, float* state,
+                                  int num_slots, int heads, int dim, int vdim, void* workspace, int64_t workspace_bytes,
+                                  void* stream) {
+  using namespace mv;
+  auto c = [](const void* x) { return static_cast<const __nv_bfloat16*>(x); };
+  const GlaChunkParams p{static_cast<__nv_bfloat16*>(out), out_stride, c(r), c(k), c(v), stride, nullptr, z_stride, 1.f, 1.f,
+                         z, c(w0), c(bonus),
+                         cu, slots, start, num_seqs, state, num_slots, heads, dim, vdim, static_cast<unsigned char*>(workspace)};
+  return run_chunks<true>("time_chunk_scan", p, tokens, workspace_bytes, static_cast<cudaStream_t>(stream));
 }

@@ -1,7 +1,8 @@
-// Prefill attention on the Blackwell tensor cores, causal, packed batch, an optional sink per head, in two forms:
+// Prefill attention on the Blackwell tensor cores, causal, packed batch, an optional sink per head, in three forms:
 //   latent attention, with keys and values expanded per head (k = [W_uk c | shared rotated part], v = W_uv c);
 //   kWin: grouped-query attention with a sliding window and a bias per distance and head; results may be turned back by
-//   their positions in pairs of neighbouring columns (values that were turned when they were stored).
+//   their positions in pairs of neighbouring columns (values that were turned when they were stored);
+//   kDiff: differential attention in chunks of the sequence: a head has two maps over the same values.
 //
 // The two 128-row problems of a CTA are two consecutive query tiles of ONE head (latent attention: every head has keys of
 // its own): they share each K/V tile.  The K operand is assembled by TMA from two tensors, 64-column boxes of the expanded
@@ -16,9 +17,13 @@
 // distance, from -256 on, with -inf where a distance is not visible, so that one lookup masks and biases a score; tiles
 // whose distances all lie at or beyond the table's last entry add that entry instead.
 //
+// kDiff: the two problems are the two maps of one head on the same query tile; a K stage holds both maps' keys.  In the end each
+// warpgroup takes half of the columns of both results: their difference, its norm over the head, and the output gate.
+//
 // Tensor-bound: FLOPs = 2 * heads * (dim + rot_dim + vdim) * (number of visible (query, key) pairs).
 #include <algorithm>
 #include "mma.cuh"
+#include "query_tile.cuh"
 #include "tcgen05.cuh"
 #include "tmap.cuh"
 #include "vec.cuh"
@@ -31,11 +36,13 @@ constexpr float kLfRescale = 8.f;                     // log2 units
 
 constexpr int kLfBefore = 256, kLfAfter = 256;        // bias table: entries in front of distance 0 and past the last one
 
-template <int NQ, int NV, bool kWin> struct LfShape {
-  static constexpr int kKStages = kWin && NQ == 3 ? 1 : 2;
+enum { LF_LATENT = 0, LF_WINDOW = 1, LF_DIFF = 2 };
+template <int NQ, int NV, int FORM> struct LfShape {
+  static constexpr bool kWin = FORM == LF_WINDOW, kDiff = FORM == LF_DIFF;
+  static constexpr int kKStages = (kWin && NQ == 3) || (kDiff && NQ == 2) ? 1 : 2;
   static constexpr int kVStages = NQ == 3 && NV == 2 && !kWin ? 1 : 2;
-  static constexpr int kQBytes = NQ * kLfBox, kVBytes = NV * kLfBox;
-  static constexpr int kSmem = (2 + kKStages) * kQBytes + kVStages * kVBytes + 1024;
+  static constexpr int kQBytes = NQ * kLfBox, kKBytes = (kDiff ? 2 : 1) * kQBytes, kVBytes = NV * kLfBox;
+  static constexpr int kSmem = 2 * kQBytes + kKStages * kKBytes + kVStages * kVBytes + 1024;
   static constexpr int kTable = (227 * 1024 - 512 - kSmem) / 4;       // floats left for the bias table
 };
 
@@ -51,6 +58,9 @@ struct LfParams {
   const float* bias; int64_t bias_stride;
   const float2* turn; int64_t table_rows;             // kWin: (vdim / 2, table_rows) cos, sin; null: results stay as they are
   const int64_t* positions;                           // of the queries
+  int chunk;                                          // kDiff
+  const __nv_bfloat16* gate; int64_t gate_stride;
+  float lambda, mult, eps;
 };
 
 enum { LB_Q = 0, LB_KFULL = 1, LB_KEMPTY = 3, LB_VFULL = 5, LB_VEMPTY = 7, LB_SFULL = 9, LB_PREADY = 11, LB_ODONE = 13,
@@ -63,12 +73,14 @@ __device__ __forceinline__ void turn_back(uint32_t& a, uint32_t& b, float2 cs) {
   b = __float_as_uint(fmaf(y, cs.x, -x * cs.y));
 }
 
-template <int NQ, int NV, bool kWin>
+template <int NQ, int NV, int FORM>
 __global__ void __launch_bounds__(kLfThreads, 1)
 latent_prefill_kernel(const __grid_constant__ CUtensorMap tm_qn, const __grid_constant__ CUtensorMap tm_qr,
                       const __grid_constant__ CUtensorMap tm_kn, const __grid_constant__ CUtensorMap tm_kr,
                       const __grid_constant__ CUtensorMap tm_v, const LfParams p) {
-  using Sh = LfShape<NQ, NV, kWin>;
+  using Sh = LfShape<NQ, NV, FORM>;
+  constexpr bool kWin = Sh::kWin, kDiff = Sh::kDiff;
+  constexpr int kRows = kDiff ? kLfTile : 2 * kLfTile, kSecond = kDiff ? 0 : kLfTile;      // queries of a CTA; where the second problem's begin
   constexpr int VS = Sh::kVStages, KS = Sh::kKStages;
   extern __shared__ unsigned char smem_raw[];
   __shared__ __align__(8) uint64_t bars[LB_COUNT];
@@ -77,57 +89,31 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap tm_qn, const __grid_co
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const uint32_t q_smem = (smem_u32(smem_raw) + 1023u) & ~1023u;      // [tile 2][box][128][128B]
   const uint32_t k_smem = q_smem + 2 * Sh::kQBytes;                   // [stage KS][box]
-  const uint32_t v_smem = k_smem + KS * Sh::kQBytes;                  // [stage VS][box]
+  const uint32_t v_smem = k_smem + KS * Sh::kKBytes;                  // [stage VS][box]
   float* s_bias = reinterpret_cast<float*>(smem_raw + (v_smem + VS * Sh::kVBytes - smem_u32(smem_raw)));     // kWin
   const uint32_t bar0 = smem_u32(bars);
   auto bar = [&](int i) { return bar0 + 8u * i; };
   volatile int* abort_flag = &s_abort;
 
-  // which (sequence, 256-row tile) is blockIdx.x: tiles of a sequence in descending order
   if (tid == 0) {
-    s_tile[0] = -1;
-    s_tile[1] = 0;
     s_abort = 0;
     s_sticky = *reinterpret_cast<volatile int*>(p.error_word);
   }
-  __syncthreads();
-  int carry = 0;
-  for (int base = 0; base < p.num_seqs; base += kLfThreads) {
-    const int s = base + tid;
-    int n = 0;
-    if (s < p.num_seqs) n = (max(p.cu_q[s + 1] - p.cu_q[s], 0) + 2 * kLfTile - 1) / (2 * kLfTile);
-    int incl = n;
-#pragma unroll
-    for (int o = 1; o < 32; o <<= 1) {
-      const int v = __shfl_up_sync(0xffffffffu, incl, o);
-      if (lane >= o) incl += v;
-    }
-    if (lane == 31) s_scan[warp] = incl;
-    __syncthreads();
-    int before = 0, tot = 0;
-    for (int w = 0; w < kLfThreads / 32; ++w) {
-      if (w < warp) before += s_scan[w];
-      tot += s_scan[w];
-    }
-    const int start = carry + before + incl - n, x = static_cast<int>(blockIdx.x);
-    if (n > 0 && x >= start && x < start + n) { s_tile[0] = s; s_tile[1] = n - 1 - (x - start); }
-    carry += tot;
-    __syncthreads();
-  }
+  find_query_tile<kLfThreads>(p.cu_q, p.num_seqs, kRows, s_tile, s_scan);
   const int seq = s_tile[0];
   if (seq < 0 || s_sticky != 0) return;      // uniform: the grid is an upper bound; an earlier wait ran out
-  const int head = blockIdx.y, kv_head = kWin ? head / p.group : head;
+  const int head = blockIdx.y, kv_head = FORM == LF_LATENT ? head : head / p.group;
   const int q_start = p.cu_q[seq], q_len = p.cu_q[seq + 1] - q_start;
   const int k_start = p.cu_k[seq], k_len = p.cu_k[seq + 1] - k_start;
-  const int q0 = s_tile[1] * 2 * kLfTile;
+  const int q0 = s_tile[1] * kRows;
   const int first_pos = k_len - q_len + q0;
   // KV tiles up to the position of each query tile's last row
   const int n_a = (k_len - q_len + min(q0 + kLfTile, q_len) + kLfTile - 1) / kLfTile;
-  const int n_b = q0 + kLfTile < q_len ? (k_len - q_len + min(q0 + 2 * kLfTile, q_len) + kLfTile - 1) / kLfTile : 0;
+  const int n_b = kDiff ? n_a : q0 + kLfTile < q_len ? (k_len - q_len + min(q0 + 2 * kLfTile, q_len) + kLfTile - 1) / kLfTile : 0;
   const int n_kv = max(n_a, n_b);
   // kWin: first KV tile of each query tile; ring positions count from lo_a
-  const int lo_a = kWin ? min(max(first_pos - p.window + 1, 0) / kLfTile, n_a - 1) : 0;
-  const int lo_b = kWin && n_b > 0 ? max(first_pos + kLfTile - p.window + 1, 0) / kLfTile : 0;
+  const int lo_a = kDiff ? first_pos / p.chunk * p.chunk / kLfTile : kWin ? min(max(first_pos - p.window + 1, 0) / kLfTile, n_a - 1) : 0;
+  const int lo_b = kDiff ? lo_a : kWin && n_b > 0 ? max(first_pos + kLfTile - p.window + 1, 0) / kLfTile : 0;
   if (kWin)
     for (int i = tid; i < kLfBefore + p.distances + kLfAfter; i += kLfThreads) {
       const int d = i - kLfBefore;
@@ -167,17 +153,19 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap tm_qn, const __grid_co
         for (int t = 0; t < tiles; ++t)
           for (int b = 0; b < NQ; ++b) {
             const uint32_t dst = q_smem + t * Sh::kQBytes + b * kLfBox;
-            const int row = q_start + q0 + t * kLfTile;
-            if (b < p.nd) tc::tma_load_3d(dst, &tm_qn, 64 * b, head, row, bar(LB_Q));
+            const int row = q_start + q0 + t * kSecond;
+            if (kDiff) tc::tma_load_3d(dst, &tm_qn, 64 * b, 2 * head + t, row, bar(LB_Q));
+            else if (b < p.nd) tc::tma_load_3d(dst, &tm_qn, 64 * b, head, row, bar(LB_Q));
             else tc::tma_load_3d(dst, &tm_qr, 64 * (b - p.nd), head, row, bar(LB_Q));
           }
         for (int i = 0; i < n_kv - lo_a; ++i) {
           const int s = i % KS, row = k_start + (lo_a + i) * kLfTile;
           tc::mbar_wait(bar(LB_KEMPTY + s), ((i / KS) & 1) ^ 1, abort_flag, p.error_word, 1);
-          tc::mbar_expect_tx(bar(LB_KFULL + s), Sh::kQBytes);
-          for (int b = 0; b < NQ; ++b) {
-            const uint32_t dst = k_smem + s * Sh::kQBytes + b * kLfBox;
-            if (b < p.nd) tc::tma_load_3d(dst, &tm_kn, 64 * b, kv_head, row, bar(LB_KFULL + s));
+          tc::mbar_expect_tx(bar(LB_KFULL + s), Sh::kKBytes);
+          for (int b = 0; b < Sh::kKBytes / kLfBox; ++b) {
+            const uint32_t dst = k_smem + s * Sh::kKBytes + b * kLfBox;
+            if (kDiff) tc::tma_load_3d(dst, &tm_kn, 64 * (b % NQ), 2 * kv_head + b / NQ, row, bar(LB_KFULL + s));
+            else if (b < p.nd) tc::tma_load_3d(dst, &tm_kn, 64 * b, kv_head, row, bar(LB_KFULL + s));
             else tc::tma_load_3d(dst, &tm_kr, 64 * (b - p.nd), 0, row, bar(LB_KFULL + s));
           }
           const int vs = i % VS;
@@ -203,7 +191,7 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap tm_qn, const __grid_co
 #pragma unroll
         for (int b = 0; b < NQ; ++b)
           tc::mma_ss_k64(tmem + t * 128, tc::desc64(q_lo + ((t * Sh::kQBytes + b * kLfBox) >> 4), tc::kDescHiSw128Sbo1024),
-                         tc::desc64(k_lo + ((s * Sh::kQBytes + b * kLfBox) >> 4), tc::kDescHiSw128Sbo1024), idesc_qk, b > 0);
+                         tc::desc64(k_lo + ((s * Sh::kKBytes + (kDiff ? t * Sh::kQBytes : 0) + b * kLfBox) >> 4), tc::kDescHiSw128Sbo1024), idesc_qk, b > 0);
         tc::commit_elected(bar(LB_SFULL + t), 0, false);
       };
       tc::mbar_wait(bar(LB_Q), 0, abort_flag, p.error_word, 3);
@@ -251,12 +239,13 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap tm_qn, const __grid_co
       const int row = (warp & 3) * 32 + lane;
       const uint32_t lane_addr = static_cast<uint32_t>((warp & 3) * 32) << 16;
       const uint32_t s_addr = tmem + lane_addr + t * 128, o_addr = tmem + lane_addr + 256 + t * 128;
+      const int low = kDiff ? (first_pos + row) / p.chunk * p.chunk : 0;      // first key of the row's chunk
       float m_used = -INFINITY, l = 0.f;
       for (int j = lo_t; j < n_t; ++j) {
         tc::mbar_wait(bar(LB_SFULL + t), (j - lo_t) & 1, abort_flag, p.error_word, 8);
         tc::fence_after_sync();
         // key 128j + col is visible to this row when col <= vis
-        const int vis = first_pos + t * kLfTile + row - j * kLfTile;
+        const int vis = first_pos + t * kSecond + row - j * kLfTile;
         uint32_t sv[4][32];
 #pragma unroll
         for (int c = 0; c < 4; ++c) tc::tmem_ld32(s_addr + c * 32, sv[c]);
@@ -283,6 +272,15 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap tm_qn, const __grid_co
                 for (int i = 0; i < 32; ++i)
                   if (vis - (c * 32 + i) >= p.window) sv[c][i] = 0xff800000u;
             }
+          }
+        } else if (kDiff) {
+          // the tile reaches past the first row's position, or begins in front of the last row's chunk
+          if (first_pos - j * kLfTile < kLfTile - 1 || (first_pos + kLfTile - 1) / p.chunk * p.chunk > j * kLfTile) {
+#pragma unroll
+            for (int c = 0; c < 4; ++c)
+#pragma unroll
+              for (int i = 0; i < 32; ++i)
+                if (c * 32 + i > vis || c * 32 + i < low - j * kLfTile) sv[c][i] = 0xff800000u;
           }
         } else if (first_pos + t * kLfTile - j * kLfTile < kLfTile - 1) {     // the tile reaches past the first row's position
 #pragma unroll
@@ -320,7 +318,7 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap tm_qn, const __grid_co
           l *= alpha;
         }
         if (grow) m_used = mx;
-        const float off = kWin && m_used == -INFINITY ? 0.f : -m_used;         // kWin: a tile in front of the row's window
+        const float off = FORM != LF_LATENT && m_used == -INFINITY ? 0.f : -m_used;         // a tile in front of the row's window or chunk
         const float2 sc2 = make_float2(p.scale_log2, p.scale_log2), nm2 = make_float2(off, off);
         float2 sums[4] = {make_float2(0.f, 0.f), make_float2(0.f, 0.f), make_float2(0.f, 0.f), make_float2(0.f, 0.f)};
 #pragma unroll
@@ -351,6 +349,52 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap tm_qn, const __grid_co
       }
       tc::mbar_wait(bar(LB_ODONE + t), (n_t - lo_t - 1) & 1, abort_flag, p.error_word, 10);
       tc::fence_after_sync();
+      if constexpr (kDiff) {
+        // queries are no longer wanted: [problem][row] factors, then [group][row] sums of squares take their place
+        float* s_f = reinterpret_cast<float*>(smem_raw + (q_smem - smem_u32(smem_raw)));
+        auto slot = [&](int u) -> float& { return s_f[u * (Sh::kQBytes / 4) + row]; };
+        slot(t) = l > 0.f ? (t ? p.lambda : 1.f) / l : 0.f;
+        tc::fence_before_sync();
+        asm volatile("bar.sync 1, 256;" ::: "memory");
+        tc::fence_after_sync();
+        const float f1 = slot(0), f2 = slot(1);
+        const uint32_t o1 = tmem + lane_addr + 256 + t * 32 * NV, o2 = o1 + 128;
+        float o[NV][32], sq = 0.f;
+#pragma unroll
+        for (int c = 0; c < NV; ++c) {
+          uint32_t u[32], v[32];
+          tc::tmem_ld32(o1 + c * 32, u);
+          tc::tmem_ld32(o2 + c * 32, v);
+          tc::wait_ld();
+#pragma unroll
+          for (int i = 0; i < 32; ++i) {
+            o[c][i] = __uint_as_float(u[i]) * f1 - __uint_as_float(v[i]) * f2;
+            sq = fmaf(o[c][i], o[c][i], sq);       // columns past vdim are zero
+          }
+        }
+        float* s_sq = s_f + kLfTile;
+        s_sq[t * (Sh::kQBytes / 4) + row] = sq;
+        asm volatile("bar.sync 1, 256;" ::: "memory");
+        sq = s_sq[row] + s_sq[Sh::kQBytes / 4 + row];
+        const float f = p.mult / sqrtf(sq / static_cast<float>(p.vdim) + p.eps);
+        if (q0 + row < q_len) {
+          const int64_t tok = q_start + q0 + row;
+          const __nv_bfloat16* gate = p.gate + tok * p.gate_stride + static_cast<int64_t>(head) * p.vdim;
+          __nv_bfloat16* orow = p.out + tok * p.out_stride + static_cast<int64_t>(head) * p.vdim;
+#pragma unroll
+          for (int c = 0; c < NV; ++c)
+#pragma unroll
+            for (int i = 0; i < 4; ++i) {
+              const int d = (t * NV + c) * 32 + i * 8;
+              if (d >= p.vdim) continue;
+              float g[8];
+              Vec<__nv_bfloat16, 8>::load(gate + d, g);
+#pragma unroll
+              for (int e = 0; e < 8; ++e) g[e] = o[c][8 * i + e] * f * sigmoid_t<__nv_bfloat16>(g[e]);
+              Vec<__nv_bfloat16, 8>::store(orow + d, g);
+            }
+        }
+      } else {
       float f = 1.f;
       if (p.sink) {
         const float sk = __bfloat162float(p.sink[head]) * 1.4426950408889634f, mm = fmaxf(m_used, sk);
@@ -386,6 +430,7 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap tm_qn, const __grid_co
           }
         }
       }
+      }
     }
   }
   __syncwarp();
@@ -414,20 +459,22 @@ latent_gather_kernel(uint4* __restrict__ out, const uint4* __restrict__ cache, c
   }
 }
 
-template <int NQ, int NV, bool kWin = false>
+template <int NQ, int NV, int FORM = LF_LATENT>
 static int launch_latent_prefill(const CUtensorMap (&tm)[5], const LfParams& p, int64_t tokens, int heads, cudaStream_t st) {
-  using Sh = LfShape<NQ, NV, kWin>;
-  const char* what = kWin ? "window_prefill" : "latent_prefill";
+  using Sh = LfShape<NQ, NV, FORM>;
+  constexpr bool kWin = FORM == LF_WINDOW;
+  constexpr int kRows = FORM == LF_DIFF ? kLfTile : 2 * kLfTile;
+  const char* what = kWin ? "window_prefill" : FORM == LF_DIFF ? "diff_prefill" : "latent_prefill";
   int smem = Sh::kSmem;
   if (kWin) {
     const int table = kLfBefore + p.distances + kLfAfter;
     if (table > Sh::kTable) return fail(MV_ERR_LIMIT, "window_prefill: %d distances (at most %d)", p.distances, Sh::kTable - kLfBefore - kLfAfter);
     smem += table * 4;
   }
-  const cudaError_t e = cudaFuncSetAttribute(latent_prefill_kernel<NQ, NV, kWin>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
+  const cudaError_t e = cudaFuncSetAttribute(latent_prefill_kernel<NQ, NV, FORM>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
   if (e != cudaSuccess) return fail(MV_ERR_CUDA, "%s: %s", what, cudaGetErrorString(e));
-  const dim3 grid(static_cast<unsigned>(tokens / (2 * kLfTile) + std::min<int64_t>(p.num_seqs, tokens)), heads);
-  latent_prefill_kernel<NQ, NV, kWin><<<grid, kLfThreads, smem, st>>>(tm[0], tm[1], tm[2], tm[3], tm[4], p);
+  const dim3 grid(static_cast<unsigned>(tokens / kRows + std::min<int64_t>(p.num_seqs, tokens)), heads);
+  latent_prefill_kernel<NQ, NV, FORM><<<grid, kLfThreads, smem, st>>>(tm[0], tm[1], tm[2], tm[3], tm[4], p);
   return check_launch(what);
 }
 
@@ -477,7 +524,7 @@ extern "C" int mv_latent_prefill(void* out, int64_t out_stride, const void* q, i
   if (rc) return rc;
   if (!rot_dim) { tm[1] = tm[0]; tm[3] = tm[2]; }
   LfParams p{static_cast<__nv_bfloat16*>(out), out_stride, vdim, cu_q, cu_k, num_seqs, nd, dim, rot_dim,
-             scale * 1.4426950408889634f, static_cast<const __nv_bfloat16*>(sink), error_word, 1, 0, 0, nullptr, 0, nullptr, 0, nullptr};
+             scale * 1.4426950408889634f, static_cast<const __nv_bfloat16*>(sink), error_word, 1, 0, 0, nullptr, 0, nullptr, 0, nullptr, 1, nullptr, 0, 0.f, 0.f, 0.f};
   auto st = static_cast<cudaStream_t>(stream);
   if (nq == 1) return nv == 1 ? launch_latent_prefill<1, 1>(tm, p, tokens, heads, st) : launch_latent_prefill<1, 2>(tm, p, tokens, heads, st);
   if (nq == 2) return nv == 1 ? launch_latent_prefill<2, 1>(tm, p, tokens, heads, st) : launch_latent_prefill<2, 2>(tm, p, tokens, heads, st);
@@ -489,9 +536,9 @@ extern "C" int mv_window_prefill_distances(int dim, int vdim) {
   using namespace mv;
   if (dim <= 0 || vdim <= 0 || dim % 8 || vdim % 8 || dim > 192 || vdim > 128) return -1;
   const int nq = (dim + 63) / 64, extra = kLfBefore + kLfAfter;
-  if (nq == 1) return (vdim <= 64 ? LfShape<1, 1, true>::kTable : LfShape<1, 2, true>::kTable) - extra;
-  if (nq == 2) return (vdim <= 64 ? LfShape<2, 1, true>::kTable : LfShape<2, 2, true>::kTable) - extra;
-  return (vdim <= 64 ? LfShape<3, 1, true>::kTable : LfShape<3, 2, true>::kTable) - extra;
+  if (nq == 1) return (vdim <= 64 ? LfShape<1, 1, LF_WINDOW>::kTable : LfShape<1, 2, LF_WINDOW>::kTable) - extra;
+  if (nq == 2) return (vdim <= 64 ? LfShape<2, 1, LF_WINDOW>::kTable : LfShape<2, 2, LF_WINDOW>::kTable) - extra;
+  return (vdim <= 64 ? LfShape<3, 1, LF_WINDOW>::kTable : LfShape<3, 2, LF_WINDOW>::kTable) - extra;
 }
 
 extern "C" int mv_window_prefill(void* out, int64_t out_stride, const void* q, int64_t q_stride, const void* k,
@@ -522,9 +569,44 @@ extern "C" int mv_window_prefill(void* out, int64_t out_stride, const void* q, i
   const int win = static_cast<int>(std::min<int64_t>(window, 1 << 30));
   LfParams p{static_cast<__nv_bfloat16*>(out), out_stride, vdim, cu_q, cu_k, num_seqs, nq, dim, 0,
              scale * 1.4426950408889634f, static_cast<const __nv_bfloat16*>(sink), error_word, heads / kv_heads, win,
-             bias ? std::min(distances, win) : 1, bias, bias_stride, reinterpret_cast<const float2*>(turn), table_rows, positions};
+             bias ? std::min(distances, win) : 1, bias, bias_stride, reinterpret_cast<const float2*>(turn), table_rows, positions,
+             1, nullptr, 0, 0.f, 0.f, 0.f};
   auto st = static_cast<cudaStream_t>(stream);
-  if (nq == 1) return nv == 1 ? launch_latent_prefill<1, 1, true>(tm, p, tokens, heads, st) : launch_latent_prefill<1, 2, true>(tm, p, tokens, heads, st);
-  if (nq == 2) return nv == 1 ? launch_latent_prefill<2, 1, true>(tm, p, tokens, heads, st) : launch_latent_prefill<2, 2, true>(tm, p, tokens, heads, st);
-  return nv == 1 ? launch_latent_prefill<3, 1, true>(tm, p, tokens, heads, st) : launch_latent_prefill<3, 2, true>(tm, p, tokens, heads, st);
+  if (nq == 1) return nv == 1 ? launch_latent_prefill<1, 1, LF_WINDOW>(tm, p, tokens, heads, st) : launch_latent_prefill<1, 2, LF_WINDOW>(tm, p, tokens, heads, st);
+  if (nq == 2) return nv == 1 ? launch_latent_prefill<2, 1, LF_WINDOW>(tm, p, tokens, heads, st) : launch_latent_prefill<2, 2, LF_WINDOW>(tm, p, tokens, heads, st);
+  return nv == 1 ? launch_latent_prefill<3, 1, LF_WINDOW>(tm, p, tokens, heads, st) : launch_latent_prefill<3, 2, LF_WINDOW>(tm, p, tokens, heads, st);
+}
+
+extern "C" int mv_diff_prefill_takes(int dim, int vdim) {
+  return dim > 0 && vdim > 0 && dim % 8 == 0 && vdim % 8 == 0 && dim <= 128 && vdim <= 128;
+}
+
+extern "C" int mv_diff_prefill(void* out, const void* q, int64_t q_stride, const void* k, int64_t k_stride, const void* v,
+                               int64_t v_stride, const int32_t* cu_q, const int32_t* cu_k, int num_seqs, int64_t tokens,
+                               int64_t keys, int64_t chunk, const void* gate, int64_t gate_stride, float lambda, float mult,
+                               float eps, int heads, int kv_heads, int dim, int vdim, float scale, int* error_word,
+                               void* stream) {
+  using namespace mv;
+  const char* w = "diff_prefill";
+  if (num_seqs < 0 || tokens < 0 || keys < tokens || heads <= 0 || kv_heads <= 0 || heads % kv_heads || chunk <= 0 || !(scale > 0.f))
+    return fail(MV_ERR_SHAPE, "diff_prefill: heads %d over %d, chunk %lld, scale %f", heads, kv_heads, static_cast<long long>(chunk), scale);
+  if (!mv_diff_prefill_takes(dim, vdim)) return fail(MV_ERR_LIMIT, "diff_prefill: dim %d vdim %d", dim, vdim);
+  if (tokens == 0 || num_seqs == 0) return MV_OK;
+  if (!out || !q || !k || !v || !cu_q || !cu_k || !gate || !error_word) return fail(MV_ERR_NULL, "diff_prefill: null pointer");
+  if (!aligned16(out) || !vec8_ok(q, q_stride, 2) || !vec8_ok(k, k_stride, 2) || !vec8_ok(v, v_stride, 2) || !vec8_ok(gate, gate_stride, 2))
+    return fail(MV_ERR_ALIGN, "diff_prefill: rows must start on 16-byte boundaries");
+  CUtensorMap tm[5];
+  int rc = make_tmap_bf16(&tm[0], q, dim, 2 * heads, tokens, dim, q_stride, 1, kLfTile, w);
+  if (!rc) rc = make_tmap_bf16(&tm[2], k, dim, 2 * kv_heads, keys, dim, k_stride, 1, kLfTile, w);
+  if (!rc) rc = make_tmap_bf16(&tm[4], v, vdim, kv_heads, keys, vdim, v_stride, 1, kLfTile, w);
+  if (rc) return rc;
+  tm[1] = tm[0];
+  tm[3] = tm[2];
+  const int nq = (dim + 63) / 64, nv = (vdim + 63) / 64;
+  LfParams p{static_cast<__nv_bfloat16*>(out), static_cast<int64_t>(heads) * vdim, vdim, cu_q, cu_k, num_seqs, nq, dim, 0,
+             scale * 1.4426950408889634f, nullptr, error_word, heads / kv_heads, 1, 1, nullptr, 0, nullptr, 0, nullptr,
+             static_cast<int>(std::min<int64_t>(chunk, 1 << 30)), static_cast<const __nv_bfloat16*>(gate), gate_stride, lambda, mult, eps};
+  auto st = static_cast<cudaStream_t>(stream);
+  if (nq == 1) return nv == 1 ? launch_latent_prefill<1, 1, LF_DIFF>(tm, p, tokens, heads, st) : launch_latent_prefill<1, 2, LF_DIFF>(tm, p, tokens, heads, st);
+  return nv == 1 ? launch_latent_prefill<2, 1, LF_DIFF>(tm, p, tokens, heads, st) : launch_latent_prefill<2, 2, LF_DIFF>(tm, p, tokens, heads, st);
 }

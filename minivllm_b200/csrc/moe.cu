@@ -12,13 +12,14 @@ namespace mv {
 constexpr int kRtThreads = 256;
 constexpr int kRtMaxPer = 32;      // experts per lane: up to 1024 experts
 
-// One warp per token: the `top` largest logits (ties: lower index) and the softmax over them.
+// One warp per token: the `top` largest logits (ties: lower index) and the softmax over them (kAll: over all experts), times
+// `scale`.
 // kPer: experts per lane.
-template <int kPer>
+template <int kPer, bool kAll>
 __global__ void __launch_bounds__(kRtThreads)
 moe_route_kernel(int32_t* __restrict__ idx, float* __restrict__ weight, const float* __restrict__ logits,
                  int64_t stride, const float* __restrict__ bias, int64_t tokens, int experts, int top, int groups,
-                 int keep) {
+                 int keep, float scale) {
   __shared__ float s_best[kRtThreads / 32][32 * kPer];      // per group of experts: its largest logit
   const int lane = threadIdx.x & 31;
   const int64_t t = static_cast<int64_t>(blockIdx.x) * (kRtThreads / 32) + (threadIdx.x >> 5);
@@ -53,6 +54,15 @@ moe_route_kernel(int32_t* __restrict__ idx, float* __restrict__ weight, const fl
     }
   }
   float first = 0.f, sum = 0.f;
+  if (kAll) {
+#pragma unroll
+    for (int i = 0; i < kPer; ++i) first = i == 0 ? z[0] : fmaxf(first, z[i]);
+#pragma unroll
+    for (int o = 16; o; o >>= 1) first = fmaxf(first, __shfl_xor_sync(0xffffffffu, first, o));
+#pragma unroll
+    for (int i = 0; i < kPer; ++i) sum += i * 32 + lane < experts ? expf(z[i] - first) : 0.f;
+    sum = warp_sum(sum);
+  }
   for (int k = 0; k < top; ++k) {
     float best = -INFINITY;
     int at = 0x7fffffff;
@@ -68,16 +78,16 @@ moe_route_kernel(int32_t* __restrict__ idx, float* __restrict__ weight, const fl
       if (oa != 0x7fffffff && (at == 0x7fffffff || ob > best || (ob == best && oa < at))) { best = ob; at = oa; }
     }
     if ((at & 31) == lane) taken |= 1u << (at >> 5);
-    if (k == 0) first = best;
+    if (!kAll && k == 0) first = best;
     const float e = expf(best - first);
-    sum += e;
+    if (!kAll) sum += e;
     if (lane == 0) {
       idx[t * top + k] = at;
       weight[t * top + k] = e;
     }
   }
   __syncwarp();
-  for (int k = lane; k < top; k += 32) weight[t * top + k] /= sum;
+  for (int k = lane; k < top; k += 32) weight[t * top + k] = weight[t * top + k] / sum * scale;
 }
 
 constexpr int kSortThreads = 256;   // entries per block
@@ -284,7 +294,7 @@ grouped_rows_kernel(T* __restrict__ out, const T* __restrict__ x, const T* __res
 }  // namespace mv
 
 extern "C" int mv_moe_route(int32_t* idx, float* weight, const float* logits, int64_t logits_stride, const float* bias,
-                            int64_t tokens, int experts, int top, int groups, int keep, void* stream) {
+                            int64_t tokens, int experts, int top, int groups, int keep, int over_all, float scale, void* stream) {
   using namespace mv;
   if (tokens < 0 || experts <= 0 || top <= 0 || top > experts) return fail(MV_ERR_SHAPE, "moe_route: experts %d top %d", experts, top);
   if (groups <= 0 || experts % groups || keep <= 0 || keep > groups || experts / groups * keep < top)
@@ -295,11 +305,11 @@ extern "C" int mv_moe_route(int32_t* idx, float* weight, const float* logits, in
   const unsigned grid = static_cast<unsigned>((tokens + kRtThreads / 32 - 1) / (kRtThreads / 32));
   auto go = [&](auto kernel) {
     kernel<<<grid, kRtThreads, 0, static_cast<cudaStream_t>(stream)>>>(idx, weight, logits, logits_stride, bias, tokens, experts, top,
-                                                                        keep < groups ? groups : 1, keep);
+                                                                        keep < groups ? groups : 1, keep, scale);
   };
-  if (experts <= 64) go(moe_route_kernel<2>);
-  else if (experts <= 256) go(moe_route_kernel<8>);
-  else go(moe_route_kernel<kRtMaxPer>);
+  if (experts <= 64) over_all ? go(moe_route_kernel<2, true>) : go(moe_route_kernel<2, false>);
+  else if (experts <= 256) over_all ? go(moe_route_kernel<8, true>) : go(moe_route_kernel<8, false>);
+  else over_all ? go(moe_route_kernel<kRtMaxPer, true>) : go(moe_route_kernel<kRtMaxPer, false>);
   return check_launch("moe_route");
 }
 

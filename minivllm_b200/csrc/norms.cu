@@ -399,6 +399,8 @@ __global__ void __launch_bounds__(kNormThreads, SRC == SRC_EXPERTS ? (kCh == 1 ?
 struct HeadNorm {
   const float* den;
   bool full_weight, sigmoid;
+  float mult;                    // of the result
+  int64_t out_stride;            // of its rows, 0: dense
 };
 
 // kGateFirst: out = group_rms_norm(y * silu(z)) * w.  Otherwise out = group_rms_norm(y / den) * w * act(z).
@@ -442,9 +444,9 @@ gated_group_norm_kernel(T* __restrict__ out, const T* __restrict__ y, int64_t y_
       if (!kGateFirst) {
         Vec<T, V>::load(z + row * z_stride + c, t);
 #pragma unroll
-        for (int e = 0; e < V; ++e) v[e] *= hn.sigmoid ? sigmoid_t<T>(t[e]) : silu_t<T>(t[e]);
+        for (int e = 0; e < V; ++e) v[e] *= (hn.sigmoid ? sigmoid_t<T>(t[e]) : silu_t<T>(t[e])) * hn.mult;
       }
-      Vec<T, V>::store(out + row * width + c, v);
+      Vec<T, V>::store(out + row * (kGateFirst || !hn.out_stride ? width : hn.out_stride) + c, v);
     }
   }
 }
@@ -493,8 +495,8 @@ head_norm_gate_kernel(T* __restrict__ out, const T* __restrict__ y, int64_t y_st
         b[k].get(g);
         Vec<T, 8>::load(wh + c, t);
 #pragma unroll
-        for (int e = 0; e < 8; ++e) v[e] = v[e] * rs * t[e] * (hn.sigmoid ? sigmoid_t<T>(g[e]) : silu_t<T>(g[e]));
-        Vec<T, 8>::store(out + row * (static_cast<int64_t>(heads) * gs) + static_cast<int64_t>(h) * gs + c, v);
+        for (int e = 0; e < 8; ++e) v[e] = v[e] * (rs * hn.mult) * t[e] * (hn.sigmoid ? sigmoid_t<T>(g[e]) : silu_t<T>(g[e]));
+        Vec<T, 8>::store(out + row * (hn.out_stride ? hn.out_stride : static_cast<int64_t>(heads) * gs) + static_cast<int64_t>(h) * gs + c, v);
       }
     }
   }
@@ -652,7 +654,7 @@ extern "C" int mv_moe_residual_norm(void* out, float* x, const void* expert_rows
 }
 
 static int gated_norm(const char* what, bool gate_first, void* out, const void* y, int64_t y_stride, const void* z, int64_t z_stride,
-                      const void* w, int64_t rows, int width, int groups, float eps, int dtype, void* stream, mv::HeadNorm hn = {}) {
+                      const void* w, int64_t rows, int width, int groups, float eps, int dtype, void* stream, mv::HeadNorm hn = {nullptr, false, false, 1.f, 0}) {
   using namespace mv;
   int rc = check_norm(what, width, groups, dtype);
   if (rc || rows == 0) return rc;
@@ -669,7 +671,7 @@ static int gated_norm(const char* what, bool gate_first, void* out, const void* 
           static_cast<const T*>(w), width, groups, eps, hn);
       return check_launch(what);
     };
-    const bool v8 = (width / groups) % 8 == 0 && vec8_ok(out, width, eb) && vec8_ok(y, y_stride, eb) && vec8_ok(z, z_stride, eb) &&
+    const bool v8 = (width / groups) % 8 == 0 && vec8_ok(out, hn.out_stride ? hn.out_stride : width, eb) && vec8_ok(y, y_stride, eb) && vec8_ok(z, z_stride, eb) &&
         aligned16(w);
     if (v8 && !gate_first && width / groups <= 1024) {
       const int gs = width / groups;
@@ -701,12 +703,12 @@ extern "C" int mv_gated_group_norm(void* out, const void* y, int64_t y_stride, c
   return gated_norm("gated_group_norm", true, out, y, y_stride, z, z_stride, w, rows, width, groups, eps, dtype, stream);
 }
 
-extern "C" int mv_head_norm_gate(void* out, const void* y, int64_t y_stride, const float* den, const void* z, int64_t z_stride,
-                                 const void* w, int full_weight, int act, int64_t rows, int width, int heads, float eps,
-                                 int dtype, void* stream) {
+extern "C" int mv_head_norm_gate(void* out, int64_t out_stride, const void* y, int64_t y_stride, const float* den, const void* z, int64_t z_stride,
+                                 const void* w, int full_weight, int act, float mult, int64_t rows, int width, int heads,
+                                 float eps, int dtype, void* stream) {
   if (act != MV_ACT_SILU && act != MV_ACT_SIGMOID) return mv::fail(MV_ERR_SHAPE, "head_norm_gate: activation %d", act);
   return gated_norm("head_norm_gate", false, out, y, y_stride, z, z_stride, w, rows, width, heads, eps, dtype, stream,
-                    {den, full_weight != 0, act == MV_ACT_SIGMOID});
+                    {den, full_weight != 0, act == MV_ACT_SIGMOID, mult, out_stride});
 }
 
 extern "C" int mv_gate_mul(void* out, const void* y, int64_t y_stride, int64_t y_head_stride, int heads,

@@ -3,6 +3,8 @@
 //   gated delta rule         S <- g S;  u = beta (v - S^T k);  S <- S + k u^T,       o = S^T q
 //   matrix memory (mLSTM)    S <- alpha S + w k v^T;  n <- alpha n + w k,            o = S^T q / (max(|n . q|, e^-m') + 1e-6)
 //     with alpha = e^(f + m - m'), w = e^(i - m'), m' = max(f + m, i) the running maximum of the gates' logarithms
+//   time mixing              o = (S + diag(u) k v^T)^T q,  S <- diag(e^(-e^z)) S + k v^T: the read-out comes before the decay,
+//     and a token's own entry enters it with the bonus u
 // Everything is computed in 32-bit, token by token, with the state in registers, so a result does not depend on how a
 // prompt is cut.
 //
@@ -32,7 +34,7 @@
 
 namespace mv {
 
-enum { SK_GLA = 0, SK_DELTA = 1, SK_MLSTM = 2 };
+enum { SK_GLA = 0, SK_DELTA = 1, SK_MLSTM = 2, SK_TIME = 3 };
 
 constexpr int log2_c(int n) { return n <= 1 ? 0 : 1 + log2_c(n / 2); }
 
@@ -137,8 +139,8 @@ template <typename Sh> struct ScanState {
       }
   }
   // One token of gated linear attention.  sk, sq, sa: K values in shared memory (sa: alpha - 1); v: this lane's columns.
-  // o receives the read-out of the columns first_held(kp) .. + HELD.
-  __device__ __forceinline__ void gla(const float* sk, const float* sq, const float* sa, const float* sv, int kp, float (&o)[Sh::HELD]) {
+  // o receives the read-out of the columns first_held(kp) .. + HELD.  kBefore: of the state before the token.
+  template <bool kBefore = false> __device__ __forceinline__ void gla(const float* sk, const float* sq, const float* sa, const float* sv, int kp, float (&o)[Sh::HELD]) {
     float2 acc[Sh::VT];
     float2 vv[Sh::VT];
 #pragma unroll
@@ -156,10 +158,16 @@ template <typename Sh> struct ScanState {
       const float4 a4 = *reinterpret_cast<const float4*>(sa + (i * Sh::KP + kp) * 4);
 #pragma unroll
       for (int v = 0; v < Sh::VT; ++v) {
+        if (kBefore) {
+          acc[v] = fma_f32x2(make_float2(q4.x, q4.y), s[2 * i][v], acc[v]);
+          acc[v] = fma_f32x2(make_float2(q4.z, q4.w), s[2 * i + 1][v], acc[v]);
+        }
         s[2 * i][v] = fma_f32x2(make_float2(k4.x, k4.y), vv[v], fma_f32x2(make_float2(a4.x, a4.y), s[2 * i][v], s[2 * i][v]));
         s[2 * i + 1][v] = fma_f32x2(make_float2(k4.z, k4.w), vv[v], fma_f32x2(make_float2(a4.z, a4.w), s[2 * i + 1][v], s[2 * i + 1][v]));
-        acc[v] = fma_f32x2(make_float2(q4.x, q4.y), s[2 * i][v], acc[v]);
-        acc[v] = fma_f32x2(make_float2(q4.z, q4.w), s[2 * i + 1][v], acc[v]);
+        if (!kBefore) {
+          acc[v] = fma_f32x2(make_float2(q4.x, q4.y), s[2 * i][v], acc[v]);
+          acc[v] = fma_f32x2(make_float2(q4.z, q4.w), s[2 * i + 1][v], acc[v]);
+        }
       }
     }
     float val[Sh::VT];
@@ -241,6 +249,7 @@ constexpr int kScanMaxK = 256;
 
 // Logarithms of the decays, in 32-bit.
 __device__ __forceinline__ float channel_log_decay(float z, float inv_tau) { return -softplus_f(-z) * inv_tau; }
+__device__ __forceinline__ float time_log_decay(float z) { return -expf(z); }
 __device__ __forceinline__ float head_log_decay(float a, float A_log, float dt_bias) { return -expf(A_log) * softplus_f(a + dt_bias); }
 constexpr float kUnitEps = 1e-6f;       // of q and k scaled to unit length
 constexpr float kMemFloor = 1e-6f;      // matrix memory: added to the denominator
@@ -256,6 +265,8 @@ template <typename T> struct ScanParams {
   const T *q, *k, *v; int64_t stride;                  // rows of a token: (kv_heads, K), (kv_heads, K), (heads, V)
   const T* z; int64_t z_stride;                        // gated linear attention: (heads, K) logits of the decay
   float inv_tau;
+  const float* zf; int64_t zf_stride;                  // time mixing: (heads, K) logarithms of the decay's rate, to be added to w0
+  const T *w0, *bonus;                                 //   (heads, K)
   const T *beta, *a; int64_t gate_stride;              // delta rule: (heads) logits of the step size and of the decay
   const T *A_log, *dt_bias;
   const float* gates; int64_t gates_stride;            // matrix memory, prompts: (heads) logits of the input gate, (heads) of the forget gate
@@ -267,19 +278,19 @@ template <typename T> struct ScanParams {
   float* state; int num_slots, heads, kv_heads, K, V;
   float q_scale;
   // step only
-  const T *gate, *norm_w; int64_t out_gate_stride; float eps;
+  const T *gate, *norm_w; int64_t out_gate_stride; float eps, out_scale;
   const T *conv_w, *conv_state; int taps, channels;    // delta rule: channels [q | k | v]
 };
 
 template <typename Sh, typename T, int W>
 __global__ void __launch_bounds__(32 * W, 16 / W) scan_kernel(const ScanParams<T> p, int cols_cta) {
-  constexpr bool kDelta = Sh::KIND == SK_DELTA, kMem = Sh::KIND == SK_MLSTM;
+  constexpr bool kDelta = Sh::KIND == SK_DELTA, kMem = Sh::KIND == SK_MLSTM, kTime = Sh::KIND == SK_TIME;
   constexpr int K = Sh::K, KL = K / 32, VL = kScanCols / 32, TT = W;      // a tile: one token per warp
   constexpr int VEC = kDelta ? 2 : 3;
   extern __shared__ __align__(16) float sm[];
   float* s_vec = sm;                                   // [2][TT][VEC][K]
   float* s_v = s_vec + 2 * TT * VEC * K;               // [2][TT][kScanCols]
-  float* s_par = s_v + 2 * TT * kScanCols;             // [2][TT][4]: decay, step size, k . q
+  float* s_par = s_v + 2 * TT * kScanCols;             // [2][TT][4]: decay, step size, k . q; time mixing: k . (u q)
   const int s = blockIdx.x, h = blockIdx.y, p0 = blockIdx.z * cols_cta, pw = min(cols_cta, p.V - p0);
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, kp = lane & (Sh::KP - 1), vp = lane / Sh::KP;
   const int kh = h / (p.heads / p.kv_heads);
@@ -294,7 +305,17 @@ __global__ void __launch_bounds__(32 * W, 16 / W) scan_kernel(const ScanParams<T
   if (work && live && st0 > 0) S.load(gS, kp, p.K, p.V, pw - c0, vec);
   else S.zero();
 
-  T rk[KL], rq[KL], rz[kDelta || kMem ? 1 : KL], rv[VL], rb[2];
+  T rk[KL], rq[KL], rv[VL], rb[2];
+  std::conditional_t<kTime, float, T> rz[kDelta || kMem ? 1 : KL];
+  float w0[kTime ? KL : 1], bonus[kTime ? KL : 1];
+  if constexpr (kTime) {
+#pragma unroll
+    for (int m = 0; m < KL; ++m) {
+      const bool ok = m * 32 + lane < p.K;
+      w0[m] = ok ? Elem<T>::to_f(p.w0[h * p.K + m * 32 + lane]) : 0.f;
+      bonus[m] = ok ? Elem<T>::to_f(p.bonus[h * p.K + m * 32 + lane]) : 0.f;
+    }
+  }
   float4 rc = make_float4(0.f, 0.f, 0.f, 0.f);
   float n[kMem ? KL : 1];                // matrix memory: this lane's entries of n
   const bool keeps_n = kMem && blockIdx.z == 0 && warp == 0;
@@ -318,7 +339,8 @@ __global__ void __launch_bounds__(32 * W, 16 / W) scan_kernel(const ScanParams<T
       const bool ok = on && j < p.K;
       rk[m] = ok ? p.k[row * p.stride + kh * p.K + j] : zero_t;
       rq[m] = ok ? p.q[row * p.stride + kh * p.K + j] : zero_t;
-      if constexpr (!kDelta && !kMem) rz[m] = ok ? p.z[row * p.z_stride + h * p.K + j] : zero_t;
+      if constexpr (kTime) rz[m] = ok ? p.zf[row * p.zf_stride + h * p.K + j] : 0.f;
+      else if constexpr (!kDelta && !kMem) rz[m] = ok ? p.z[row * p.z_stride + h * p.K + j] : zero_t;
     }
 #pragma unroll
     for (int m = 0; m < VL; ++m) {
@@ -350,6 +372,11 @@ __global__ void __launch_bounds__(32 * W, 16 / W) scan_kernel(const ScanParams<T
         vecs[j] = kf * write;
         vecs[K + j] = qf * p.q_scale;
         vecs[2 * K + j] = alpha_m1;
+      } else if constexpr (kTime) {
+        vecs[j] = kf;
+        vecs[K + j] = qf;
+        vecs[2 * K + j] = expm1f(time_log_decay(rz[m] + w0[m]));
+        kq = fmaf(kf * bonus[m], qf, kq);
       } else {
         vecs[j] = kf;
         vecs[K + j] = qf * p.q_scale;
@@ -358,6 +385,10 @@ __global__ void __launch_bounds__(32 * W, 16 / W) scan_kernel(const ScanParams<T
     }
 #pragma unroll
     for (int m = 0; m < VL; ++m) s_v[(buf * TT + warp) * kScanCols + m * 32 + lane] = Elem<T>::to_f(rv[m]);
+    if (kTime) {
+      kq = warp_sum(kq);
+      if (lane == 0) s_par[(buf * TT + warp) * 4] = kq;
+    }
     if (kDelta) {
       kk = warp_sum(kk);
       qq = warp_sum(qq);
@@ -395,7 +426,12 @@ __global__ void __launch_bounds__(32 * W, 16 / W) scan_kernel(const ScanParams<T
           const float4 par = *reinterpret_cast<const float4*>(s_par + (buf * TT + t) * 4);
           S.delta(vecs, vecs + K, sv, par.x, par.y, 1.f, 1.f, par.z, kp, o);
         } else {
-          S.gla(vecs, vecs + K, vecs + 2 * K, sv, kp, o);
+          S.template gla<kTime>(vecs, vecs + K, vecs + 2 * K, sv, kp, o);
+        }
+        if constexpr (kTime) {
+          const float own = s_par[(buf * TT + t) * 4];
+#pragma unroll
+          for (int j = 0; j < Sh::HELD; ++j) o[j] = fmaf(own, sv[Sh::first_held(kp) + j], o[j]);
         }
 #pragma unroll
         for (int j = 0; j < Sh::HELD; ++j)
@@ -484,7 +520,7 @@ __device__ __forceinline__ void mem_advance(const ScanParams<T>& p, int h, int s
 template <int KIND, typename T>
 __device__ __forceinline__ void step_vectors(const ScanParams<T>& p, int s, int h, int slot, int st0, int K, int vpad, float* s_k,
                                              float* s_q, float* s_a, float* s_v, const MemFactors& mem) {
-  constexpr bool kDelta = KIND == SK_DELTA, kMem = KIND == SK_MLSTM;
+  constexpr bool kDelta = KIND == SK_DELTA, kMem = KIND == SK_MLSTM, kTime = KIND == SK_TIME;
   const int kh = h / (p.heads / p.kv_heads);
   for (int i = threadIdx.x; i < K + K + vpad; i += blockDim.x) {
     const int part = i < K ? 0 : i < 2 * K ? 1 : 2, j = part == 0 ? i : part == 1 ? i - K : i - 2 * K;
@@ -503,7 +539,7 @@ __device__ __forceinline__ void step_vectors(const ScanParams<T>& p, int s, int 
           for (int n = 0; n < p.taps - 1; ++n) acc = fmaf(Elem<T>::to_f(wc[n]), Elem<T>::to_f(cs[static_cast<int64_t>(n) * p.channels]), acc);
         acc = fmaf(Elem<T>::to_f(wc[p.taps - 1]), x, acc);
         x = Elem<T>::to_f(Elem<T>::from_f(silu_t<T>(acc)));       // rounded as the prompt path stores it
-      } else if (part == 1) {
+      } else if (part == 1 && !kTime) {
         x *= p.q_scale;
       } else if (kMem && part == 0) {
         x *= mem.write;
@@ -511,7 +547,9 @@ __device__ __forceinline__ void step_vectors(const ScanParams<T>& p, int s, int 
     }
     (part == 0 ? s_k : part == 1 ? s_q : s_v)[j] = x;
     if (kMem && part == 0) s_a[j] = mem.alpha_m1;
-    if (!kDelta && !kMem && part == 0)
+    if (kTime && part == 0)
+      s_a[j] = ok ? expm1f(time_log_decay(p.zf[static_cast<int64_t>(s) * p.zf_stride + h * p.K + j] + Elem<T>::to_f(p.w0[h * p.K + j]))) : 0.f;
+    if (!kDelta && !kMem && !kTime && part == 0)
       s_a[j] = ok ? expm1f(channel_log_decay(Elem<T>::to_f(p.z[static_cast<int64_t>(s) * p.z_stride + h * p.K + j]), p.inv_tau)) : 0.f;
   }
 }
@@ -537,11 +575,18 @@ __device__ __forceinline__ StepFactors step_factors(const ScanParams<T>& p, int 
   return f;
 }
 
+// Time mixing: what a token's own entry adds to its read-out, per value.  Every warp for itself.
+template <typename T> __device__ __forceinline__ float own_entry(const ScanParams<T>& p, int h, const float* s_k, const float* s_q) {
+  float acc = 0.f;
+  for (int j = threadIdx.x & 31; j < p.K; j += 32) acc = fmaf(s_k[j] * Elem<T>::to_f(p.bonus[h * p.K + j]), s_q[j], acc);
+  return warp_sum(acc);
+}
+
 // Norm of the head's read-out and output gate; matrix memory divides first (s_nq: the terms of n . q).
 template <int KIND, typename T>
 __device__ __forceinline__ void step_output(const ScanParams<T>& p, int s, int h, const float* s_o, T* out, const float* s_nq,
                                             const MemFactors& mem) {
-  constexpr bool kMem = KIND == SK_MLSTM;
+  constexpr bool kMem = KIND == SK_MLSTM, kTime = KIND == SK_TIME;
   float inv = 1.f;
   if (kMem) {
     float dot = 0.f;
@@ -552,17 +597,17 @@ __device__ __forceinline__ void step_output(const ScanParams<T>& p, int s, int h
   for (int j = threadIdx.x & 31; j < p.V; j += 32) acc = fmaf(s_o[j] * inv, s_o[j] * inv, acc);
   const float rs = inv / sqrtf(warp_sum(acc) / static_cast<float>(p.V) + p.eps);
   const T* gate = p.gate + static_cast<int64_t>(s) * p.out_gate_stride + static_cast<int64_t>(h) * p.V;
-  const T* w = p.norm_w + (kMem ? static_cast<int64_t>(h) * p.V : 0);
+  const T* w = p.norm_w + (kMem || kTime ? static_cast<int64_t>(h) * p.V : 0);
   for (int j = threadIdx.x; j < p.V; j += blockDim.x) {
     const float g = Elem<T>::to_f(gate[j]);
-    out[j] = Elem<T>::from_f(s_o[j] * rs * Elem<T>::to_f(w[j]) * (kMem ? sigmoid_t<T>(g) : silu_t<T>(g)));
+    out[j] = Elem<T>::from_f(s_o[j] * rs * Elem<T>::to_f(w[j]) * (kMem ? sigmoid_t<T>(g) : silu_t<T>(g)) * (kTime ? p.out_scale : 1.f));
   }
 }
 
 // Any sizes: the state in the prompt kernel's layout.
 template <typename Sh, typename T>
 __global__ void __launch_bounds__(256, 1) step_kernel(const ScanParams<T> p) {
-  constexpr bool kDelta = Sh::KIND == SK_DELTA, kMem = Sh::KIND == SK_MLSTM;
+  constexpr bool kDelta = Sh::KIND == SK_DELTA, kMem = Sh::KIND == SK_MLSTM, kTime = Sh::KIND == SK_TIME;
   constexpr int K = Sh::K;
   extern __shared__ __align__(16) float sm[];
   const int vpad = (p.V + Sh::CW - 1) / Sh::CW * Sh::CW;
@@ -584,6 +629,7 @@ __global__ void __launch_bounds__(256, 1) step_kernel(const ScanParams<T> p) {
   if constexpr (kMem) mem_advance(p, h, slot, st0, mem, s_k, s_q, s_nq);
   StepFactors f{};
   if (kDelta) f = step_factors(p, s, h, K, s_k, s_q);
+  const float own = kTime ? own_entry(p, h, s_k, s_q) : 0.f;
   const bool writes = (!kDelta || (kp & (Sh::KP / 2))) && (kp & (Sh::LOW - 1)) == 0;
   ScanState<Sh> S;
   for (int cb = warp; cb * Sh::CW < p.V; cb += warps) {
@@ -592,10 +638,13 @@ __global__ void __launch_bounds__(256, 1) step_kernel(const ScanParams<T> p) {
     else S.zero();
     float o[Sh::HELD];
     if constexpr (kDelta) S.delta(s_k, s_q, s_v + c0, f.gm1, f.beta, f.ks, f.qs, f.kq, kp, o);
-    else S.gla(s_k, s_q, s_a, s_v + c0, kp, o);
+    else S.template gla<kTime>(s_k, s_q, s_a, s_v + c0, kp, o);
     if (writes)
 #pragma unroll
-      for (int j = 0; j < Sh::HELD; ++j) s_o[c0 + Sh::first_held(kp) + j] = o[j];
+      for (int j = 0; j < Sh::HELD; ++j) {
+        const int c = c0 + Sh::first_held(kp) + j;
+        s_o[c] = kTime ? fmaf(own, s_v[c], o[j]) : o[j];
+      }
     S.store(gS + c0, kp, p.K, p.V, p.V - c0, vec);
   }
   __syncthreads();
@@ -608,7 +657,7 @@ __global__ void __launch_bounds__(256, 1) step_kernel(const ScanParams<T> p) {
 constexpr int kStHold = 8, kStThreads4 = 512;
 template <int KIND, typename T>
 __global__ void __launch_bounds__(kStThreads4, 2) step_quad_kernel(const ScanParams<T> p, int vpad) {
-  constexpr bool kDelta = KIND == SK_DELTA, kMem = KIND == SK_MLSTM;
+  constexpr bool kDelta = KIND == SK_DELTA, kMem = KIND == SK_MLSTM, kTime = KIND == SK_TIME;
   extern __shared__ __align__(16) float sm[];
   const int K = (p.K + 3) & ~3, nthr = blockDim.x, tid = threadIdx.x, s = blockIdx.x, h = blockIdx.y;
   const int PQ = p.V / 4, rows = nthr / PQ, q = tid % PQ, r = tid / PQ;
@@ -653,17 +702,19 @@ __global__ void __launch_bounds__(kStThreads4, 2) step_quad_kernel(const ScanPar
         if (on && n < p.K) {
           const float a = s_a[n], k = s_k[n];
           const float4 old = x[i];
+          if (kTime) add(s_q[n], old, aq);
           add(a, old, x[i]);
           add(k, v, x[i]);
           gS[n * PQ] = x[i];
-          add(s_q[n], x[i], aq);
+          if (!kTime) add(s_q[n], x[i], aq);
         }
       }
     }
     if (on) red[r * PQ + q] = aq;
+    const float own = kTime ? own_entry(p, h, s_k, s_q) : 0.f;
     __syncthreads();
     for (int i = tid; i < p.V; i += nthr) {
-      float o = 0.f;
+      float o = kTime ? own * s_v[i] : 0.f;
       for (int k = 0; k < rows; ++k) o += reinterpret_cast<const float*>(red)[k * p.V + i];
       s_o[i] = o;
     }
@@ -748,7 +799,7 @@ template <int KIND, typename T> static int run_step(const ScanParams<T>& p, int 
     const int quads = p.V / 4, K = (p.K + 3) & ~3;
     const int threads = std::min(kStThreads4, std::max(128, (quads * ((p.K + kStHold - 1) / kStHold) + 31) / 32 * 32));
     const int fit = std::max(threads, (quads + 31) / 32 * 32), rows = fit / quads;
-    const size_t smem = sizeof(float) * ((KIND == SK_DELTA ? 2 : KIND == SK_GLA ? 3 : 4) * K + 2 * p.V + (KIND == SK_DELTA ? 2 : 1) * static_cast<size_t>(rows) * p.V);
+    const size_t smem = sizeof(float) * ((KIND == SK_DELTA ? 2 : KIND == SK_MLSTM ? 4 : 3) * K + 2 * p.V + (KIND == SK_DELTA ? 2 : 1) * static_cast<size_t>(rows) * p.V);
     if (smem <= 48 * 1024) {
       step_quad_kernel<KIND, T><<<dim3(num_seqs, p.heads), fit, smem, st>>>(p, p.V);
       return check_launch("state_step");
@@ -757,7 +808,7 @@ template <int KIND, typename T> static int run_step(const ScanParams<T>& p, int 
   return scan_dispatch<KIND>(p.K, [&](auto sh) {
     using Sh = decltype(sh);
     const int blocks = (p.V + Sh::CW - 1) / Sh::CW, warps = std::min(8, blocks);
-    const size_t smem = sizeof(float) * ((KIND == SK_DELTA ? 2 : KIND == SK_GLA ? 3 : 4) * Sh::K + 2 * static_cast<size_t>(blocks) * Sh::CW);
+    const size_t smem = sizeof(float) * ((KIND == SK_DELTA ? 2 : KIND == SK_MLSTM ? 4 : 3) * Sh::K + 2 * static_cast<size_t>(blocks) * Sh::CW);
     if (smem > 48 * 1024) return fail(MV_ERR_LIMIT, "state_step: vdim %d", p.V);
     step_kernel<Sh, T><<<dim3(num_seqs, p.heads), 32 * warps, smem, st>>>(p);
     return check_launch("state_step");

@@ -5,6 +5,11 @@
 // neighbouring columns (values that were turned by their own positions when they were stored).
 //
 // kv_norm_store_kernel        RMS norm over all query rows and over all key rows of a token, scatter of [k | v]
+// Two more forms of attention over the same kind of cache run on the kernel for any sizes (and on kernels of their own,
+// talk_attention.cu, diff_attention.cu):
+//   capped scores, a bias that grows with the logarithm of the distance, every weight head's result for every value head;
+//   keys in `maps` heads per value head, positions that see their own chunk of the sequence only.
+//
 // qkv_rope_store_kernel       RMS norm and rotation per query and key head, rotation of the values, scatter of [k | v]
 // window_attention_rows_kernel  any sizes, bf16 or fp32, token by token
 // window_decode_kernel        one token per sequence on mma.sync: HBM-bound on the rows inside the window
@@ -124,14 +129,14 @@ __device__ __forceinline__ void turn_back(float& a, float& b, float2 cs) {
 
 template <typename T> struct RopeStoreParams {
   T *q; const T *k, *v; int64_t stride;        // (tokens, heads * dim), (tokens, kv_heads * dim), (tokens, kv_heads * vdim)
-  const T *q_weight, *k_weight, *temp;         // (dim), (dim), (heads) or null
+  const T *q_weight, *k_weight, *temp;         // (dim), (dim; null: keys are stored as they are), (heads) or null
   const float *cos_t, *sin_t; int dims;        // (table_rows, dims / 2)
   const float *vcos_t, *vsin_t;                // (table_rows, vdim / 2), null: values are stored as they are
   int64_t table_rows;
   const int64_t* positions;
   T *kv_out, *cache; const int64_t* slot_mapping; int64_t num_slots;
   int64_t tokens;
-  int heads, kv_heads, dim, vdim;
+  int heads, kv_heads, v_heads, dim, vdim;
   float eps;
 };
 
@@ -139,7 +144,7 @@ template <typename T> struct RopeStoreParams {
 // value heads.
 template <typename T, int V, int L, int kCh>
 __global__ void __launch_bounds__(kKnThreads) qkv_rope_store_kernel(const RopeStoreParams<T> p) {
-  const int lane = threadIdx.x & (L - 1), per = p.heads + 2 * p.kv_heads, row = p.kv_heads * (p.dim + p.vdim);
+  const int lane = threadIdx.x & (L - 1), per = p.heads + p.kv_heads + p.v_heads, row = p.kv_heads * p.dim + p.v_heads * p.vdim;
   const uint32_t items = static_cast<uint32_t>(p.tokens * per), step = gridDim.x * (kKnThreads / L);      // the host checks the range
   for (uint32_t i0 = blockIdx.x * (kKnThreads / L); i0 < items; i0 += step) {
     const uint32_t i = i0 + threadIdx.x / L, row_i = i / static_cast<uint32_t>(per);
@@ -168,8 +173,8 @@ __global__ void __launch_bounds__(kKnThreads) qkv_rope_store_kernel(const RopeSt
     }
 #pragma unroll
     for (int o = L / 2; o; o >>= 1) acc += __shfl_xor_sync(0xffffffffu, acc, o);
-    const float rs = is_v ? 1.f : 1.f / sqrtf(acc / static_cast<float>(n) + p.eps);
     const T* weight = is_q ? p.q_weight : p.k_weight;
+    const float rs = 1.f / sqrtf(acc / static_cast<float>(n) + p.eps);
     const float f = is_q && p.temp && on ? Elem<T>::to_f(p.temp[head]) : 1.f;
     const float* co = is_v ? p.vcos_t : p.cos_t;
     const float* si = is_v ? p.vsin_t : p.sin_t;
@@ -189,7 +194,7 @@ __global__ void __launch_bounds__(kKnThreads) qkv_rope_store_kernel(const RopeSt
     for (int k = 0; k < kCh; ++k) {
       const int c = (k * L + lane) * V;
       if (!on || c >= n) continue;
-      if (!is_v) {
+      if (!is_v && weight) {
         if constexpr (V == 8) {
           float w[8];
           Vec<T, 8>::load(weight + c, w);
@@ -232,7 +237,13 @@ template <typename T> struct WindowParams {
   int64_t window;
   float scale;
   const float2* turn; int64_t table_rows;                      // (vdim / 2, table_rows) cos, sin: results are turned back; null: not
+  // rows only
+  float cap; const float *r1, *r2;           // cap > 0: score = cap tanh(score / cap) - r1[h] ln(1 + r2[h] distance)
+  int cross;                                 // value heads of which every head's result is wanted: out (tokens, heads, cross, vdim); 0: its own
+  int maps; int64_t chunk;                   // key heads per value head (query heads: [head][map]); chunk > 0: positions see their own chunk
+  float* out_f;                              // fp32 results instead of out
   // decode
+  const T* gate; int64_t gate_stride; float lambda, mult, eps;   // two maps: their difference, normed, times mult and sigmoid(gate)
   int splits;
   float *part_ml, *part_o;                   // (batch, splits, heads, 2) and (.., vdim)
 };
@@ -244,8 +255,11 @@ __global__ void __launch_bounds__(kWaThreads) window_attention_rows_kernel(const
   extern __shared__ __align__(16) float sm[];
   const int group = p.heads / p.kv_heads, chunks = (group + kWaHeads - 1) / kWaHeads;
   const int kv = blockIdx.y / chunks, g0 = (blockIdx.y - kv * chunks) * kWaHeads;
-  const int h0 = kv * group + g0, nh = min(kWaHeads, group - g0);
-  const int D = p.dim, VD = p.vdim, row = p.kv_heads * (D + VD);
+  const int nh = min(kWaHeads, group - g0);
+  const int D = p.dim, VD = p.vdim, v_heads = p.kv_heads / p.maps, row = p.kv_heads * D + v_heads * VD;
+  const int vh = p.cross ? blockIdx.z : kv / p.maps;
+  // query heads over key head kv: one per head of the group, `maps` apart
+  auto head_at = [&](int i) { return (kv / p.maps * group + g0 + i) * p.maps + kv % p.maps; };
   float* sq = sm;                               // [kWaHeads][D]
   float* sk = sq + kWaHeads * D;                // [kWaKeys][D + 1]
   float* sv = sk + kWaKeys * (D + 1);           // [kWaKeys][VD]
@@ -256,14 +270,14 @@ __global__ void __launch_bounds__(kWaThreads) window_attention_rows_kernel(const
   const int32_t* table = p.tables + static_cast<int64_t>(seq) * p.bt_stride;
   const int64_t pos = p.positions[t];
   const int nk = static_cast<int>(min(pos + 1, static_cast<int64_t>(p.max_blocks) * p.block_size));
-  const int first = static_cast<int>(max(pos - p.window + 1, static_cast<int64_t>(0)));
+  const int first = static_cast<int>(max(p.chunk ? pos / p.chunk * p.chunk : pos - p.window + 1, static_cast<int64_t>(0)));
   for (int i = tid; i < kWaHeads * D; i += kWaThreads) {
     const int h = i / D, j = i - h * D;
-    sq[i] = h < nh ? Elem<T>::to_f(p.q[t * p.q_stride + static_cast<int64_t>(h0 + h) * D + j]) : 0.f;
+    sq[i] = h < nh ? Elem<T>::to_f(p.q[t * p.q_stride + static_cast<int64_t>(head_at(h)) * D + j]) : 0.f;
   }
   // the sink is one more score without a value: it opens the running maximum and sum
   if (tid < kWaHeads) {
-    s_m[tid] = tid < nh && p.sink ? Elem<T>::to_f(p.sink[h0 + tid]) : -INFINITY;
+    s_m[tid] = tid < nh && p.sink ? Elem<T>::to_f(p.sink[head_at(tid)]) : -INFINITY;
     s_l[tid] = tid < nh && p.sink ? 1.f : 0.f;
   }
   float acc[kWaHeads][kWaPer];
@@ -280,11 +294,12 @@ __global__ void __launch_bounds__(kWaThreads) window_attention_rows_kernel(const
       const bool ok = phys >= 0 && phys < p.num_blocks;
       const T* src = p.cache + (static_cast<int64_t>(ok ? phys : 0) * p.block_size + (at - blk * p.block_size)) * row;
       for (int i = lane; i < D; i += 32) sk[k * (D + 1) + i] = ok ? Elem<T>::to_f(src[kv * D + i]) : 0.f;
-      for (int i = lane; i < VD; i += 32) sv[k * VD + i] = ok ? Elem<T>::to_f(src[p.kv_heads * D + kv * VD + i]) : 0.f;
+      for (int i = lane; i < VD; i += 32) sv[k * VD + i] = ok ? Elem<T>::to_f(src[p.kv_heads * D + vh * VD + i]) : 0.f;
       if (lane < kWaHeads) {
         float b = ok ? 0.f : -INFINITY;
         if (ok && p.bias && lane < nh)
-          b = p.bias[(h0 + lane) * p.bias_stride + min(static_cast<int>(pos) - at, p.distances - 1)];
+          b = p.bias[head_at(lane) * p.bias_stride + min(static_cast<int>(pos) - at, p.distances - 1)];
+        if (ok && p.r1 && lane < nh) b = -p.r1[head_at(lane)] * log1pf(p.r2[head_at(lane)] * static_cast<float>(static_cast<int>(pos) - at));
         ss[lane * kWaKeys + k] = b;
       }
     }
@@ -295,7 +310,9 @@ __global__ void __launch_bounds__(kWaThreads) window_attention_rows_kernel(const
       float s = 0.f;
       for (int i = half; i < D; i += 2) s = fmaf(a[i], b[i], s);
       s += __shfl_xor_sync(0xffffffffu, s, 1);
-      if (half == 0) ss[h * kWaKeys + k] += s * p.scale;     // -inf stays -inf
+      s *= p.scale;
+      if (p.cap > 0.f) s = p.cap * tanhf(s / p.cap);
+      if (half == 0) ss[h * kWaKeys + k] += s;     // -inf stays -inf
     }
     __syncthreads();
     if (warp < kWaHeads) {
@@ -345,7 +362,11 @@ __global__ void __launch_bounds__(kWaThreads) window_attention_rows_kernel(const
           acc[h][i] = fmaf(acc[h][i], cs.x, d & 1 ? -other * cs.y : other * cs.y);
         }
       }
-      if (d < VD) p.out[(static_cast<int64_t>(t) * p.heads + h0 + h) * VD + d] = Elem<T>::from_f(acc[h][i] * inv);
+      if (d < VD) {
+        const int64_t at = (p.cross ? (static_cast<int64_t>(t) * p.heads + head_at(h)) * p.cross + vh : static_cast<int64_t>(t) * p.heads + head_at(h)) * VD + d;
+        if (p.out_f) p.out_f[at] = acc[h][i] * inv;
+        else p.out[at] = Elem<T>::from_f(acc[h][i] * inv);
+      }
     }
   }
 }
@@ -354,41 +375,70 @@ __global__ void __launch_bounds__(kWaThreads) window_attention_rows_kernel(const
 // One CTA per (piece of the window, KV head and tile of 16 query heads, sequence): four warps stream 16-key tiles of
 // their own through cp.async rings; the query heads are the rows of m16n8k16 products.  Attention weights enter their
 // product as value and rounding residue.
+//
+// MAPS = 2: every head has two maps, with queries and keys of their own and the same values.  The upper eight rows are the
+// heads' first maps, the lower eight the second ones; the rows of the other map are left out of each product with keys.
 constexpr int kWdWarps = 4, kWdThreads = 32 * kWdWarps, kWdStages = 3, kWdTile = 16;
 constexpr float kWdNeg = -1e30f;
 
-template <int KD, int VD> struct WdShape {
-  static constexpr int kK = kWdTile * KD * 2, kV = kWdTile * VD * 2, kStage = kK + kV, kWarp = kWdStages * kStage;
+template <int KD, int VD, int MAPS = 1> struct WdShape {
+  static constexpr int kK = MAPS * kWdTile * KD * 2, kV = kWdTile * VD * 2, kStage = kK + kV, kWarp = kWdStages * kStage;
   static constexpr int kRing = kWdWarps * kWarp, kStride = VD + 8;
   static constexpr int kMerge = kWdWarps * 16 * (kStride + 2) * 4;
   static constexpr int kSmem = kRing > kMerge ? kRing : kMerge;
 };
 
-template <int KD, int VD>
-__global__ void __launch_bounds__(kWdThreads, KD + VD > 256 ? 1 : 2)
+// What becomes of the two maps' results of a row: a1 - lambda a2, its RMS norm over the head, factor and gate.  One warp;
+// get(d) gives the difference in columns d and d + 1.
+template <typename T, typename F>
+__device__ __forceinline__ void diff_finish(const WindowParams<T>& p, int64_t row, int h, int lane, F&& get) {
+  constexpr int kHold = 4;               // vdim up to 256
+  float2 o[kHold];
+  float acc = 0.f;
+#pragma unroll
+  for (int i = 0; i < kHold; ++i) {
+    const int d = (i * 32 + lane) * 2;
+    o[i] = d < p.vdim ? get(d) : make_float2(0.f, 0.f);
+    acc = fmaf(o[i].x, o[i].x, fmaf(o[i].y, o[i].y, acc));
+  }
+  const float f = p.mult / sqrtf(warp_sum(acc) / static_cast<float>(p.vdim) + p.eps);
+#pragma unroll
+  for (int i = 0; i < kHold; ++i) {
+    const int d = (i * 32 + lane) * 2;
+    if (d >= p.vdim) continue;
+    const T *g = p.gate + row * p.gate_stride + static_cast<int64_t>(h) * p.vdim + d;
+    T* out = p.out + (row * p.heads + h) * p.vdim + d;
+    out[0] = Elem<T>::from_f(o[i].x * f * sigmoid_t<T>(Elem<T>::to_f(g[0])));
+    out[1] = Elem<T>::from_f(o[i].y * f * sigmoid_t<T>(Elem<T>::to_f(g[1])));
+  }
+}
+
+template <int KD, int VD, int MAPS>
+__global__ void __launch_bounds__(kWdThreads, MAPS * KD + VD > 256 ? 1 : 2)
 window_decode_kernel(const WindowParams<__nv_bfloat16> p) {
   using T = __nv_bfloat16;
-  using S = WdShape<KD, VD>;
+  using S = WdShape<KD, VD, MAPS>;
+  constexpr int R = 16 / MAPS;           // heads per tile of rows
   using Mma = Mma16816<T>;
   constexpr int KSTEPS = KD / 16, NT = VD / 8, KC = KD / 8, VC = VD / 8;
   extern __shared__ __align__(128) unsigned char smem[];
   __shared__ uint32_t s_mask[kWdWarps][kWdStages];
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, g = lane >> 2, t = lane & 3;
-  const int group = p.heads / p.kv_heads, mtiles = (group + 15) / 16;
+  const int group = p.heads / p.kv_heads, mtiles = (group + R - 1) / R;
   const int kv = blockIdx.y / mtiles, mt = blockIdx.y - kv * mtiles, b = blockIdx.z, split = blockIdx.x;
-  const int rows = min(16, group - mt * 16), h0 = kv * group + mt * 16;
+  const int rows = min(R, group - mt * R), h0 = kv * group + mt * R;
   const int64_t pos64 = p.positions[b];
   const int pos = static_cast<int>(pos64);
   const int nk = static_cast<int>(min(pos64 + 1, static_cast<int64_t>(p.max_blocks) * p.block_size));
-  const int lo = static_cast<int>(max(pos64 - p.window + 1, static_cast<int64_t>(0)));
+  const int lo = static_cast<int>(max(MAPS > 1 ? pos64 / p.chunk * p.chunk : pos64 - p.window + 1, static_cast<int64_t>(0)));
   const int span = max(nk - lo, 0);
   const int len = ((span + p.splits - 1) / p.splits + kWdTile - 1) / kWdTile * kWdTile;
   const int k_begin = lo + split * len, k_end = min(k_begin + len, nk);
   const int tiles = k_end > k_begin ? (k_end - k_begin + kWdTile - 1) / kWdTile : 0;
   const int my_tiles = tiles > warp ? (tiles - warp + kWdWarps - 1) / kWdWarps : 0;
   const int32_t* table = p.tables + static_cast<int64_t>(b) * p.bt_stride;
-  const int64_t row_elems = static_cast<int64_t>(p.kv_heads) * (p.dim + p.vdim);
-  const T *k_base = p.cache + kv * p.dim, *v_base = p.cache + p.kv_heads * p.dim + kv * p.vdim;
+  const int64_t row_elems = static_cast<int64_t>(p.kv_heads) * (MAPS * p.dim + p.vdim);
+  const T *k_base = p.cache + kv * MAPS * p.dim, *v_base = p.cache + p.kv_heads * MAPS * p.dim + kv * p.vdim;
   const uint32_t ring = smem_u32(smem) + warp * S::kWarp;
   const int kc_real = p.dim / 8, vc_real = p.vdim / 8;
 
@@ -405,11 +455,11 @@ window_decode_kernel(const WindowParams<__nv_bfloat16> p) {
       if (lane == 0) s_mask[warp][stage] = live;
       const uint32_t kd = ring + stage * S::kStage, vd = kd + S::kK;
 #pragma unroll
-      for (int c0 = 0; c0 < kWdTile * KC; c0 += 32) {
-        const int r = (c0 + lane) / KC, c = (c0 + lane) % KC;
+      for (int c0 = 0; c0 < MAPS * kWdTile * KC; c0 += 32) {
+        const int m = c0 / (kWdTile * KC), r = (c0 + lane) / KC % kWdTile, c = (c0 + lane) % KC;
         const int64_t src = __shfl_sync(0xffffffffu, at, r);
         const bool ok = src >= 0 && c < kc_real;
-        cp_async16(kd + r * (KD * 2) + ((c ^ (r & 7)) << 4), ok ? k_base + src + c * 8 : p.cache, ok ? 16 : 0);
+        cp_async16(kd + (m * kWdTile + r) * (KD * 2) + ((c ^ (r & 7)) << 4), ok ? k_base + src + m * p.dim + c * 8 : p.cache, ok ? 16 : 0);
       }
 #pragma unroll
       for (int c0 = 0; c0 < kWdTile * VC; c0 += 32) {
@@ -426,10 +476,10 @@ window_decode_kernel(const WindowParams<__nv_bfloat16> p) {
 
   uint32_t qa[KSTEPS][4];
   {
-    const T* qb = p.q + b * p.q_stride + static_cast<int64_t>(h0) * p.dim;
-    const bool v0 = g < rows, v1 = g + 8 < rows;
-    const uint32_t* q0 = reinterpret_cast<const uint32_t*>(qb + static_cast<int64_t>(g) * p.dim);
-    const uint32_t* q1 = reinterpret_cast<const uint32_t*>(qb + static_cast<int64_t>(g + 8) * p.dim);
+    const T* qb = p.q + b * p.q_stride + static_cast<int64_t>(h0) * MAPS * p.dim;
+    const bool v0 = g < rows, v1 = MAPS > 1 ? v0 : g + 8 < rows;
+    const uint32_t* q0 = reinterpret_cast<const uint32_t*>(qb + static_cast<int64_t>(MAPS * g) * p.dim);
+    const uint32_t* q1 = reinterpret_cast<const uint32_t*>(qb + static_cast<int64_t>(MAPS > 1 ? 2 * g + 1 : g + 8) * p.dim);
     const int half = p.dim / 2;
 #pragma unroll
     for (int ks = 0; ks < KSTEPS; ++ks) {
@@ -465,6 +515,18 @@ window_decode_kernel(const WindowParams<__nv_bfloat16> p) {
         ldmatrix_x4(kb, kd + row * (KD * 2) + (((2 * ks + csel) ^ (row & 7)) << 4));
         Mma::run(s[0], qa[ks], kb[0], kb[1]);
         Mma::run(s[1], qa[ks], kb[2], kb[3]);
+      }
+      if constexpr (MAPS > 1) {
+        float s2[2][4] = {};
+#pragma unroll
+        for (int ks = 0; ks < KSTEPS; ++ks) {
+          uint32_t kb[4];
+          ldmatrix_x4(kb, kd + (kWdTile + row) * (KD * 2) + (((2 * ks + csel) ^ (row & 7)) << 4));
+          Mma::run(s2[0], qa[ks], kb[0], kb[1]);
+          Mma::run(s2[1], qa[ks], kb[2], kb[3]);
+        }
+#pragma unroll
+        for (int n = 0; n < 2; ++n) { s[n][2] = s2[n][2]; s[n][3] = s2[n][3]; }
       }
     }
     issue(i + kWdStages - 1);
@@ -555,6 +617,53 @@ window_decode_kernel(const WindowParams<__nv_bfloat16> p) {
     }
   }
   __syncthreads();
+  if constexpr (MAPS > 1) {
+    auto scales = [&](int r, float (&f)[kWdWarps], float& M) {     // factors of the warps' parts of a row; returns its sum
+      M = kWdNeg;
+#pragma unroll
+      for (int w = 0; w < kWdWarps; ++w) M = fmaxf(M, sML[(w * 16 + r) * 2]);
+      float L = 0.f;
+#pragma unroll
+      for (int w = 0; w < kWdWarps; ++w) {
+        f[w] = fast_exp2(sML[(w * 16 + r) * 2] - M);
+        L = fmaf(f[w], sML[(w * 16 + r) * 2 + 1], L);
+      }
+      return L;
+    };
+    auto joined = [&](int r, const float (&f)[kWdWarps], int d) {
+      float2 acc = make_float2(0.f, 0.f);
+#pragma unroll
+      for (int w = 0; w < kWdWarps; ++w) {
+        const float2 o2 = *reinterpret_cast<const float2*>(sO + (w * 16 + r) * S::kStride + d);
+        acc.x = fmaf(f[w], o2.x, acc.x);
+        acc.y = fmaf(f[w], o2.y, acc.y);
+      }
+      return acc;
+    };
+    for (int r = warp; r < rows; r += kWdWarps) {
+      float f1[kWdWarps], f2[kWdWarps], M1, M2;
+      const float L1 = scales(r, f1, M1), L2 = scales(r + 8, f2, M2);
+      if (p.splits == 1) {
+        const float i1 = L1 > 0.f ? 1.f / L1 : 0.f, i2 = L2 > 0.f ? p.lambda / L2 : 0.f;
+        diff_finish(p, b, h0 + r, lane, [&](int d) {
+          const float2 a1 = joined(r, f1, d), a2 = joined(r + 8, f2, d);
+          return make_float2(a1.x * i1 - a2.x * i2, a1.y * i1 - a2.y * i2);
+        });
+      } else {
+#pragma unroll
+        for (int m = 0; m < 2; ++m) {
+          const int64_t pi = ((static_cast<int64_t>(b) * p.splits + split) * p.heads + h0 + r) * 2 + m;
+          for (int d = lane * 2; d < p.vdim; d += 64)
+            *reinterpret_cast<float2*>(p.part_o + pi * p.vdim + d) = m ? joined(r + 8, f2, d) : joined(r, f1, d);
+          if (lane == 0) {
+            p.part_ml[pi * 2] = m ? M2 : M1;
+            p.part_ml[pi * 2 + 1] = m ? L2 : L1;
+          }
+        }
+      }
+    }
+    return;
+  }
   const int half = p.vdim / 2;           // a thread has pairs of neighbouring columns
   const int64_t angle = p.turn ? table_row(pos64, p.table_rows) : 0;
   for (int i = tid; i < rows * half; i += kWdThreads) {
@@ -622,21 +731,71 @@ __global__ void __launch_bounds__(128) window_join_kernel(const WindowParams<__n
   }
 }
 
-template <int KD, int VD> static int launch_window_decode(const WindowParams<__nv_bfloat16>& p, int batch, cudaStream_t st) {
-  const int smem = WdShape<KD, VD>::kSmem;
-  const cudaError_t e = cudaFuncSetAttribute(window_decode_kernel<KD, VD>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
+// The same for two maps: a warp per sequence and head.
+__global__ void __launch_bounds__(128) diff_join_kernel(const WindowParams<__nv_bfloat16> p, int batch) {
+  const int i = blockIdx.x * 4 + (threadIdx.x >> 5), lane = threadIdx.x & 31, b = i / p.heads, h = i - b * p.heads;
+  if (b >= batch) return;
+  const int64_t first = (static_cast<int64_t>(b) * p.splits * p.heads + h) * 2, step = static_cast<int64_t>(p.heads) * 2;
+  float M[2] = {kWdNeg, kWdNeg}, L[2] = {0.f, 0.f};
+#pragma unroll
+  for (int m = 0; m < 2; ++m) {
+    for (int s = 0; s < p.splits; ++s) M[m] = fmaxf(M[m], p.part_ml[(first + s * step + m) * 2]);
+    for (int s = 0; s < p.splits; ++s) {
+      const float* ml = p.part_ml + (first + s * step + m) * 2;
+      L[m] = fmaf(fast_exp2(ml[0] - M[m]), ml[1], L[m]);
+    }
+  }
+  const float i1 = L[0] > 0.f ? 1.f / L[0] : 0.f, i2 = L[1] > 0.f ? p.lambda / L[1] : 0.f;
+  diff_finish(p, b, h, lane, [&](int d) {
+    float2 acc = make_float2(0.f, 0.f);
+    for (int s = 0; s < p.splits; ++s) {
+      const int64_t pi = first + s * step;
+      const float f1 = fast_exp2(p.part_ml[pi * 2] - M[0]) * i1, f2 = fast_exp2(p.part_ml[pi * 2 + 2] - M[1]) * i2;
+      const float2 a1 = *reinterpret_cast<const float2*>(p.part_o + pi * p.vdim + d), a2 = *reinterpret_cast<const float2*>(p.part_o + (pi + 1) * p.vdim + d);
+      acc.x += f1 * a1.x - f2 * a2.x;
+      acc.y += f1 * a1.y - f2 * a2.y;
+    }
+    return acc;
+  });
+}
+
+// Difference, norm and gate for results in fp32, (tokens, heads, 2, vdim): a warp per token and head.
+template <typename T> struct DiffParams {
+  T* out; const float* a; const T* gate; int64_t gate_stride; int64_t tokens; int heads, vdim; float lambda, mult, eps;
+};
+template <typename T> __global__ void __launch_bounds__(256) diff_norm_gate_kernel(const DiffParams<T> p) {
+  const int lane = threadIdx.x & 31;
+  for (int64_t i = static_cast<int64_t>(blockIdx.x) * 8 + (threadIdx.x >> 5); i < p.tokens * p.heads; i += static_cast<int64_t>(gridDim.x) * 8) {
+    const int64_t t = i / p.heads, h = i - t * p.heads;
+    const float *a1 = p.a + i * 2 * p.vdim, *a2 = a1 + p.vdim;
+    float acc = 0.f;
+    for (int d = lane; d < p.vdim; d += 32) {
+      const float o = a1[d] - p.lambda * a2[d];
+      acc = fmaf(o, o, acc);
+    }
+    const float f = p.mult / sqrtf(warp_sum(acc) / static_cast<float>(p.vdim) + p.eps);
+    const T* g = p.gate + t * p.gate_stride + h * p.vdim;
+    for (int d = lane; d < p.vdim; d += 32)
+      p.out[i * p.vdim + d] = Elem<T>::from_f((a1[d] - p.lambda * a2[d]) * f * sigmoid_t<T>(Elem<T>::to_f(g[d])));
+  }
+}
+
+template <int KD, int VD, int MAPS = 1> static int launch_window_decode(const WindowParams<__nv_bfloat16>& p, int batch, cudaStream_t st) {
+  const int smem = WdShape<KD, VD, MAPS>::kSmem;
+  const cudaError_t e = cudaFuncSetAttribute(window_decode_kernel<KD, VD, MAPS>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
   if (e != cudaSuccess) return fail(MV_ERR_CUDA, "window_decode: %s", cudaGetErrorString(e));
-  const int mtiles = (p.heads / p.kv_heads + 15) / 16;
-  window_decode_kernel<KD, VD><<<dim3(p.splits, p.kv_heads * mtiles, batch), kWdThreads, smem, st>>>(p);
+  const int mtiles = (p.heads / p.kv_heads + 16 / MAPS - 1) / (16 / MAPS);
+  window_decode_kernel<KD, VD, MAPS><<<dim3(p.splits, p.kv_heads * mtiles, batch), kWdThreads, smem, st>>>(p);
   int rc = check_launch("window_decode");
   if (rc || p.splits == 1) return rc;
-  window_join_kernel<<<dim3(p.heads, batch), 128, 0, st>>>(p);
+  if (MAPS > 1) diff_join_kernel<<<static_cast<unsigned>((static_cast<int64_t>(batch) * p.heads + 3) / 4), 128, 0, st>>>(p, batch);
+  else window_join_kernel<<<dim3(p.heads, batch), 128, 0, st>>>(p);
   return check_launch("window_join");
 }
 
 // Pieces per sequence: enough CTAs to fill the GPU twice, none of less than 64 keys.  Depends on shapes only.
-static int window_splits(int batch, int heads, int kv_heads, int64_t most_keys) {
-  const int64_t units = static_cast<int64_t>(batch) * kv_heads * ((heads / kv_heads + 15) / 16);
+static int window_splits(int batch, int heads, int kv_heads, int64_t most_keys, int rows = 16) {
+  const int64_t units = static_cast<int64_t>(batch) * kv_heads * ((heads / kv_heads + rows - 1) / rows);
   const int64_t want = (2 * kNumSMs + units - 1) / std::max<int64_t>(units, 1);
   return static_cast<int>(std::max<int64_t>(1, std::min<int64_t>({want, most_keys / 64, 64})));
 }
@@ -683,18 +842,19 @@ extern "C" int mv_qkv_rope_store(void* q, const void* k, const void* v, int64_t 
                                  const void* k_weight, const void* temp, const float* cos_t, const float* sin_t, int dims,
                                  const float* vcos_t, const float* vsin_t, int64_t table_rows, const int64_t* positions,
                                  void* kv_out, void* cache, const int64_t* slot_mapping, int64_t num_slots, int64_t tokens,
-                                 int heads, int kv_heads, int dim, int vdim, float eps, int dtype, void* stream) {
+                                 int heads, int kv_heads, int v_heads, int dim, int vdim, float eps, int dtype, void* stream) {
   using namespace mv;
   if (dtype != MV_BF16 && dtype != MV_F32) return fail(MV_ERR_DTYPE, "qkv_rope_store: dtype %d", dtype);
-  if (tokens < 0 || heads <= 0 || kv_heads < 0 || dim <= 0 || vdim < 0 || (kv_heads && vdim <= 0) || dims < 0 || dims > dim || dims % 2 ||
-      (vcos_t && vdim % 2) || table_rows <= 0)
-    return fail(MV_ERR_SHAPE, "qkv_rope_store: heads %d over %d, dim %d (%d rotated), vdim %d", heads, kv_heads, dim, dims, vdim);
+  if (tokens < 0 || heads < 0 || kv_heads < 0 || !kv_heads != !v_heads || v_heads < 0 || heads + kv_heads == 0 || dim <= 0 || vdim < 0 ||
+      (kv_heads && vdim <= 0) || dims < 0 || dims > dim || dims % 2 || (vcos_t && vdim % 2) || table_rows <= 0)
+    return fail(MV_ERR_SHAPE, "qkv_rope_store: heads %d over %d and %d, dim %d (%d rotated), vdim %d", heads, kv_heads, v_heads, dim, dims, vdim);
   const int widest = kv_heads ? std::max(dim, vdim) : dim;
   if (widest > 1024) return fail(MV_ERR_LIMIT, "qkv_rope_store: dim %d, vdim %d (at most 1024)", dim, vdim);
-  if (tokens * (heads + 2 * static_cast<int64_t>(kv_heads)) >= 1LL << 31) return fail(MV_ERR_LIMIT, "qkv_rope_store: %lld tokens", static_cast<long long>(tokens));
+  const int64_t items = tokens * (heads + static_cast<int64_t>(kv_heads) + v_heads);
+  if (items >= 1LL << 31) return fail(MV_ERR_LIMIT, "qkv_rope_store: %lld tokens", static_cast<long long>(tokens));
   if (tokens == 0) return MV_OK;
-  if (!q || !q_weight || !positions || (dims && (!cos_t || !sin_t)) || !vcos_t != !vsin_t ||
-      (kv_heads && (!k || !v || !k_weight)) || (cache && !slot_mapping))
+  if ((heads && (!q || !q_weight)) || !positions || (dims && (!cos_t || !sin_t)) || !vcos_t != !vsin_t ||
+      (kv_heads && (!k || !v)) || (cache && !slot_mapping))
     return fail(MV_ERR_NULL, "qkv_rope_store: null pointer");
   auto run = [&](auto tag) {
     using T = decltype(tag);
@@ -702,9 +862,9 @@ extern "C" int mv_qkv_rope_store(void* q, const void* k, const void* v, int64_t 
     auto c = [](const void* x) { return static_cast<const T*>(x); };
     RopeStoreParams<T> p{static_cast<T*>(q), c(k), c(v), stride, c(q_weight), c(k_weight), c(temp), cos_t, sin_t, dims, vcos_t, vsin_t,
                          table_rows, positions, static_cast<T*>(kv_out), static_cast<T*>(cache), slot_mapping, num_slots, tokens,
-                         heads, kv_heads, dim, vdim, eps};
+                         heads, kv_heads, v_heads, dim, vdim, eps};
     auto go = [&](auto kernel, int lanes) {
-      const int64_t blocks = (tokens * (heads + 2 * kv_heads) + kKnThreads / lanes - 1) / (kKnThreads / lanes);
+      const int64_t blocks = (items + kKnThreads / lanes - 1) / (kKnThreads / lanes);
       kernel<<<static_cast<unsigned>(std::min<int64_t>(blocks, kNumSMs * 64)), kKnThreads, 0, static_cast<cudaStream_t>(stream)>>>(p);
       return check_launch("qkv_rope_store");
     };
@@ -720,38 +880,80 @@ extern "C" int mv_qkv_rope_store(void* q, const void* k, const void* v, int64_t 
   return dtype == MV_F32 ? run(float{}) : run(__nv_bfloat16{});
 }
 
+// What the forms of attention on the kernel for any sizes differ in.
+struct RowsForm {
+  const float* bias = nullptr; int64_t bias_stride = 0; int distances = 1; const void* sink = nullptr;
+  const float* turn = nullptr; int64_t table_rows = 0;
+  float cap = 0.f; const float *r1 = nullptr, *r2 = nullptr; int cross = 0, maps = 1; int64_t chunk = 0; float* out_f = nullptr;
+};
+static int attention_rows(const char* what, void* out, const void* q, int64_t q_stride, const void* cache,
+                          const int32_t* block_tables, int64_t bt_stride, int max_blocks, int block_size, int64_t num_blocks,
+                          const int32_t* cu_q, int num_seqs, const int64_t* positions, int64_t tokens, int heads, int kv_heads,
+                          int dim, int vdim, int64_t window, float scale, const RowsForm& f, int dtype, void* stream) {
+  using namespace mv;
+  if (dtype != MV_BF16 && dtype != MV_F32) return fail(MV_ERR_DTYPE, "%s: dtype %d", what, dtype);
+  const int rc = check_window(what, heads, kv_heads, dim, vdim, window, block_size);
+  if (rc) return rc;
+  if (!check_turn(f.turn, f.table_rows, vdim)) return fail(MV_ERR_SHAPE, "%s: rotation of %d columns", what, vdim);
+  if (vdim > kWaThreads * kWaPer) return fail(MV_ERR_LIMIT, "%s: vdim %d (at most %d)", what, vdim, kWaThreads * kWaPer);
+  if (f.bias && f.distances <= 0) return fail(MV_ERR_SHAPE, "%s: %d distances", what, f.distances);
+  if (tokens <= 0) return tokens < 0 ? fail(MV_ERR_SHAPE, "%s: tokens", what) : static_cast<int>(MV_OK);
+  if (!(out || f.out_f) || !q || !cache || !block_tables || !positions) return fail(MV_ERR_NULL, "%s: null pointer", what);
+  const size_t smem = sizeof(float) * (static_cast<size_t>(kWaHeads) * dim + static_cast<size_t>(kWaKeys) * (dim + 1 + vdim) + kWaHeads * kWaKeys);
+  if (smem > 227 * 1024) return fail(MV_ERR_LIMIT, "%s: dim %d, vdim %d", what, dim, vdim);
+  auto run = [&](auto tag) {
+    using T = decltype(tag);
+    const cudaError_t e = cudaFuncSetAttribute(window_attention_rows_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem));
+    if (e != cudaSuccess) return fail(MV_ERR_CUDA, "%s: %s", what, cudaGetErrorString(e));
+    WindowParams<T> p{};
+    p.out = static_cast<T*>(out); p.q = static_cast<const T*>(q); p.q_stride = q_stride; p.cache = static_cast<const T*>(cache);
+    p.tables = block_tables; p.bt_stride = bt_stride; p.max_blocks = max_blocks; p.block_size = block_size; p.num_blocks = num_blocks;
+    p.cu_q = cu_q; p.num_seqs = num_seqs; p.positions = positions; p.bias = f.bias; p.bias_stride = f.bias_stride; p.distances = f.distances;
+    p.sink = static_cast<const T*>(f.sink); p.heads = heads; p.kv_heads = kv_heads; p.dim = dim; p.vdim = vdim; p.window = window; p.scale = scale;
+    p.turn = reinterpret_cast<const float2*>(f.turn); p.table_rows = f.table_rows;
+    p.cap = f.cap; p.r1 = f.r1; p.r2 = f.r2; p.cross = f.cross; p.maps = f.maps; p.chunk = f.chunk; p.out_f = f.out_f;
+    const int chunks = (heads / kv_heads + kWaHeads - 1) / kWaHeads;
+    window_attention_rows_kernel<T><<<dim3(static_cast<unsigned>(tokens), kv_heads * chunks, f.cross ? f.cross : 1), kWaThreads, smem, static_cast<cudaStream_t>(stream)>>>(p);
+    return check_launch(what);
+  };
+  return dtype == MV_F32 ? run(float{}) : run(__nv_bfloat16{});
+}
+
 extern "C" int mv_window_attention_rows(void* out, const void* q, int64_t q_stride, const void* cache,
                                         const int32_t* block_tables, int64_t bt_stride, int max_blocks, int block_size,
                                         int64_t num_blocks, const int32_t* cu_q, int num_seqs, const int64_t* positions,
                                         const float* bias, int64_t bias_stride, int distances, const void* sink,
                                         const float* turn, int64_t table_rows, int64_t tokens, int heads, int kv_heads,
                                         int dim, int vdim, int64_t window, float scale, int dtype, void* stream) {
-  using namespace mv;
-  if (dtype != MV_BF16 && dtype != MV_F32) return fail(MV_ERR_DTYPE, "window_attention_rows: dtype %d", dtype);
-  const int rc = check_window("window_attention_rows", heads, kv_heads, dim, vdim, window, block_size);
-  if (rc) return rc;
-  if (!check_turn(turn, table_rows, vdim)) return fail(MV_ERR_SHAPE, "window_attention_rows: rotation of %d columns", vdim);
-  if (vdim > kWaThreads * kWaPer) return fail(MV_ERR_LIMIT, "window_attention_rows: vdim %d (at most %d)", vdim, kWaThreads * kWaPer);
-  if (bias && distances <= 0) return fail(MV_ERR_SHAPE, "window_attention_rows: %d distances", distances);
-  if (tokens <= 0) return tokens < 0 ? fail(MV_ERR_SHAPE, "window_attention_rows: tokens") : static_cast<int>(MV_OK);
-  if (!out || !q || !cache || !block_tables || !positions) return fail(MV_ERR_NULL, "window_attention_rows: null pointer");
-  const size_t smem = sizeof(float) * (static_cast<size_t>(kWaHeads) * dim + static_cast<size_t>(kWaKeys) * (dim + 1 + vdim) + kWaHeads * kWaKeys);
-  if (smem > 227 * 1024) return fail(MV_ERR_LIMIT, "window_attention_rows: dim %d, vdim %d", dim, vdim);
-  auto run = [&](auto tag) {
-    using T = decltype(tag);
-    const cudaError_t e = cudaFuncSetAttribute(window_attention_rows_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem));
-    if (e != cudaSuccess) return fail(MV_ERR_CUDA, "window_attention_rows: %s", cudaGetErrorString(e));
-    WindowParams<T> p{};
-    p.out = static_cast<T*>(out); p.q = static_cast<const T*>(q); p.q_stride = q_stride; p.cache = static_cast<const T*>(cache);
-    p.tables = block_tables; p.bt_stride = bt_stride; p.max_blocks = max_blocks; p.block_size = block_size; p.num_blocks = num_blocks;
-    p.cu_q = cu_q; p.num_seqs = num_seqs; p.positions = positions; p.bias = bias; p.bias_stride = bias_stride; p.distances = distances;
-    p.sink = static_cast<const T*>(sink); p.heads = heads; p.kv_heads = kv_heads; p.dim = dim; p.vdim = vdim; p.window = window; p.scale = scale;
-    p.turn = reinterpret_cast<const float2*>(turn); p.table_rows = table_rows;
-    const int chunks = (heads / kv_heads + kWaHeads - 1) / kWaHeads;
-    window_attention_rows_kernel<T><<<dim3(static_cast<unsigned>(tokens), kv_heads * chunks), kWaThreads, smem, static_cast<cudaStream_t>(stream)>>>(p);
-    return check_launch("window_attention_rows");
-  };
-  return dtype == MV_F32 ? run(float{}) : run(__nv_bfloat16{});
+  RowsForm f;
+  f.bias = bias; f.bias_stride = bias_stride; f.distances = distances; f.sink = sink; f.turn = turn; f.table_rows = table_rows;
+  return attention_rows("window_attention_rows", out, q, q_stride, cache, block_tables, bt_stride, max_blocks, block_size, num_blocks, cu_q,
+                        num_seqs, positions, tokens, heads, kv_heads, dim, vdim, window, scale, f, dtype, stream);
+}
+
+extern "C" int mv_talk_attention_rows(float* out, const void* q, int64_t q_stride, const void* cache,
+                                      const int32_t* block_tables, int64_t bt_stride, int max_blocks, int block_size,
+                                      int64_t num_blocks, const int32_t* cu_q, int num_seqs, const int64_t* positions,
+                                      const float* r1, const float* r2, float cap, int64_t tokens, int heads, int kv_heads,
+                                      int dim, int vdim, float scale, int dtype, void* stream) {
+  RowsForm f;
+  if (!(cap > 0.f)) return mv::fail(MV_ERR_SHAPE, "talk_attention_rows: cap %f", cap);
+  if (!r1 || !r2) return mv::fail(MV_ERR_NULL, "talk_attention_rows: null pointer");
+  f.r1 = r1; f.r2 = r2; f.cap = cap; f.cross = kv_heads; f.out_f = out;
+  return attention_rows("talk_attention_rows", nullptr, q, q_stride, cache, block_tables, bt_stride, max_blocks, block_size, num_blocks, cu_q,
+                        num_seqs, positions, tokens, heads, kv_heads, dim, vdim, 1LL << 40, scale, f, dtype, stream);
+}
+
+extern "C" int mv_diff_attention_rows(float* out, const void* q, int64_t q_stride, const void* cache,
+                                      const int32_t* block_tables, int64_t bt_stride, int max_blocks, int block_size,
+                                      int64_t num_blocks, const int32_t* cu_q, int num_seqs, const int64_t* positions,
+                                      int64_t chunk, int64_t tokens, int heads, int kv_heads, int dim, int vdim, float scale,
+                                      int dtype, void* stream) {
+  RowsForm f;
+  if (chunk <= 0) return mv::fail(MV_ERR_SHAPE, "diff_attention_rows: chunk %lld", static_cast<long long>(chunk));
+  f.maps = 2; f.chunk = chunk; f.out_f = out;
+  return attention_rows("diff_attention_rows", nullptr, q, q_stride, cache, block_tables, bt_stride, max_blocks, block_size, num_blocks, cu_q,
+                        num_seqs, positions, tokens, 2 * heads, 2 * kv_heads, dim, vdim, 1LL << 40, scale, f, dtype, stream);
 }
 
 // Bytes of scratch, or -1 when the kernel does not take the sizes.
@@ -802,4 +1004,70 @@ extern "C" int mv_window_decode(void* out, const void* q, int64_t q_stride, cons
   if (dim <= 64) return go(std::integral_constant<int, 64>{});
   if (dim <= 128) return go(std::integral_constant<int, 128>{});
   return go(std::integral_constant<int, 256>{});
+}
+
+// ------------------------------------------------------------------------------------------------ two maps per head
+static int64_t diff_most_keys(int64_t chunk, int max_blocks, int block_size) {
+  return std::max<int64_t>(1, std::min<int64_t>(chunk, static_cast<int64_t>(max_blocks) * block_size));
+}
+// Bytes of scratch, or -1 when the kernel does not take the sizes.
+extern "C" int64_t mv_diff_decode_workspace_bytes(int batch, int heads, int kv_heads, int dim, int vdim, int64_t most_keys) {
+  using namespace mv;
+  if (batch < 0 || batch > 65535 || heads <= 0 || kv_heads <= 0 || heads % kv_heads || dim <= 0 || vdim <= 0 || dim % 8 || vdim % 8 ||
+      dim > 128 || vdim > 256 || most_keys <= 0)
+    return -1;
+  const int splits = window_splits(batch, heads, kv_heads, most_keys, 8);
+  return splits == 1 ? 0 : static_cast<int64_t>(batch) * splits * heads * 2 * (vdim + 2) * 4;
+}
+
+extern "C" int mv_diff_decode(void* out, const void* q, int64_t q_stride, const void* cache, const int32_t* block_tables,
+                              int64_t bt_stride, int max_blocks, int block_size, int64_t num_blocks,
+                              const int64_t* positions, int64_t chunk, const void* gate, int64_t gate_stride, float lambda,
+                              float mult, float eps, int batch, int heads, int kv_heads, int dim, int vdim, float scale,
+                              void* workspace, int64_t workspace_bytes, void* stream) {
+  using namespace mv;
+  const int rc = check_window("diff_decode", heads, kv_heads, dim, vdim, chunk, block_size);
+  if (rc) return rc;
+  const int64_t most = diff_most_keys(chunk, max_blocks, block_size), need = mv_diff_decode_workspace_bytes(batch, heads, kv_heads, dim, vdim, most);
+  if (need < 0) return fail(MV_ERR_LIMIT, "diff_decode: dim %d, vdim %d, batch %d", dim, vdim, batch);
+  if (batch == 0) return MV_OK;
+  if (!out || !q || !cache || !block_tables || !positions || !gate) return fail(MV_ERR_NULL, "diff_decode: null pointer");
+  if (!aligned16(cache) || (reinterpret_cast<uintptr_t>(q) & 3u) || (reinterpret_cast<uintptr_t>(out) & 3u) || q_stride % 2)
+    return fail(MV_ERR_ALIGN, "diff_decode: alignment");
+  if (need > 0 && (!workspace || workspace_bytes < need)) return fail(MV_ERR_WORKSPACE, "diff_decode: workspace");
+  WindowParams<__nv_bfloat16> p{};
+  p.out = static_cast<__nv_bfloat16*>(out); p.q = static_cast<const __nv_bfloat16*>(q); p.q_stride = q_stride;
+  p.cache = static_cast<const __nv_bfloat16*>(cache);
+  p.tables = block_tables; p.bt_stride = bt_stride; p.max_blocks = max_blocks; p.block_size = block_size; p.num_blocks = num_blocks;
+  p.positions = positions; p.distances = 1; p.heads = heads; p.kv_heads = kv_heads; p.dim = dim; p.vdim = vdim; p.scale = scale;
+  p.window = 1LL << 40; p.maps = 2; p.chunk = chunk;
+  p.gate = static_cast<const __nv_bfloat16*>(gate); p.gate_stride = gate_stride; p.lambda = lambda; p.mult = mult; p.eps = eps;
+  p.splits = window_splits(batch, heads, kv_heads, most, 8);
+  p.part_ml = static_cast<float*>(workspace);
+  p.part_o = p.part_ml ? p.part_ml + static_cast<int64_t>(batch) * p.splits * heads * 4 : nullptr;
+  auto st = static_cast<cudaStream_t>(stream);
+  auto go = [&](auto kd) {
+    constexpr int KD = decltype(kd)::value;
+    if (vdim <= 64) return launch_window_decode<KD, 64, 2>(p, batch, st);
+    if (vdim <= 128) return launch_window_decode<KD, 128, 2>(p, batch, st);
+    return launch_window_decode<KD, 256, 2>(p, batch, st);
+  };
+  return dim <= 64 ? go(std::integral_constant<int, 64>{}) : go(std::integral_constant<int, 128>{});
+}
+
+extern "C" int mv_diff_norm_gate(void* out, const float* a, const void* gate, int64_t gate_stride, float lambda, float mult,
+                                 float eps, int64_t tokens, int heads, int vdim, int dtype, void* stream) {
+  using namespace mv;
+  if (dtype != MV_BF16 && dtype != MV_F32) return fail(MV_ERR_DTYPE, "diff_norm_gate: dtype %d", dtype);
+  if (tokens < 0 || heads <= 0 || vdim <= 0) return fail(MV_ERR_SHAPE, "diff_norm_gate: heads %d, vdim %d", heads, vdim);
+  if (tokens == 0) return MV_OK;
+  if (!out || !a || !gate) return fail(MV_ERR_NULL, "diff_norm_gate: null pointer");
+  const unsigned grid = static_cast<unsigned>(std::min<int64_t>((tokens * heads + 7) / 8, kNumSMs * 32));
+  auto run = [&](auto tag) {
+    using T = decltype(tag);
+    diff_norm_gate_kernel<T><<<grid, 256, 0, static_cast<cudaStream_t>(stream)>>>(
+        {static_cast<T*>(out), a, static_cast<const T*>(gate), gate_stride, tokens, heads, vdim, lambda, mult, eps});
+    return check_launch("diff_norm_gate");
+  };
+  return dtype == MV_F32 ? run(float{}) : run(__nv_bfloat16{});
 }

@@ -12,6 +12,7 @@ from .dafotar import DafotarConfig, DafotarForCausalLM
 from .fozerax import FozeraxConfig, FozeraxForCausalLM
 from .qwen3 import Qwen3Config, Qwen3ForCausalLM
 from .sipazen import SipazenConfig, SipazenForCausalLM
+from .subivik import SubivikConfig, SubivikForCausalLM
 from .weights import SafetensorsWeights
 
 
@@ -29,6 +30,7 @@ FAMILIES = {f.name: f for f in (
     ModelFamily("Sipazen", SipazenConfig, SipazenForCausalLM, "sipazen", loads_folders=True),
     ModelFamily("Fozerax", FozeraxConfig, FozeraxForCausalLM, "fozerax", loads_folders=True),
     ModelFamily("Dafotar", DafotarConfig, DafotarForCausalLM, "dafotar", loads_folders=True),
+    ModelFamily("Subivik", SubivikConfig, SubivikForCausalLM, "subivik", loads_folders=True),
 )}
 DEFAULT_FAMILY = "Qwen3ForCausalLM"
 

@@ -91,9 +91,9 @@ def gated_group_norm(y, z, weight, groups, eps):
     return out
 
 
-def head_norm_gate(y, z, weight, heads, eps, out=None, den=None, act="silu"):
-    """norm(y / den) * weight * act(z), rows in `heads` runs of channels; den (rows, heads) fp32 or None; weight has one run's
-    length, or a row's; act silu or sigmoid."""
+def head_norm_gate(y, z, weight, heads, eps, out=None, den=None, act="silu", mult=1.0):
+    """norm(y / den) * weight * act(z) * mult, rows in `heads` runs of channels; den (rows, heads) fp32 or None; weight has one
+    run's length, or a row's; act silu or sigmoid; out may have any row stride."""
     _cabi.require_cuda(y, z, weight, den)
     yp, ys = _rows(y, "y")
     zp, zs = _rows(z, "z")
@@ -103,7 +103,7 @@ def head_norm_gate(y, z, weight, heads, eps, out=None, den=None, act="silu"):
     if not full and weight.numel() * heads != y.shape[1]:
         raise ValueError("the norm's weight has neither a head's nor a row's length")
     _cabi.check(_cabi.lib().mv_head_norm_gate(
-        out.data_ptr(), yp, ys, _ptr(den), zp, zs, weight.data_ptr(), int(full), ACTS[act], y.shape[0], y.shape[1], heads, eps,
+        *_rows(out, "out"), yp, ys, _ptr(den), zp, zs, weight.data_ptr(), int(full), ACTS[act], mult, y.shape[0], y.shape[1], heads, eps,
         _cabi.layer_dtype_code(y.dtype), _cabi.stream_ptr()))
     return out
 

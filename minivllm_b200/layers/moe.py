@@ -16,16 +16,17 @@ from .group_norm import ACTS, gate_mul, moe_residual_norm
 from .linear import StackedLinear, router_logits
 
 
-def route(logits, bias, top, groups=1, keep=1):
+def route(logits, bias, top, groups=1, keep=1, over_all=False, scale=1.0):
     """fp32 logits (tokens, experts) -> (idx int32, weight fp32), both (tokens, top), best first.  Of `groups` equal runs
-    of experts only the `keep` with the largest maxima are chosen from."""
+    of experts only the `keep` with the largest maxima are chosen from.  Weights are `scale` times a softmax over the chosen
+    experts, or with `over_all` over all."""
     _cabi.require_cuda(logits)
     tokens, experts = logits.shape
     idx = torch.empty((tokens, top), dtype=torch.int32, device=logits.device)
     weight = torch.empty((tokens, top), dtype=torch.float32, device=logits.device)
     _cabi.check(_cabi.lib().mv_moe_route(idx.data_ptr(), weight.data_ptr(), logits.data_ptr(), logits.stride(0),
                                          bias.data_ptr() if bias is not None else None, tokens, experts, top, groups,
-                                         keep, _cabi.stream_ptr()))
+                                         keep, int(over_all), scale, _cabi.stream_ptr()))
     return idx, weight
 
 
@@ -76,10 +77,12 @@ def grouped_linear(x, weight, offsets, gated=False, tensor_cores=None, act="silu
 
 
 class MixtureOfExperts(nn.Module):
-    """spec: {'router': {'experts', 'top', 'groups': {'count', 'keep'} or absent}, 'expert': {'ff', 'limit' with the
-    clamped activation}, 'shared': the same or absent}; `load(name, shape)` returns a tensor of the layer's feed-forward."""
+    """spec: {'router': {'experts', 'top', 'groups': {'count', 'keep'} or absent, 'scale' of the weights or absent}, 'expert':
+    {'ff', 'limit' with the clamped activation}, 'shared': the same or absent}; `load(name, shape)` returns a tensor of the
+    layer's feed-forward.  `over_all`: weights are probabilities among all experts, not among the chosen."""
 
-    def __init__(self, spec, width, load, extra=None, act="silu", router_bias=True, shared_gate=True):
+    def __init__(self, spec, width, load, extra=None, act="silu", router_bias=True, shared_gate=True,
+                 over_all=False):
         super().__init__()
         self.experts, self.top = spec["router"]["experts"], spec["router"]["top"]
         groups = spec["router"].get("groups") or {"count": 1, "keep": 1}
@@ -87,6 +90,7 @@ class MixtureOfExperts(nn.Module):
         if self.experts % self.groups or not 0 < self.keep <= self.groups or \
                 not 0 < self.top <= self.experts // self.groups * self.keep:
             raise ValueError(f"moe: top {self.top} of {self.experts} experts in {self.groups} groups, {self.keep} kept")
+        self.over_all, self.scale = over_all, float(spec["router"].get("scale", 1.0))
         ff = spec["expert"]["ff"]
         self.act, self.limit = act, float(spec["expert"].get("limit", 0.0))
         param = lambda t: nn.Parameter(t, requires_grad=False)
@@ -112,16 +116,21 @@ class MixtureOfExperts(nn.Module):
             self.shared_down = param(load("shared.down", (width, sff)))
         self.stacked = StackedLinear(parts) if parts else None
 
+    def routed(self, h):
+        """h (tokens, width) -> (rows, pos, weight): token t's experts' results are rows[pos[t, k]], to be summed with
+        weight[t, k]."""
+        idx, weight = route(router_logits(h, self.router_w), self.router_b, self.top, self.groups, self.keep, self.over_all,
+                            self.scale)
+        pos, row_token, offsets = sort_by_expert(idx, self.experts)
+        act = grouped_linear(gather_rows(h, row_token), self.gate_up_w, offsets, gated=True, act=self.act,
+                             limit=self.limit)
+        return grouped_linear(act, self.down_w, offsets), pos, weight
+
     def forward(self, h, x, gate_bias, w_post, w_next, mult, groups, eps):
         """h: the sublayer's input, x: residual stream (updated in place).  Returns the next sublayer's input.  The
         residual gate, if any, is the stacked part 'residual_gate'."""
         p = self.stacked(h) if self.stacked is not None else {}
-        idx, weight = route(router_logits(h, self.router_w), self.router_b, self.top, self.groups,
-                            self.keep)
-        pos, row_token, offsets = sort_by_expert(idx, self.experts)
-        act = grouped_linear(gather_rows(h, row_token), self.gate_up_w, offsets, gated=True, act=self.act,
-                             limit=self.limit)
-        rows = grouped_linear(act, self.down_w, offsets)
+        rows, pos, weight = self.routed(h)
         shared = None
         if self.shared_down is not None:
             shared = F.linear(gate_mul(p["shared_up"], p["shared_gate"], self.act, limit=self.shared_limit),

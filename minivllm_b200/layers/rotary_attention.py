@@ -42,16 +42,19 @@ def _reorder(w, heads, order, dim=0):
 
 
 def qkv_rope_store(q, k, v, q_weight, k_weight, temp, eps, positions, table, dims, vtable, heads, kv_heads, cache=None,
-                   slot_mapping=None, packed=False):
+                   slot_mapping=None, packed=False, v_heads=None):
     """Norms and rotates q in place; [k | v], normed and rotated, goes to the cache and, with `packed`, to the returned
-    (tokens, row) tensor.  k and v None: queries only.  table, vtable: (cos, sin) or None.  See mv_qkv_rope_store."""
+    (tokens, row) tensor.  k and v None: queries only; q None: keys and values only; k_weight None: keys without a norm; v_heads:
+    value heads, when they are not as many as the key heads.  table, vtable: (cos, sin) or None.  See mv_qkv_rope_store."""
     _cabi.require_cuda(q, k, v, q_weight, k_weight, temp, cache, positions)
-    if k is not None and not q.stride(0) == k.stride(0) == v.stride(0):
+    if len({t.stride(0) for t in (q, k, v) if t is not None}) > 1:
         raise ValueError("q, k and v must share a row stride")
-    tokens, dim = q.shape[0], q.shape[1] // heads
-    G = kv_heads if k is not None else 0
-    vdim = v.shape[1] // G if G else 0
-    out = torch.empty((tokens, G * (dim + vdim)), dtype=q.dtype, device=q.device) if packed else None
+    any_, G = q if q is not None else k, kv_heads if k is not None else 0
+    VG = (v_heads or G) if G else 0
+    heads = heads if q is not None else 0
+    tokens, dim = any_.shape[0], any_.shape[1] // (heads or G)
+    vdim = v.shape[1] // VG if G else 0
+    out = torch.empty((tokens, G * dim + VG * vdim), dtype=any_.dtype, device=any_.device) if packed else None
     ptr = lambda t: t.data_ptr() if t is not None else None
     cos, sin = table if table is not None else (None, None)
     vcos, vsin = vtable if vtable is not None and G else (None, None)
@@ -59,10 +62,10 @@ def qkv_rope_store(q, k, v, q_weight, k_weight, temp, eps, positions, table, dim
     if not G:
         cache = None
     _cabi.check(_cabi.lib().mv_qkv_rope_store(
-        q.data_ptr(), ptr(k), ptr(v), q.stride(0), q_weight.data_ptr(), ptr(k_weight) if G else None, ptr(temp), ptr(cos), ptr(sin),
+        ptr(q), ptr(k), ptr(v), any_.stride(0), ptr(q_weight), ptr(k_weight) if G else None, ptr(temp), ptr(cos), ptr(sin),
         dims, ptr(vcos), ptr(vsin), min(rows) if rows else 1, positions.data_ptr(), ptr(out), ptr(cache),
         slot_mapping.data_ptr() if cache is not None else None, cache.shape[0] * cache.shape[1] if cache is not None else 0,
-        tokens, heads, G, dim, vdim, eps, _cabi.layer_dtype_code(q.dtype), _cabi.stream_ptr()))
+        tokens, heads, G, VG, dim, vdim, eps, _cabi.layer_dtype_code(any_.dtype), _cabi.stream_ptr()))
     return out
 
 

@@ -116,9 +116,17 @@ def window_prefill(q, kv, cu_q, cu_k, kv_heads, dim, vdim, window, scale, bias=N
 
 def window_keys(ctx, window, device):
     """Keys that the portions of a step can see through a window: (cu_k, first position of each sequence, total)."""
-    key = ("window_keys", window)
+    return _portion_keys(ctx, ("window_keys", window), lambda behind: max(0, behind - window + 1), device)
+
+
+def chunk_keys(ctx, size, device):
+    """The same for positions that see their own chunk of the sequence."""
+    return _portion_keys(ctx, ("chunk_keys", size), lambda behind: behind // size * size, device)
+
+
+def _portion_keys(ctx, key, first_of, device):
     if key not in ctx.memo:
-        first = [max(0, behind - window + 1) for behind, _ in ctx.portion_spans]
+        first = [first_of(behind) for behind, _ in ctx.portion_spans]
         cu = [0]
         for f, (behind, n) in zip(first, ctx.portion_spans):
             cu.append(cu[-1] + behind + n - f)
