@@ -249,7 +249,8 @@ constexpr int kScanMaxK = 256;
 
 // Logarithms of the decays, in 32-bit.
 __device__ __forceinline__ float channel_log_decay(float z, float inv_tau) { return -softplus_f(-z) * inv_tau; }
-__device__ __forceinline__ float time_log_decay(float z) { return -expf(z); }
+// A decay below e^-40 is none that fp32 could tell from zero; sums of logarithms stay small enough for their differences.
+__device__ __forceinline__ float time_log_decay(float z) { return -fminf(expf(z), 40.f); }
 __device__ __forceinline__ float head_log_decay(float a, float A_log, float dt_bias) { return -expf(A_log) * softplus_f(a + dt_bias); }
 constexpr float kUnitEps = 1e-6f;       // of q and k scaled to unit length
 constexpr float kMemFloor = 1e-6f;      // matrix memory: added to the denominator

@@ -226,7 +226,7 @@ def random_weights(config, seed=0, rank=5):
             a, b = m["left"], m["right"]
             H, G, d, vd = a["heads"], a["kv_heads"], a["dim"], a["vdim"]
             q = p + "left."
-            w.update({q + "q": mat(H * d, W, 1.5), q + "k": mat(G * d, W, 1.5), q + "v": mat(G * vd, W, 1.5),
+            w.update({q + "q": mat(H * d, W, 3.0), q + "k": mat(G * d, W, 3.0), q + "v": mat(G * vd, W, 1.5),
                       q + "r1": torch.rand(H, generator=g) * 1.2, q + "r2": torch.rand(H, generator=g) + 0.1,
                       q + "talk": torch.eye(H) + mat(H, H, 0.8), q + "o": mat(W, H * vd)})
             H, K = b["heads"], b["dim"]
