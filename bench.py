@@ -793,9 +793,9 @@ def main():
     ap.add_argument("--steps", type=int, default=None)
     ap.add_argument("--warmup", type=int, default=None)
     ap.add_argument("--impl", default="ours", choices=["ours", "reference"])
-    ap.add_argument("--workload", default="engine", choices=["engine", "decode", "allreduce", "ops", "sipazen", "fozerax", "dafotar"])
+    ap.add_argument("--workload", default="engine", choices=["engine", "decode", "allreduce", "ops", "sipazen", "fozerax", "dafotar", "subivik"])
     ap.add_argument("--case", default=None, help="operator case of --workload ops: " + ", ".join(OP_CASES) +
-                    "; of --workload sipazen, fozerax or dafotar: one of its kernels")
+                    "; of --workload sipazen, fozerax, dafotar or subivik: one of its kernels")
     ap.add_argument("--cpu-seconds", type=float, default=10.0)
     ap.add_argument("--no-extras", action="store_true", help="skip the secondary operator numbers and the CPU leg")
     ap.add_argument("--small", action="store_true",
@@ -810,7 +810,7 @@ def main():
         if not ours:
             args.steps = min(args.steps, 2)      # each CPU step is ~20-40 s of host work
             args.warmup = min(args.warmup, 1)    # (a short pass that touches every weight once)
-    elif args.workload in ("sipazen", "fozerax", "dafotar"):
+    elif args.workload in ("sipazen", "fozerax", "dafotar", "subivik"):
         args.steps, args.warmup = 20 if args.steps is None else args.steps, 3
     elif args.workload == "ops":
         args.case = args.case or "store_kvcache_bf16"
@@ -854,6 +854,9 @@ def main():
     elif args.workload == "dafotar":
         import bench_dafotar
         line = bench_dafotar.run(device, pk, args.steps, args.case)
+    elif args.workload == "subivik":
+        import bench_subivik
+        line = bench_subivik.run(device, pk, args.steps, args.case)
     elif args.workload == "ops":
         line = run_ops(args, device, pk)
     else:
