@@ -11,11 +11,12 @@ import torch
 
 
 def _median_ms(fn, iters, warmup=3):
-    """Median device time of single calls."""
+    """Median device time of single calls, queued behind a pause of some 20 ms so that the host's own time stays out of it."""
     for _ in range(warmup):
         fn()
     torch.cuda.synchronize()
     ev = [(torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)) for _ in range(iters)]
+    torch.cuda._sleep(40_000_000)
     for a, b in ev:
         a.record()
         fn()

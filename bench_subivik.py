@@ -44,7 +44,7 @@ def _wave(dev):
 
 
 def _sfu(d, weights, per_weight):
-    """Fraction of the special-function unit's rate at the SM clock's maximum that the given weights want."""
+    """Fraction of the special-function unit's rate, at the SM clock's maximum, that the given weights take up."""
     d["frac_sfu"] = weights * per_weight / (d["us"] * 1e-6) / (148 * SFU_PER_SM_CLOCK * 1965e6)
     return d
 
@@ -64,7 +64,7 @@ def kernel_talk_prefill(dev, pk, iters=20, heads=16, kv=4, dim=128, vdim=128):
     d = _line(ms, pk, flops=2.0 * heads * (dim + vdim) * pairs, nbytes=2 * T * (heads * dim + kv * (dim + vdim) + heads * kv * vdim))
     passes = -(-kv // (4 // (vdim // 64)))
     d["frac_bf16_made"] = 2.0 * heads * (passes * dim + kv * vdim) * pairs / ms / 1e9 / pk["bf16_tflops"]
-    return _sfu(d, passes * heads * pairs, 3)
+    return _sfu(d, passes * heads * pairs, 1.875)
 
 
 def kernel_head_mix(dev, pk, iters=20, rows=16384, heads=16, kv=4, vdim=128):

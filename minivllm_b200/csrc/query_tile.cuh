@@ -39,4 +39,28 @@ __device__ __forceinline__ void find_query_tile(const int32_t* cu_q, int num_seq
   }
 }
 
+// Tile x of the same order, by every warp for itself: false without a tile.
+__device__ __forceinline__ bool find_query_tile_warp(const int32_t* cu_q, int num_seqs, int rows, int x, int& seq, int& tile) {
+  const int lane = threadIdx.x & 31;
+  int base = 0;
+  for (int b = 0; b < num_seqs; b += 32) {
+    const int s = b + lane, n = s < num_seqs ? (max(cu_q[s + 1] - cu_q[s], 0) + rows - 1) / rows : 0;
+    int incl = n;
+#pragma unroll
+    for (int o = 1; o < 32; o <<= 1) {
+      const int v = __shfl_up_sync(0xffffffffu, incl, o);
+      if (lane >= o) incl += v;
+    }
+    const uint32_t past = __ballot_sync(0xffffffffu, base + incl > x);
+    if (past) {
+      const int at = __ffs(past) - 1;
+      seq = b + at;
+      tile = base + __shfl_sync(0xffffffffu, incl, at) - 1 - x;
+      return true;
+    }
+    base += __shfl_sync(0xffffffffu, incl, 31);
+  }
+  return false;
+}
+
 }  // namespace mv

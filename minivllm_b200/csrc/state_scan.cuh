@@ -517,10 +517,10 @@ __device__ __forceinline__ void mem_advance(const ScanParams<T>& p, int h, int s
 }
 
 // The vectors of a token for the step kernels: K (padded) values of k and q, gated linear attention's alpha - 1, V (padded)
-// values of v; the delta rule's go through the convolution, matrix memory's k takes its factor.
+// values of v; the delta rule's go through the convolution, matrix memory's k takes its factor; time mixing: s_u = k times the bonus.
 template <int KIND, typename T>
 __device__ __forceinline__ void step_vectors(const ScanParams<T>& p, int s, int h, int slot, int st0, int K, int vpad, float* s_k,
-                                             float* s_q, float* s_a, float* s_v, const MemFactors& mem) {
+                                             float* s_q, float* s_a, float* s_v, const MemFactors& mem, float* s_u) {
   constexpr bool kDelta = KIND == SK_DELTA, kMem = KIND == SK_MLSTM, kTime = KIND == SK_TIME;
   const int kh = h / (p.heads / p.kv_heads);
   for (int i = threadIdx.x; i < K + K + vpad; i += blockDim.x) {
@@ -548,6 +548,7 @@ __device__ __forceinline__ void step_vectors(const ScanParams<T>& p, int s, int 
     }
     (part == 0 ? s_k : part == 1 ? s_q : s_v)[j] = x;
     if (kMem && part == 0) s_a[j] = mem.alpha_m1;
+    if (kTime && part == 0) s_u[j] = ok ? x * Elem<T>::to_f(p.bonus[h * p.K + j]) : 0.f;
     if (kTime && part == 0)
       s_a[j] = ok ? expm1f(time_log_decay(p.zf[static_cast<int64_t>(s) * p.zf_stride + h * p.K + j] + Elem<T>::to_f(p.w0[h * p.K + j]))) : 0.f;
     if (!kDelta && !kMem && !kTime && part == 0)
@@ -577,16 +578,28 @@ __device__ __forceinline__ StepFactors step_factors(const ScanParams<T>& p, int 
 }
 
 // Time mixing: what a token's own entry adds to its read-out, per value.  Every warp for itself.
-template <typename T> __device__ __forceinline__ float own_entry(const ScanParams<T>& p, int h, const float* s_k, const float* s_q) {
+__device__ __forceinline__ float own_entry(int K, const float* s_u, const float* s_q) {
   float acc = 0.f;
-  for (int j = threadIdx.x & 31; j < p.K; j += 32) acc = fmaf(s_k[j] * Elem<T>::to_f(p.bonus[h * p.K + j]), s_q[j], acc);
+  for (int j = threadIdx.x & 31; j < K; j += 32) acc = fmaf(s_u[j], s_q[j], acc);
   return warp_sum(acc);
 }
 
-// Norm of the head's read-out and output gate; matrix memory divides first (s_nq: the terms of n . q).
+template <typename T> __device__ __forceinline__ const T* step_gate(const ScanParams<T>& p, int s, int h) {
+  return p.gate + static_cast<int64_t>(s) * p.out_gate_stride + static_cast<int64_t>(h) * p.V;
+}
+template <int KIND, typename T> __device__ __forceinline__ const T* step_weight(const ScanParams<T>& p, int h) {
+  return p.norm_w + (KIND == SK_MLSTM || KIND == SK_TIME ? static_cast<int64_t>(h) * p.V : 0);
+}
+template <int KIND, typename T> __device__ __forceinline__ void step_ahead(const ScanParams<T>& p, int s, int h, T (&first)[2]) {
+  const int j = threadIdx.x;
+  first[0] = j < p.V ? step_gate<T>(p, s, h)[j] : Elem<T>::from_f(0.f);
+  first[1] = j < p.V ? step_weight<KIND, T>(p, h)[j] : Elem<T>::from_f(0.f);
+}
+// Norm of the head's read-out and output gate; matrix memory divides first (s_nq: the terms of n . q).  `first`: gate and weight
+// of this thread's first column, fetched ahead.
 template <int KIND, typename T>
 __device__ __forceinline__ void step_output(const ScanParams<T>& p, int s, int h, const float* s_o, T* out, const float* s_nq,
-                                            const MemFactors& mem) {
+                                            const MemFactors& mem, const T (&first)[2]) {
   constexpr bool kMem = KIND == SK_MLSTM, kTime = KIND == SK_TIME;
   float inv = 1.f;
   if (kMem) {
@@ -597,11 +610,11 @@ __device__ __forceinline__ void step_output(const ScanParams<T>& p, int s, int h
   float acc = 0.f;
   for (int j = threadIdx.x & 31; j < p.V; j += 32) acc = fmaf(s_o[j] * inv, s_o[j] * inv, acc);
   const float rs = inv / sqrtf(warp_sum(acc) / static_cast<float>(p.V) + p.eps);
-  const T* gate = p.gate + static_cast<int64_t>(s) * p.out_gate_stride + static_cast<int64_t>(h) * p.V;
-  const T* w = p.norm_w + (kMem || kTime ? static_cast<int64_t>(h) * p.V : 0);
+  const T *gate = step_gate<T>(p, s, h), *w = step_weight<KIND, T>(p, h);
   for (int j = threadIdx.x; j < p.V; j += blockDim.x) {
-    const float g = Elem<T>::to_f(gate[j]);
-    out[j] = Elem<T>::from_f(s_o[j] * rs * Elem<T>::to_f(w[j]) * (kMem ? sigmoid_t<T>(g) : silu_t<T>(g)) * (kTime ? p.out_scale : 1.f));
+    const bool ahead = j == static_cast<int>(threadIdx.x);
+    const float g = Elem<T>::to_f(ahead ? first[0] : gate[j]), wj = Elem<T>::to_f(ahead ? first[1] : w[j]);
+    out[j] = Elem<T>::from_f(s_o[j] * rs * wj * (kMem ? sigmoid_t<T>(g) : silu_t<T>(g)) * (kTime ? p.out_scale : 1.f));
   }
 }
 
@@ -623,14 +636,16 @@ __global__ void __launch_bounds__(256, 1) step_kernel(const ScanParams<T> p) {
   }
   const bool vec = p.V % 4 == 0;
   float* gS = p.state + (static_cast<int64_t>(slot) * p.heads + h) * p.K * p.V;
+  T first[2];
+  step_ahead<Sh::KIND>(p, s, h, first);
   MemFactors mem{};
   if constexpr (kMem) mem = mem_factors(p, s, h, slot, st0);
-  step_vectors<Sh::KIND>(p, s, h, slot, st0, K, vpad, s_k, s_q, s_a, s_v, mem);
+  step_vectors<Sh::KIND>(p, s, h, slot, st0, K, vpad, s_k, s_q, s_a, s_v, mem, s_nq);
   __syncthreads();
   if constexpr (kMem) mem_advance(p, h, slot, st0, mem, s_k, s_q, s_nq);
   StepFactors f{};
   if (kDelta) f = step_factors(p, s, h, K, s_k, s_q);
-  const float own = kTime ? own_entry(p, h, s_k, s_q) : 0.f;
+  const float own = kTime ? own_entry(p.K, s_nq, s_q) : 0.f;
   const bool writes = (!kDelta || (kp & (Sh::KP / 2))) && (kp & (Sh::LOW - 1)) == 0;
   ScanState<Sh> S;
   for (int cb = warp; cb * Sh::CW < p.V; cb += warps) {
@@ -649,7 +664,7 @@ __global__ void __launch_bounds__(256, 1) step_kernel(const ScanParams<T> p) {
     S.store(gS + c0, kp, p.K, p.V, p.V - c0, vec);
   }
   __syncthreads();
-  step_output<Sh::KIND>(p, s, h, s_o, out, s_nq, mem);
+  step_output<Sh::KIND>(p, s, h, s_o, out, s_nq, mem, first);
 }
 
 // vdim a multiple of four: a thread has four columns of every rows-th row of S, so that a warp reads whole lines, and the
@@ -664,8 +679,8 @@ __global__ void __launch_bounds__(kStThreads4, 2) step_quad_kernel(const ScanPar
   const int PQ = p.V / 4, rows = nthr / PQ, q = tid % PQ, r = tid / PQ;
   const bool on = r < rows;
   float *s_k = sm, *s_q = s_k + K, *s_a = s_q + K, *s_v = s_a + (kDelta ? 0 : K), *s_o = s_v + vpad;
-  float* s_nq = s_o + vpad;                                      // matrix memory
-  float4* red = reinterpret_cast<float4*>(s_nq + (kMem ? K : 0));        // [rows][PQ], twice for the delta rule
+  float* s_nq = s_o + vpad;                                      // matrix memory, time mixing
+  float4* red = reinterpret_cast<float4*>(s_nq + (kMem || kTime ? K : 0));        // [rows][PQ], twice for the delta rule
   const int slot = p.slots[s], st0 = p.start[s];
   T* out = p.out + static_cast<int64_t>(s) * p.out_stride + static_cast<int64_t>(h) * p.V;
   if (slot < 0 || slot >= p.num_slots || st0 < 0) {
@@ -683,9 +698,11 @@ __global__ void __launch_bounds__(kStThreads4, 2) step_quad_kernel(const ScanPar
     }
   };
   fetch(0);                              // in flight while the vectors are made
+  T first[2];
+  step_ahead<KIND>(p, s, h, first);
   MemFactors mem{};
   if constexpr (kMem) mem = mem_factors(p, s, h, slot, st0);
-  step_vectors<KIND>(p, s, h, slot, st0, K, vpad, s_k, s_q, s_a, s_v, mem);
+  step_vectors<KIND>(p, s, h, slot, st0, K, vpad, s_k, s_q, s_a, s_v, mem, s_nq);
   __syncthreads();
   if constexpr (kMem) mem_advance(p, h, slot, st0, mem, s_k, s_q, s_nq);
   const float4 v = on ? *reinterpret_cast<const float4*>(s_v + q * 4) : zero;
@@ -712,7 +729,7 @@ __global__ void __launch_bounds__(kStThreads4, 2) step_quad_kernel(const ScanPar
       }
     }
     if (on) red[r * PQ + q] = aq;
-    const float own = kTime ? own_entry(p, h, s_k, s_q) : 0.f;
+    const float own = kTime ? own_entry(p.K, s_nq, s_q) : 0.f;
     __syncthreads();
     for (int i = tid; i < p.V; i += nthr) {
       float o = kTime ? own * s_v[i] : 0.f;
@@ -771,7 +788,7 @@ __global__ void __launch_bounds__(kStThreads4, 2) step_quad_kernel(const ScanPar
     }
   }
   __syncthreads();
-  step_output<KIND>(p, s, h, s_o, out, s_nq, mem);
+  step_output<KIND>(p, s, h, s_o, out, s_nq, mem, first);
 }
 
 template <typename Sh, typename T, int W>
@@ -800,7 +817,7 @@ template <int KIND, typename T> static int run_step(const ScanParams<T>& p, int 
     const int quads = p.V / 4, K = (p.K + 3) & ~3;
     const int threads = std::min(kStThreads4, std::max(128, (quads * ((p.K + kStHold - 1) / kStHold) + 31) / 32 * 32));
     const int fit = std::max(threads, (quads + 31) / 32 * 32), rows = fit / quads;
-    const size_t smem = sizeof(float) * ((KIND == SK_DELTA ? 2 : KIND == SK_MLSTM ? 4 : 3) * K + 2 * p.V + (KIND == SK_DELTA ? 2 : 1) * static_cast<size_t>(rows) * p.V);
+    const size_t smem = sizeof(float) * ((KIND == SK_DELTA ? 2 : KIND == SK_GLA ? 3 : 4) * K + 2 * p.V + (KIND == SK_DELTA ? 2 : 1) * static_cast<size_t>(rows) * p.V);
     if (smem <= 48 * 1024) {
       step_quad_kernel<KIND, T><<<dim3(num_seqs, p.heads), fit, smem, st>>>(p, p.V);
       return check_launch("state_step");
@@ -809,7 +826,7 @@ template <int KIND, typename T> static int run_step(const ScanParams<T>& p, int 
   return scan_dispatch<KIND>(p.K, [&](auto sh) {
     using Sh = decltype(sh);
     const int blocks = (p.V + Sh::CW - 1) / Sh::CW, warps = std::min(8, blocks);
-    const size_t smem = sizeof(float) * ((KIND == SK_DELTA ? 2 : KIND == SK_MLSTM ? 4 : 3) * Sh::K + 2 * static_cast<size_t>(blocks) * Sh::CW);
+    const size_t smem = sizeof(float) * ((KIND == SK_DELTA ? 2 : KIND == SK_GLA ? 3 : 4) * Sh::K + 2 * static_cast<size_t>(blocks) * Sh::CW);
     if (smem > 48 * 1024) return fail(MV_ERR_LIMIT, "state_step: vdim %d", p.V);
     step_kernel<Sh, T><<<dim3(num_seqs, p.heads), 32 * warps, smem, st>>>(p);
     return check_launch("state_step");
