@@ -304,6 +304,26 @@ def test_scores_at_the_cap(dtype):
         _close(out, torch.stack([mixed[h] @ v[:, h // 2].double() for h in range(H)], 1).flatten(1), tol, "decode")
 
 
+@pytest.mark.parametrize("lens", [[2, 3] * 600, [1300, 2, 700, 129, 128, 127, 257]], ids=["many", "long"])
+def test_prefill_over_many_units(lens):
+    """More sequences than the prefill kernel keeps bounds of, and more units of work than there are SMs; portions behind a past
+    of their own.  Against the kernel for any sizes."""
+    from minivllm_b200.layers import talk_attention as TA
+    H, G, d, vd, bs, cap = 6, 3, 64, 64, 16, 20.0
+    behind = [(7 * i) % 40 for i in range(len(lens))]
+    total = [n + b for n, b in zip(lens, behind)]
+    rows = [_rnd(i, n, G * (d + vd)).bfloat16() for i, n in enumerate(total)]
+    q, r1, r2 = 2.0 * _rnd(5, sum(lens), H * d), torch.rand(H).cuda(), torch.rand(H).cuda()
+    cache, tables = _paged(rows, bs, torch.bfloat16)
+    q, packed = q.bfloat16().cuda(), torch.cat(rows).cuda()
+    pos = torch.cat([torch.arange(b, b + n) for n, b in zip(lens, behind)]).cuda()
+    args = (G, d, vd, 0.3, r1, r2, cap)
+    want = TA.talk_attention_rows(q, cache, tables, _cu(lens), pos, *args)
+    got = TA.talk_prefill(q, packed[:, :G * d], packed[:, G * d:], _cu(lens), _cu(total), *args)
+    _close(got, want.cpu(), 1.2e-2)
+    assert int(TA._error_word(q.device).item()) == 0
+
+
 def test_a_long_past():
     """One token behind 9,000 others: the only key that matters is the first, the weights reach it past all the others."""
     from minivllm_b200.layers import talk_attention as TA
