@@ -7,7 +7,7 @@ from oracle import subivik_oracle as oracle
 from tests.sipazen_cases import error
 
 
-def _par(left, right, cap=20.0, scale=None, left_scale=0.8, right_scale=0.5):
+def _par(left, right, cap=18.0, scale=None, left_scale=0.9, right_scale=0.6):
     """left (heads, kv_heads, dim, vdim), right (heads, dim)."""
     H, G, d, vd = left
     return "parallel", {"left": {"heads": H, "kv_heads": G, "dim": d, "vdim": vd, "softcap": cap,
@@ -15,7 +15,7 @@ def _par(left, right, cap=20.0, scale=None, left_scale=0.8, right_scale=0.5):
                         "right": {"heads": right[0], "dim": right[1]}, "left_scale": left_scale, "right_scale": right_scale}
 
 
-def _att(heads, kv, dim, vdim, chunk, diff=0.6, scale=None, kv_from=None):
+def _att(heads, kv, dim, vdim, chunk, diff=0.55, scale=None, kv_from=None):
     m = {"heads": heads, "kv_heads": kv, "dim": dim, "vdim": vdim, "mask": {"size": chunk}, "diff": diff,
          "scale": scale if scale is not None else dim ** -0.5}
     if kv_from is not None:
@@ -23,7 +23,7 @@ def _att(heads, kv, dim, vdim, chunk, diff=0.6, scale=None, kv_from=None):
     return "attention", m
 
 
-def _moe(experts, top, ff, scale=1.5):
+def _moe(experts, top, ff, scale=1.7):
     return {"kind": "moe", "expert": {"ff": ff}, "router": {"experts": experts, "top": top, "scale": scale}}
 
 
@@ -50,7 +50,7 @@ def odd():
 def even():
     """Sizes that the tensor-core kernels take, chunks shorter and longer than a tile of keys."""
     return _config(320, 192, [
-        (_par((8, 4, 64, 128), (3, 64)), None),
+        (_par((6, 3, 64, 128), (3, 64)), None),
         (_att(8, 2, 64, 128, 33), _dense(256)),
         (_par((6, 2, 128, 64), (1, 128), cap=30.0), _moe(16, 4, 40)),
         (_att(8, 2, 64, 128, 150, diff=0.4, kv_from=1), _moe(8, 2, 64, scale=2.5)),

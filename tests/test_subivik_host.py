@@ -77,7 +77,7 @@ def test_constants_of_a_layer():
     assert abs(m.layers[2].mixer.lam - float(want)) < 1e-6 and m.layers[2].mixer.mult == 1 - 0.3
     p, q = (oracle.softplus(x) for x in d["l4.mlp.act"])
     assert abs(m.layers[4].mlp.a - float(p)) < 1e-6 and abs(m.layers[4].mlp.b - 0.5 - float(q)) < 1e-6
-    assert m.layers[0].mlp.scale == 1.5 and m.layers[0].mlp.over_all
+    assert m.layers[0].mlp.scale == 1.7 and m.layers[0].mlp.over_all
     f = position_frequencies(7, "cpu")
     assert f.dtype == torch.float64 and f.numel() == 4 and float(f[3]) == 10000.0 ** (-6 / 7)
 
